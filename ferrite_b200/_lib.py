@@ -52,6 +52,12 @@ SIGNATURES = {
     "fb_argmax": (_i, [_p, _i64, _i64, _i64, _p, _p, _p]),
     "fb_rope_kv_write_packed": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _p, _p, _i64, _i64, _p, _p, _p, _f, _p, _i64, _p, _i64, _p]),
     "fb_decode_attention_packed": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _p, _i64, _p, _p, _i64, _i, _p, _i64, _p, _sz, _p]),
+    "fb_latent_put": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _i, _p, _p, _f, _p, _f, _p, _p, _i, _p, _i64, _p, _i64, _p]),
+    "fb_rotate_pairs": (_i, [_i, _p, _i64, _i, _i64, _i64, _i, _i, _p, _f, _p, _p, _i64, _i64, _p]),
+    "fb_latent_attention_workspace_bytes": (_sz, [_i, _i64, _i, _i, _i, _i64, _i]),
+    "fb_latent_attention": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _p, _i64, _p, _i64, _p, _i64, _i, _f, _p, _p, _i64, _p, _sz, _p]),
+    "fb_decay_scan": (_i, [_i, _p, _i64, _i, _i, _i, _p, _p, _i, _i64, _i64, _p, _i64, _p, _i64, _p]),
+    "fb_gated_rmsnorm": (_i, [_p, _i64, _i64, _i64, _i, _p, _i64, _p, _f, _p, _i64, _p]),
     "fb_peer_reduce_add": (_i, [_p, _p, _i, _i, _p, _i64, _p, _p, _p]),
 }
 

@@ -8,7 +8,7 @@ batch) that is carried out either on the host in numpy (`bits()`: what the oracl
 (`device(rt)`: every piece is copied up as it lies in the file and transposed / joined there by this library's strided
 copy kernel, so an 8 B-parameter model's transposes cost no host time); `llama.upload` then casts each matrix to its
 block-float format on the device.  Covered: Llama / SmolLM / Qwen3 dense models and Mixtral- and Qwen3-style mixtures
-(BF16 or F32 tensors).  Not covered, and refused by name: Gated DeltaNet blocks, gated attention, biases, MXFP4 experts.
+(BF16 or F32 tensors), and the designs models.py names by config.json's "architecture", whose modules name their weights.  Not covered, and refused by name: Gated DeltaNet blocks, gated attention, biases, MXFP4 experts.
 """
 import json
 import os
@@ -17,7 +17,7 @@ import struct
 
 import numpy as np
 
-from . import llama
+from . import llama, models
 
 
 def safetensors(path):
@@ -90,6 +90,27 @@ def stack(ws):
                   lambda rt: (lambda xs: xs[0].cat(*xs[1:], axis=0))([w.device(rt) for w in ws]))
 
 
+def rows(*ws):
+    """Matrices one above the other (stored out x in: projections of the same rows side by side)."""
+    return Weight(lambda: np.ascontiguousarray(np.concatenate([w.bits() for w in ws], -2)),
+                  lambda rt: (lambda xs: xs[0].cat(*xs[1:], axis=1))([w.device(rt) for w in ws]))
+
+
+def batched(w, n):
+    """A matrix cut along its rows into a batch of n (a head's own each)."""
+    return Weight(lambda: (lambda b: b.reshape(n, b.shape[-2] // n, b.shape[-1]))(w.bits()), lambda rt: (lambda x: x.reshape(n, x.rows // n, x.cols))(w.device(rt)))
+
+
+def turned(w):
+    """A stored out x in matrix as x @ w takes it; on the device a view, so each output column's weights lie together."""
+    return Weight(lambda: np.ascontiguousarray(np.swapaxes(w.bits(), -1, -2)), lambda rt: w.device(rt).T)
+
+
+def columns_together(w):
+    """A matrix that x @ w takes as it is, laid out on the device as `turned` leaves one: each output column's weights together."""
+    return Weight(w.bits, lambda rt: (w.device(rt).T + 0).realize().T)
+
+
 def read_json(path):
     with open(path, encoding="utf-8") as f:
         return json.load(f)
@@ -98,6 +119,9 @@ def read_json(path):
 def config(folder, places=4096):
     """A model's config.json as a decode-path config (models/llama.py:545-570), for the families covered here."""
     j = read_json(os.path.join(folder, "config.json"))
+    family = models.of_json(j)
+    if family is not llama:
+        return family.config(j, places)
     j = j.get("text_config", j)
     rope = j.get("rope_parameters") or (j.get("rope_scaling") or {}) | {"rope_theta": j["rope_theta"]}
     theta, kind = rope.pop("rope_theta"), rope.pop("type", None)
@@ -148,6 +172,9 @@ def load(folder, places=4096):
     for file in files:
         header, data = safetensors(os.path.join(folder, file))
         tensors |= {name: (data, t) for name, t in header.items() if name != "__metadata__"}
+    family = models.of(c)
+    if family is not llama:
+        return c, family.weights(tensors, c)
     for full, (data, t) in tensors.items():
         name = full.removeprefix("model.").removeprefix("language_model.").removesuffix(".weight")
         for part in ("self_attn.", "mlp.", "block_sparse_moe."):

@@ -16,7 +16,7 @@ constexpr int EW_MAX_INPUTS = 8, EW_MAX_OPS = 48, EW_STACK = 12;
 enum EwOp {
   EW_LOAD = 0, EW_CONST = 1,
   EW_ADD = 10, EW_SUB, EW_MUL, EW_MAX, EW_CMPLT, EW_CMPNE, EW_KEEP, EW_DROP, EW_DIV, EW_MIN,
-  EW_EXP = 30, EW_LOG, EW_SIN, EW_COS, EW_SQRT, EW_RECIP, EW_RELU, EW_EXP2, EW_LOG2, EW_BF16, EW_TRUNC, EW_NEG
+  EW_EXP = 30, EW_LOG, EW_SIN, EW_COS, EW_SQRT, EW_RECIP, EW_RELU, EW_EXP2, EW_LOG2, EW_BF16, EW_TRUNC, EW_NEG, EW_TANH
 };
 
 struct EwOperand {
@@ -68,6 +68,7 @@ __global__ void __launch_bounds__(256) elementwise_kernel(const __grid_constant_
           case EW_BF16: x = bf16_bits_to_float(float_to_bf16_bits(x)); break;
           case EW_TRUNC: x = truncf(x); break;
           case EW_NEG: x = -x; break;
+          case EW_TANH: x = tanhf(x); break;
         }
         st[sp - 1] = x;
         continue;

@@ -1,0 +1,35 @@
+// bf16 / fp32 values behind one name, for the kernels that run in either: a pointer's type says how its values are stored,
+// arithmetic is fp32 throughout.
+#pragma once
+#include "common.cuh"
+
+namespace fb {
+
+__device__ __forceinline__ float value_of(float x) { return x; }
+__device__ __forceinline__ float value_of(uint16_t x) { return bf16_bits_to_float(x); }
+__device__ __forceinline__ void store_value(float* p, float v) { *p = v; }
+__device__ __forceinline__ void store_value(uint16_t* p, float v) { *p = (uint16_t)float_to_bf16_bits(v); }
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+
+// sum over a block of up to 1024 threads (whole warps); every thread gets it.  `red` is 32 floats of shared memory
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  __syncthreads();  // (the words may still be read from a sum before)
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float total = 0.f;
+  for (int w = 0; w < (int)(blockDim.x + 31) / 32; ++w) total += red[w];
+  return total;
+}
+
+// cos and sin of place * freq, times mag.  The angle is formed in double and brought into one turn there, so that a far
+// place's angle is as exact as a near one's.
+__device__ __forceinline__ void turn_of(int place, double freq, float mag, float& c, float& s) {
+  const double turns = (double)place * freq * 0.15915494309189535;  // / (2 pi)
+  float a = (float)((turns - rint(turns)) * 6.283185307179586);
+  sincosf(a, &s, &c);
+  c *= mag, s *= mag;
+}
+
+}  // namespace fb

@@ -17,7 +17,7 @@ from . import ops
 from .tensor import BFP, Tensor, jit  # noqa: F401  (jit re-exported: `from ferrite_b200.llama import jit`)
 
 # a config's fields past a plain Llama's, as a plain Llama has them (models/llama.py:541-543)
-DEFAULTS = dict(head_dim=None, rope=None, sliding=None, k=0, experts=0, moe=0, norm_topk=True, tied=False, precision=None, places=4096,
+DEFAULTS = dict(family="llama", head_dim=None, rope=None, sliding=None, k=0, experts=0, moe=0, norm_topk=True, tied=False, precision=None, places=4096,
                 ffn=None, vocab=None, qk_norm=False, tp=None)
 
 
@@ -63,9 +63,9 @@ def weight_format(name, prec):
     return "bf16"
 
 
-def upload(rt, weights, prec=None):
+def upload(rt, weights, prec=None, weight_format=weight_format):
     """name -> Tensor from name -> numpy arrays of bf16 values, each cast on the device to its format
-    (models/llama.py:628-640).  qk_norm / qk_on arrive as the reference stacks them ([heads, 1, hd])."""
+    (models/llama.py:628-640; weight_format: another family's own).  qk_norm / qk_on arrive as the reference stacks them ([heads, 1, hd])."""
     t = {}
     for name, w in weights.items():
         f = weight_format(name, prec)
@@ -358,7 +358,9 @@ def forward(ids, places, w, c, caches, slots=None, every=False, length=None):
     for l in range(c.layers):
         x = layer(x, blocks[l], c, rotary, seen, caches[l], rows, live, slots)
     h = rms(x, w["norm"], c)
-    if not (slots or every):
+    if isinstance(every, Tensor):  # the rows it names (int32, on the device)
+        h = h.realize().gather(every)
+    elif not (slots or every):
         h = h.realize()[:, x.rows - 1:, :]
     return h.matmul(w["embed.T"], dtype="fp32")
 
@@ -367,10 +369,11 @@ def prefill(ids, w, c, caches, tokens, on):
     """A prompt from place 0 in chunks of `tokens` (models/llama.py:498-504): a chunk's keys and values are in the caches
     before the next chunk attends, so the scores are a chunk's rows by the places so far, never the prompt squared.
     on: makes the int32 row tensor forward takes from a list.  Returns the logits for the token after the prompt."""
-    out = None
+    from . import models
+    out, step = None, models.of(c).forward
     for first in range(0, len(ids), tokens):
         chunk = list(ids[first:first + tokens])
-        out = forward(on(chunk), on(list(range(first, first + len(chunk)))), w, c, caches)
+        out = step(on(chunk), on(list(range(first, first + len(chunk)))), w, c, caches)
     return out
 
 
@@ -390,8 +393,8 @@ def slot(c, caches, u, slots):
 def zeros(rt, dtype="bf16"):
     """zeros of a shape on the device, for kv_cache (models/llama.py:656-658)."""
     def make(shape, d=None):
-        t = Tensor(rt, shape[1], shape[2], batch=shape[0], dtype=dtype)
-        (t.packed.data if dtype in BFP else t.buf).zero_()  # (a block float of zero bytes is zeros)
+        t = Tensor(rt, shape[1], shape[2], batch=shape[0], dtype=d or dtype)
+        (t.packed.data if t.dtype in BFP else t.buf).zero_()  # (a block float of zero bytes is zeros)
         return t
     return make
 

@@ -1,0 +1,24 @@
+"""The model families this library serves.  A family is a module with the decode path's calls - config, weights, upload,
+precision, forward, kv_cache, slot - and everything that drives a model (the checkpoint reader, the engine, the command
+line) finds it here: by a config's `family`, or, when a checkpoint is opened, by config.json."""
+import importlib
+
+FAMILIES = {"llama": "llama", "binutar": "binutar"}  # a config's family -> its module of this package
+ARCHITECTURES = {"Binutar": "binutar"}  # config.json's "architecture" -> family (Hugging Face configs, which have none, are Llama-like)
+
+
+def module(family):
+    assert family in FAMILIES, f"no model family {family!r}: {', '.join(sorted(FAMILIES))}"
+    return importlib.import_module("." + FAMILIES[family], __package__)
+
+
+def of(c):
+    """The family module of a model's config."""
+    return module(getattr(c, "family", "llama"))
+
+
+def of_json(j):
+    """The family module of a parsed config.json."""
+    name = j.get("architecture")
+    assert name is None or name in ARCHITECTURES, f"architecture {name!r} is not served here: {', '.join(sorted(ARCHITECTURES))}"
+    return module(ARCHITECTURES.get(name, "llama"))

@@ -6,6 +6,7 @@ from . import _lib
 from ._lib import BF16, BFP4, BFP8, FP32, check, lib
 
 _TORCH = {"bf16": torch.bfloat16, "fp32": torch.float32, "int32": torch.int32}
+_CODES = {torch.bfloat16: BF16, torch.float32: FP32, torch.int32: _lib.INT32}
 
 KERNELS = [0]  # kernels of this library launched so far by this process (every wrapper below counts its own)
 
@@ -261,4 +262,53 @@ def linear_indexed(x, w, index, out, sum_slots=False, x_slot_rows=0, out_slot_st
                                   _ptr(residual), residual.stride(0) if residual is not None else 0, _ptr(row_scale), _ptr(ws),
                                   ws.numel() if ws is not None else 0, _stream()))
     count(2 if norm_w is not None else 1)
+    return out
+
+
+def latent_put(down, q_rank, kv_rank, rot, dims, q_norm, kv_norm, eps, freq, mag, places, rows, cache, q_out):
+    """The norms, the turn and the cache write after a joint down-projection (fb_latent_put)."""
+    check(lib().fb_latent_put(_CODES[down.dtype], down.data_ptr(), down.shape[0], down.stride(0), q_rank, kv_rank, rot, dims, _ptr(q_norm), kv_norm.data_ptr(), eps,
+                              freq.data_ptr(), mag, places.data_ptr(), rows.data_ptr(), _CODES[cache.dtype], _ptr(q_out), q_out.stride(0) if q_out is not None else 0,
+                              cache.data_ptr(), cache.shape[0], _stream()))
+    count()
+
+
+def rotate_pairs(x, rotation, places, out):
+    """x [heads, T, width] -> out, the first columns of each head turned (fb_rotate_pairs)."""
+    freq, dims, mag = rotation
+    check(lib().fb_rotate_pairs(_CODES[x.dtype], x.data_ptr(), x.shape[1], x.shape[0], x.stride(1), x.stride(0), x.shape[2], dims, freq.data_ptr(), mag,
+                                places.data_ptr(), out.data_ptr(), out.stride(1), out.stride(0), _stream()))
+    count()
+    return out
+
+
+def latent_attention(q, cache, base, last, heads, rank, scale, sink, max_keys, chunk, row0=0, out=None):
+    """q [T, heads * (rank + rot)] over cache [rows, rank + rot] (fb_latent_attention)."""
+    T, rot = q.shape[0], cache.shape[1] - rank
+    if out is None:
+        out = torch.empty(T, heads * rank, dtype=q.dtype, device=q.device)
+    assert cache.is_contiguous() and last.numel() == T and (base is None or base.numel() == T) and last.dtype == torch.int32
+    code = _CODES[q.dtype]
+    need = lib().fb_latent_attention_workspace_bytes(code, T, heads, rank, rot, max_keys, int(chunk))
+    ws = attention_workspace(q.device, need)
+    check(lib().fb_latent_attention(code, q.data_ptr(), T, q.stride(0), heads, rank, rot, cache.data_ptr(), cache.shape[0], _ptr(base), row0, last.data_ptr(), max_keys,
+                                    int(chunk), scale, _ptr(sink), out.data_ptr(), out.stride(0), _ptr(ws) if need else None, ws.numel() if need else 0, _stream()))
+    count(2 if need else 1)
+    return out
+
+
+def decay_scan(qkv, heads, dim, vdim, decay, places, dead, state, out):
+    """Linear attention with decay over state [sequences, heads * dim, vdim] (fb_decay_scan)."""
+    sequences = state.shape[0]
+    assert state.stride(2) == 1 and state.stride(1) == vdim and places.dtype == torch.int32 and places.numel() == qkv.shape[0]
+    check(lib().fb_decay_scan(_CODES[qkv.dtype], qkv.data_ptr(), qkv.stride(0), heads, dim, vdim, decay.data_ptr(), places.data_ptr(), dead, sequences,
+                              qkv.shape[0] // sequences, state.data_ptr(), state.stride(0), out.data_ptr(), out.stride(0), _stream()))
+    count()
+    return out
+
+
+def gated_rmsnorm(x, gate, w, eps, out):
+    check(lib().fb_gated_rmsnorm(x.data_ptr(), x.shape[0], x.shape[1], x.stride(0), _CODES[gate.dtype], gate.data_ptr(), gate.stride(0), w.data_ptr(), eps,
+                                 out.data_ptr(), out.stride(0), _stream()))
+    count()
     return out

@@ -90,7 +90,9 @@ class Engine:
     """Several requests decoding together in the slots of one KV cache (models/serve.py:247-330).  The device work sits
     behind `backend`: prefill(u, ids, first, t) runs a chunk of slot u's prompt at places first.. and gives the head of
     its last token's logits; decode(ids, places, ts) runs one token of every slot and gives every slot's head.  A free
-    slot's token is 0 at its part's last place, which marks it not live (models/llama.py:448-449).
+    slot's token is 0 at its part's last place, which marks it not live (models/llama.py:448-449).  A backend whose model
+    keeps a recurrent state says `rewinds = False`: what a slot holds then serves a new prompt only if all of it is the
+    prompt's beginning.
 
         admit(r)   into the free slot that already holds the most of r's prompt (a slot keeps its last request's keys:
                    a shared system prompt is prefilled once), ties to the one used longest ago;
@@ -106,11 +108,16 @@ class Engine:
     def admit(self, r):
         free = [u for u, b in enumerate(self.busy) if b is None]
         assert free and len(r.ids) < self.places, "a free slot, and a prompt shorter than a slot's places"
-        u = max(free, key=lambda u: (reach(self.held[u], r.ids), -self.used[u]))
+        u = max(free, key=lambda u: (self.kept(u, r.ids), -self.used[u]))
         self.used[u], self.busy[u] = max(self.used) + 1, r
-        n = reach(self.held[u], r.ids)
+        n = self.kept(u, r.ids)
         self.held[u], r.cached = r.ids[:n], n
         return u
+
+    def kept(self, u, ids):
+        """How much of the prompt ids free slot u already holds and can go on from."""
+        n = reach(self.held[u], ids)
+        return n if n == len(self.held[u]) or getattr(self.backend, "rewinds", True) else 0
 
     def fill(self, u):
         r, at = self.busy[u], len(self.held[u])
@@ -153,22 +160,21 @@ class Engine:
 
 
 class DeviceBackend:
-    """The engine's device side: the slots' shared KV cache, a prompt's chunk through forward over the slot's own rows
-    (the prefill-shaped attention), and one recorded step for a token of every slot, each followed by `heads` so that
-    only 64 values, 64 tokens and a log-sum-exp per row are read back."""
+    """The engine's device side for any family (models.py): the slots' shared caches, a prompt's chunk through forward over
+    the slot's own part (the prefill-shaped attention), and one recorded step for a token of every slot, each followed by
+    `heads` so that only 64 values, 64 tokens and a log-sum-exp per row are read back.  prompt and token give the logits
+    themselves."""
 
     def __init__(self, rt, weights, c, slots, places):
-        from . import llama
+        from . import llama, models
         from .tensor import jit
-        self.rt, self.w, self.c, self.slots, self.llama = rt, weights, c, slots, llama
-        self.part = places
-        self.kv = llama.kv_cache(c, slots * places, llama.zeros(rt))
-        self.parts = [llama.slot(c, self.kv, u, slots) for u in range(slots)]
-
-        def step(ids, at, t):
-            logits = llama.forward(ids, at, weights, c, self.kv, slots).realize()
-            return self._pack(heads(logits[0], t))
-        self.step = jit(step)
+        self.rt, self.w, self.c, self.slots, self.model = rt, weights, c, slots, models.of(c)
+        self.part, self.rewinds = places, getattr(self.model, "REWINDS", True)
+        self.kv = self.model.kv_cache(c, slots * places, llama.zeros(rt), slots)
+        self.parts = [self.model.slot(c, self.kv, u, slots) for u in range(slots)]
+        forward = lambda ids, at: self.model.forward(ids, at, weights, c, self.kv, slots).realize()
+        self.logits_step = jit(forward)
+        self.step = jit(lambda ids, at, t: self._pack(heads(forward(ids, at)[0], t)))
 
     def _pack(self, h):
         """values | ids | lse side by side in one fp32 matrix (token ids below 2^24 are exact in fp32): one readback."""
@@ -182,9 +188,69 @@ class DeviceBackend:
     def on(self, row, dtype="int32"):
         return Tensor.of(self.rt, [row], dtype)
 
+    def prompt(self, u, ids, first, every=False):
+        """The logits after a chunk of slot u's prompt at places first.. (every: a list of the chunk's tokens: after those)."""
+        every = self.on(every) if isinstance(every, list) else every
+        return self.model.forward(self.on(ids), self.on(list(range(first, first + len(ids)))), self.w, self.c, self.parts[u], every=every).realize()
+
+    def token(self, ids, places):
+        """The logits after one token of every slot (a free slot's: 0 at the last place)."""
+        return self.logits_step(self.on(ids), self.on(places))
+
     def prefill(self, u, ids, first, t):
-        out = self.llama.forward(self.on(ids), self.on(list(range(first, first + len(ids)))), self.w, self.c, self.parts[u])
+        out = self.prompt(u, ids, first)
         return self._unpack(self._pack(heads(out, Tensor.of(self.rt, [[t]], "fp32"))))[0]
 
     def decode(self, ids, places, ts):
         return self._unpack(self.step(self.on(ids), self.on(places), Tensor.of(self.rt, [[t] for t in ts], "fp32")))
+
+
+class Replay:
+    """Given tokens through the engine's device side, step by step, for their logits: nothing is sampled.  A request's first
+    tokens take a free slot; a step in which every request brings one more token is a decode step of all slots together
+    (the recorded one), any other runs each request's tokens as a chunk of its prompt."""
+
+    def __init__(self, rt, weights, c, places, chunk=2048):
+        self.make = lambda slots: DeviceBackend(rt, weights, c, slots, places + 2)
+        self.chunk, self.backend, self.slot, self.held = chunk, None, {}, {}
+
+    def admit(self, names):
+        """Slots for new requests; more are made when too few are free, which takes that no request is under way."""
+        slots = self.backend.slots if self.backend else 0
+        free = [u for u in range(slots) if u not in self.slot.values()]
+        if len(names) > len(free):
+            assert not self.slot, "every slot is taken"
+            self.backend = None  # (its caches go before the larger ones are made)
+            self.backend = self.make(len(names))
+            free = list(range(len(names)))
+        for name, u in zip(names, free):
+            self.slot[name], self.held[name] = u, 0
+
+    def step(self, entries):
+        """entries: (name, tokens, wanted places among them).  The wanted logits, numpy [wanted, vocabulary], in their order."""
+        self.admit([name for name, _, _ in entries if name not in self.slot])
+        b, out = self.backend, []
+        if all(len(tokens) == 1 and self.held[name] for name, tokens, _ in entries):
+            ids, places = [0] * b.slots, [b.part - 1] * b.slots
+            for name, tokens, _ in entries:
+                ids[self.slot[name]], places[self.slot[name]] = tokens[0], self.held[name]
+                self.held[name] += 1
+            logits = b.token(ids, places)
+            if any(want for _, _, want in entries):
+                a = logits.numpy()[0]
+                out = [a[self.slot[name]] for name, _, want in entries for _ in want]
+        else:
+            for name, tokens, want in entries:
+                for at in range(0, len(tokens), self.chunk):
+                    ids = tokens[at:at + self.chunk]
+                    here = [i - at for i in want if at <= i < at + len(ids)]
+                    logits = b.prompt(self.slot[name], ids, self.held[name], here or False)
+                    self.held[name] += len(ids)
+                    if here:
+                        out.extend(logits.numpy()[0])
+        return np.stack(out) if out else None
+
+    def end(self, name):
+        """The request is finished: its slot is free."""
+        if name in self.slot:
+            del self.slot[name], self.held[name]

@@ -36,7 +36,7 @@ FIDELITY = 4  # accepted and ignored, as the numpy reference ignores it (models/
 # elementwise opcodes of fb_elementwise (include/ferrite_b200.h)
 _BINARY = {"add": 10, "sub": 11, "mul": 12, "max": 13, "cmplt": 14, "cmpne": 15, "keep": 16, "drop": 17, "div": 18, "min": 19}
 _UNARY = {"exp": 30, "log": 31, "sin": 32, "cos": 33, "sqrt": 34, "recip": 35, "relu": 36, "exp2": 37, "log2": 38, "round_bf16": 39,
-          "trunc": 40, "neg": 41}
+          "trunc": 40, "neg": 41, "tanh": 42}
 _ELEMENTWISE = set(_BINARY) | set(_UNARY) | {"cast"}
 _MAX_OPS, _MAX_INPUTS, _MAX_STACK = 48, 8, 12
 
@@ -199,6 +199,7 @@ class Tensor:
     def reciprocal(self): return self._unary("recip")
     def exp(self): return self._unary("exp")
     def log(self): return self._unary("log")
+    def tanh(self): return self._unary("tanh")
     def relu(self): return self._unary("relu")
     def rsqrt(self): return self.sqrt().reciprocal()
     def maximum(self, x): return self._binop("max", x)
@@ -494,6 +495,10 @@ class Tensor:
         self.rt.launched("touched", 1)
         return experts, out
 
+    def silu_columns(self, n):
+        """self with its first n columns through SiLU (a joint projection of activated and plain parts); fuses into a matmul."""
+        return self._lazy("silu_columns", (self,), self.shape, self.dtype, n=n)
+
     # ---------------------------------------------------------------- a decode step's two fused kernels
 
     def rope_put(self, cos, sin, places, rows, cache, heads, kv, qk_norm=None, eps=1e-5):
@@ -537,6 +542,68 @@ class Tensor:
                              max_keys=min(length or cache.rows, cache.rows),
                              window=window or 0, out=out.buf[0])
         self.rt.launched("attention")
+        return out
+
+    # ---------------------------------------------------------------- latent attention and decaying linear attention
+
+    def latent_put(self, rotation, places, rows, cache, q_rank, q_norm, kv_norm, eps):
+        """self: a joint down-projection [1, tokens, query latent | key-value latent | shared key part | ...].  One kernel norms
+        both latents, turns the key part and puts (key-value latent | key part) into `cache` ([1, size, kv_rank + rot]) at
+        `rows`; returns the normed query latent, as the cache is stored.  rotation: (frequencies on the device, their
+        number of columns, factor) of mixers.rotation; places, rows: int32 rows read on the device."""
+        x, places, rows = self.realize(), places.realize(), rows.realize()
+        kv_rank = kv_norm.cols
+        rot = cache.cols - kv_rank
+        assert x.batch == 1 and x.buf.stride(2) == 1 and x.cols >= q_rank + cache.cols and cache.buf.is_contiguous(), f"{self.shape} into a cache {cache.shape}"
+        assert q_norm is None or (q_norm.cols == q_rank and q_norm.dtype == "fp32") and kv_norm.dtype == "fp32" and places.cols == rows.cols == x.rows
+        freq, dims, mag = rotation
+        out = Tensor(self.rt, x.rows, q_rank, dtype=cache.dtype) if q_rank else None
+        ops.latent_put(x.buf[0], q_rank, kv_rank, rot, dims, None if q_norm is None else q_norm.buf, kv_norm.buf, eps, freq, mag, places.buf.reshape(-1),
+                       rows.buf.reshape(-1), cache.buf[0], None if out is None else out.buf[0])
+        self.rt.launched("latent put")
+        return out
+
+    def rotate_pairs(self, rotation, places, into=None):
+        """self: [heads, tokens, width], each head's first columns turned pair by pair by its token's angle (the rest as they
+        are), into `into` (a view of the same shape) or a tensor of its own."""
+        x, places = self.realize(), places.realize()
+        into = into if into is not None else Tensor(self.rt, x.rows, x.cols, batch=x.batch, dtype=x.dtype)
+        assert into.shape == x.shape and into.dtype == x.dtype and x.buf.stride(2) == into.buf.stride(2) == 1 and places.cols == x.rows
+        ops.rotate_pairs(x.buf, rotation, places.buf.reshape(-1), into.buf)
+        self.rt.launched("rotate pairs")
+        return into
+
+    def attend_latent(self, cache, base, last, rank, scale, sink=None, length=None, chunk=False):
+        """self: [1, tokens, heads (rank + rot)], each head's query in the latents' space and its turned part.  Token t attends
+        the cache rows base[t] .. base[t] + last[t]: one row is key (all of it) and value (its first `rank` columns) of every
+        head.  sink: a number per head that joins the softmax's denominator.  chunk: the tokens are one sequence's, its first
+        cache row 0.  Returns [1, tokens, heads rank]: weighted sums of latents."""
+        q, last = self.realize(), last.realize()
+        heads = q.cols // cache.cols
+        assert q.batch == cache.batch == 1 and q.cols % cache.cols == 0 and q.dtype == cache.dtype and q.buf.stride(2) == 1, f"{q.shape} over a cache {cache.shape}"
+        out = Tensor(self.rt, q.rows, heads * rank, dtype=q.dtype)
+        ops.latent_attention(q.buf[0], cache.buf[0], None if chunk else base.realize().buf.reshape(-1), last.buf.reshape(-1), heads, rank, scale,
+                             None if sink is None else sink.buf, min(length or cache.rows, cache.rows), chunk, out=out.buf[0])
+        self.rt.launched("latent attention")
+        return out
+
+    def decay_scan(self, heads, dim, vdim, decay, places, state, dead=-1):
+        """self: rows of q | k | v (| more) of one sequence, or one row of each of state.batch sequences; state: fp32 [sequences,
+        heads dim, vdim], read and written.  S = decay S + k v^T, o = S^T q per head; a sequence at place 0 starts from
+        zeros, one at place `dead` is left alone.  Returns fp32 [1, tokens, heads vdim]."""
+        x, places = self.realize(), places.realize()
+        assert x.batch == 1 and x.buf.stride(2) == 1 and state.dtype == "fp32" and state.shape[1:] == (heads * dim, vdim) and x.rows % state.batch == 0
+        out = Tensor(self.rt, x.rows, heads * vdim, dtype="fp32")
+        ops.decay_scan(x.buf[0], heads, dim, vdim, decay.buf, places.buf.reshape(-1), dead, state.buf, out.buf[0])
+        self.rt.launched("decay scan")
+        return out
+
+    def gated_rms(self, gate, w, eps):
+        """RMSNorm of self (fp32 rows) by w, times the sigmoid of gate, as gate is stored."""
+        x, gate = self.realize(), gate.realize()
+        out = Tensor(self.rt, x.rows, x.cols, dtype=gate.dtype)
+        ops.gated_rmsnorm(x.buf[0], gate.buf[0], w.buf, eps, out.buf[0])
+        self.rt.launched("gated rmsnorm")
         return out
 
     def greedy(self, values=None):
@@ -586,6 +653,9 @@ def _realize(t, into=None):
             return
         if _run_rmsnorm(t, into):
             return
+        found = _match_dyt(t)
+        if found:  # (what it stands on is read by others too - the residual stream: computed once, not inside this expression)
+            found[0].realize()
         _run_elementwise(t, into)
     elif op == "reduce_sum" and t.args["axis"] == 0 and _match_experts(t.srcs[0]):
         _run_experts(t, _match_experts(t.srcs[0]), None, into)
@@ -606,6 +676,12 @@ def _realize(t, into=None):
         t.owner = mm
         if into is not None:
             _copy(t, into)
+    elif op == "silu_columns":
+        src = t.srcs[0].realize()
+        out = (src + 0).realize()
+        part = out[:, :, :t.args["n"]]
+        part.assign(part.silu())
+        _done(t, buf=out.buf)
     elif op == "repeat":
         src, n = t.srcs[0].realize(), t.args["n"]
         out = Tensor(t.rt, t.rows, t.cols, batch=t.batch, dtype=t.dtype)
@@ -667,6 +743,20 @@ def _run_rmsnorm(t, into):
     t.rt.launched("rmsnorm")
     _done(t, buf=out.buf)
     return True
+
+
+def _match_dyt(t):
+    """(x, alpha, w, b) if t is tanh(alpha x) w + b as mixers.dyt writes it, or a cast of it, else None."""
+    if isinstance(t, Tensor) and t.op == "cast":
+        t = t.srcs[0]
+    if not (isinstance(t, Tensor) and t.op == "add" and isinstance(t.srcs[0], Tensor) and t.srcs[0].op == "mul"):
+        return None
+    (th, w), b = t.srcs[0].srcs, t.srcs[1]
+    vector = lambda v: isinstance(v, Tensor) and v.op is None and v.dtype == "fp32" and v.shape == (1, 1, t.cols)
+    if not (isinstance(th, Tensor) and th.op == "tanh" and th.srcs[0].op == "mul" and vector(w) and vector(b)):
+        return None
+    x, alpha = th.srcs[0].srcs
+    return (x, alpha, w, b) if isinstance(alpha, Tensor) and alpha.op is None and alpha.dtype == "fp32" and alpha.shape == (1, 1, 1) else None
 
 
 def _match_silu_of(g):
@@ -892,8 +982,22 @@ def _program(t, inputs, code, consts, depth=1):
     return most
 
 
+def _realize_leaves(t, seen):
+    """Compute what the elementwise tree under t reads before the tree is looked at: a leaf's own inputs may be part of the
+    tree as well (a residual stream under the branch that is added to it), and are then realized instead of inlined."""
+    if not isinstance(t, Tensor) or t.op is None or id(t) in seen:
+        return
+    seen.add(id(t))
+    if t.op not in _ELEMENTWISE:
+        t.realize()
+        return
+    for src in reversed(t.srcs):
+        _realize_leaves(src, seen)
+
+
 def _run_elementwise(t, into=None):
     inputs, code, consts = [], [], []
+    _realize_leaves(t, set())
     _program(t, inputs, code, consts)
     assert len(code) <= _MAX_OPS and len(inputs) <= _MAX_INPUTS, "an expression too large for one kernel even after splitting"
     out = into if into is not None else Tensor(t.rt, t.rows, t.cols, batch=t.batch, dtype=t.dtype)

@@ -282,7 +282,7 @@ int fb_group(const int32_t* ids, int64_t rows, int k, int n, int32_t* order, int
 /* One fused elementwise expression (ferrite fuses a tree into one kernel, ferrite/compiler.py:699-738).  The
  * expression is a postfix program of n_ops (op, arg) pairs: op 0 pushes input `arg`, op 1 pushes consts_host[position];
  * 10.. are binary (add sub mul max cmplt cmpne keep drop div min), 30.. unary (exp log sin cos sqrt recip relu exp2
- * log2 round-to-bf16 trunc neg).  Computed in fp32, rounded once at the store. */
+ * log2 round-to-bf16 trunc neg tanh).  Computed in fp32, rounded once at the store. */
 int fb_elementwise(int n_ops, const int32_t* program_host, const float* consts_host, int n_inputs, const void* const* inputs_host,
                    const int64_t* strides_host, const int32_t* dtypes_host, void* out, const int64_t* out_strides_host,
                    int out_dtype, int64_t batch, int64_t rows, int64_t cols, void* stream);
@@ -295,6 +295,45 @@ int fb_reduce(int is_max, const void* in, const int64_t* in_strides_host, int in
  * repeats a matrix): Tensor.matmul without a block-float B (ferrite/tensor.py:443-485); fp32 accumulation. */
 int fb_matmul(const void* a, const int64_t* a_strides_host, int a_dtype, const void* b, const int64_t* b_strides_host, int b_dtype,
               void* c, const int64_t* c_strides_host, int c_dtype, int64_t batch, int64_t M, int64_t N, int64_t K, void* stream);
+
+/* ---- attention over a cache of latents, rotation of neighbouring pairs, linear attention with decay ------- */
+
+/* After a joint down-projection (row t of `down`: q_rank columns of the query latent, kv_rank of the key-value latent, rot
+ * of the key part that all heads share): q_out[t] = RMSNorm(query latent) * q_norm (q_rank 0: a design without one), and
+ * cache row rows[t] = RMSNorm(key-value latent) * kv_norm | the key part, its first `dims` columns turned pair by pair (2i,
+ * 2i + 1) by places[t] * freq[i] with cos and sin times `mag`.  Norms and angles in fp32 or better; in_dtype: how `down`
+ * is stored, dtype: q_out and the cache.  A row outside the cache is not written. */
+int fb_latent_put(int in_dtype, const void* down, int64_t T, int64_t ld, int q_rank, int kv_rank, int rot, int dims, const float* q_norm,
+                  const float* kv_norm, float eps, const double* freq, float mag, const int32_t* places, const int32_t* rows, int dtype,
+                  void* q_out, int64_t ld_q, void* cache, int64_t cache_rows, void* stream);
+
+/* The same turn for each head of x (head h of token t at x + t * x_row + h * x_head, `width` columns, the first `dims` of
+ * them turned, the rest copied) into out (strides alike). */
+int fb_rotate_pairs(int dtype, const void* x, int64_t T, int heads, int64_t x_row, int64_t x_head, int width, int dims, const double* freq,
+                    float mag, const int32_t* places, void* out, int64_t o_row, int64_t o_head, void* stream);
+
+/* Attention whose keys and values are one row of cache [cache_rows, rank + rot] a token, shared by all heads: head h of token t
+ * has its query at q + t * ld_q + h * (rank + rot), scores are scale * (query . row), the output (out + t * ld_o + h * rank) is
+ * the softmax-weighted sum of the rows' first `rank` columns.  Token t sees the rows base[t] + row0 + 0 .. last[t] (base null:
+ * row0 alone).  sink (fp32 [heads], or null): exp(sink[h]) joins head h's denominator once, unscaled and without a value.
+ * chunk: the tokens are consecutive ones of one sequence (they may share the rows they read).  max_keys: an upper bound of
+ * last[t] + 1.  workspace: fb_latent_attention_workspace_bytes bytes. */
+size_t fb_latent_attention_workspace_bytes(int dtype, int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk);
+int fb_latent_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int rank, int rot, const void* cache, int64_t cache_rows,
+                        const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk, float scale, const float* sink,
+                        void* out, int64_t ld_o, void* workspace, size_t workspace_bytes, void* stream);
+
+/* Linear attention with a decay per head, token after token: S = decay[h] * S + k v^T, out = S^T q, over `sequences`
+ * sequences of `tokens` tokens each, one sequence's rows after the other's.  qkv row: q (heads x dim) | k (heads x dim) |
+ * v (heads x vdim).  state: fp32 [heads, dim, vdim] per sequence, state_stride elements apart, read and left for the next
+ * call.  A sequence whose first token stands at place 0 starts from zeros; one whose first token stands at place `dead`
+ * (-1: none) has no token: its state is left alone and its output is 0. */
+int fb_decay_scan(int dtype, const void* qkv, int64_t ld, int heads, int dim, int vdim, const float* decay, const int32_t* places, int dead,
+                  int64_t sequences, int64_t tokens, float* state, int64_t state_stride, float* out, int64_t ld_o, void* stream);
+
+/* out = RMSNorm(x) * w * sigmoid(gate), row by row; x, w fp32, gate and out of `dtype` */
+int fb_gated_rmsnorm(const float* x, int64_t rows, int64_t cols, int64_t ldx, int dtype, const void* gate, int64_t ld_g, const float* w, float eps,
+                     void* out, int64_t ldo, void* stream);
 
 /* ---- several GPUs -------------------------------------------------------------------------------------- */
 
