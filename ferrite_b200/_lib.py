@@ -16,6 +16,15 @@ LINEAR_AUTO, LINEAR_TCGEN05, LINEAR_GEMV, LINEAR_MMA, LINEAR_PERSISTENT, LINEAR_
 
 _p, _i, _i64, _f, _sz = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_float, ctypes.c_size_t
 
+DENSE_NONE, DENSE_SILU, DENSE_GLU, DENSE_GATE, DENSE_DYT_ADD = 0, 1, 2, 3, 4  # fb_dense_epilogue_kind
+
+
+class DenseEpilogue(ctypes.Structure):
+    """fb_dense_epilogue of include/ferrite_b200.h, field by field."""
+    _fields_ = [("kind", _i), ("act_cols", _i64), ("limit", _f), ("slope", _f), ("gate", _p), ("ld_gate", _i64), ("residual", _p), ("ld_residual", _i64),
+                ("alpha", _p), ("w", _p), ("b", _p), ("h_out", _p), ("ld_h", _i64), ("alpha2", _p), ("w2", _p), ("b2", _p)]
+
+
 # name -> (restype, argtypes); one entry per declaration in include/ferrite_b200.h
 SIGNATURES = {
     "fb_version": (_i, []),
@@ -52,6 +61,8 @@ SIGNATURES = {
     "fb_argmax": (_i, [_p, _i64, _i64, _i64, _p, _p, _p]),
     "fb_rope_kv_write_packed": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _p, _p, _i64, _i64, _p, _p, _p, _f, _p, _i64, _p, _i64, _p]),
     "fb_decode_attention_packed": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _p, _i64, _p, _p, _i64, _i, _p, _i64, _p, _sz, _p]),
+    "fb_dense_supports": (_i, [_p, _i64, _i64, _p, _i64, _i64, _i64, _i64, _i]),
+    "fb_dense": (_i, [_p, _i64, _i64, _i64, _i64, _p, _i64, _i64, _i64, _i64, _p, _i, _i64, _i64, _p, _i, _p]),
     "fb_latent_put": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _i, _p, _p, _f, _p, _f, _p, _p, _i, _p, _i64, _p, _i64, _p]),
     "fb_rotate_pairs": (_i, [_i, _p, _i64, _i, _i64, _i64, _i, _i, _p, _f, _p, _p, _i64, _i64, _p]),
     "fb_latent_attention_workspace_bytes": (_sz, [_i, _i64, _i, _i, _i, _i64, _i]),

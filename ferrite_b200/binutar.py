@@ -189,5 +189,6 @@ def random_weights(rt, c, prec=None, seed=0, scale=0.02):
     matrix("head", c.vocab, c.dim)
     embed = torch.empty(c.vocab, c.dim, dtype=torch.float32, device=rt.device).normal_(0, 1, generator=gen)
     w["embed"] = Tensor(rt, c.vocab, c.dim, dtype=c.dtype, buf=embed.to(torch.float32 if c.dtype == "fp32" else torch.bfloat16).view(1, c.vocab, c.dim))
+    llama.settle(rt, w)
     w["_blocks"] = [llama.block(w, f"l{l}.") for l in range(c.layers)]
     return w

@@ -18,6 +18,8 @@ int launch_status(const char* what);  // cudaGetLastError() -> FB_OK / FB_ERR_LA
 int status_word_tcgen05();
 int status_word_peer();
 int status_word_gemv_stream();
+int status_word_dense();
+int status_word_latent();
 
 #define FB_REQUIRE(cond, ...)            \
   do {                                   \

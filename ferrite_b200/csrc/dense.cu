@@ -1,0 +1,345 @@
+// fb_dense: activations by bf16 weights on the 5th-generation tensor cores, both operands by TMA.
+//
+// The weights are the MMA's A operand (a tile of 128 output columns = the 128 accumulator lanes in tensor memory), the
+// tokens its N dimension (16 .. 256), so one kernel serves a decode step of a few tokens - bound by the stream of weights -
+// and a prompt's hundreds, bound by the MMAs.  Both operands arrive K-major in 128-byte swizzled rows: no unpacking, no
+// transposition, and the CTA's threads touch nothing but the accumulators.
+//
+//   warp 8      asks for the tiles: [128 x 64] of weights and [tokens x 64] of activations a step, a ring of 4 to 10 steps
+//   warp 9      issues the MMAs (4 x K = 16 a step), one accumulator of two in tensor memory a tile
+//   warps 0-7   the epilogue: a warp has a quarter of the lanes and half of the tokens; it empties one accumulator while the
+//               MMAs fill the other
+//
+// CTAs are persistent: tiles are dealt out round robin, the ring and the accumulators run on across tile borders.  Where
+// the tiles are too few to fill the GPU, K is split over the CTAs of a cluster (2, 4 or 8): each leaves its sums in shared
+// memory, each then takes a share of the tokens and adds the others' sums to its own in rank order (the same every run).
+//
+// What follows a matmul in its model runs on the accumulators (fb_dense_epilogue): SiLU on the first columns, a clamped
+// gated unit (gate and up rows alternate in runs of 16 inside a tile, so a pair is 16 lanes apart), a gate per head, and the
+// Dynamic Tanh - residual add - Dynamic Tanh between two branches, which needs no sum over the row and therefore no
+// kernel of its own.  Every wait is bounded (sm100.cuh).
+#include "sm100.cuh"
+#include "tma_host.cuh"
+#include "values.cuh"
+
+namespace fb {
+
+namespace {
+
+constexpr int D_EPI_WARPS = 8, D_WARP_LOAD = 8, D_WARP_MMA = 9, D_THREADS = 10 * 32;
+constexpr int D_A_BYTES = 128 * 128;  // 128 weight rows of 64 values
+constexpr int D_MAX_STAGES = 10;
+constexpr size_t D_SMEM = 200 * 1024;
+
+enum DenseWait { DW_EMPTY = 301, DW_FULL, DW_ACC_FULL, DW_ACC_EMPTY, DW_DRAIN };
+
+struct DenseParams {
+  int64_t M, N;  // N: output columns of W (gate and up together)
+  int nt, stages, tmem_cols, steps, splits, steps_per_split;
+  int tiles_m, tiles_n, tiles;  // tiles: all batch entries'
+  void* out;
+  int out_dtype;
+  int64_t ldo, out_batch;
+  int settled;
+  fb_dense_epilogue e;
+};
+
+struct DenseTile {
+  int m, n, b;
+};
+__device__ __forceinline__ DenseTile tile_of(const DenseParams& p, int id) {  // tokens fastest: tiles that share weights run together
+  const int rest = id / p.tiles_m;
+  return {id % p.tiles_m, rest % p.tiles_n, rest / p.tiles_n};
+}
+
+// one value of the result: column n of token t (GLU: v the gate, up its partner); the caller has checked the bounds
+template <int EPI>
+__device__ __forceinline__ void emit(const DenseParams& p, int b, int64_t t, int64_t n, float v, float up, float res, float gate) {
+  if constexpr (EPI == FB_DENSE_DYT_ADD) {
+    const float x = res + (tanhf(*p.e.alpha * v) * p.e.w[n] + p.e.b[n]);
+    static_cast<float*>(p.out)[t * p.ldo + n] = x;
+    if (p.e.h_out) static_cast<uint16_t*>(p.e.h_out)[t * p.e.ld_h + n] = (uint16_t)float_to_bf16_bits(tanhf(*p.e.alpha2 * x) * p.e.w2[n] + p.e.b2[n]);
+    return;
+  }
+  if constexpr (EPI == FB_DENSE_SILU) {
+    if (n < p.e.act_cols) v = v / (1.f + __expf(-v));
+  }
+  if constexpr (EPI == FB_DENSE_GLU) {
+    const float g = fminf(v, p.e.limit), u = fminf(fmaxf(up, -p.e.limit), p.e.limit);
+    v = g / (1.f + __expf(-p.e.slope * g)) * (u + 1.f);
+  }
+  if constexpr (EPI == FB_DENSE_GATE) v *= gate;
+  const int64_t at = b * p.out_batch + t * p.ldo + n;
+  if (p.out_dtype == FB_FP32) static_cast<float*>(p.out)[at] = v;
+  else static_cast<uint16_t*>(p.out)[at] = (uint16_t)float_to_bf16_bits(v);
+}
+
+template <int EPI>
+__global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx, const DenseParams p) {
+  extern __shared__ uint8_t dense_smem[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dense_smem) + 1023) & ~uintptr_t(1023));
+  __shared__ uint64_t bars[2 * D_MAX_STAGES + 4];
+  __shared__ uint32_t tmem_slot[2];  // the allocation's address, the abort flag
+  uint64_t *full = bars, *empty = bars + D_MAX_STAGES, *acc_full = bars + 2 * D_MAX_STAGES, *acc_empty = acc_full + 2;
+  const uint32_t abort_flag = smem_u32(tmem_slot + 1);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int S = p.stages, nt = p.nt, stage_bytes = D_A_BYTES + nt * 128;
+  const int s0 = blockIdx.y * p.steps_per_split, n_steps = min(p.steps - s0, p.steps_per_split);
+
+  griddep_launch_dependents();
+  if (tid == 0) {
+    for (int s = 0; s < S; ++s) mbar_init(smem_u32(full + s), 1), mbar_init(smem_u32(empty + s), 1);
+    for (int s = 0; s < 2; ++s) mbar_init(smem_u32(acc_full + s), 1), mbar_init(smem_u32(acc_empty + s), D_EPI_WARPS);
+    tmem_slot[1] = 0;
+    fence_barrier_init();
+  }
+  if (warp == D_WARP_MMA) tmem_alloc(smem_u32(tmem_slot), p.tmem_cols);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_slot[0];
+
+  if (warp == D_WARP_LOAD && lane == 0) {
+    prefetch_tensormap(&tw), prefetch_tensormap(&tx);
+    auto weights = [&](const DenseTile& t, int k, int slot) {
+      const uint32_t bar = smem_u32(full + slot), dst = smem_u32(smem + slot * stage_bytes);
+      mbar_expect_tx(bar, (uint32_t)stage_bytes);
+      if (EPI == FB_DENSE_GLU) tma_load_4d(dst, &tw, 64 * k, 0, 0, 4 * t.n, bar);
+      else tma_load_3d(dst, &tw, 64 * k, 128 * t.n, t.b, bar);
+    };
+    int early = 0;
+    if (p.settled && (int)blockIdx.x < p.tiles) {
+      const DenseTile t = tile_of(p, blockIdx.x);
+      for (early = 0; early < min(S, n_steps); ++early) weights(t, s0 + early, early);
+    }
+    griddep_wait();  // the activations come from the kernel before
+    int i = 0, slot = 0;
+    uint32_t phase = 0;
+    bool ok = true;
+    for (int id = blockIdx.x; id < p.tiles && ok; id += gridDim.x) {
+      const DenseTile t = tile_of(p, id);
+      for (int k = 0; k < n_steps && ok; ++k, ++i) {
+        if (i >= early) {
+          ok = mbar_wait(smem_u32(empty + slot), phase ^ 1, abort_flag, DW_EMPTY);
+          if (!ok) break;
+          weights(t, s0 + k, slot);
+        }
+        tma_load_3d(smem_u32(smem + slot * stage_bytes + D_A_BYTES), &tx, 64 * (s0 + k), nt * t.m, t.b, smem_u32(full + slot));
+        if (++slot == S) slot = 0, phase ^= 1;
+      }
+    }
+    if (!ok)  // given up: the copies under way land before this CTA's shared memory is anyone else's
+      for (int s = 0; s < S; ++s) {
+        const long long start = clock64();
+        const uint32_t parity = s < slot ? phase : phase ^ 1;
+        while (i > s && !mbar_try_wait(smem_u32(full + s), parity) && clock64() - start < WAIT_CLOCKS) {
+        }
+      }
+  } else if (warp == D_WARP_MMA && lane == 0) {
+    const uint32_t idesc = umma_idesc_bf16(nt, false, false);
+    const uint64_t d0 = umma_smem_desc(smem_u32(smem), 16, 1024);
+    int slot = 0, n = 0;
+    uint32_t phase = 0;
+    for (int id = blockIdx.x; id < p.tiles; id += gridDim.x, ++n) {
+      const uint32_t acc = tmem + (n & 1) * nt;
+      mbar_wait(smem_u32(acc_empty + (n & 1)), ((n >> 1) & 1) ^ 1, abort_flag, DW_ACC_EMPTY);
+      tc_fence_after();
+      for (int k = 0; k < n_steps; ++k) {
+        mbar_wait(smem_u32(full + slot), phase, abort_flag, DW_FULL);
+        tc_fence_after();
+        const uint64_t da = d0 + (uint32_t)(slot * stage_bytes >> 4), dx = da + (D_A_BYTES >> 4);
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) umma_bf16(acc, da + 2 * kk, dx + 2 * kk, idesc, k | kk);
+        umma_commit(smem_u32(empty + slot));
+        if (++slot == S) slot = 0, phase ^= 1;
+      }
+      umma_commit(smem_u32(acc_full + (n & 1)));
+    }
+  } else if (warp < D_EPI_WARPS) {
+    griddep_wait();
+    const int q = warp & 3, half = nt / 2, col0 = (warp >> 2) * half, row = 32 * q + lane;
+    int n = 0;
+    for (int id = blockIdx.x; id < p.tiles; id += gridDim.x, ++n) {
+      const DenseTile t = tile_of(p, id);
+      mbar_wait(smem_u32(acc_full + (n & 1)), (n >> 1) & 1, abort_flag, DW_ACC_FULL);
+      tc_fence_after();
+      const uint32_t acc = tmem + ((uint32_t)(32 * q) << 16) + (n & 1) * nt + col0;
+      const int64_t t0 = (int64_t)nt * t.m + col0;
+      if (p.splits > 1) {  // this CTA's part of the sums, token by token, for the cluster to read
+        float* ex = reinterpret_cast<float*>(smem);
+        for (int c = 0; c < half; c += 8) {
+          float v[8];
+          tmem_ld8(acc + c, v);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) ex[(col0 + c + e) * 128 + row] = v[e];
+        }
+      } else {
+        const int64_t col = EPI == FB_DENSE_GLU ? 64 * (int64_t)t.n + 16 * q + (lane & 15) : 128 * (int64_t)t.n + row;
+        const bool live = col < (EPI == FB_DENSE_GLU ? p.N / 2 : p.N);
+        for (int c = 0; c < half && t0 + c < p.M; c += 8) {
+          float v[8], extra[8];
+          tmem_ld8_nowait(acc + c, v);
+          if constexpr (EPI == FB_DENSE_DYT_ADD || EPI == FB_DENSE_GATE) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+              const int64_t tt = t0 + c + e;
+              extra[e] = 0.f;
+              if (tt < p.M && live) extra[e] = EPI == FB_DENSE_GATE ? p.e.gate[tt * p.e.ld_gate + t.b] : p.e.residual[tt * p.e.ld_residual + col];
+            }
+          }
+          tmem_ld_wait();
+          if constexpr (EPI == FB_DENSE_GLU) {
+            // lanes 0-15 hold gates, 16-31 their ups: the low half takes the first four tokens, the high half the others
+            const bool high = lane >= 16;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float got = __shfl_xor_sync(0xffffffffu, high ? v[e] : v[e + 4], 16);
+              const int64_t tt = t0 + c + e + (high ? 4 : 0);
+              if (tt < p.M && live) emit<EPI>(p, t.b, tt, col, high ? got : v[e], high ? v[e + 4] : got, 0.f, 0.f);
+            }
+          } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+              const int64_t tt = t0 + c + e;
+              if (tt < p.M && live) {
+                if constexpr (EPI == FB_DENSE_GATE) emit<EPI>(p, t.b, tt, col, v[e], 0.f, 0.f, 1.f / (1.f + __expf(-extra[e])));
+                else emit<EPI>(p, t.b, tt, col, v[e], 0.f, EPI == FB_DENSE_DYT_ADD ? extra[e] : 0.f, 0.f);
+              }
+            }
+          }
+        }
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(acc_empty + (n & 1)));
+    }
+  }
+  __syncwarp();
+
+  if (p.splits > 1) {
+    cluster_barrier();  // every CTA's sums are in its shared memory
+    if (warp < D_EPI_WARPS) {
+      const DenseTile t = tile_of(p, blockIdx.x);
+      const int share = (nt + p.splits - 1) / p.splits, first = blockIdx.y * share, last = min(nt, first + share);
+      const int row = tid & 127;
+      const int64_t col = EPI == FB_DENSE_GLU ? 64 * (int64_t)t.n + (row >> 5) * 16 + (row & 15) : 128 * (int64_t)t.n + row;
+      const bool live = col < (EPI == FB_DENSE_GLU ? p.N / 2 : p.N) && (EPI != FB_DENSE_GLU || !(row & 16));
+      for (int c = first + (tid >> 7); c < last; c += 2) {
+        const int64_t tt = (int64_t)nt * t.m + c;
+        if (tt >= p.M || !live) continue;
+        const uint32_t at = smem_u32(smem) + (uint32_t)(c * 128 + row) * 4;
+        float v = 0.f, up = 0.f, res = 0.f, gate = 0.f;
+        if constexpr (EPI == FB_DENSE_DYT_ADD) res = p.e.residual[tt * p.e.ld_residual + col];
+        if constexpr (EPI == FB_DENSE_GATE) gate = 1.f / (1.f + __expf(-p.e.gate[tt * p.e.ld_gate + t.b]));
+        for (int s = 0; s < p.splits; ++s) {
+          v += load_cluster_f32(at, s);
+          if constexpr (EPI == FB_DENSE_GLU) up += load_cluster_f32(at + 64, s);
+        }
+        emit<EPI>(p, t.b, tt, col, v, up, res, gate);
+      }
+    }
+    cluster_barrier();  // the others have read what they need of this CTA's shared memory
+  }
+  __syncthreads();
+  if (warp == D_WARP_MMA) {
+    tc_fence_after();
+    tmem_dealloc(tmem, p.tmem_cols);
+  }
+}
+
+template <int EPI>
+int launch_dense(const CUtensorMap& tw, const CUtensorMap& tx, const DenseParams& p, int grid, size_t smem, cudaStream_t s) {
+  static std::atomic<uint64_t> opted{0};
+  if (first_on_device(opted)) cudaFuncSetAttribute(dense_kernel<EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = dim3((unsigned)grid, (unsigned)p.splits), cfg.blockDim = dim3(D_THREADS), cfg.dynamicSmemBytes = smem, cfg.stream = s;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  attr[1].id = cudaLaunchAttributeClusterDimension;
+  attr[1].val.clusterDim.x = 1, attr[1].val.clusterDim.y = (unsigned)p.splits, attr[1].val.clusterDim.z = 1;
+  cfg.attrs = attr, cfg.numAttrs = p.splits > 1 ? 2 : 1;
+  cudaLaunchKernelEx(&cfg, dense_kernel<EPI>, tw, tx, p);
+  return launch_status("fb_dense");
+}
+
+}  // namespace
+
+int status_word_dense() { return read_and_clear_status_word(); }
+
+}  // namespace fb
+
+extern "C" int fb_dense_supports(const void* x, int64_t ldx, int64_t x_batch, const void* W, int64_t ldw, int64_t w_batch, int64_t K, int64_t N, int kind) {
+  return K >= 8 && K % 8 == 0 && N >= 1 && ldx % 8 == 0 && ldw % 8 == 0 && x_batch % 8 == 0 && w_batch % 8 == 0 && ldx >= K && ldw >= K && (uintptr_t)x % 16 == 0 &&
+         (uintptr_t)W % 16 == 0 && (kind != FB_DENSE_GLU || N % 32 == 0) && fb::tma_encoder() != nullptr;
+}
+
+extern "C" int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_t x_batch, const void* W, int64_t N, int64_t ldw, int64_t w_batch, int64_t batch,
+                        void* out, int out_dtype, int64_t ldo, int64_t out_batch, const fb_dense_epilogue* epilogue_host, int settled, void* stream) {
+  using namespace fb;
+  FB_REQUIRE(x && W && out && M >= 1 && batch >= 1 && M < (1 << 30) && N < (1 << 30), "fb_dense: null pointer or empty");
+  const fb_dense_epilogue e = epilogue_host ? *epilogue_host : fb_dense_epilogue{};
+  FB_REQUIRE(e.kind >= FB_DENSE_NONE && e.kind <= FB_DENSE_DYT_ADD, "fb_dense: unknown epilogue %d", e.kind);
+  FB_REQUIRE(K >= 8 && K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && x_batch % 8 == 0 && w_batch % 8 == 0 && ldx >= K && ldw >= K && (uintptr_t)x % 16 == 0 &&
+                 (uintptr_t)W % 16 == 0 && N >= 1,
+             "fb_dense: rows of x and W 16-byte aligned, K a multiple of 8 (K %lld, row strides %lld and %lld)", (long long)K, (long long)ldx, (long long)ldw);
+  FB_REQUIRE(out_dtype == FB_BF16 || out_dtype == FB_FP32, "fb_dense: out is bf16 or fp32");
+  FB_REQUIRE(e.kind != FB_DENSE_GLU || (N % 32 == 0 && batch == 1), "fb_dense: a gated unit takes one matrix of whole runs of 16 gate rows and as many up rows");
+  FB_REQUIRE(e.kind != FB_DENSE_GATE || e.gate, "fb_dense: no gate given");
+  FB_REQUIRE(e.kind != FB_DENSE_DYT_ADD || (e.residual && e.alpha && e.w && e.b && out_dtype == FB_FP32 && batch == 1 && (!e.h_out || (e.alpha2 && e.w2 && e.b2))),
+             "fb_dense: a Dynamic Tanh and add takes its vectors, a residual and an fp32 result");
+  FB_REQUIRE(tma_encoder() != nullptr, "fb_dense: no CUDA driver");
+  const int64_t out_cols = e.kind == FB_DENSE_GLU ? N / 2 : N;
+  FB_REQUIRE(ldo >= out_cols, "fb_dense: rows of out too close");
+  DenseParams p{};
+  p.M = M, p.N = N, p.e = e, p.out = out, p.out_dtype = out_dtype, p.ldo = ldo, p.out_batch = out_batch, p.settled = settled;
+  p.tiles_m = (int)ceil_div(M, 256);
+  p.nt = (int)ceil_div(ceil_div(M, p.tiles_m), 16) * 16;
+  p.tiles_m = (int)ceil_div(M, p.nt);
+  p.tiles_n = (int)ceil_div(out_cols, e.kind == FB_DENSE_GLU ? 64 : 128);
+  FB_REQUIRE((int64_t)p.tiles_m * p.tiles_n * batch < (1 << 30), "fb_dense: too many tiles");
+  p.tiles = (int)(p.tiles_m * p.tiles_n * batch);
+  p.steps = (int)ceil_div(K, 64);
+  p.tmem_cols = 32;
+  while (p.tmem_cols < 2 * p.nt) p.tmem_cols *= 2;
+  const int stage_bytes = D_A_BYTES + p.nt * 128;
+  p.stages = (int)(D_SMEM / stage_bytes);
+  p.stages = p.stages > D_MAX_STAGES ? D_MAX_STAGES : p.stages;
+  // K over the CTAs of a cluster where the tiles alone leave SMs idle: the split with the least modelled time
+  const int sms = sm_count_of_device();
+  p.splits = 1;
+  double best = 1e30;
+  for (int s = 1; s <= 8; s *= 2) {
+    if (s > 1 && (p.tiles * s > sms || p.steps < 2 * s)) break;
+    const int per = (int)ceil_div(p.steps, s);
+    if ((int)ceil_div(p.steps, per) != s) continue;
+    const double step = 0.12 + 0.001 * p.nt + 0.25 * (double)(p.tiles * s < sms ? p.tiles * s : sms) / sms;  // us: latency-bound at first, then the stream's share
+    const double cost = (double)ceil_div((int64_t)p.tiles * s, sms) * (per * step + 0.5) + (s > 1 ? 1.0 : 0.0);
+    if (cost < best) best = cost, p.splits = s;
+  }
+  p.steps_per_split = (int)ceil_div(p.steps, p.splits);
+  const int grid = p.splits > 1 ? p.tiles : p.tiles < sms ? p.tiles : sms;
+  CUtensorMap tw, tx;
+  if (e.kind == FB_DENSE_GLU) {
+    const int64_t dims[4] = {K, 16, 2, N / 32}, strides[3] = {ldw, N / 2 * ldw, 16 * ldw};
+    const int box[4] = {64, 16, 2, 4};
+    if (int rc = tma_map_bf16(&tw, W, 4, dims, strides, box, "fb_dense (weights)")) return rc;
+  } else {
+    const int64_t dims[3] = {K, N, batch}, strides[2] = {ldw, batch > 1 ? w_batch : ldw};
+    const int box[3] = {64, 128, 1};
+    if (int rc = tma_map_bf16(&tw, W, 3, dims, strides, box, "fb_dense (weights)")) return rc;
+  }
+  const int64_t dims[3] = {K, M, batch}, strides[2] = {ldx, batch > 1 && x_batch ? x_batch : ldx};
+  FB_REQUIRE(batch == 1 || x_batch > 0, "fb_dense: a batch takes rows of its own an entry");
+  const int box[3] = {64, p.nt, 1};
+  if (int rc = tma_map_bf16(&tx, x, 3, dims, strides, box, "fb_dense (activations)")) return rc;
+  const size_t smem = 1024 + (size_t)p.stages * stage_bytes;
+  const auto s = (cudaStream_t)stream;
+  switch (e.kind) {
+    case FB_DENSE_SILU: return launch_dense<FB_DENSE_SILU>(tw, tx, p, grid, smem, s);
+    case FB_DENSE_GLU: return launch_dense<FB_DENSE_GLU>(tw, tx, p, grid, smem, s);
+    case FB_DENSE_GATE: return launch_dense<FB_DENSE_GATE>(tw, tx, p, grid, smem, s);
+    case FB_DENSE_DYT_ADD: return launch_dense<FB_DENSE_DYT_ADD>(tw, tx, p, grid, smem, s);
+    default: return launch_dense<FB_DENSE_NONE>(tw, tx, p, grid, smem, s);
+  }
+}

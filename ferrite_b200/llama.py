@@ -78,7 +78,16 @@ def upload(rt, weights, prec=None, weight_format=weight_format):
         x = Tensor.of(rt, a)
         f = weight_format(name, prec)
         t[name] = x.cast(f).realize() if f != "bf16" else x
-    return t
+    return settle(rt, t)
+
+
+def settle(rt, weights):
+    """Wait for the weights and mark them as complete: a matmul may then fetch them while the kernel before it still runs."""
+    torch.cuda.synchronize(rt.device)
+    for t in weights.values():
+        if isinstance(t, Tensor):
+            t.settled = True
+    return weights
 
 
 def rms(x, w, c):

@@ -1,5 +1,7 @@
 """Thin typed wrappers over the C ABI: torch tensors own the device memory, every call is one or two
 kernel launches on torch's current CUDA stream.  No arithmetic happens in Python or in torch here."""
+import ctypes
+
 import torch
 
 from . import _lib
@@ -310,5 +312,23 @@ def decay_scan(qkv, heads, dim, vdim, decay, places, dead, state, out):
 def gated_rmsnorm(x, gate, w, eps, out):
     check(lib().fb_gated_rmsnorm(x.data_ptr(), x.shape[0], x.shape[1], x.stride(0), _CODES[gate.dtype], gate.data_ptr(), gate.stride(0), w.data_ptr(), eps,
                                  out.data_ptr(), out.stride(0), _stream()))
+    count()
+    return out
+
+
+def dense_supports(x, w, kind=_lib.DENSE_NONE):
+    """Whether fb_dense takes x [batch, M, K] by w [batch, K, N], both bf16 views, w with each column's values together."""
+    return x.dtype == w.dtype == torch.bfloat16 and x.stride(2) == 1 and w.stride(1) == 1 and bool(
+        lib().fb_dense_supports(x.data_ptr(), x.stride(1), x.stride(0) if x.shape[0] > 1 else 0, w.data_ptr(), w.stride(2), w.stride(0) if w.shape[0] > 1 else 0,
+                                w.shape[1], w.shape[2], kind))
+
+
+def dense(x, w, out, settled=False, /, kind=_lib.DENSE_NONE, **extra):
+    """x [batch, M, K] @ w [batch, K, N] into out [batch, M, columns] by fb_dense; extra: the fields of the epilogue's struct."""
+    e = _lib.DenseEpilogue(kind=kind, **extra)
+    batch = x.shape[0]
+    assert out.stride(2) == 1 and out.shape[0] == batch == w.shape[0] and out.shape[1] == x.shape[1]
+    check(lib().fb_dense(x.data_ptr(), x.shape[1], w.shape[1], x.stride(1), x.stride(0) if batch > 1 else 0, w.data_ptr(), w.shape[2], w.stride(2),
+                         w.stride(0) if batch > 1 else 0, batch, out.data_ptr(), _CODES[out.dtype], out.stride(1), out.stride(0), ctypes.byref(e), int(settled), _stream()))
     count()
     return out

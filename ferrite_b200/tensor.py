@@ -649,7 +649,7 @@ def _realize(t, into=None):
             bf = Tensor(t.rt, t.rows, t.cols, batch=t.batch, buf=ops.dequantize(src.packed))
             _done(t, buf=bf.buf if t.dtype == "bf16" else bf.cast(t.dtype).realize().buf)
             return
-        if _fused_linear(t, into):
+        if _fused_linear(t, into) or _fused_dense(t, into):
             return
         if _run_rmsnorm(t, into):
             return
@@ -677,6 +677,8 @@ def _realize(t, into=None):
         if into is not None:
             _copy(t, into)
     elif op == "silu_columns":
+        if _dense(t, t.srcs[0], into, _lib.DENSE_SILU, act_cols=t.args["n"]):
+            return
         src = t.srcs[0].realize()
         out = (src + 0).realize()
         part = out[:, :, :t.args["n"]]
@@ -757,6 +759,117 @@ def _match_dyt(t):
         return None
     x, alpha = th.srcs[0].srcs
     return (x, alpha, w, b) if isinstance(alpha, Tensor) and alpha.op is None and alpha.dtype == "fp32" and alpha.shape == (1, 1, 1) else None
+
+
+def _match_clamped_glu(t):
+    """(matmul, limit, slope) if t is mixers.clamped_glu over the halves of one matmul not yet computed, else None."""
+    if not (t.op == "mul" and all(isinstance(s, Tensor) for s in t.srcs)):
+        return None
+    act, plus = t.srcs
+    if not (act.op == "mul" and isinstance(act.srcs[1], Tensor) and act.srcs[1].op == "recip" and plus.op == "add" and _is_const(plus.srcs[1], 1)):
+        return None
+    g, u = act.srcs[0], plus.srcs[0]
+    one = act.srcs[1].srcs[0]
+    if not (one.op == "add" and _is_const(one.srcs[1], 1) and one.srcs[0].op == "exp"):
+        return None
+    neg = one.srcs[0].srcs[0]
+    if not (neg.op == "mul" and _is_const(neg.srcs[1], -1) and neg.srcs[0].op == "mul" and neg.srcs[0].srcs[0] is g and _is_const(neg.srcs[0].srcs[1])):
+        return None
+    if not (isinstance(u, Tensor) and g.op == "min" and u.op == "min" and isinstance(u.srcs[0], Tensor) and u.srcs[0].op == "max"):
+        return None
+    limit, gate, up = g.srcs[1], g.srcs[0], u.srcs[0].srcs[0]
+    if not (_is_const(limit) and _is_const(u.srcs[1], limit) and _is_const(u.srcs[0].srcs[1], -limit) and gate.op == up.op == "cols" and gate.srcs[0] is up.srcs[0]):
+        return None
+    mm = gate.srcs[0]
+    if gate.args["start"] != 0 or up.args["start"] != gate.cols or 2 * gate.cols != mm.cols:
+        return None
+    return mm, float(limit), float(neg.srcs[0].srcs[1])
+
+
+def _match_gated(t):
+    """(matmul, gate) if t is matmul * gate.sigmoid(), a number a row of each of the matmul's batch, else None."""
+    if t.op != "mul" or not all(isinstance(s, Tensor) for s in t.srcs):
+        return None
+    mm, s = t.srcs
+    if mm.op != "matmul" or s.op != "recip" or s.srcs[0].op != "add" or not _is_const(s.srcs[0].srcs[1], 1) or s.srcs[0].srcs[0].op != "exp":
+        return None
+    neg = s.srcs[0].srcs[0].srcs[0]
+    if not (neg.op == "mul" and _is_const(neg.srcs[1], -1) and isinstance(neg.srcs[0], Tensor) and neg.srcs[0].op is None):
+        return None
+    gate = neg.srcs[0]
+    return (mm, gate) if gate.dtype == "fp32" and gate.shape == (mm.batch, mm.rows, 1) and (mm.batch == 1 or gate.buf.stride(0) == 1) else None
+
+
+def _dense(t, mm, into, kind, **extra):
+    """t by fb_dense where mm is a matmul, not yet computed, by bf16 weights whose columns each lie together (a turned matrix as
+    a checkpoint stores it), with an epilogue; else False.  extra: the epilogue's fields, tensors by name."""
+    if mm.op != "matmul" or len(mm.srcs) != 2:
+        return False
+    a, w = mm.srcs
+    if not (a.dtype == "bf16" and w.dtype == "bf16" and w.op is None and a.batch == w.batch and w.buf.stride(1) == 1 and w.rows % 8 == 0 and w.buf.stride(2) % 8 == 0):
+        return False
+    if kind == _lib.DENSE_GLU and w.cols % 32:
+        return False
+    x = a.realize()
+    if not ops.dense_supports(x.buf, w.buf, kind):
+        x = (x + 0).realize()
+        if not ops.dense_supports(x.buf, w.buf, kind):
+            return False
+    out = into if into is not None and into.buf.stride(2) == 1 and into.dtype == t.dtype else Tensor(t.rt, t.rows, t.cols, batch=t.batch, dtype=t.dtype)
+    fields, keep = {}, []
+    for name, v in extra.items():
+        if isinstance(v, Tensor):
+            v = v.realize()
+            keep.append(v)
+            fields[name] = v.buf.data_ptr()
+            if name in ("residual", "gate", "h_out"):
+                fields["ld_" + name.removesuffix("_out")] = v.buf.stride(1)
+        elif v is not None:
+            fields[name] = v
+    ops.dense(x.buf, w.buf, out.buf, getattr(w, "settled", False), kind=kind, **fields)
+    t.rt.launched("dense" + ("", " silu", " glu", " gate", " dyt add")[kind])
+    _done(t, buf=out.buf)
+    if into is not None and out is not into:
+        _copy(t, into)
+    return True
+
+
+def _fused_dense(t, into, hand_on=None):
+    """t as one fb_dense call with an epilogue, where its tree is a gated unit, a gated output, or a branch's end - the Dynamic
+    Tanh over a matmul, added to the residual stream; else False.  hand_on: the Dynamic Tanh (its tensors, and where its
+    result goes) that the next branch starts with: the same kernel computes it."""
+    inner = t.srcs[0] if t.op == "cast" and t.dtype == "bf16" else t
+    if not isinstance(inner, Tensor) or inner.op is None:
+        return False
+    if inner.op == "mul" and t.dtype == "bf16":
+        found = _match_clamped_glu(inner)
+        if found:
+            return _dense(t, found[0], into, _lib.DENSE_GLU, limit=found[1], slope=found[2])
+        found = _match_gated(inner)
+        if found:
+            return _dense(t, found[0], into, _lib.DENSE_GATE, gate=found[1])
+    if t.op == "cast" and t.dtype == "bf16" and t.batch == 1:
+        found = _match_dyt(inner)
+        if found and found[0].op == "add" and found[0].dtype == "fp32":
+            h = into if into is not None and into.buf.stride(2) == 1 else Tensor(t.rt, t.rows, t.cols)
+            if _fused_dense(found[0], None, (h, *found[1:])):
+                _done(t, buf=h.buf)
+                if into is not None and h is not into:
+                    _copy(t, into)
+                return True
+    if t.op == "add" and t.dtype == "fp32" and t.batch == 1:
+        for x, y in (t.srcs, t.srcs[::-1]):
+            found = _match_dyt(y) if isinstance(y, Tensor) and y.op == "add" else None
+            if found and isinstance(x, Tensor) and x.dtype == "fp32" and x.shape == t.shape and found[0].op == "matmul" and found[0].dtype == "fp32":
+                mm, alpha, w, b = found
+                mm.srcs[0].realize()  # (it may stand on x itself: then x is computed by now, and not once more)
+                x = x.realize()
+                x = x if x.buf.stride(2) == 1 else (x + 0).realize()
+                extra = dict(residual=x, alpha=alpha, w=w, b=b)
+                if hand_on:
+                    extra |= dict(h_out=hand_on[0], alpha2=hand_on[1], w2=hand_on[2], b2=hand_on[3])
+                return _dense(t, mm, into, _lib.DENSE_DYT_ADD, **extra)
+    return False
 
 
 def _match_silu_of(g):
@@ -860,6 +973,8 @@ def _run_matmul(t, into):
         return _linear(t, t, "none", None, into)
     if len(t.srcs) == 3:
         return _run_indexed_matmul(t, into)
+    if _dense(t, t, into, _lib.DENSE_NONE):
+        return
     a, b = t.srcs[0].realize(), t.srcs[1]
     if b.dtype in BFP:  # a batch of block floats, or an fp32 A: by the values, through the general kernel
         b = b.cast("bf16")

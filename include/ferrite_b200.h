@@ -141,6 +141,38 @@ int fb_linear_chained(int fmt, const void* x, int64_t M, int64_t K, int64_t ldx,
                       const void* next_norm_w, void* xn_out, int64_t ld_xn, float* sumsq_out, void* workspace, size_t workspace_bytes,
                       void* stream);
 
+/* ---- matmul by bf16 weights whose output columns each lie together (W [N, K], as checkpoints store a linear layer): x [M, K]
+ * bf16 @ W^T on the tcgen05 tensor cores, fp32 accumulation, with one of these after it: */
+enum fb_dense_epilogue_kind {
+  FB_DENSE_NONE = 0,
+  FB_DENSE_SILU = 1,    /* the first act_cols columns through SiLU */
+  FB_DENSE_GLU = 2,     /* W holds gate rows, then as many up rows: out = g sigmoid(slope g) (u + 1), g = min(gate, limit), u = up in -limit .. limit;
+                           out is [M, N / 2] */
+  FB_DENSE_GATE = 3,    /* times sigmoid(gate[t * ld_gate + batch entry]) */
+  FB_DENSE_DYT_ADD = 4  /* out (fp32) = residual + tanh(alpha acc) w + b, and, with h_out given, h_out (bf16) = tanh(alpha2 out) w2 + b2: a Dynamic
+                           Tanh on a branch, the residual add, and the Dynamic Tanh that the next branch starts with */
+};
+typedef struct {
+  int kind;
+  int64_t act_cols;
+  float limit, slope;
+  const float* gate;
+  int64_t ld_gate;
+  const float* residual;
+  int64_t ld_residual;
+  const float *alpha, *w, *b; /* alpha: one number on the device; w, b: [N] */
+  void* h_out;
+  int64_t ld_h;
+  const float *alpha2, *w2, *b2;
+} fb_dense_epilogue;
+/* batch independent matmuls: x, W and out move on by x_batch, w_batch and out_batch elements an entry (x_batch 0: all take the
+ * same rows).  ldx, ldw, x_batch, w_batch multiples of 8 elements, x and W 16-byte aligned, K a multiple of 8 (GLU: N / 2 a
+ * multiple of 16); fb_dense_supports says whether a call qualifies.  settled: W was complete before the kernel launched
+ * before this one (loaded weights): its first tiles are then fetched while that kernel drains. */
+int fb_dense_supports(const void* x, int64_t ldx, int64_t x_batch, const void* W, int64_t ldw, int64_t w_batch, int64_t K, int64_t N, int kind);
+int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_t x_batch, const void* W, int64_t N, int64_t ldw, int64_t w_batch, int64_t batch,
+             void* out, int out_dtype, int64_t ldo, int64_t out_batch, const fb_dense_epilogue* epilogue_host, int settled, void* stream);
+
 /* Tensor.matmul(index=) (ferrite/tensor.py:450-460; ferrite/compiler.py:704-706): a mixture of experts' matmul.  W is
  * a batch of n_experts packed [K, N] matrices fb_packed_bytes(fmt, K, N) apart; index[slot] (int32, read on the
  * device, so a replayed step follows its tokens' choices) picks one for each of n_slots slots, and a slot that picks
