@@ -28,7 +28,7 @@ extern "C" int fb_version(void) { return 1; }
 extern "C" const char* fb_last_error(void) { return fb::g_error; }
 
 extern "C" int fb_status_word(void) {
-  const int codes[] = {fb::status_word_tcgen05(), fb::status_word_peer(), fb::status_word_gemv_stream(), fb::status_word_dense()};  // (all read, so all are cleared)
+  const int codes[] = {fb::status_word_tcgen05(), fb::status_word_peer(), fb::status_word_gemv_stream(), fb::status_word_dense(), fb::status_word_latent()};  // (all read, so all are cleared)
   for (int code : codes)
     if (code) return code;
   return 0;

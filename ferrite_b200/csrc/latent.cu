@@ -200,8 +200,7 @@ extern "C" int fb_rotate_pairs(int dtype, const void* x, int64_t T, int heads, i
 }
 
 extern "C" size_t fb_latent_attention_workspace_bytes(int dtype, int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk) {
-  (void)dtype, (void)T, (void)heads, (void)rank, (void)rot, (void)max_keys, (void)chunk;
-  return 0;
+  return dtype == FB_BF16 && heads >= 1 && rank >= 1 && rot >= 0 ? fb::latent_tcgen05_workspace(T, heads, rank, rot, max_keys, chunk) : 0;
 }
 
 extern "C" int fb_latent_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int rank, int rot, const void* cache, int64_t cache_rows,
@@ -213,6 +212,7 @@ extern "C" int fb_latent_attention(int dtype, const void* q, int64_t T, int64_t 
   FB_REQUIRE(rank <= 32 * fb::LAT_COLS, "fb_latent_attention: latents of up to %d columns", 32 * fb::LAT_COLS);
   fb::LatentArgs a{q, T, ld_q, heads, rank, rot, cache, cache_rows, base, row0, last, max_keys, chunk, scale, sink, out, ld_o, workspace, workspace_bytes};
   const auto s = (cudaStream_t)stream;
+  if (dtype == FB_BF16 && fb::latent_tcgen05_supports(a)) return fb::latent_tcgen05(a, s);
   if (dtype == FB_FP32) return rank <= 256 ? fb::launch_latent<float, 8>(a, s) : fb::launch_latent<float, fb::LAT_COLS>(a, s);
   return rank <= 256 ? fb::launch_latent<uint16_t, 8>(a, s) : fb::launch_latent<uint16_t, fb::LAT_COLS>(a, s);
 }

@@ -23,4 +23,9 @@ struct LatentArgs {
   size_t workspace_bytes;
 };
 
+// latent_tcgen05.cu: bf16 rows on the tensor cores
+bool latent_tcgen05_supports(const LatentArgs& a);
+size_t latent_tcgen05_workspace(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk);
+int latent_tcgen05(const LatentArgs& a, cudaStream_t s);
+
 }  // namespace fb

@@ -1,0 +1,405 @@
+// fb_latent_attention on the 5th-generation tensor cores (bf16 rows).
+//
+// All heads of a token read the same cache row, and one row is key and value at once, so the unit of work is a tile of up
+// to 64 query ROWS - (token, head) pairs that see keys of one sequence: a decode step's heads of a token, or consecutive
+// pairs of a prompt's chunk - by tiles of 64 cache rows, each brought in by TMA once and used twice from shared memory:
+//
+//   scores    S [rows, 64 keys]    = Q [rows, W] . K^T       Q is the MMA's A operand (its 128 lanes read past the last row:
+//                                                            lanes of no row, never looked at), the keys its N dimension
+//   sums      O^T [128 columns of the latent, rows] += V^T P^T   the same tile of cache rows as A operand, now with the
+//                                                            latent's columns as lanes; P from shared memory as B
+//
+// so a softmax thread owns a row's 64 scores of a tile outright (tcgen05.ld; no exchange between threads), and the sums of a
+// 512-column latent by 64 rows take half of tensor memory.  The sums stand under a reference maximum that moves only when a
+// row's scores outgrow it by a factor of 256; then (rarely after the first tiles) the accumulators are rescaled.
+//
+//   warps 0-3   softmax; rescaling; the result        warp 4   TMA        warp 5   MMAs
+//
+// The ring holds two to four tiles of cache rows.  With three or more the next tile's scores are computed while this
+// tile's softmax runs.  Few row tiles are split along the keys over more CTAs; latent_combine_kernel merges the parts and adds
+// the sink, which is one more part with a maximum and no value.  Every wait is bounded (sm100.cuh).
+#include "latent.cuh"
+#include "sm100.cuh"
+#include "tma_host.cuh"
+
+namespace fb {
+
+namespace {
+
+constexpr int L_KEYS = 64, L_ROWS = 64, L_WARP_LOAD = 4, L_WARP_MMA = 5, L_THREADS = 6 * 32, L_MAX_BUFS = 4;
+constexpr int L_CHUNK = L_KEYS * 128;  // 64 cache rows of 64 columns
+constexpr size_t L_SMEM = 225 * 1024;
+constexpr float L_SLACK = 8.f;  // log2 of how far scores may outgrow the reference maximum
+
+enum LatentWait { LW_Q = 401, LW_K_EMPTY, LW_K_FULL, LW_S, LW_P, LW_PV, LW_DRAIN };
+
+struct LatentParams {
+  LatentArgs a;
+  int nr, chunks, blocks, bufs, tmem_cols, splits, tiles_per_token;  // tiles_per_token: 0 for a chunk (tiles run through its rows)
+  float scale_log2;
+  float *part_o, *part_ml;  // [tile, split, 64, rank] and [tile, split, 64, 2]
+};
+
+__device__ __forceinline__ void tmem_st16(uint32_t taddr, const float v[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};" ::"r"(taddr),
+      "r"(__float_as_uint(v[0])), "r"(__float_as_uint(v[1])), "r"(__float_as_uint(v[2])), "r"(__float_as_uint(v[3])), "r"(__float_as_uint(v[4])),
+      "r"(__float_as_uint(v[5])), "r"(__float_as_uint(v[6])), "r"(__float_as_uint(v[7])), "r"(__float_as_uint(v[8])), "r"(__float_as_uint(v[9])),
+      "r"(__float_as_uint(v[10])), "r"(__float_as_uint(v[11])), "r"(__float_as_uint(v[12])), "r"(__float_as_uint(v[13])), "r"(__float_as_uint(v[14])),
+      "r"(__float_as_uint(v[15]))
+      : "memory");
+}
+__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+
+// a barrier of the four softmax warps; true if any of their threads brings a true
+__device__ __forceinline__ bool softmax_any(bool mine) {
+  uint32_t any;
+  asm volatile("{\n.reg .pred p, q;\nsetp.ne.u32 q, %1, 0;\nbarrier.cta.red.or.aligned.pred p, 1, 128, q;\nselp.u32 %0, 1, 0, p;\n}" : "=r"(any) : "r"((uint32_t)mine) : "memory");
+  return any != 0;
+}
+__device__ __forceinline__ void softmax_sync() { asm volatile("barrier.cta.sync.aligned 1, 128;" ::: "memory"); }
+
+// where a row tile stands: its first (token, head) pair, how many, and the keys it reads
+struct RowTile {
+  int64_t first_row, seq_first;
+  int rows, keys;
+};
+__device__ __forceinline__ RowTile row_tile(const LatentParams& p, int tile) {
+  const LatentArgs& a = p.a;
+  RowTile r;
+  int64_t t0, t1;
+  if (p.tiles_per_token) {
+    const int g = tile % p.tiles_per_token;
+    t0 = t1 = tile / p.tiles_per_token;
+    r.first_row = t0 * a.heads + g * L_ROWS, r.rows = min(L_ROWS, a.heads - g * L_ROWS);
+  } else {
+    r.first_row = (int64_t)tile * L_ROWS, r.rows = (int)min((int64_t)L_ROWS, a.T * a.heads - r.first_row);
+    t0 = r.first_row / a.heads, t1 = (r.first_row + r.rows - 1) / a.heads;
+  }
+  r.seq_first = (a.base ? a.base[t0] : 0) + a.row0;
+  int last = -1;
+  for (int64_t t = t0; t <= t1; ++t) last = max(last, a.last[t]);
+  const int64_t room = r.seq_first < 0 ? 0 : a.cache_rows - r.seq_first;
+  r.keys = (int)max((int64_t)0, min((int64_t)last + 1, room));
+  return r;
+}
+
+__global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk, const LatentParams p) {
+  extern __shared__ uint8_t latent_smem[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(latent_smem) + 1023) & ~uintptr_t(1023));
+  __shared__ uint64_t bars[2 * L_MAX_BUFS + 5];
+  __shared__ uint32_t tmem_slot[2];  // the allocation's address, the abort flag
+  __shared__ float row_scale[L_ROWS];
+  uint64_t *k_full = bars, *k_empty = bars + L_MAX_BUFS, *q_full = bars + 2 * L_MAX_BUFS, *s_full = q_full + 1, *p_full = q_full + 3, *pv_done = q_full + 4;
+  const uint32_t abort_flag = smem_u32(tmem_slot + 1);
+  const LatentArgs& a = p.a;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int nr = p.nr, C = p.chunks, NB = p.bufs;
+  const int tile = p.tiles_per_token ? blockIdx.x : gridDim.x - 1 - blockIdx.x, split = blockIdx.y;  // (a chunk's longest rows first)
+  const uint32_t sQ = smem_u32(smem), sK = sQ + C * nr * 128, tile_bytes = C * L_CHUNK, sP = sK + NB * tile_bytes;
+
+  griddep_launch_dependents();
+  if (tid == 0) {
+    for (int i = 0; i < NB; ++i) mbar_init(smem_u32(k_full + i), 1), mbar_init(smem_u32(k_empty + i), 1);
+    mbar_init(smem_u32(q_full), 1), mbar_init(smem_u32(s_full), 1), mbar_init(smem_u32(s_full + 1), 1);
+    mbar_init(smem_u32(p_full), 4), mbar_init(smem_u32(pv_done), 1);
+    tmem_slot[1] = 0;
+    fence_barrier_init();
+  }
+  if (warp == L_WARP_MMA) tmem_alloc(smem_u32(tmem_slot), p.tmem_cols);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_slot[0], tS = tmem, tO = tmem + 2 * L_KEYS;
+  griddep_wait();
+
+  const RowTile r = row_tile(p, tile);
+  // this CTA's run of whole tiles of keys
+  const int all = (r.keys + L_KEYS - 1) / L_KEYS, per = (all + p.splits - 1) / p.splits;
+  const int first_tile = split * per, n_tiles = max(0, min(all, first_tile + per) - first_tile);
+
+  if (warp == L_WARP_LOAD && lane == 0) {
+    if (n_tiles) {
+      prefetch_tensormap(&tq), prefetch_tensormap(&tk);
+      mbar_expect_tx(smem_u32(q_full), (uint32_t)(C * nr * 128));
+      for (int c = 0; c < C; ++c) tma_load_2d(sQ + c * nr * 128, &tq, 64 * c, (int)r.first_row, smem_u32(q_full));
+    }
+    int buf = 0, i = 0;
+    uint32_t phase = 0;
+    bool ok = true;
+    for (; i < n_tiles; ++i) {
+      ok = mbar_wait(smem_u32(k_empty + buf), phase ^ 1, abort_flag, LW_K_EMPTY);
+      if (!ok) break;
+      mbar_expect_tx(smem_u32(k_full + buf), tile_bytes);
+      for (int c = 0; c < C; ++c)
+        tma_load_2d(sK + buf * tile_bytes + c * L_CHUNK, &tk, 64 * c, (int)(r.seq_first + (int64_t)(first_tile + i) * L_KEYS), smem_u32(k_full + buf));
+      if (++buf == NB) buf = 0, phase ^= 1;
+    }
+    if (!ok)  // given up: the copies under way land before this CTA's shared memory is anyone else's
+      for (int b = 0; b < NB && b < i; ++b) {
+        const long long start = clock64();
+        while (!mbar_try_wait(smem_u32(k_full + b), b < buf ? phase : phase ^ 1) && clock64() - start < WAIT_CLOCKS) {
+        }
+      }
+  } else if (warp == L_WARP_MMA && lane == 0 && n_tiles) {
+    const uint32_t idesc_s = umma_idesc_bf16(L_KEYS, false, false), idesc_o = umma_idesc_bf16(nr, true, false);
+    const uint64_t dq0 = umma_smem_desc(sQ, 16, 1024), dk0 = umma_smem_desc(sK, 16, 1024), dv0 = umma_smem_desc(sK, L_CHUNK, 1024), dp = umma_smem_desc(sP, 16, 1024);
+    const uint32_t q_chunk = (uint32_t)(nr * 128) >> 4, k_chunk = L_CHUNK >> 4, k_tile = tile_bytes >> 4;
+    int sbuf = 0;  // the ring's place of the next scores
+    uint32_t sphase = 0;
+    auto scores = [&](int t) {
+      mbar_wait(smem_u32(k_full + sbuf), sphase, abort_flag, LW_K_FULL);
+      tc_fence_after();
+      for (int c = 0; c < C; ++c)
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk)
+          umma_bf16(tS + (t & 1) * L_KEYS, dq0 + c * q_chunk + 2 * kk, dk0 + sbuf * k_tile + c * k_chunk + 2 * kk, idesc_s, c | kk);
+      umma_commit(smem_u32(s_full + (t & 1)));
+      if (++sbuf == NB) sbuf = 0, sphase ^= 1;
+    };
+    mbar_wait(smem_u32(q_full), 0, abort_flag, LW_Q);
+    scores(0);
+    int vbuf = 0;
+    for (int t = 0; t < n_tiles; ++t) {
+      if (NB >= 3 && t + 1 < n_tiles) scores(t + 1);
+      mbar_wait(smem_u32(p_full), t & 1, abort_flag, LW_P);
+      tc_fence_after();
+      for (int b = 0; b < p.blocks; ++b)
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk)  // 16 keys each
+          umma_bf16(tO + b * nr, dv0 + vbuf * k_tile + 2 * b * k_chunk + kk * (2048 >> 4), dp + 2 * kk, idesc_o, t | kk);
+      umma_commit(smem_u32(k_empty + vbuf));
+      umma_commit(smem_u32(pv_done));
+      if (++vbuf == NB) vbuf = 0;
+      if (NB < 3 && t + 1 < n_tiles) scores(t + 1);
+    }
+  } else if (warp < 4) {
+    const int row = tid;  // lane `row` of the scores
+    const bool live = row < r.rows;
+    const int place = live ? a.last[(r.first_row + row) / a.heads] : -1;
+    const uint32_t lanes = (uint32_t)(32 * warp) << 16;
+    float m = -INFINITY, l = 0.f;  // the reference maximum (in units of log2) and the sum under it
+    for (int t = 0; t < n_tiles; ++t) {
+      mbar_wait(smem_u32(s_full + (t & 1)), (t >> 1) & 1, abort_flag, LW_S);
+      tc_fence_after();
+      float s[L_KEYS];
+      float corr = 1.f;
+      bool moved = false;
+      if (32 * warp < nr) {
+        tmem_ld32_nowait(tS + lanes + (t & 1) * L_KEYS, s);
+        tmem_ld32_nowait(tS + lanes + (t & 1) * L_KEYS + 32, s + 32);
+        tmem_ld_wait();
+        const int seen = min(place, r.keys - 1) + 1 - (first_tile + t) * L_KEYS;  // the tile's first `seen` keys
+        float top = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < L_KEYS; ++j) {
+          s[j] = j < seen ? s[j] * p.scale_log2 : -INFINITY;
+          top = fmaxf(top, s[j]);
+        }
+        if (top > m + L_SLACK || (m == -INFINITY && top > m)) {
+          corr = exp2f(m - top);  // (0 from -infinity)
+          m = top, moved = t > 0;
+        }
+        const float at = m == -INFINITY ? 0.f : m;
+        float sum = 0.f;
+#pragma unroll
+        for (int j = 0; j < L_KEYS; ++j) {
+          s[j] = exp2f(s[j] - at);
+          sum += s[j];
+        }
+        l = l * corr + sum;
+      }
+      if (t > 0) {  // the sums and P are free once the last tile's MMAs are done
+        mbar_wait(smem_u32(pv_done), (t - 1) & 1, abort_flag, LW_PV);
+        tc_fence_after();
+      }
+      if (row < L_ROWS) row_scale[row] = corr;
+      if (softmax_any(moved)) {
+        for (int b = 0; b < p.blocks; ++b)
+          for (int c = 0; c < nr; c += 16) {
+            float v[16];
+            tmem_ld16_nowait(tO + lanes + b * nr + c, v);
+            tmem_ld_wait();
+#pragma unroll
+            for (int e = 0; e < 16; ++e) v[e] *= row_scale[c + e];
+            tmem_st16(tO + lanes + b * nr + c, v);
+          }
+        tmem_st_wait();
+      }
+      if (row < nr) {
+#pragma unroll
+        for (int c = 0; c < 8; ++c)
+          st_shared_v4(sP + row * 128 + ((c ^ (row & 7)) << 4), pack_bf16x2(s[8 * c], s[8 * c + 1]), pack_bf16x2(s[8 * c + 2], s[8 * c + 3]),
+                       pack_bf16x2(s[8 * c + 4], s[8 * c + 5]), pack_bf16x2(s[8 * c + 6], s[8 * c + 7]));
+      }
+      fence_proxy_async();
+      tc_fence_before();
+      softmax_sync();  // (row_scale has been read by all before a next tile writes it)
+      if (lane == 0) mbar_arrive(smem_u32(p_full));
+    }
+    // ---- the result
+    if (n_tiles) {
+      mbar_wait(smem_u32(pv_done), (n_tiles - 1) & 1, abort_flag, LW_PV);
+      tc_fence_after();
+    }
+    const int64_t part = (int64_t)tile * p.splits + split;
+    if (row < L_ROWS) {
+      if (p.splits > 1) {
+        p.part_ml[(part * L_ROWS + row) * 2] = m, p.part_ml[(part * L_ROWS + row) * 2 + 1] = l;
+        row_scale[row] = 1.f;
+      } else {
+        float f = 1.f, total = l;
+        if (a.sink && live) {
+          const float sink = a.sink[(r.first_row + row) % a.heads] * 1.4426950408889634f, top = fmaxf(m, sink);
+          f = exp2f(m - top), total = l * f + exp2f(sink - top);
+        }
+        row_scale[row] = total > 0.f ? f / total : 0.f;
+      }
+    }
+    softmax_sync();
+    for (int b = 0; b < p.blocks && (n_tiles || p.splits == 1); ++b) {
+      const int d = 128 * b + tid;
+      for (int c = 0; c < nr && c < r.rows; c += 16) {
+        float v[16];
+        if (n_tiles) {
+          tmem_ld16_nowait(tO + lanes + b * nr + c, v);
+          tmem_ld_wait();
+        }
+        if (d >= a.rank) continue;
+#pragma unroll
+        for (int e = 0; e < 16; ++e) {
+          if (c + e >= r.rows) break;
+          if (p.splits > 1) p.part_o[(part * L_ROWS + c + e) * a.rank + d] = v[e];
+          else static_cast<uint16_t*>(a.out)[(r.first_row + c + e) * a.rank + d] = (uint16_t)float_to_bf16_bits(n_tiles ? v[e] * row_scale[c + e] : 0.f);
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == L_WARP_MMA) {
+    tc_fence_after();
+    tmem_dealloc(tmem, p.tmem_cols);
+  }
+}
+
+// a block per (token, head): its splits' sums weighted by their maxima, the sink beside them
+__global__ void __launch_bounds__(128) latent_combine_kernel(const LatentParams p) {
+  griddep_launch_dependents();
+  griddep_wait();
+  const LatentArgs& a = p.a;
+  const int64_t id = blockIdx.x;
+  int64_t tile;
+  int row;
+  if (p.tiles_per_token) {
+    const int h = (int)(id % a.heads);
+    tile = id / a.heads * p.tiles_per_token + h / L_ROWS, row = h % L_ROWS;
+  } else {
+    tile = id / L_ROWS, row = (int)(id % L_ROWS);
+  }
+  const float* ml = p.part_ml + (tile * p.splits * L_ROWS + row) * 2;
+  const float sink = a.sink ? a.sink[id % a.heads] * 1.4426950408889634f : -INFINITY;
+  float m = sink;
+  for (int s = 0; s < p.splits; ++s) m = fmaxf(m, ml[s * L_ROWS * 2]);
+  const float at = m == -INFINITY ? 0.f : m;
+  float total = exp2f(sink - at);
+  for (int s = 0; s < p.splits; ++s) total += ml[s * L_ROWS * 2 + 1] * exp2f(ml[s * L_ROWS * 2] - at);
+  const float inv = total > 0.f ? 1.f / total : 0.f;
+  for (int d = threadIdx.x; d < a.rank; d += blockDim.x) {
+    float acc = 0.f;
+    for (int s = 0; s < p.splits; ++s)
+      if (ml[s * L_ROWS * 2 + 1] > 0.f) acc += p.part_o[((tile * p.splits + s) * L_ROWS + row) * a.rank + d] * exp2f(ml[s * L_ROWS * 2] - at);
+    static_cast<uint16_t*>(a.out)[id * a.rank + d] = (uint16_t)float_to_bf16_bits(acc * inv);
+  }
+}
+
+// sizes and launch shape; false: not for this kernel
+bool make_latent_plan(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk, LatentParams& p) {
+  const int W = rank + rot;
+  if (W % 8 || rank > 512 || max_keys < 1) return false;
+  const int64_t rows = chunk ? T * heads : heads;
+  p.nr = rows >= L_ROWS ? L_ROWS : (int)ceil_div(rows, 16) * 16;
+  p.chunks = (int)ceil_div(W, 64), p.blocks = (int)ceil_div(rank, 128);
+  const size_t fixed = 2048 + (size_t)p.chunks * p.nr * 128 + L_ROWS * 128, tile = (size_t)p.chunks * L_CHUNK;
+  if (fixed + 2 * tile > L_SMEM) return false;
+  p.bufs = (int)((L_SMEM - fixed) / tile);
+  p.bufs = p.bufs > L_MAX_BUFS ? L_MAX_BUFS : p.bufs;
+  // (an A operand reads 128 rows from a Q chunk's start, and two 64-column chunks from a cache tile's last: both stay within the ring and P)
+  const int cols = 2 * L_KEYS + p.blocks * p.nr;
+  p.tmem_cols = 32;
+  while (p.tmem_cols < cols) p.tmem_cols *= 2;
+  if (p.tmem_cols > 512) return false;
+  p.tiles_per_token = chunk ? 0 : (int)ceil_div(heads, L_ROWS);
+  const int64_t tiles = chunk ? ceil_div(rows, L_ROWS) : T * p.tiles_per_token;
+  if (tiles > (1 << 20)) return false;
+  const int sms = sm_count_of_device();
+  const int64_t key_tiles = ceil_div(max_keys, L_KEYS);
+  int best = 1;
+  double best_cost = 1e30;
+  for (int s = 1; s <= 32 && s <= key_tiles; ++s) {  // tiles of keys a CTA, plus its fixed cost in the same unit, by rounds of CTAs
+    const double cost = (double)ceil_div(tiles * s, sms) * ((double)ceil_div(key_tiles, s) + 2.5) + (s > 1 ? 1.5 + 0.05 * s : 0.0);
+    if (cost < best_cost - 1e-9) best_cost = cost, best = s;
+  }
+  p.splits = best;
+  return true;
+}
+
+int64_t latent_tiles(const LatentParams& p, int64_t T, int heads) { return p.tiles_per_token ? T * p.tiles_per_token : ceil_div(T * heads, L_ROWS); }
+
+}  // namespace
+
+size_t latent_tcgen05_workspace(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk) {
+  LatentParams p{};
+  if (T < 1 || !make_latent_plan(T, heads, rank, rot, max_keys, chunk, p) || p.splits == 1) return 0;
+  return (size_t)latent_tiles(p, T, heads) * p.splits * L_ROWS * (rank + 2) * sizeof(float);
+}
+
+bool latent_tcgen05_supports(const LatentArgs& a) {
+  LatentParams p{};
+  return tma_encoder() != nullptr && a.ld_q == (int64_t)a.heads * (a.rank + a.rot) && a.ld_o == (int64_t)a.heads * a.rank && (uintptr_t)a.q % 16 == 0 &&
+         (uintptr_t)a.cache % 16 == 0 && a.cache_rows < (1ll << 31) && a.T * a.heads < (1ll << 31) && make_latent_plan(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, p);
+}
+
+int latent_tcgen05(const LatentArgs& a, cudaStream_t s) {
+  LatentParams p{};
+  p.a = a;
+  make_latent_plan(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, p);
+  p.scale_log2 = a.scale * 1.4426950408889634f;
+  const int64_t tiles = latent_tiles(p, a.T, a.heads);
+  if (p.splits > 1) {
+    const size_t need = latent_tcgen05_workspace(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk);
+    if (!a.workspace || a.workspace_bytes < need) {
+      set_error("fb_latent_attention: workspace of %zu bytes needed, %zu given", need, a.workspace_bytes);
+      return FB_ERR_MEMORY;
+    }
+    p.part_o = (float*)a.workspace, p.part_ml = p.part_o + (size_t)tiles * p.splits * L_ROWS * a.rank;
+  }
+  const int W = a.rank + a.rot;
+  CUtensorMap tq, tk;
+  const int64_t qd[2] = {W, a.T * a.heads}, kd[2] = {W, a.cache_rows}, stride[1] = {W};
+  const int qb[2] = {64, p.nr}, kb[2] = {64, L_KEYS};
+  if (int rc = tma_map_bf16(&tq, a.q, 2, qd, stride, qb, "fb_latent_attention (queries)")) return rc;
+  if (int rc = tma_map_bf16(&tk, a.cache, 2, kd, stride, kb, "fb_latent_attention (cache)")) return rc;
+  static std::atomic<uint64_t> opted{0};
+  if (first_on_device(opted)) cudaFuncSetAttribute(latent_tcgen05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = dim3((unsigned)tiles, (unsigned)p.splits), cfg.blockDim = dim3(L_THREADS), cfg.stream = s;
+  cfg.dynamicSmemBytes = 1024 + (size_t)p.chunks * p.nr * 128 + (size_t)p.bufs * p.chunks * L_CHUNK + L_ROWS * 128;
+  // (room for what an A operand reads past Q's last rows where the ring is short)
+  const size_t reach = 1024 + (size_t)(p.chunks - 1) * p.nr * 128 + 128 * 128;
+  if (cfg.dynamicSmemBytes < reach) cfg.dynamicSmemBytes = reach;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr, cfg.numAttrs = 1;
+  cudaLaunchKernelEx(&cfg, latent_tcgen05_kernel, tq, tk, p);
+  if (p.splits > 1) {
+    cfg.gridDim = dim3((unsigned)(a.T * a.heads)), cfg.blockDim = dim3(128), cfg.dynamicSmemBytes = 0;
+    cudaLaunchKernelEx(&cfg, latent_combine_kernel, p);
+  }
+  return launch_status("fb_latent_attention");
+}
+
+int status_word_latent() { return read_and_clear_status_word(); }
+
+}  // namespace fb
