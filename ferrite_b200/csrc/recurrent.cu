@@ -1,8 +1,10 @@
 // Linear attention with a fixed decay per head: S_t = decay S_(t-1) + k_t v_t^T (fp32, a [dim, vdim] matrix a head and
 // sequence), o_t = S_t^T q_t, and the gated RMSNorm that follows it.
 //
-//   fb_decay_scan       token after token: a decode step's one token a sequence, and prompts in fp32 or of odd sizes
+//   fb_decay_scan       token after token: a decode step's one token a sequence, and prompts in fp32 or of odd sizes; bf16
+//                       prompts in chunks of 64 tokens on tensor-core MMAs (decay_chunk_kernel)
 //   fb_gated_rmsnorm    RMSNorm over all the heads' outputs together, times the sigmoid of a gate
+#include "mma_sync.cuh"
 #include "values.cuh"
 
 namespace fb {
@@ -81,6 +83,203 @@ __global__ void decay_scan_kernel(const ScanArgs a) {
   }
 }
 
+// ---- a prompt in chunks of 64 tokens.  Within a chunk that starts from the state S,
+//     o_i = decay^(i+1) S^T q_i + sum over j <= i of decay^(i-j) (q_i . k_j) v_j,    S' = decay^n S + sum decay^(n-1-j) k_j v_j^T,
+// all of it matrix products.  A CTA walks one sequence's chunks for one head and 32 of its value columns, with its part of the
+// state in registers as the accumulators of the last product.  q, k and v are bf16 as they come; what is not - the state, the
+// decayed scores, the decayed values - enters a product as two bf16 parts, so the recurrence keeps fp32's range and 16 bits
+// of mantissa in every factor, with sums in fp32.
+constexpr int CH_TOKENS = 64, CH_COLS = 32, CH_PITCH = CH_COLS * 2 + 16;  // (rows an odd number of 16-byte pieces apart: no bank conflicts)
+
+template <int TILES>  // 16-row tiles of the state a warp owns
+__global__ void __launch_bounds__(128) decay_chunk_kernel(const ScanArgs a) {
+  griddep_launch_dependents();
+  griddep_wait();
+  extern __shared__ __align__(128) uint8_t chunk_smem[];
+  __shared__ float power[CH_TOKENS + 1];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, v0 = blockIdx.x * CH_COLS;
+  const int dim = a.dim, pitch = dim * 2 + 16, pieces = dim / 8;
+  const int64_t seq = blockIdx.z, t0 = seq * a.tokens;
+  const uint32_t sQ = smem_addr(chunk_smem), sK = sQ + 2 * CH_TOKENS * pitch, sV = sK + 2 * CH_TOKENS * pitch;
+  const uint32_t sS = sV + 2 * CH_TOKENS * CH_PITCH, sW = sS + 2 * dim * CH_PITCH;  // the state, the decayed values: high parts, then low
+  uint8_t* generic = chunk_smem - sQ;  // + a shared address
+  const uint16_t* qkv = static_cast<const uint16_t*>(a.qkv);
+  const int64_t q_at = (int64_t)h * dim, k_at = ((int64_t)a.heads + h) * dim, v_at = 2 * (int64_t)a.heads * dim + (int64_t)h * a.vdim + v0;
+  const int place = a.places[t0];
+  for (int e = tid; e <= CH_TOKENS; e += 128) power[e] = (float)pow((double)a.decay[h], (double)e);
+
+  auto load = [&](int64_t c, int buf) {
+    for (int i = tid; i < CH_TOKENS * pieces; i += 128) {
+      const int r = i / pieces, ch = i % pieces;
+      const int64_t t = c * CH_TOKENS + r;
+      const bool in = t < a.tokens;
+      const uint16_t* x = qkv + (t0 + (in ? t : 0)) * a.ld + ch * 8;
+      cp_async16_or_zero(sQ + (buf * CH_TOKENS + r) * pitch + ch * 16, x + q_at, in ? 16 : 0);
+      cp_async16_or_zero(sK + (buf * CH_TOKENS + r) * pitch + ch * 16, x + k_at, in ? 16 : 0);
+    }
+    for (int i = tid; i < CH_TOKENS * CH_COLS / 8; i += 128) {
+      const int r = i / (CH_COLS / 8), ch = i % (CH_COLS / 8);
+      const int64_t t = c * CH_TOKENS + r;
+      const bool in = t < a.tokens && v0 + ch * 8 < a.vdim;
+      cp_async16_or_zero(sV + (buf * CH_TOKENS + r) * CH_PITCH + ch * 16, in ? qkv + (t0 + t) * a.ld + v_at + ch * 8 : qkv, in ? 16 : 0);
+    }
+    cp_async_commit();
+  };
+  load(0, 0);
+
+  float* state = a.state + seq * a.state_stride + (int64_t)h * dim * a.vdim;
+  float S[TILES][CH_COLS / 8][4];
+  auto each_state = [&](auto&& f) {  // f(value, row, column) for the pairs of this thread's part of the state
+#pragma unroll
+    for (int i = 0; i < TILES; ++i)
+#pragma unroll
+      for (int n = 0; n < CH_COLS / 8; ++n)
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+          const int row = 16 * (warp + 4 * i) + (lane >> 2) + 8 * g, col = n * 8 + (lane & 3) * 2;
+          if (row < dim) f(S[i][n][2 * g], S[i][n][2 * g + 1], row, col);
+        }
+  };
+#pragma unroll
+  for (int i = 0; i < TILES; ++i)
+#pragma unroll
+    for (int n = 0; n < CH_COLS / 8; ++n) S[i][n][0] = S[i][n][1] = S[i][n][2] = S[i][n][3] = 0.f;
+  if (place != 0)
+    each_state([&](float& x, float& y, int row, int col) {
+      if (v0 + col < a.vdim) {  // (vdim is even)
+        const float2 v = *reinterpret_cast<const float2*>(state + (int64_t)row * a.vdim + v0 + col);
+        x = v.x, y = v.y;
+      }
+    });
+
+  const int64_t chunks = (a.tokens + CH_TOKENS - 1) / CH_TOKENS;
+  const int m = lane >> 3, m_row = lane & 7;
+  for (int64_t c = 0; c < chunks; ++c) {
+    const int buf = (int)(c & 1), n = (int)min((int64_t)CH_TOKENS, a.tokens - c * CH_TOKENS);
+    cp_async_wait<0>();
+    __syncthreads();
+    if (c + 1 < chunks) load(c + 1, buf ^ 1);
+    each_state([&](float& x, float& y, int row, int col) {
+      uint32_t high, low;
+      split_bf16x2(x, y, high, low);
+      *reinterpret_cast<uint32_t*>(generic + sS + row * CH_PITCH + col * 2) = high;
+      *reinterpret_cast<uint32_t*>(generic + sS + (dim + row) * CH_PITCH + col * 2) = low;
+    });
+    for (int i = tid; i < CH_TOKENS * CH_COLS / 2; i += 128) {  // decay^(n-1-j) v_j
+      const int j = i / (CH_COLS / 2), at = j * CH_PITCH + (i % (CH_COLS / 2)) * 4;
+      const uint32_t v = *reinterpret_cast<const uint32_t*>(generic + sV + buf * CH_TOKENS * CH_PITCH + at);
+      const float f = j < n ? power[n - 1 - j] : 0.f;
+      uint32_t high, low;
+      split_bf16x2(f * bf16_bits_to_float(v & 0xffffu), f * bf16_bits_to_float(v >> 16), high, low);
+      *reinterpret_cast<uint32_t*>(generic + sW + at) = high;
+      *reinterpret_cast<uint32_t*>(generic + sW + CH_TOKENS * CH_PITCH + at) = low;
+    }
+    __syncthreads();
+
+    const uint32_t q = sQ + buf * CH_TOKENS * pitch, k = sK + buf * CH_TOKENS * pitch, v = sV + buf * CH_TOKENS * CH_PITCH;
+    const int i0 = 16 * warp, row0 = i0 + (lane >> 2);  // this warp's tokens; this thread's are row0 and row0 + 8
+    if (i0 < n) {
+      float o[CH_COLS / 8][4];
+#pragma unroll
+      for (int d = 0; d < CH_COLS / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
+      for (int kt = 0; kt < dim / 16; ++kt) {  // S^T q
+        uint32_t qa[4];
+        ldmatrix_x4(q + (i0 + (m & 1) * 8 + m_row) * pitch + (2 * kt + (m >> 1)) * 16, qa);
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int d = 0; d < CH_COLS / 8; d += 2) {
+            uint32_t b[4];
+            ldmatrix_x4_trans(sS + (part * dim + kt * 16 + (m & 1) * 8 + m_row) * CH_PITCH + (d + (m >> 1)) * 16, b);
+            mma_bf16(o[d], qa, b[0], b[1]);
+            mma_bf16(o[d + 1], qa, b[2], b[3]);
+          }
+      }
+#pragma unroll
+      for (int d = 0; d < CH_COLS / 8; ++d) {
+        o[d][0] *= power[row0 + 1], o[d][1] *= power[row0 + 1];
+        o[d][2] *= power[row0 + 9], o[d][3] *= power[row0 + 9];
+      }
+      for (int js = 0; js <= warp; ++js) {  // 16 earlier tokens at a time (the last 16: this warp's own)
+        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        for (int kt = 0; kt < dim / 16; ++kt) {
+          uint32_t qa[4], b[4];
+          ldmatrix_x4(q + (i0 + (m & 1) * 8 + m_row) * pitch + (2 * kt + (m >> 1)) * 16, qa);
+          ldmatrix_x4(k + (16 * js + (m >> 1) * 8 + m_row) * pitch + (2 * kt + (m & 1)) * 16, b);
+          mma_bf16(s[0], qa, b[0], b[1]);
+          mma_bf16(s[1], qa, b[2], b[3]);
+        }
+        uint32_t high[4], low[4];
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+          for (int g = 0; g < 2; ++g) {
+            const int i = row0 + 8 * g, j = 16 * js + nt * 8 + (lane & 3) * 2;
+            const float x = j <= i ? s[nt][2 * g] * power[i - j] : 0.f, y = j + 1 <= i ? s[nt][2 * g + 1] * power[i - j - 1] : 0.f;
+            split_bf16x2(x, y, high[2 * nt + g], low[2 * nt + g]);
+          }
+#pragma unroll
+        for (int d = 0; d < CH_COLS / 8; d += 2) {
+          uint32_t b[4];
+          ldmatrix_x4_trans(v + (16 * js + (m & 1) * 8 + m_row) * CH_PITCH + (d + (m >> 1)) * 16, b);
+          mma_bf16(o[d], high, b[0], b[1]);
+          mma_bf16(o[d], low, b[0], b[1]);
+          mma_bf16(o[d + 1], high, b[2], b[3]);
+          mma_bf16(o[d + 1], low, b[2], b[3]);
+        }
+      }
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        const int i = row0 + 8 * g;
+        float* out = a.out + (t0 + c * CH_TOKENS + i) * a.ld_o + (int64_t)h * a.vdim + v0;
+#pragma unroll
+        for (int d = 0; d < CH_COLS / 8; ++d) {
+          const int col = d * 8 + (lane & 3) * 2;
+          if (i < n && v0 + col < a.vdim) *reinterpret_cast<float2*>(out + col) = make_float2(o[d][2 * g], o[d][2 * g + 1]);
+        }
+      }
+    }
+    // the state after the chunk
+#pragma unroll
+    for (int i = 0; i < TILES; ++i) {
+      const int tile = warp + 4 * i;
+      if (16 * tile >= dim) continue;
+#pragma unroll
+      for (int d = 0; d < CH_COLS / 8; ++d)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[i][d][e] *= power[n];
+      for (int js = 0; js < (n + 15) / 16; ++js) {
+        uint32_t ka[4];
+        ldmatrix_x4_trans(k + (16 * js + (m >> 1) * 8 + m_row) * pitch + (2 * tile + (m & 1)) * 16, ka);
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int d = 0; d < CH_COLS / 8; d += 2) {
+            uint32_t b[4];
+            ldmatrix_x4_trans(sW + (part * CH_TOKENS + 16 * js + (m & 1) * 8 + m_row) * CH_PITCH + (d + (m >> 1)) * 16, b);
+            mma_bf16(S[i][d], ka, b[0], b[1]);
+            mma_bf16(S[i][d + 1], ka, b[2], b[3]);
+          }
+      }
+    }
+  }
+  each_state([&](float& x, float& y, int row, int col) {
+    if (v0 + col < a.vdim) *reinterpret_cast<float2*>(state + (int64_t)row * a.vdim + v0 + col) = make_float2(x, y);
+  });
+}
+
+static size_t chunk_smem_bytes(int dim) {
+  return 4 * (size_t)CH_TOKENS * (dim * 2 + 16) + 4 * (size_t)CH_TOKENS * CH_PITCH + 2 * (size_t)dim * CH_PITCH;
+}
+
+template <int TILES>
+static int launch_chunks(const ScanArgs& a, int64_t sequences, cudaStream_t s) {
+  static std::atomic<uint64_t> opted{0};
+  if (first_on_device(opted)) cudaFuncSetAttribute(decay_chunk_kernel<TILES>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+  decay_chunk_kernel<TILES><<<dim3((unsigned)ceil_div(a.vdim, CH_COLS), (unsigned)a.heads, (unsigned)sequences), 128, chunk_smem_bytes(a.dim), s>>>(a);
+  return launch_status("fb_decay_scan (chunks)");
+}
+
 template <typename Act>
 __global__ void __launch_bounds__(256) gated_rmsnorm_kernel(const float* x, int64_t ldx, const void* gate, int64_t ld_g, const float* w, float eps,
                                                             int64_t cols, void* out, int64_t ldo) {
@@ -106,6 +305,12 @@ extern "C" int fb_decay_scan(int dtype, const void* qkv, int64_t ld, int heads, 
   FB_REQUIRE(ld >= (int64_t)heads * (2 * dim + vdim) && ld_o >= (int64_t)heads * vdim && state_stride >= (int64_t)heads * dim * vdim && sequences <= 65535 && heads <= 65535,
              "fb_decay_scan: row strides too small");
   fb::ScanArgs a{qkv, ld, heads, dim, vdim, decay, places, dead, tokens, state, state_stride, out, ld_o};
+  // (a few tokens are done sooner one by one)
+  if (dtype == FB_BF16 && tokens >= 16 && dead < 0 && dim % 16 == 0 && dim <= 256 && vdim % 8 == 0 && ld % 8 == 0 && ld_o % 2 == 0 && state_stride % 2 == 0 &&
+      (uintptr_t)qkv % 16 == 0 && (uintptr_t)state % 8 == 0 && (uintptr_t)out % 8 == 0) {
+    const auto s = (cudaStream_t)stream;
+    return dim <= 64 ? fb::launch_chunks<1>(a, sequences, s) : dim <= 128 ? fb::launch_chunks<2>(a, sequences, s) : fb::launch_chunks<4>(a, sequences, s);
+  }
   const int groups = (dim + fb::SCAN_ROWS - 1) / fb::SCAN_ROWS;
   const dim3 grid((unsigned)fb::ceil_div(vdim, 32), (unsigned)heads, (unsigned)sequences);
   const size_t smem = (2 * (size_t)dim + 2 * groups * 32) * sizeof(float);
