@@ -3,6 +3,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--workload llama8b|smollm] [--layers L] [--impl reference]
     python bench.py --matmul 32,4096,14336,bfp8,6      (one isolated matmul, a few calls: what the ncu captures run)
     python bench.py --attend 32,32,8,128,2048,6        (the decode attention alone, likewise)
+    python bench.py --design binutar                   (prefill, decode and kernels of that design beside the Llama decoder)
 
 The default workload is the Llama-3.1-8B-shape batched decode (32 sequences, 2048 tokens of context each, bfp8 weights,
 bf16 KV cache), tensor-parallel over N GPUs with an NCCL all-reduce after o_proj and down_proj.  A step is one decode
@@ -63,6 +64,8 @@ def parse():
     ap.add_argument("--sweep", type=int, default=1, help="0: leave the isolated matmul sweep out of the line (a profiling run)")
     ap.add_argument("--attend", default="", help="T,H,KV,hd,context[,calls]: only the decode attention, e.g. 32,32,8,128,2048,6")
     ap.add_argument("--matmul", default="", help="M,K,N,fmt[,calls]: only that isolated matmul (RMSNorm + SwiGLU fused), e.g. 32,4096,14336,bfp8,6")
+    ap.add_argument("--design", default="", help="binutar[:SIZE]: instead of the workload, prefill and decode of that design at sizes like a real model's layers, "
+                                                 "and each of its kernels, beside the Llama decoder at equal size (one GPU)")
     return ap.parse_args()
 
 
@@ -407,6 +410,259 @@ def one_attention(spec):
     print(json.dumps({"attend": spec, "calls": calls, "us_per_call_eager": e0.elapsed_time(e1) * 1e3 / calls, "kv_bytes_per_call": kv_bytes}))
 
 
+# layers of the sizes real models have, latent and linear mixers in turn, a Llama-like decoder of the same width, depth and MLP
+# beside each (its attention at that width's usual head counts)
+DESIGN_SIZES = {
+    "4096": dict(width=4096, layers=8, ff=14336, vocab=32000, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=1536, kv=8),
+    "2560": dict(width=2560, layers=8, ff=6400, vocab=32000, heads=32, dim=64, rot_dim=32, vdim=64, kv_rank=256, q_rank=768, kv=8),
+}
+
+
+def design_models(s, places):
+    """(Binutar config, Llama config) of one size."""
+    from ferrite_b200 import binutar, llama
+    rot = dict(base=10000.0, dims=s["rot_dim"], scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0))
+    latent = dict(heads=s["heads"], dim=s["dim"], rot_dim=s["rot_dim"], vdim=s["vdim"], kv_rank=s["kv_rank"], q_rank=s["q_rank"], rot=rot, scale=(s["dim"] + s["rot_dim"]) ** -0.5)
+    linear = dict(heads=s["heads"], dim=s["dim"], vdim=s["vdim"], decay=[1 - 2.0 ** -(2 + 6 * h / s["heads"]) for h in range(s["heads"])])
+    mlp = dict(kind="dense", ff=s["ff"], limit=7.0)
+    blocks = [dict(type="lightning", mixer=linear, mlp=mlp) if i % 2 else dict(type="latent_attention", mixer=latent, mlp=mlp) for i in range(s["layers"])]
+    return (binutar.model(vocab=s["vocab"], dim=s["width"], eps=1e-5, blocks=blocks, places=places),
+            llama.model(dim=s["width"], heads=s["heads"], kv=s["kv"], head_dim=128 if s["dim"] == 128 else 64, layers=s["layers"], vocab=s["vocab"], ffn=s["ff"], theta=10000.0,
+                        eps=1e-5, places=places))
+
+
+def timed(calls, copies, call):
+    """Microseconds of call(i), i running round `copies` sets of inputs, from a replayed graph of `calls` of them."""
+    import torch
+    for i in range(3):
+        call(i % copies)
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for i in range(calls):
+            call(i % copies)
+    best = 1e30
+    for _ in range(3):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        graph.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        best = min(best, e0.elapsed_time(e1) * 1e3 / calls)
+    return best
+
+
+def design_steps(rt, c, prec, S, ctx, prompt, steps):
+    """Decode of S sequences at ctx tokens each (a recorded step, picks fed back on the device) and one sequence's prompt."""
+    import torch
+    from ferrite_b200 import llama, models
+    from ferrite_b200.tensor import Tensor, jit
+    family = models.of(c)
+    w = family.random_weights(rt, c, prec)
+    part = ctx + 64 + steps
+    part += -part % 64
+    kv = family.kv_cache(c, S * part, llama.zeros(rt), S)
+    gen = torch.Generator(device=rt.device).manual_seed(1)
+    for t in kv:  # (what the prompts would have left)
+        t.buf.normal_(0, 1, generator=gen)
+    on = lambda row: Tensor.of(rt, [row], "int32")
+    step = jit(lambda ids, at: llama.next_tokens(family.forward(ids, at, w, c, kv, S), c))
+    ids, one = on([1] * S), Tensor.of(rt, [[1] * S], "int32")
+    bump = jit(lambda p: p + one)
+    at = on([ctx] * S)
+    before = rt.launches
+    for i in range(4):
+        out = step(ids, at)
+        ids.buf.copy_(out.buf)
+        at = bump(at)
+        if i == 0:
+            names = rt.profile(before)
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(steps):
+        out = step(ids, at)
+        ids.buf.copy_(out.buf)
+        at = bump(at)
+    e1.record()
+    torch.cuda.synchronize()
+    ms = e0.elapsed_time(e1) / steps
+    rows = {"decode": {"sequences": S, "context": ctx, "ms_per_step": ms, "tokens/s": 1e3 * S / ms, "launches": dict(names)}, "prefill": []}
+    alone = family.kv_cache(c, prompt + 64, llama.zeros(rt), 1)
+    tokens = [int(v) for v in np.random.default_rng(0).integers(0, c.vocab, prompt)]
+    for chunk in (prompt, 512, 128):
+        tries = []
+        for _ in range(3):
+            torch.cuda.synchronize()
+            e0.record()
+            llama.next_tokens(llama.prefill(tokens, w, c, alone, chunk, on), c)
+            e1.record()
+            torch.cuda.synchronize()
+            tries.append(e0.elapsed_time(e1))
+        rows["prefill"].append({"prompt": prompt, "chunk": chunk, "ms": min(tries), "tokens/s": 1e3 * prompt / min(tries)})
+    rt.wait()
+    return rows
+
+
+def design_kernels(rt, s, T, ctx, peaks):
+    """Each kernel of a layer at T tokens - a decode step of T sequences, or (ctx 0) a prompt of T tokens - alone, over inputs that
+    together exceed L2, with the part of its roofline that it reaches: bytes by the measured copy bandwidth or products by the
+    measured bf16 rate, whichever takes longer.  Then the Llama decoder's like kernels."""
+    import torch
+    from ferrite_b200 import _lib, ops
+    dev, gen = rt.device, torch.Generator(device=rt.device).manual_seed(0)
+    bf = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.float32).normal_(0, 1, generator=gen).bfloat16()
+    f32 = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.float32).normal_(0, 1, generator=gen)
+    rows, prompt = [], ctx == 0
+    d, H, dim, rd, vd, rank, qr, ff = (s[k] for k in ("width", "heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank", "ff"))
+
+    def row(name, us, nbytes, flops=0.0, like=None):
+        floor = max(nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6)
+        rows.append({"kernel": name, "us": round(us, 2), "roofline_us": round(floor, 2), "frac": round(floor / us, 3)} | ({"like": like} if like else {}))
+
+    def dense(name, K, N, batch=1, kind=_lib.DENSE_NONE, out_dtype=torch.bfloat16, like="fb_linear"):
+        copies = max(1, min(16, int(3e8 // (2 * batch * K * N))))
+        ws = [bf(batch, N, K) for _ in range(copies)]
+        x = bf(T, batch, K).permute(1, 0, 2)
+        cols = N // 2 if kind == _lib.DENSE_GLU else N
+        out = torch.empty(T, batch, cols, device=dev, dtype=out_dtype).permute(1, 0, 2)
+        v, extra, more = f32(N), {}, 0
+        if kind == _lib.DENSE_SILU:
+            extra = dict(act_cols=N // 2)
+        if kind == _lib.DENSE_GLU:
+            extra = dict(limit=7.0, slope=1.702)
+        if kind == _lib.DENSE_GATE:
+            g = f32(T, batch)
+            extra = dict(gate=g.data_ptr(), ld_gate=batch)
+        if kind == _lib.DENSE_DYT_ADD:
+            res, h = f32(T, N), bf(T, N)
+            extra = dict(residual=res.data_ptr(), ld_residual=N, alpha=v.data_ptr(), w=v.data_ptr(), b=v.data_ptr(), h_out=h.data_ptr(), ld_h=N, alpha2=v.data_ptr(),
+                         w2=v.data_ptr(), b2=v.data_ptr())
+            more = 6 * T * N
+        us = timed(40, copies, lambda i: ops.dense(x, ws[i].transpose(1, 2), out, True, kind, **extra))
+        row(f"fb_dense {name} {batch}x[{K}, {N}]" if batch > 1 else f"fb_dense {name} [{K}, {N}]", us,
+            2 * batch * K * N + 2 * T * batch * K + out.element_size() * T * batch * cols + more, 2.0 * T * batch * K * N, like)
+
+    dense("in", d, qr + rank + rd + H, out_dtype=torch.float32)
+    dense("uq", qr, H * (dim + rd))
+    dense("uk by head", dim, rank, H)
+    dense("uv by head, gate", rank, vd, H, _lib.DENSE_GATE)
+    dense("o, dyt, add, dyt", H * vd, d, 1, _lib.DENSE_DYT_ADD, torch.float32)
+    dense("qkvg, silu", d, 2 * H * (dim + vd), 1, _lib.DENSE_SILU)
+    dense("gate_up, clamped unit", d, 2 * ff, 1, _lib.DENSE_GLU)
+    dense("down, dyt, add, dyt", ff, d, 1, _lib.DENSE_DYT_ADD, torch.float32)
+    dense("head", d, s["vocab"], out_dtype=torch.float32)
+
+    W, keys = rank + rd, T if prompt else ctx
+    part = keys + -keys % 64
+    caches = [bf((1 if prompt else T) * part, W) for _ in range(4)]
+    q, o, sink = bf(T, H * W), torch.empty(T, H * rank, device=dev, dtype=torch.bfloat16), f32(H)
+    base = torch.arange(T, device=dev, dtype=torch.int32) * part
+    last = torch.arange(T, device=dev, dtype=torch.int32) if prompt else torch.full((T,), ctx - 1, device=dev, dtype=torch.int32)
+    pairs = T * (T + 1) / 2 if prompt else T * ctx
+    us = timed(20, 4, lambda i: ops.latent_attention(q, caches[i], None if prompt else base, last, H, rank, 0.1, sink, keys, prompt, out=o))
+    row("fb_latent_attention", us, 2 * ((1 if prompt else T) * keys * W + T * H * (W + rank)), 2.0 * pairs * H * (W + rank), "attention")
+    if prompt:  # (the same attention with keys and values made first: fewer products, and what a kernel of that form would be held to)
+        row("fb_latent_attention, counted as keys and values of a head", us, 0, 2.0 * pairs * H * (dim + rd + vd), "attention")
+
+    down, places = f32(T, qr + W + H), last if prompt else torch.full((T,), ctx - 1, device=dev, dtype=torch.int32)
+    at, freq, cq = (places if prompt else base + places), torch.ones(rd // 2, device=dev, dtype=torch.float64), bf(T, qr)
+    us = timed(40, 1, lambda i: ops.latent_put(down, qr, rank, rd, rd, f32_ones(dev, qr), f32_ones(dev, rank), 1e-5, freq, 1.0, places, at, caches[0], cq))
+    row("fb_latent_put", us, T * (qr + W) * 6, like="fb_rope_kv_write")
+    qh, q3 = bf(T, H, dim + rd), q.view(T, H, W).permute(1, 0, 2)
+    us = timed(40, 1, lambda i: ops.rotate_pairs(qh.permute(1, 0, 2)[:, :, dim:], (freq, rd, 1.0), places, q3[:, :, rank:]))
+    row("fb_rotate_pairs", us, 4 * T * H * rd, like="fb_rope_kv_write")
+
+    n = 2 * H * (dim + vd)
+    qkvg, out, decay = bf(T, n), f32(T, H * vd), torch.full((H,), 0.95, device=dev)
+    states = [f32(1 if prompt else T, H * dim, vd) for _ in range(1 if prompt else 4)]
+    us = timed(20, len(states), lambda i: ops.decay_scan(qkvg, H, dim, vd, decay, places, -1 if prompt else keys + 9, states[i], out))
+    row("fb_decay_scan", us, T * H * (2 * (2 * dim + vd) + 4 * vd) + (1 if prompt else T) * H * dim * vd * 8, 2.0 * T * H * 2 * dim * vd)
+    g, h = qkvg[:, n - H * vd:], bf(T, H * vd)
+    us = timed(40, 1, lambda i: ops.gated_rmsnorm(out, g, f32_ones(dev, H * vd), 1e-5, h))
+    row("fb_gated_rmsnorm", us, T * H * vd * 8, like="fb_rmsnorm")
+    return rows
+
+
+_ONES = {}
+
+
+def f32_ones(dev, n):
+    import torch
+    if (dev, n) not in _ONES:
+        _ONES[dev, n] = torch.ones(n, device=dev)
+    return _ONES[dev, n]
+
+
+def llama_kernels(rt, s, T, ctx, peaks):
+    """The Llama decoder's kernels at the same size (bfp8 weights, as it serves them), likewise."""
+    import torch
+    from ferrite_b200 import ops
+    dev, gen = rt.device, torch.Generator(device=rt.device).manual_seed(0)
+    bf = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.float32).normal_(0, 1, generator=gen).bfloat16()
+    rows, prompt = [], ctx == 0
+    d, H, KV, ff, hd = s["width"], s["heads"], s["kv"], s["ff"], 128 if s["dim"] == 128 else 64
+
+    def row(name, us, nbytes, flops=0.0):
+        floor = max(nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6)
+        rows.append({"kernel": name, "us": round(us, 2), "roofline_us": round(floor, 2), "frac": round(floor / us, 3)})
+
+    for name, K, N, epilogue, norm in (("qkv, rms", d, (H + 2 * KV) * hd, "none", True), ("o, add", H * hd, d, "residual", False), ("gate_up, rms, swiglu", d, 2 * ff, "swiglu", True),
+                                       ("down, add", ff, d, "residual", False), ("head, rms", d, s["vocab"], "none", True)):
+        copies = max(1, min(16, int(3e8 // (1.0625 * K * N))))
+        ws = [ops.quantize(bf(K, N), "bfp8") for _ in range(copies)]
+        x, g, res = bf(T, K), bf(K), bf(T, N)
+        cols = N // 2 if epilogue == "swiglu" else N
+        out = torch.empty(T, cols, device=dev, dtype=torch.bfloat16)
+        us = timed(40 if not prompt else 8, copies, lambda i: ops.linear(x, ws[i], out=out, norm_w=g if norm else None, epilogue=epilogue, residual=res if epilogue == "residual" else None))
+        row(f"fb_linear bfp8 {name} [{K}, {N}]", us, 1.0625 * K * N + 2 * T * K + 2 * T * cols + (2 * T * N if epilogue == "residual" else 0), 2.0 * T * K * N)
+    keys = T if prompt else ctx
+    part = keys + -keys % 64
+    caches = [bf(2 * KV, (1 if prompt else T) * part, hd) for _ in range(4)]
+    q, o = bf(T, H * hd), torch.empty(T, H * hd, device=dev, dtype=torch.bfloat16)
+    base = torch.arange(T, device=dev, dtype=torch.int32) * part
+    last = torch.arange(T, device=dev, dtype=torch.int32) if prompt else torch.full((T,), ctx - 1, device=dev, dtype=torch.int32)
+    pairs = T * (T + 1) / 2 if prompt else T * ctx
+    if prompt:
+        us = timed(8, 4, lambda i: ops.prefill_attention(q, caches[i], 0, last, H, KV, hd, keys, out=o))
+    else:
+        us = timed(20, 4, lambda i: ops.decode_attention(q, caches[i], base, last, H, KV, hd, keys, out=o))
+    row("fb_prefill_attention" if prompt else "fb_decode_attention", us, 2 * ((1 if prompt else T) * keys * 2 * KV * hd + 2 * T * H * hd), 4.0 * pairs * H * hd)
+    qkv, cos = bf(T, (H + 2 * KV) * hd), bf(keys + 1, hd)
+    at = last if prompt else base + last
+    us = timed(40, 1, lambda i: ops.rope_kv_write(qkv, cos, cos, last, at, caches[0], H, KV, hd, q_out=q))
+    row("fb_rope_kv_write", us, 4 * T * (H + 2 * KV) * hd)
+    x, g = bf(T, d), bf(d)
+    us = timed(40, 1, lambda i: ops.rmsnorm(x, g, 1e-5, out=o[:, :d] if H * hd >= d else None))
+    row("fb_rmsnorm", us, 4 * T * d)
+    return rows
+
+
+def run_design(args):
+    """--design: one JSON line a size."""
+    import torch
+    from ferrite_b200 import binutar, llama
+    from ferrite_b200.tensor import Runtime
+    name, _, size = args.design.partition(":")
+    assert name == "binutar" and args.gpus == 1, "--design binutar[:SIZE], one GPU"
+    rt, (peaks, kind) = Runtime(0), measured_peaks()
+    S, ctx, prompt = 32, 2048, 2048
+    for key in [size] if size else DESIGN_SIZES:
+        s = DESIGN_SIZES[key]
+        clocks = Clocks(0)
+        clocks.start()
+        line = {"design": name, "size": key, "shape": s, "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "source": kind}, "weights": "random"}
+        b, l = design_models(s, ctx + 256)
+        line["binutar bf16"] = design_steps(rt, b, binutar.precision(b, "bf16"), S, ctx, prompt, args.steps)
+        line["binutar bfp8"] = design_steps(rt, b, binutar.precision(b, "bfp8"), S, ctx, prompt, args.steps)
+        line["llama bfp8"] = design_steps(rt, l, llama.precision(l, "bfp8"), S, ctx, prompt, args.steps)
+        for what, T, at in (("decode", S, ctx), ("prefill", prompt, 0)):
+            line["kernels " + what] = {"binutar": design_kernels(rt, s, T, at, peaks), "llama": llama_kernels(rt, s, T, at, peaks)}
+            torch.cuda.empty_cache()
+        line["clocks"] = clocks.summary()
+        print(json.dumps(line), flush=True)
+
+
 def matmul_sweep(device, peak_gbs, calls=200):
     """the isolated block-float matmul, RMSNorm prologue and SwiGLU epilogue fused, K = 4096,
     M in {1, 8, 32, 128}, N in {4096, 14336}, bfp8 and bfp4.  `calls` back-to-back calls (one recorded graph) rotate
@@ -557,5 +813,7 @@ if __name__ == "__main__":
         one_matmul(a.matmul)
     elif a.attend:
         one_attention(a.attend)
+    elif a.design:
+        run_design(a)
     else:
         run_reference(a) if a.impl == "reference" else run_ferrite(a)

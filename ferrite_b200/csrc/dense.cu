@@ -52,17 +52,33 @@ __device__ __forceinline__ DenseTile tile_of(const DenseParams& p, int id) {  //
   return {id % p.tiles_m, rest % p.tiles_n, rest / p.tiles_n};
 }
 
+// what the epilogue needs of a column, read once a tile
+struct Column {
+  float alpha, w, b, alpha2, w2, b2;
+};
+template <int EPI>
+__device__ __forceinline__ Column column_of(const DenseParams& p, int64_t n, bool live) {
+  Column c{};
+  if constexpr (EPI == FB_DENSE_DYT_ADD) {
+    if (live) {
+      c.alpha = *p.e.alpha, c.w = p.e.w[n], c.b = p.e.b[n];
+      if (p.e.h_out) c.alpha2 = *p.e.alpha2, c.w2 = p.e.w2[n], c.b2 = p.e.b2[n];
+    }
+  }
+  return c;
+}
+
 // one value of the result: column n of token t (GLU: v the gate, up its partner); the caller has checked the bounds
 template <int EPI>
-__device__ __forceinline__ void emit(const DenseParams& p, int b, int64_t t, int64_t n, float v, float up, float res, float gate) {
+__device__ __forceinline__ void emit(const DenseParams& p, const Column& c, int b, int64_t t, int64_t n, float v, float up, float res, float gate) {
   if constexpr (EPI == FB_DENSE_DYT_ADD) {
-    const float x = res + (tanhf(*p.e.alpha * v) * p.e.w[n] + p.e.b[n]);
+    const float x = res + fmaf(tanh_of(c.alpha * v), c.w, c.b);
     static_cast<float*>(p.out)[t * p.ldo + n] = x;
-    if (p.e.h_out) static_cast<uint16_t*>(p.e.h_out)[t * p.e.ld_h + n] = (uint16_t)float_to_bf16_bits(tanhf(*p.e.alpha2 * x) * p.e.w2[n] + p.e.b2[n]);
+    if (p.e.h_out) static_cast<uint16_t*>(p.e.h_out)[t * p.e.ld_h + n] = (uint16_t)float_to_bf16_bits(fmaf(tanh_of(c.alpha2 * x), c.w2, c.b2));
     return;
   }
   if constexpr (EPI == FB_DENSE_SILU) {
-    if (n < p.e.act_cols) v = v / (1.f + __expf(-v));
+    if (n < p.e.act_cols) v = __fdividef(v, 1.f + __expf(-v));
   }
   if constexpr (EPI == FB_DENSE_GLU) {
     const float g = fminf(v, p.e.limit), u = fminf(fmaxf(up, -p.e.limit), p.e.limit);
@@ -176,6 +192,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
       } else {
         const int64_t col = EPI == FB_DENSE_GLU ? 64 * (int64_t)t.n + 16 * q + (lane & 15) : 128 * (int64_t)t.n + row;
         const bool live = col < (EPI == FB_DENSE_GLU ? p.N / 2 : p.N);
+        const Column mine = column_of<EPI>(p, col, live);
         for (int c = 0; c < half && t0 + c < p.M; c += 8) {
           float v[8], extra[8];
           tmem_ld8_nowait(acc + c, v);
@@ -195,15 +212,15 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
             for (int e = 0; e < 4; ++e) {
               const float got = __shfl_xor_sync(0xffffffffu, high ? v[e] : v[e + 4], 16);
               const int64_t tt = t0 + c + e + (high ? 4 : 0);
-              if (tt < p.M && live) emit<EPI>(p, t.b, tt, col, high ? got : v[e], high ? v[e + 4] : got, 0.f, 0.f);
+              if (tt < p.M && live) emit<EPI>(p, mine, t.b, tt, col, high ? got : v[e], high ? v[e + 4] : got, 0.f, 0.f);
             }
           } else {
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
               const int64_t tt = t0 + c + e;
               if (tt < p.M && live) {
-                if constexpr (EPI == FB_DENSE_GATE) emit<EPI>(p, t.b, tt, col, v[e], 0.f, 0.f, 1.f / (1.f + __expf(-extra[e])));
-                else emit<EPI>(p, t.b, tt, col, v[e], 0.f, EPI == FB_DENSE_DYT_ADD ? extra[e] : 0.f, 0.f);
+                if constexpr (EPI == FB_DENSE_GATE) emit<EPI>(p, mine, t.b, tt, col, v[e], 0.f, 0.f, 1.f / (1.f + __expf(-extra[e])));
+                else emit<EPI>(p, mine, t.b, tt, col, v[e], 0.f, EPI == FB_DENSE_DYT_ADD ? extra[e] : 0.f, 0.f);
               }
             }
           }
@@ -224,6 +241,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
       const int row = tid & 127;
       const int64_t col = EPI == FB_DENSE_GLU ? 64 * (int64_t)t.n + (row >> 5) * 16 + (row & 15) : 128 * (int64_t)t.n + row;
       const bool live = col < (EPI == FB_DENSE_GLU ? p.N / 2 : p.N) && (EPI != FB_DENSE_GLU || !(row & 16));
+      const Column mine = column_of<EPI>(p, col, live);
       for (int c = first + (tid >> 7); c < last; c += 2) {
         const int64_t tt = (int64_t)nt * t.m + c;
         if (tt >= p.M || !live) continue;
@@ -231,11 +249,18 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
         float v = 0.f, up = 0.f, res = 0.f, gate = 0.f;
         if constexpr (EPI == FB_DENSE_DYT_ADD) res = p.e.residual[tt * p.e.ld_residual + col];
         if constexpr (EPI == FB_DENSE_GATE) gate = 1.f / (1.f + __expf(-p.e.gate[tt * p.e.ld_gate + t.b]));
-        for (int s = 0; s < p.splits; ++s) {
-          v += load_cluster_f32(at, s);
-          if constexpr (EPI == FB_DENSE_GLU) up += load_cluster_f32(at + 64, s);
+        float part[8], upper[8];  // (all on their way before the first is needed)
+#pragma unroll
+        for (int s = 0; s < 8; ++s) {
+          part[s] = upper[s] = 0.f;
+          if (s < p.splits) {
+            part[s] = load_cluster_f32(at, s);
+            if constexpr (EPI == FB_DENSE_GLU) upper[s] = load_cluster_f32(at + 64, s);
+          }
         }
-        emit<EPI>(p, t.b, tt, col, v, up, res, gate);
+#pragma unroll
+        for (int s = 0; s < 8; ++s) v += part[s], up += upper[s];
+        emit<EPI>(p, mine, t.b, tt, col, v, up, res, gate);
       }
     }
     cluster_barrier();  // the others have read what they need of this CTA's shared memory

@@ -9,11 +9,12 @@
 //   sums      O^T [128 columns of the latent, rows] += V^T P^T   the same tile of cache rows as A operand, now with the
 //                                                            latent's columns as lanes; P from shared memory as B
 //
-// so a softmax thread owns a row's 64 scores of a tile outright (tcgen05.ld; no exchange between threads), and the sums of a
+// so a softmax thread owns a row's scores (tcgen05.ld; two threads agree on a row's maximum, nothing else is exchanged), and the sums of a
 // 512-column latent by 64 rows take half of tensor memory.  The sums stand under a reference maximum that moves only when a
 // row's scores outgrow it by a factor of 256; then (rarely after the first tiles) the accumulators are rescaled.
 //
-//   warps 0-3   softmax; rescaling; the result        warp 4   TMA        warp 5   MMAs
+//   warps 0-7   softmax (two warps share 32 rows, half a tile's keys each); rescaling; the result
+//   warp 8      TMA          warp 9   MMAs (written out tile by tile: a loop around each would cost more than the MMA)
 //
 // The ring holds two to four tiles of cache rows.  With three or more the next tile's scores are computed while this
 // tile's softmax runs.  Few row tiles are split along the keys over more CTAs; latent_combine_kernel merges the parts and adds
@@ -26,9 +27,10 @@ namespace fb {
 
 namespace {
 
-constexpr int L_KEYS = 64, L_ROWS = 64, L_WARP_LOAD = 4, L_WARP_MMA = 5, L_THREADS = 6 * 32, L_MAX_BUFS = 4;
+constexpr int L_KEYS = 64, L_ROWS = 64, L_WARP_LOAD = 8, L_WARP_MMA = 9, L_SOFTMAX = 256, L_THREADS = 10 * 32, L_MAX_BUFS = 4;
 constexpr int L_CHUNK = L_KEYS * 128;  // 64 cache rows of 64 columns
 constexpr size_t L_SMEM = 225 * 1024;
+constexpr int L_MAX_CHUNKS = 9, L_MAX_BLOCKS = 4;  // rows of up to 576 columns, latents of up to 512
 constexpr float L_SLACK = 8.f;  // log2 of how far scores may outgrow the reference maximum
 
 enum LatentWait { LW_Q = 401, LW_K_EMPTY, LW_K_FULL, LW_S, LW_P, LW_PV, LW_DRAIN };
@@ -51,13 +53,19 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const float v[16]) {
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-// a barrier of the four softmax warps; true if any of their threads brings a true
+// a barrier of the softmax warps; true if any of their threads brings a true
 __device__ __forceinline__ bool softmax_any(bool mine) {
   uint32_t any;
-  asm volatile("{\n.reg .pred p, q;\nsetp.ne.u32 q, %1, 0;\nbarrier.cta.red.or.aligned.pred p, 1, 128, q;\nselp.u32 %0, 1, 0, p;\n}" : "=r"(any) : "r"((uint32_t)mine) : "memory");
+  asm volatile("{\n.reg .pred p, q;\nsetp.ne.u32 q, %1, 0;\nbarrier.cta.red.or.aligned.pred p, 1, 256, q;\nselp.u32 %0, 1, 0, p;\n}" : "=r"(any) : "r"((uint32_t)mine) : "memory");
   return any != 0;
 }
-__device__ __forceinline__ void softmax_sync() { asm volatile("barrier.cta.sync.aligned 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void softmax_sync() { asm volatile("barrier.cta.sync.aligned 1, 256;" ::: "memory"); }
+
+__device__ __forceinline__ float exp2_fast(float x) {  // (0 from -infinity)
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
 // where a row tile stands: its first (token, head) pair, how many, and the keys it reads
 struct RowTile {
@@ -89,7 +97,7 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(latent_smem) + 1023) & ~uintptr_t(1023));
   __shared__ uint64_t bars[2 * L_MAX_BUFS + 5];
   __shared__ uint32_t tmem_slot[2];  // the allocation's address, the abort flag
-  __shared__ float row_scale[L_ROWS];
+  __shared__ float row_scale[L_ROWS], row_top[2][2][L_ROWS];  // per row: a factor; each half's maximum, two tiles' of them
   uint64_t *k_full = bars, *k_empty = bars + L_MAX_BUFS, *q_full = bars + 2 * L_MAX_BUFS, *s_full = q_full + 1, *p_full = q_full + 3, *pv_done = q_full + 4;
   const uint32_t abort_flag = smem_u32(tmem_slot + 1);
   const LatentArgs& a = p.a;
@@ -102,7 +110,7 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
   if (tid == 0) {
     for (int i = 0; i < NB; ++i) mbar_init(smem_u32(k_full + i), 1), mbar_init(smem_u32(k_empty + i), 1);
     mbar_init(smem_u32(q_full), 1), mbar_init(smem_u32(s_full), 1), mbar_init(smem_u32(s_full + 1), 1);
-    mbar_init(smem_u32(p_full), 4), mbar_init(smem_u32(pv_done), 1);
+    mbar_init(smem_u32(p_full), L_SOFTMAX / 32), mbar_init(smem_u32(pv_done), 1);
     tmem_slot[1] = 0;
     fence_barrier_init();
   }
@@ -150,10 +158,14 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
     auto scores = [&](int t) {
       mbar_wait(smem_u32(k_full + sbuf), sphase, abort_flag, LW_K_FULL);
       tc_fence_after();
-      for (int c = 0; c < C; ++c)
+      const uint64_t dk = dk0 + sbuf * k_tile;
+      const uint32_t to = tS + (t & 1) * L_KEYS;
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk)
-          umma_bf16(tS + (t & 1) * L_KEYS, dq0 + c * q_chunk + 2 * kk, dk0 + sbuf * k_tile + c * k_chunk + 2 * kk, idesc_s, c | kk);
+      for (int c = 0; c < L_MAX_CHUNKS; ++c) {
+        if (c >= C) break;
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) umma_bf16(to, dq0 + c * q_chunk + 2 * kk, dk + c * k_chunk + 2 * kk, idesc_s, c | kk);
+      }
       umma_commit(smem_u32(s_full + (t & 1)));
       if (++sbuf == NB) sbuf = 0, sphase ^= 1;
     };
@@ -164,59 +176,65 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
       if (NB >= 3 && t + 1 < n_tiles) scores(t + 1);
       mbar_wait(smem_u32(p_full), t & 1, abort_flag, LW_P);
       tc_fence_after();
-      for (int b = 0; b < p.blocks; ++b)
+      const uint64_t dv = dv0 + vbuf * k_tile;
+#pragma unroll
+      for (int b = 0; b < L_MAX_BLOCKS; ++b) {
+        if (b >= p.blocks) break;
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk)  // 16 keys each
-          umma_bf16(tO + b * nr, dv0 + vbuf * k_tile + 2 * b * k_chunk + kk * (2048 >> 4), dp + 2 * kk, idesc_o, t | kk);
+          umma_bf16(tO + b * nr, dv + 2 * b * k_chunk + kk * (2048 >> 4), dp + 2 * kk, idesc_o, t | kk);
+      }
       umma_commit(smem_u32(k_empty + vbuf));
       umma_commit(smem_u32(pv_done));
       if (++vbuf == NB) vbuf = 0;
       if (NB < 3 && t + 1 < n_tiles) scores(t + 1);
     }
-  } else if (warp < 4) {
-    const int row = tid;  // lane `row` of the scores
+  } else if (warp < L_SOFTMAX / 32) {
+    const int half = warp >> 2, row = 32 * (warp & 3) + lane;  // lane `row` of the scores, keys 32 half .. of a tile
     const bool live = row < r.rows;
     const int place = live ? a.last[(r.first_row + row) / a.heads] : -1;
-    const uint32_t lanes = (uint32_t)(32 * warp) << 16;
-    float m = -INFINITY, l = 0.f;  // the reference maximum (in units of log2) and the sum under it
+    const uint32_t lanes = (uint32_t)(32 * (warp & 3)) << 16;
+    float m = -INFINITY, l = 0.f;  // the reference maximum (in units of log2) and this half's sum under it
     for (int t = 0; t < n_tiles; ++t) {
       mbar_wait(smem_u32(s_full + (t & 1)), (t >> 1) & 1, abort_flag, LW_S);
       tc_fence_after();
-      float s[L_KEYS];
-      float corr = 1.f;
-      bool moved = false;
-      if (32 * warp < nr) {
-        tmem_ld32_nowait(tS + lanes + (t & 1) * L_KEYS, s);
-        tmem_ld32_nowait(tS + lanes + (t & 1) * L_KEYS + 32, s + 32);
+      float s[32];
+      float top = -INFINITY;
+      if (32 * (warp & 3) < nr) {
+        tmem_ld32_nowait(tS + lanes + (t & 1) * L_KEYS + 32 * half, s);
         tmem_ld_wait();
-        const int seen = min(place, r.keys - 1) + 1 - (first_tile + t) * L_KEYS;  // the tile's first `seen` keys
-        float top = -INFINITY;
+        const int seen = min(place, r.keys - 1) + 1 - (first_tile + t) * L_KEYS - 32 * half;  // the first `seen` of these keys
+        float tops[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        if (__all_sync(0xffffffffu, seen >= 32)) {
 #pragma unroll
-        for (int j = 0; j < L_KEYS; ++j) {
-          s[j] = j < seen ? s[j] * p.scale_log2 : -INFINITY;
-          top = fmaxf(top, s[j]);
+          for (int j = 0; j < 32; ++j) s[j] *= p.scale_log2, tops[j & 3] = fmaxf(tops[j & 3], s[j]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) s[j] = j < seen ? s[j] * p.scale_log2 : -INFINITY, tops[j & 3] = fmaxf(tops[j & 3], s[j]);
         }
-        if (top > m + L_SLACK || (m == -INFINITY && top > m)) {
-          corr = exp2f(m - top);  // (0 from -infinity)
-          m = top, moved = t > 0;
-        }
+        top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
+        if (row < L_ROWS) row_top[t & 1][half][row] = top;
+      }
+      const bool grown = top > m + L_SLACK;  // (from -infinity: anything at all)
+      const bool any = softmax_any(grown);
+      float corr = 1.f;
+      if (row < nr) {
+        top = fmaxf(top, row_top[t & 1][half ^ 1][row]);
+        if (top > m + L_SLACK) corr = exp2_fast(m - top), m = top;
         const float at = m == -INFINITY ? 0.f : m;
-        float sum = 0.f;
+        float sums[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int j = 0; j < L_KEYS; ++j) {
-          s[j] = exp2f(s[j] - at);
-          sum += s[j];
-        }
-        l = l * corr + sum;
+        for (int j = 0; j < 32; ++j) s[j] = exp2_fast(s[j] - at), sums[j & 3] += s[j];
+        l = l * corr + ((sums[0] + sums[1]) + (sums[2] + sums[3]));
       }
       if (t > 0) {  // the sums and P are free once the last tile's MMAs are done
         mbar_wait(smem_u32(pv_done), (t - 1) & 1, abort_flag, LW_PV);
         tc_fence_after();
-      }
-      if (row < L_ROWS) row_scale[row] = corr;
-      if (softmax_any(moved)) {
-        for (int b = 0; b < p.blocks; ++b)
-          for (int c = 0; c < nr; c += 16) {
+        if (any) {
+          if (row < L_ROWS && half == 0) row_scale[row] = corr;
+          softmax_sync();
+          for (int i = half; i < p.blocks * (nr / 16); i += 2) {
+            const int b = i / (nr / 16), c = i % (nr / 16) * 16;
             float v[16];
             tmem_ld16_nowait(tO + lanes + b * nr + c, v);
             tmem_ld_wait();
@@ -224,54 +242,68 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
             for (int e = 0; e < 16; ++e) v[e] *= row_scale[c + e];
             tmem_st16(tO + lanes + b * nr + c, v);
           }
-        tmem_st_wait();
+          tmem_st_wait();
+        }
       }
       if (row < nr) {
 #pragma unroll
-        for (int c = 0; c < 8; ++c)
-          st_shared_v4(sP + row * 128 + ((c ^ (row & 7)) << 4), pack_bf16x2(s[8 * c], s[8 * c + 1]), pack_bf16x2(s[8 * c + 2], s[8 * c + 3]),
+        for (int c = 0; c < 4; ++c)
+          st_shared_v4(sP + row * 128 + (((4 * half + c) ^ (row & 7)) << 4), pack_bf16x2(s[8 * c], s[8 * c + 1]), pack_bf16x2(s[8 * c + 2], s[8 * c + 3]),
                        pack_bf16x2(s[8 * c + 4], s[8 * c + 5]), pack_bf16x2(s[8 * c + 6], s[8 * c + 7]));
       }
       fence_proxy_async();
       tc_fence_before();
-      softmax_sync();  // (row_scale has been read by all before a next tile writes it)
+      __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(p_full));
     }
-    // ---- the result
+    // ---- the result: through the ring's shared memory, from where the tile's rows - one piece of memory - leave in one copy
     if (n_tiles) {
       mbar_wait(smem_u32(pv_done), (n_tiles - 1) & 1, abort_flag, LW_PV);
       tc_fence_after();
     }
+    if (row < L_ROWS && half == 1) row_top[0][1][row] = l;
+    softmax_sync();
     const int64_t part = (int64_t)tile * p.splits + split;
-    if (row < L_ROWS) {
+    if (row < L_ROWS && half == 0) {
+      l += row_top[0][1][row];
+      float f = 1.f;
       if (p.splits > 1) {
         p.part_ml[(part * L_ROWS + row) * 2] = m, p.part_ml[(part * L_ROWS + row) * 2 + 1] = l;
-        row_scale[row] = 1.f;
       } else {
-        float f = 1.f, total = l;
+        float total = l;
         if (a.sink && live) {
           const float sink = a.sink[(r.first_row + row) % a.heads] * 1.4426950408889634f, top = fmaxf(m, sink);
           f = exp2f(m - top), total = l * f + exp2f(sink - top);
         }
-        row_scale[row] = total > 0.f ? f / total : 0.f;
+        f = total > 0.f ? f / total : 0.f;
       }
+      row_scale[row] = f;
     }
     softmax_sync();
-    for (int b = 0; b < p.blocks && (n_tiles || p.splits == 1); ++b) {
-      const int d = 128 * b + tid;
-      for (int c = 0; c < nr && c < r.rows; c += 16) {
+    if (n_tiles || p.splits == 1) {
+      for (int i = half; i < p.blocks * (nr / 16); i += 2) {
+        const int b = i / (nr / 16), c = i % (nr / 16) * 16, d = 128 * b + row;
         float v[16];
         if (n_tiles) {
           tmem_ld16_nowait(tO + lanes + b * nr + c, v);
           tmem_ld_wait();
+        } else {
+#pragma unroll
+          for (int e = 0; e < 16; ++e) v[e] = 0.f;
         }
         if (d >= a.rank) continue;
 #pragma unroll
         for (int e = 0; e < 16; ++e) {
-          if (c + e >= r.rows) break;
-          if (p.splits > 1) p.part_o[(part * L_ROWS + c + e) * a.rank + d] = v[e];
-          else static_cast<uint16_t*>(a.out)[(r.first_row + c + e) * a.rank + d] = (uint16_t)float_to_bf16_bits(n_tiles ? v[e] * row_scale[c + e] : 0.f);
+          const uint32_t at = (uint32_t)((c + e) * a.rank + d);
+          if (p.splits > 1) asm volatile("st.shared.f32 [%0], %1;" ::"r"(sK + at * 4), "f"(v[e]) : "memory");
+          else asm volatile("st.shared.u16 [%0], %1;" ::"r"(sK + at * 2), "h"((uint16_t)float_to_bf16_bits(v[e] * row_scale[c + e])) : "memory");
         }
+      }
+      fence_proxy_async();
+      softmax_sync();
+      if (tid == 0) {
+        if (p.splits > 1) bulk_copy_s2g(p.part_o + part * L_ROWS * a.rank, sK, (uint32_t)(r.rows * a.rank * 4));
+        else bulk_copy_s2g(static_cast<uint16_t*>(a.out) + r.first_row * a.rank, sK, (uint32_t)(r.rows * a.rank * 2));
       }
     }
   }
@@ -316,11 +348,11 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentParams 
 // sizes and launch shape; false: not for this kernel
 bool make_latent_plan(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk, LatentParams& p) {
   const int W = rank + rot;
-  if (W % 8 || rank > 512 || max_keys < 1) return false;
+  if (W % 8 || rank % 8 || W > 64 * L_MAX_CHUNKS || rank > 128 * L_MAX_BLOCKS || max_keys < 1) return false;
   const int64_t rows = chunk ? T * heads : heads;
   p.nr = rows >= L_ROWS ? L_ROWS : (int)ceil_div(rows, 16) * 16;
   p.chunks = (int)ceil_div(W, 64), p.blocks = (int)ceil_div(rank, 128);
-  const size_t fixed = 2048 + (size_t)p.chunks * p.nr * 128 + L_ROWS * 128, tile = (size_t)p.chunks * L_CHUNK;
+  const size_t fixed = 1024 + (size_t)p.chunks * p.nr * 128 + L_ROWS * 128, tile = (size_t)p.chunks * L_CHUNK;
   if (fixed + 2 * tile > L_SMEM) return false;
   p.bufs = (int)((L_SMEM - fixed) / tile);
   p.bufs = p.bufs > L_MAX_BUFS ? L_MAX_BUFS : p.bufs;
@@ -357,7 +389,7 @@ size_t latent_tcgen05_workspace(int64_t T, int heads, int rank, int rot, int64_t
 bool latent_tcgen05_supports(const LatentArgs& a) {
   LatentParams p{};
   return tma_encoder() != nullptr && a.ld_q == (int64_t)a.heads * (a.rank + a.rot) && a.ld_o == (int64_t)a.heads * a.rank && (uintptr_t)a.q % 16 == 0 &&
-         (uintptr_t)a.cache % 16 == 0 && a.cache_rows < (1ll << 31) && a.T * a.heads < (1ll << 31) && make_latent_plan(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, p);
+         (uintptr_t)a.cache % 16 == 0 && (uintptr_t)a.out % 16 == 0 && a.cache_rows < (1ll << 31) && a.T * a.heads < (1ll << 31) && make_latent_plan(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, p);
 }
 
 int latent_tcgen05(const LatentArgs& a, cudaStream_t s) {
@@ -381,7 +413,7 @@ int latent_tcgen05(const LatentArgs& a, cudaStream_t s) {
   if (int rc = tma_map_bf16(&tq, a.q, 2, qd, stride, qb, "fb_latent_attention (queries)")) return rc;
   if (int rc = tma_map_bf16(&tk, a.cache, 2, kd, stride, kb, "fb_latent_attention (cache)")) return rc;
   static std::atomic<uint64_t> opted{0};
-  if (first_on_device(opted)) cudaFuncSetAttribute(latent_tcgen05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+  if (first_on_device(opted)) cudaFuncSetAttribute(latent_tcgen05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)L_SMEM);
   cudaLaunchConfig_t cfg{};
   cfg.gridDim = dim3((unsigned)tiles, (unsigned)p.splits), cfg.blockDim = dim3(L_THREADS), cfg.stream = s;
   cfg.dynamicSmemBytes = 1024 + (size_t)p.chunks * p.nr * 128 + (size_t)p.bufs * p.chunks * L_CHUNK + L_ROWS * 128;

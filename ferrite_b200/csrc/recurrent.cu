@@ -280,19 +280,41 @@ static int launch_chunks(const ScanArgs& a, int64_t sequences, cudaStream_t s) {
   return launch_status("fb_decay_scan (chunks)");
 }
 
+// a block a row; up to NORM_KEPT values a thread stay in registers between the sum and the result
+constexpr int NORM_THREADS = 512, NORM_KEPT = 16;
+
 template <typename Act>
-__global__ void __launch_bounds__(256) gated_rmsnorm_kernel(const float* x, int64_t ldx, const void* gate, int64_t ld_g, const float* w, float eps,
-                                                            int64_t cols, void* out, int64_t ldo) {
+__global__ void __launch_bounds__(NORM_THREADS) gated_rmsnorm_kernel(const float* x, int64_t ldx, const void* gate, int64_t ld_g, const float* w, float eps,
+                                                                     int64_t cols, void* out, int64_t ldo) {
   griddep_launch_dependents();
   griddep_wait();
   __shared__ float red[32];
   const int64_t t = blockIdx.x;
-  float ss = 0.f;
-  for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) ss = fmaf(x[t * ldx + c], x[t * ldx + c], ss);
-  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)cols + eps);
   const Act* g = static_cast<const Act*>(gate) + t * ld_g;
-  for (int64_t c = threadIdx.x; c < cols; c += blockDim.x)
-    store_value(static_cast<Act*>(out) + t * ldo + c, x[t * ldx + c] * r * w[c] * sigmoid_f(value_of(g[c])));
+  Act* o = static_cast<Act*>(out) + t * ldo;
+  x += t * ldx;
+  float v[NORM_KEPT], gw[NORM_KEPT], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NORM_KEPT; ++i) {
+    const int64_t c = threadIdx.x + i * NORM_THREADS;
+    v[i] = gw[i] = 0.f;
+    if (c < cols) v[i] = x[c], gw[i] = value_of(g[c]);
+  }
+#pragma unroll
+  for (int i = 0; i < NORM_KEPT; ++i) ss = fmaf(v[i], v[i], ss);
+  for (int64_t c = threadIdx.x + NORM_KEPT * NORM_THREADS; c < cols; c += NORM_THREADS) ss = fmaf(x[c], x[c], ss);
+#pragma unroll
+  for (int i = 0; i < NORM_KEPT; ++i) {
+    const int64_t c = threadIdx.x + i * NORM_THREADS;
+    if (c < cols) gw[i] = sigmoid_f(gw[i]) * w[c];
+  }
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)cols + eps);
+#pragma unroll
+  for (int i = 0; i < NORM_KEPT; ++i) {
+    const int64_t c = threadIdx.x + i * NORM_THREADS;
+    if (c < cols) store_value(o + c, v[i] * r * gw[i]);
+  }
+  for (int64_t c = threadIdx.x + NORM_KEPT * NORM_THREADS; c < cols; c += NORM_THREADS) store_value(o + c, x[c] * r * w[c] * sigmoid_f(value_of(g[c])));
 }
 
 }  // namespace fb
@@ -323,7 +345,7 @@ extern "C" int fb_gated_rmsnorm(const float* x, int64_t rows, int64_t cols, int6
                                 void* out, int64_t ldo, void* stream) {
   FB_REQUIRE(x && gate && w && out && rows >= 1 && cols >= 1 && ldx >= cols && ld_g >= cols && ldo >= cols, "fb_gated_rmsnorm: bad arguments");
   FB_REQUIRE(dtype == FB_BF16 || dtype == FB_FP32, "fb_gated_rmsnorm: bf16 or fp32");
-  if (dtype == FB_FP32) fb::gated_rmsnorm_kernel<float><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(x, ldx, gate, ld_g, w, eps, cols, out, ldo);
-  else fb::gated_rmsnorm_kernel<uint16_t><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(x, ldx, gate, ld_g, w, eps, cols, out, ldo);
+  if (dtype == FB_FP32) fb::gated_rmsnorm_kernel<float><<<(unsigned)rows, fb::NORM_THREADS, 0, (cudaStream_t)stream>>>(x, ldx, gate, ld_g, w, eps, cols, out, ldo);
+  else fb::gated_rmsnorm_kernel<uint16_t><<<(unsigned)rows, fb::NORM_THREADS, 0, (cudaStream_t)stream>>>(x, ldx, gate, ld_g, w, eps, cols, out, ldo);
   return fb::launch_status("fb_gated_rmsnorm");
 }

@@ -12,6 +12,14 @@ __device__ __forceinline__ void store_value(uint16_t* p, float v) { *p = (uint16
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
+// tanh by one exponential, and by its power series where that would cancel: about 2e-7 of the result either way
+__device__ __forceinline__ float tanh_of(float x) {
+  const float y = x * x;
+  const float near = x * fmaf(y, fmaf(y, fmaf(y, fmaf(y, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
+  const float far = 1.f - __fdividef(2.f, 1.f + __expf(2.f * fminf(fmaxf(x, -15.f), 15.f)));
+  return y < 0.04f ? near : far;
+}
+
 // sum over a block of up to 1024 threads (whole warps); every thread gets it.  `red` is 32 floats of shared memory
 __device__ __forceinline__ float block_sum(float v, float* red) {
   v = warp_sum(v);
