@@ -98,7 +98,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
   __shared__ uint32_t tmem_slot[2];  // the allocation's address, the abort flag
   uint64_t *full = bars, *empty = bars + D_MAX_STAGES, *acc_full = bars + 2 * D_MAX_STAGES, *acc_empty = acc_full + 2;
   const uint32_t abort_flag = smem_u32(tmem_slot + 1);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, warp = uniform_warp(), lane = tid & 31;
   const int S = p.stages, nt = p.nt, stage_bytes = D_A_BYTES + nt * 128;
   const int s0 = blockIdx.y * p.steps_per_split, n_steps = min(p.steps - s0, p.steps_per_split);
 
@@ -151,7 +151,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
         while (i > s && !mbar_try_wait(smem_u32(full + s), parity) && clock64() - start < WAIT_CLOCKS) {
         }
       }
-  } else if (warp == D_WARP_MMA && lane == 0) {
+  } else if (warp == D_WARP_MMA) {
     const uint32_t idesc = umma_idesc_bf16(nt, false, false);
     const uint64_t d0 = umma_smem_desc(smem_u32(smem), 16, 1024);
     int slot = 0, n = 0;
@@ -165,11 +165,11 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
         tc_fence_after();
         const uint64_t da = d0 + (uint32_t)(slot * stage_bytes >> 4), dx = da + (D_A_BYTES >> 4);
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) umma_bf16(acc, da + 2 * kk, dx + 2 * kk, idesc, k | kk);
-        umma_commit(smem_u32(empty + slot));
+        for (int kk = 0; kk < 4; ++kk) umma_bf16_warp(acc, da + 2 * kk, dx + 2 * kk, idesc, k | kk);
+        umma_commit_warp(smem_u32(empty + slot));
         if (++slot == S) slot = 0, phase ^= 1;
       }
-      umma_commit(smem_u32(acc_full + (n & 1)));
+      umma_commit_warp(smem_u32(acc_full + (n & 1)));
     }
   } else if (warp < D_EPI_WARPS) {
     griddep_wait();

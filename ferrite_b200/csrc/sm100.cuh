@@ -130,6 +130,12 @@ __device__ __forceinline__ float load_cluster_f32(uint32_t local_addr, uint32_t 
   return v;
 }
 
+__device__ __forceinline__ void load_cluster_v4(uint32_t local_addr, uint32_t rank, float v[4]) {
+  uint32_t remote;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local_addr), "r"(rank));
+  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v[0]), "=f"(v[1]), "=f"(v[2]), "=f"(v[3]) : "r"(remote) : "memory");
+}
+
 // ---- tensor memory
 __device__ __forceinline__ void tmem_alloc(uint32_t slot_smem, uint32_t cols) {  // whole warp; cols a power of two >= 32
   asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(slot_smem), "r"(cols) : "memory");
@@ -148,6 +154,21 @@ __device__ __forceinline__ void umma_bf16(uint32_t d_tmem, uint64_t a_desc, uint
       "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
+// The same two by a whole warp whose lanes agree: one elected lane issues.  With nothing in the warp diverging the compiler
+// keeps descriptors in uniform registers, where the MMA wants them: 40 cycles an MMA of few columns instead of 53 from a
+// loop that one lane runs alone.
+__device__ __forceinline__ void umma_bf16_warp(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n.reg .pred p, one;\nelect.sync _|one, 0xffffffff;\nsetp.ne.b32 p, %4, 0;\n@one tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}" ::"r"(d_tmem),
+      "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+__device__ __forceinline__ void umma_commit_warp(uint32_t bar) {
+  asm volatile("{\n.reg .pred one;\nelect.sync _|one, 0xffffffff;\n@one tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n}" ::"r"(bar)
+               : "memory");
+}
+// a thread's warp, as a number the compiler knows to be the warp's
+__device__ __forceinline__ int uniform_warp() { return __shfl_sync(0xffffffffu, (int)(threadIdx.x >> 5), 0); }
 // the mbarrier gets one arrival when every MMA issued before this by the thread has finished
 __device__ __forceinline__ void umma_commit(uint32_t bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
