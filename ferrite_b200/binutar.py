@@ -13,7 +13,7 @@ import numpy as np
 import torch
 
 from . import llama, mixers
-from .tensor import Tensor
+from .tensor import BFP, Tensor
 
 REWINDS = False  # a linear mixer's state cannot be taken back to an earlier token: a slot's prefix is reused whole or not at all
 GLU_SLOPE = 1.702
@@ -48,12 +48,24 @@ def config(j, places=4096):
     return model(vocab=j["vocab"], dim=j["width"], eps=j["norm"]["eps"], blocks=j["layers"], places=places)
 
 
+def projections(c, l):
+    """{op: (rows, columns)} of layer l's projections as x @ w takes them."""
+    b, m, d = c.blocks[l], c.blocks[l].mixer, c.dim
+    if b.type == "latent_attention":
+        out = {"in": (d, m.q_rank + m.kv_rank + m.rot_dim + m.heads), "uq": (m.q_rank, m.heads * (m.dim + m.rot_dim))}
+    else:
+        out = {"qkvg": (d, 2 * m.heads * (m.dim + m.vdim))}
+    return out | {"o": (m.heads * m.vdim, d)} | ({"gate_up": (d, 2 * b.mlp.ff), "down": (b.mlp.ff, d)} if b.mlp else {})
+
+
 def precision(c, mode="bf16", kv=None):
     """{(op, block): (format, phases)} as llama.precision's: mode bf16, fp32 (everything in fp32), bfp8 or bfp4 (the block-float
-    formats for the large projections; a head's own matrices, which act on the query and the weighted latents, stay bf16)."""
+    formats for the large projections; a head's own matrices, which act on the query and the weighted latents, stay bf16, and
+    so does a matrix that has no whole runs of 16 columns)."""
     assert kv in (None, "bf16", "fp32"), "the latents are cached as the activations are kept"
-    p = {(op, l): (mode, 4) for l in range(c.layers) for op in ("in", "uq", "o", "qkvg", "gate_up", "down")}
-    p["head", None] = (mode, 4)
+    fmt = lambda k, n: "bf16" if mode in BFP and (n % 16 or k % 4) else mode
+    p = {(op, l): (fmt(*shape), 4) for l in range(c.layers) for op, shape in projections(c, l).items()}
+    p["head", None] = (fmt(c.dim, c.vocab), 4)
     p["act", None] = ("fp32" if mode == "fp32" else "bf16", None)
     return p
 

@@ -335,7 +335,7 @@ extern "C" int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_
   p.splits = 1;
   double best = 1e30;
   for (int s = 1; s <= 8; s *= 2) {
-    if (s > 1 && (p.tiles * s > sms || p.steps < 2 * s)) break;
+    if (s > 1 && (p.tiles * s > (s == 8 ? 128 : sms) || p.steps < 2 * s)) break;  // (one round: clusters of eight leave some SMs unused)
     const int per = (int)ceil_div(p.steps, s);
     if ((int)ceil_div(p.steps, per) != s) continue;
     const double step = 0.12 + 0.001 * p.nt + 0.25 * (double)(p.tiles * s < sms ? p.tiles * s : sms) / sms;  // us: latency-bound at first, then the stream's share

@@ -75,7 +75,7 @@ struct RotateArgs {
 
 // a block per token; the angles are made once and kept in shared memory for all the heads
 template <typename Act>
-__global__ void __launch_bounds__(128) rotate_pairs_kernel(const RotateArgs a) {
+__global__ void __launch_bounds__(512) rotate_pairs_kernel(const RotateArgs a) {
   griddep_launch_dependents();
   griddep_wait();
   extern __shared__ float turns[];  // [dims / 2] cos, [dims / 2] sin
@@ -194,8 +194,8 @@ extern "C" int fb_rotate_pairs(int dtype, const void* x, int64_t T, int heads, i
   FB_REQUIRE(dims >= 0 && dims % 2 == 0 && dims <= width && dims <= 8192, "fb_rotate_pairs: an even number of a head's columns turn");
   FB_REQUIRE(dtype == FB_BF16 || dtype == FB_FP32, "fb_rotate_pairs: bf16 or fp32");
   fb::RotateArgs a{x, x_row, x_head, out, o_row, o_head, heads, width, dims, freq, mag, places};
-  if (dtype == FB_FP32) fb::rotate_pairs_kernel<float><<<(unsigned)T, 128, dims * 4, (cudaStream_t)stream>>>(a);
-  else fb::rotate_pairs_kernel<uint16_t><<<(unsigned)T, 128, dims * 4, (cudaStream_t)stream>>>(a);
+  if (dtype == FB_FP32) fb::rotate_pairs_kernel<float><<<(unsigned)T, 512, dims * 4, (cudaStream_t)stream>>>(a);
+  else fb::rotate_pairs_kernel<uint16_t><<<(unsigned)T, 512, dims * 4, (cudaStream_t)stream>>>(a);
   return fb::launch_status("fb_rotate_pairs");
 }
 
