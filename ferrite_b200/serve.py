@@ -172,11 +172,13 @@ class DeviceBackend:
         self.part, self.rewinds = places, getattr(self.model, "REWINDS", True)
         self.kv = self.model.kv_cache(c, slots * places, llama.zeros(rt), slots)
         self.parts = [self.model.slot(c, self.kv, u, slots) for u in range(slots)]
-        forward = lambda ids, at: self.model.forward(ids, at, weights, c, self.kv, slots).realize()
+        kv, model, pack = self.kv, self.model, self._pack  # (the recorded steps hold these, not the backend: it goes, with its caches, when nobody holds it)
+        forward = lambda ids, at: model.forward(ids, at, weights, c, kv, slots).realize()
         self.logits_step = jit(forward)
-        self.step = jit(lambda ids, at, t: self._pack(heads(forward(ids, at)[0], t)))
+        self.step = jit(lambda ids, at, t: pack(heads(forward(ids, at)[0], t)))
 
-    def _pack(self, h):
+    @staticmethod
+    def _pack(h):
         """values | ids | lse side by side in one fp32 matrix (token ids below 2^24 are exact in fp32): one readback."""
         values, ids, lse = h
         return values.cat(ids.float(), lse, axis=2).realize()

@@ -15,6 +15,7 @@ There is no CPU path: without the CUDA library the import of `_lib` raises.
 `jit` replays a recorded step as one CUDA graph (ferrite/tensor.py:788-810 replays a recorded block of launches).
 """
 import array
+import gc
 import math
 
 import numpy as np
@@ -1154,8 +1155,15 @@ def jit(f):
             inputs = [x.realize() for x in xs]
             torch.cuda.synchronize()
             graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph, capture_error_mode="thread_local"):  # (other threads, NCCL's watchdog, may touch CUDA meanwhile)
-                out = f(*inputs).realize()
+            collects = gc.isenabled()
+            gc.collect()
+            gc.disable()  # (a recording that nobody holds any more may not be taken down while another is made)
+            try:
+                with torch.cuda.graph(graph, capture_error_mode="thread_local"):  # (other threads, NCCL's watchdog, may touch CUDA meanwhile)
+                    out = f(*inputs).realize()
+            finally:
+                if collects:
+                    gc.enable()
             graph.replay()
             state.update(inputs=inputs, graph=graph, out=out)
             return out
