@@ -280,10 +280,29 @@ static int launch_chunks(const ScanArgs& a, int64_t sequences, cudaStream_t s) {
   return launch_status("fb_decay_scan (chunks)");
 }
 
-// a block a row; up to NORM_KEPT values a thread stay in registers between the sum and the result
-constexpr int NORM_THREADS = 512, NORM_KEPT = 16;
+// a block a row.  V: columns a thread takes at once (4 where rows are aligned); up to NORM_KEPT such pieces a thread stay in
+// registers between the sum and the result, a wider row is read again
+constexpr int NORM_THREADS = 256, NORM_KEPT = 4;
 
-template <typename Act>
+__device__ __forceinline__ void load4(const float* p, float v[4]) {
+  const float4 x = *reinterpret_cast<const float4*>(p);
+  v[0] = x.x, v[1] = x.y, v[2] = x.z, v[3] = x.w;
+}
+__device__ __forceinline__ void load4(const uint16_t* p, float v[4]) {
+  const uint2 x = *reinterpret_cast<const uint2*>(p);
+  v[0] = bf16_bits_to_float(x.x & 0xffffu), v[1] = bf16_bits_to_float(x.x >> 16), v[2] = bf16_bits_to_float(x.y & 0xffffu), v[3] = bf16_bits_to_float(x.y >> 16);
+}
+__device__ __forceinline__ void store4(float* p, const float v[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(uint16_t* p, const float v[4]) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]));
+}
+template <int V, typename T>
+__device__ __forceinline__ void load_piece(const T* p, float v[V]) {
+  if constexpr (V == 4) load4(p, v);
+  else v[0] = value_of(*p);
+}
+
+template <typename Act, int V>
 __global__ void __launch_bounds__(NORM_THREADS) gated_rmsnorm_kernel(const float* x, int64_t ldx, const void* gate, int64_t ld_g, const float* w, float eps,
                                                                      int64_t cols, void* out, int64_t ldo) {
   griddep_launch_dependents();
@@ -293,28 +312,44 @@ __global__ void __launch_bounds__(NORM_THREADS) gated_rmsnorm_kernel(const float
   const Act* g = static_cast<const Act*>(gate) + t * ld_g;
   Act* o = static_cast<Act*>(out) + t * ldo;
   x += t * ldx;
-  float v[NORM_KEPT], gw[NORM_KEPT], ss = 0.f;
+  const int64_t c0 = threadIdx.x * V, step = NORM_THREADS * V, kept = NORM_KEPT * step;
+  float v[NORM_KEPT][V], f[NORM_KEPT][V], ss = 0.f;
 #pragma unroll
-  for (int i = 0; i < NORM_KEPT; ++i) {
-    const int64_t c = threadIdx.x + i * NORM_THREADS;
-    v[i] = gw[i] = 0.f;
-    if (c < cols) v[i] = x[c], gw[i] = value_of(g[c]);
-  }
+  for (int i = 0; i < NORM_KEPT; ++i)
+    if (c0 + i * step < cols) load_piece<V>(x + c0 + i * step, v[i]), load_piece<V>(g + c0 + i * step, f[i]);
 #pragma unroll
-  for (int i = 0; i < NORM_KEPT; ++i) ss = fmaf(v[i], v[i], ss);
-  for (int64_t c = threadIdx.x + NORM_KEPT * NORM_THREADS; c < cols; c += NORM_THREADS) ss = fmaf(x[c], x[c], ss);
+  for (int i = 0; i < NORM_KEPT; ++i)
+    if (c0 + i * step < cols) {
+      float ws[V];
+      load_piece<V>(w + c0 + i * step, ws);
 #pragma unroll
-  for (int i = 0; i < NORM_KEPT; ++i) {
-    const int64_t c = threadIdx.x + i * NORM_THREADS;
-    if (c < cols) gw[i] = sigmoid_f(gw[i]) * w[c];
-  }
+      for (int e = 0; e < V; ++e) ss = fmaf(v[i][e], v[i][e], ss), f[i][e] = sigmoid_f(f[i][e]) * ws[e];
+    }
+  for (int64_t c = c0 + kept; c < cols; c += step)
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(x[c + e], x[c + e], ss);
   const float r = 1.f / sqrtf(block_sum(ss, red) / (float)cols + eps);
 #pragma unroll
-  for (int i = 0; i < NORM_KEPT; ++i) {
-    const int64_t c = threadIdx.x + i * NORM_THREADS;
-    if (c < cols) store_value(o + c, v[i] * r * gw[i]);
-  }
-  for (int64_t c = threadIdx.x + NORM_KEPT * NORM_THREADS; c < cols; c += NORM_THREADS) store_value(o + c, x[c] * r * w[c] * sigmoid_f(value_of(g[c])));
+  for (int i = 0; i < NORM_KEPT; ++i)
+    if (c0 + i * step < cols) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) v[i][e] *= r * f[i][e];
+      if constexpr (V == 4) store4(o + c0 + i * step, v[i]);
+      else store_value(o + c0 + i * step, v[i][0]);
+    }
+  for (int64_t c = c0 + kept; c < cols; c += step)
+#pragma unroll
+    for (int e = 0; e < V; ++e) store_value(o + c + e, x[c + e] * r * w[c + e] * sigmoid_f(value_of(g[c + e])));
+}
+
+template <typename Act>
+static int launch_gated_rmsnorm(const float* x, int64_t rows, int64_t cols, int64_t ldx, const void* gate, int64_t ld_g, const float* w, float eps, void* out,
+                                int64_t ldo, cudaStream_t s) {
+  const bool pieces = cols % 4 == 0 && ldx % 4 == 0 && ld_g % 4 == 0 && ldo % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+                      (uintptr_t)gate % (4 * sizeof(Act)) == 0 && (uintptr_t)out % (4 * sizeof(Act)) == 0;
+  if (pieces) gated_rmsnorm_kernel<Act, 4><<<(unsigned)rows, NORM_THREADS, 0, s>>>(x, ldx, gate, ld_g, w, eps, cols, out, ldo);
+  else gated_rmsnorm_kernel<Act, 1><<<(unsigned)rows, NORM_THREADS, 0, s>>>(x, ldx, gate, ld_g, w, eps, cols, out, ldo);
+  return launch_status("fb_gated_rmsnorm");
 }
 
 }  // namespace fb
@@ -345,7 +380,6 @@ extern "C" int fb_gated_rmsnorm(const float* x, int64_t rows, int64_t cols, int6
                                 void* out, int64_t ldo, void* stream) {
   FB_REQUIRE(x && gate && w && out && rows >= 1 && cols >= 1 && ldx >= cols && ld_g >= cols && ldo >= cols, "fb_gated_rmsnorm: bad arguments");
   FB_REQUIRE(dtype == FB_BF16 || dtype == FB_FP32, "fb_gated_rmsnorm: bf16 or fp32");
-  if (dtype == FB_FP32) fb::gated_rmsnorm_kernel<float><<<(unsigned)rows, fb::NORM_THREADS, 0, (cudaStream_t)stream>>>(x, ldx, gate, ld_g, w, eps, cols, out, ldo);
-  else fb::gated_rmsnorm_kernel<uint16_t><<<(unsigned)rows, fb::NORM_THREADS, 0, (cudaStream_t)stream>>>(x, ldx, gate, ld_g, w, eps, cols, out, ldo);
-  return fb::launch_status("fb_gated_rmsnorm");
+  return dtype == FB_FP32 ? fb::launch_gated_rmsnorm<float>(x, rows, cols, ldx, gate, ld_g, w, eps, out, ldo, (cudaStream_t)stream)
+                          : fb::launch_gated_rmsnorm<uint16_t>(x, rows, cols, ldx, gate, ld_g, w, eps, out, ldo, (cudaStream_t)stream);
 }

@@ -72,3 +72,27 @@ def test_empty_shapes_need_no_workspace_and_static_attention_refuses_them():
     assert rc == -1 and b"at least one token" in lib.fb_last_error()
     rc = lib.fb_rope_kv_write(16, 1, 256, 2, 1, 48, 16, 16, 48, 8, 16, 16, 16, 1e-5, 16, 96, 16, 64, 64 * 48, None)
     assert rc == -1 and b"multiple of 64" in lib.fb_last_error()
+
+
+def test_dense_latent_and_decay_entry_points_refuse_bad_arguments_without_a_gpu():
+    import ctypes
+    lib = _lib.lib()
+    rc = lib.fb_dense(16, 4, 60, 64, 0, 16, 32, 64, 0, 1, 16, _lib.BF16, 32, 0, None, 0, None)
+    assert rc == -1 and b"multiple of 8" in lib.fb_last_error()
+    e = _lib.DenseEpilogue(kind=9)
+    rc = lib.fb_dense(16, 4, 64, 64, 0, 16, 32, 64, 0, 1, 16, _lib.BF16, 32, 0, ctypes.byref(e), 0, None)
+    assert rc == -1 and b"unknown epilogue" in lib.fb_last_error()
+    e = _lib.DenseEpilogue(kind=_lib.DENSE_DYT_ADD)
+    rc = lib.fb_dense(16, 4, 64, 64, 0, 16, 32, 64, 0, 1, 16, _lib.FP32, 32, 0, ctypes.byref(e), 0, None)
+    assert rc == -1 and b"its vectors" in lib.fb_last_error()
+    assert lib.fb_dense_supports(8, 64, 0, 16, 64, 0, 64, 32, _lib.DENSE_NONE) == 0, "a row of x that is not 16-byte aligned"
+    rc = lib.fb_latent_put(_lib.FP32, 16, 2, 100, 40, 40, 21, 8, 16, 16, 1e-5, 16, 1.0, 16, 16, _lib.BF16, 16, 40, 16, 64, None)
+    assert rc == -1 and b"within the key part" in lib.fb_last_error()
+    rc = lib.fb_rotate_pairs(_lib.BF16, 16, 2, 4, 64, 16, 16, 5, 16, 1.0, 16, 16, 64, 16, None)
+    assert rc == -1 and b"even number" in lib.fb_last_error()
+    rc = lib.fb_latent_attention(_lib.BF16, 16, 2, 100, 4, 32, 8, 16, 64, 16, 0, 16, 64, 0, 1.0, None, 16, 128, None, 0, None)
+    assert rc == -1 and b"row strides too small" in lib.fb_last_error()
+    rc = lib.fb_decay_scan(_lib.BF16, 16, 4096, 2, 600, 64, 16, 16, -1, 1, 4, 16, 2 * 600 * 64, 16, 128, None)
+    assert rc == -1 and b"up to 512" in lib.fb_last_error()
+    rc = lib.fb_gated_rmsnorm(16, 2, 64, 32, _lib.BF16, 16, 64, 16, 1e-5, 16, 64, None)
+    assert rc == -1

@@ -39,3 +39,10 @@ def test_cpu_sample_runs_a_mixture_block():
     finally:
         del bench.WORKLOADS["_tiny_moe"]
     assert out["value"] > 0 and out["kind"] in ("port", "reference") and np.isfinite(out["seconds_per_step_scaled"])
+
+
+def test_design_models_are_of_equal_size():
+    for s in bench.DESIGN_SIZES.values():
+        b, l = bench.design_models(s, 512)
+        assert (b.dim, b.vocab, b.layers) == (l.dim, l.vocab, l.layers) and all(e.mlp.ff == l.ffn for e in b.blocks)
+        assert [e.type for e in b.blocks[:2]] == ["latent_attention", "lightning"] and b.blocks[0].mixer.heads == l.heads

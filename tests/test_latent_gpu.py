@@ -164,11 +164,12 @@ def test_decay_scan(cuda, H, dim, vdim, dtype):
     assert torch.equal(state[2], left) and not three_out[2].any(), "a slot without a token keeps its state"
 
 
-def test_gated_rmsnorm(cuda):
+@pytest.mark.parametrize("cols,skip", [(333, 7), (96, 8), (2048, 0), (6000, 4), (5001, 3)])
+def test_gated_rmsnorm(cuda, cols, skip):
     rng = np.random.default_rng(6)
     for dtype, tol in ((torch.float32, 2e-5), (torch.bfloat16, 8e-3)):
-        x, g, w = draw(rng, 5, 333, dtype=torch.float32), draw(rng, 5, 340, dtype=dtype), draw(rng, 333, dtype=torch.float32)
-        out = torch.empty(5, 333, dtype=dtype, device=cuda)
-        ops.gated_rmsnorm(x.to(cuda), g.to(cuda)[:, 7:], w.to(cuda), 1e-4, out)
-        want = oracle.rms(x.numpy().astype(f64), w.numpy(), 1e-4) * oracle.sigmoid(g.float().numpy().astype(f64)[:, 7:])
+        x, g, w = draw(rng, 5, cols, dtype=torch.float32), draw(rng, 5, cols + skip, dtype=dtype), draw(rng, cols, dtype=torch.float32)
+        out = torch.empty(5, cols, dtype=dtype, device=cuda)
+        ops.gated_rmsnorm(x.to(cuda), g.to(cuda)[:, skip:], w.to(cuda), 1e-4, out)
+        want = oracle.rms(x.numpy().astype(f64), w.numpy(), 1e-4) * oracle.sigmoid(g.float().numpy().astype(f64)[:, skip:])
         np.testing.assert_allclose(out.float().cpu().numpy(), want, rtol=tol, atol=tol)
