@@ -18,8 +18,9 @@ MODES = {"bfloat16": "bf16", "float32": "fp32", "bfp8": "bfp8", "bfp4": "bfp4"}
 
 def load(folder, dtype, places):
     """A runtime, a checkpoint's config and its weights on the device."""
-    from . import checkpoint, models
+    from . import build, checkpoint, models
     from .tensor import Runtime
+    build.ensure(models.family_of_json(checkpoint.read_json(os.path.join(folder, "config.json"))), MODES[dtype])  # (where it is missing)
     rt = Runtime(0)
     c, w = checkpoint.load(folder, places)
     family = models.of(c)

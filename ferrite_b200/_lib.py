@@ -80,6 +80,12 @@ class FerriteError(RuntimeError):
 _lib = None
 
 
+def _left_out(name):
+    def call(*_):
+        raise ImportError(f"{LIB_PATH} was built without {name}: run `python -m ferrite_b200.build`")
+    return call
+
+
 def lib():
     """The loaded library (loads it on first use)."""
     global _lib
@@ -88,7 +94,10 @@ def lib():
             raise ImportError(f"{LIB_PATH} is not built: run `python -m ferrite_b200.build` (the CUDA library is the only compute path)")
         _lib = ctypes.CDLL(LIB_PATH)
         for name, (res, args) in SIGNATURES.items():
-            fn = getattr(_lib, name)
+            fn = getattr(_lib, name, None)
+            if fn is None:  # a library that was built for one model family: what it leaves out says so when it is called
+                setattr(_lib, name, _left_out(name))
+                continue
             fn.restype, fn.argtypes = res, args
     return _lib
 

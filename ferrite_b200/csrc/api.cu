@@ -6,6 +6,12 @@
 
 namespace fb {
 
+static int (*g_status_word_of[16])();
+static int g_status_words;
+StatusWord::StatusWord(int (*read_and_clear)()) {
+  if (g_status_words < 16) g_status_word_of[g_status_words++] = read_and_clear;
+}
+
 static thread_local char g_error[512] = "";
 
 void set_error(const char* fmt, ...) {
@@ -28,8 +34,10 @@ extern "C" int fb_version(void) { return 1; }
 extern "C" const char* fb_last_error(void) { return fb::g_error; }
 
 extern "C" int fb_status_word(void) {
-  const int codes[] = {fb::status_word_tcgen05(), fb::status_word_peer(), fb::status_word_gemv_stream(), fb::status_word_dense(), fb::status_word_latent()};  // (all read, so all are cleared)
-  for (int code : codes)
-    if (code) return code;
-  return 0;
+  int first = 0;
+  for (int i = 0; i < fb::g_status_words; ++i) {  // (all read, so all are cleared)
+    const int code = fb::g_status_word_of[i]();
+    first = first ? first : code;
+  }
+  return first;
 }

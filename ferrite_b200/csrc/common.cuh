@@ -14,12 +14,11 @@ namespace fb {
 // fb_status and leaves the reason here (fb_last_error()).
 void set_error(const char* fmt, ...);
 int launch_status(const char* what);  // cudaGetLastError() -> FB_OK / FB_ERR_LAUNCH with the message kept
-// the status words of the kernels that wait (each reads and clears its own): 0, or the code of the wait that gave up
-int status_word_tcgen05();
-int status_word_peer();
-int status_word_gemv_stream();
-int status_word_dense();
-int status_word_latent();
+// The status words of the kernels that wait: 0, or the code of the wait that gave up; each translation unit with such
+// kernels reads and clears its own and says so by one of these at file scope (fb_status_word() asks them all)
+struct StatusWord {
+  explicit StatusWord(int (*read_and_clear)());
+};
 
 #define FB_REQUIRE(cond, ...)            \
   do {                                   \

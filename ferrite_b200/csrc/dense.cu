@@ -290,7 +290,7 @@ int launch_dense(const CUtensorMap& tw, const CUtensorMap& tx, const DenseParams
 
 }  // namespace
 
-int status_word_dense() { return read_and_clear_status_word(); }
+static const StatusWord g_status_reader(read_and_clear_status_word);
 
 }  // namespace fb
 

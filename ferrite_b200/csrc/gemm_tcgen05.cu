@@ -1084,4 +1084,4 @@ int linear_tcgen05_indexed(const LinearArgs& a, const IndexedArgs& ix, cudaStrea
 
 }  // namespace fb
 
-int fb::status_word_tcgen05() { return fb::read_and_clear_status_word(); }
+static const fb::StatusWord g_status_reader(fb::read_and_clear_status_word);

@@ -282,6 +282,6 @@ int linear_gemv_stream(const LinearArgs& a, cudaStream_t s) {
   return a.fmt == FB_BFP8 ? launch<FB_BFP8>(p, pl.ctas, smem, s) : launch<FB_BFP4>(p, pl.ctas, smem, s);
 }
 
-int status_word_gemv_stream() { return read_and_clear_status_word(); }
+static const StatusWord g_status_reader(read_and_clear_status_word);
 
 }  // namespace fb

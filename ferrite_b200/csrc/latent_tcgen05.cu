@@ -537,6 +537,6 @@ int latent_tcgen05(const LatentArgs& a, cudaStream_t s) {
   return launch_status("fb_latent_attention");
 }
 
-int status_word_latent() { return read_and_clear_status_word(); }
+static const StatusWord g_status_reader(read_and_clear_status_word);
 
 }  // namespace fb

@@ -121,7 +121,7 @@ __global__ void __launch_bounds__(256) peer_reduce_add_kernel(const PeerArgs a) 
 
 }  // namespace
 
-int status_word_peer() { return read_and_clear_status_word(); }
+static const StatusWord g_status_reader(read_and_clear_status_word);
 
 }  // namespace fb
 

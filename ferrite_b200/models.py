@@ -17,8 +17,13 @@ def of(c):
     return module(getattr(c, "family", "llama"))
 
 
-def of_json(j):
-    """The family module of a parsed config.json."""
+def family_of_json(j):
+    """The family of a parsed config.json."""
     name = j.get("architecture")
     assert name is None or name in ARCHITECTURES, f"architecture {name!r} is not served here: {', '.join(sorted(ARCHITECTURES))}"
-    return module(ARCHITECTURES.get(name, "llama"))
+    return ARCHITECTURES.get(name, "llama")
+
+
+def of_json(j):
+    """The family module of a parsed config.json."""
+    return module(family_of_json(j))

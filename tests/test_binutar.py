@@ -183,3 +183,33 @@ def test_command_line_asks_for_a_model():
     with pytest.raises(SystemExit):
         main(["replay", "--model", "x", "--out", "y", "--dtype", "float16"])
     json.dumps(models.CONFIGS)  # (a config is plain JSON)
+
+
+def test_the_library_is_built_for_a_family_and_completed_later(tmp_path, monkeypatch):
+    # the compiler played by a function that writes files: which sources are compiled and linked, and when
+    from ferrite_b200 import build
+    for name, at in (("OBJ", "obj"), ("LIB", "lib/lib.so"), ("LINKED", "lib/sources.txt")):
+        monkeypatch.setattr(build, name, str(tmp_path / at))
+    compiled, linked = [], []
+
+    def compile_one(name):
+        compiled.append(name)
+        return name, ""
+
+    def run(cmd, **_):
+        linked.append([o.split("/")[-1] for o in cmd if o.endswith(".o")])
+        open(build.LIB, "w").close()
+        return NS(returncode=0, stdout="", stderr="")
+    monkeypatch.setattr(build, "compile_one", compile_one)
+    monkeypatch.setattr(build.subprocess, "run", run)
+    need = build.FAMILY_SOURCES["binutar"]
+    assert set(need) < set(build.sources())
+    build.ensure("binutar")
+    assert sorted(compiled) == sorted(need) and len(linked[-1]) == len(need) and build.linked() == sorted(need)
+    build.ensure("binutar", "fp32")
+    assert len(linked) == 1, "nothing is missing"
+    build.ensure("binutar", "bfp8")
+    assert len(linked) == 2 and len(linked[-1]) == len(build.sources()) and build.linked() == build.sources()
+    build.ensure("llama")
+    build.ensure("binutar")
+    assert len(linked) == 2
