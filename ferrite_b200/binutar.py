@@ -12,7 +12,7 @@ from types import SimpleNamespace
 import numpy as np
 import torch
 
-from . import llama, mixers
+from . import llama, mixers, models
 from .tensor import BFP, Tensor
 
 REWINDS = False  # a linear mixer's state cannot be taken back to an earlier token: a slot's prefix is reused whole or not at all
@@ -21,14 +21,10 @@ MIXERS = {"latent_attention": (mixers.latent_attention, mixers.latent_cache), "l
 DEFAULTS = dict(family="binutar", places=4096, dtype="bf16", precision=None)
 
 
-def _sizes(x):
-    return SimpleNamespace(**{k: _sizes(v) if isinstance(v, dict) else v for k, v in x.items()})
-
-
 def model(**c):
     """A config from config.json's fields (vocab, width, norm, layers) and this library's (places, dtype, precision)."""
     c = SimpleNamespace(**DEFAULTS | c)
-    c.blocks = [_sizes(e) for e in c.blocks]
+    c.blocks = [models.sizes(e) for e in c.blocks]
     for i, b in enumerate(c.blocks):
         assert b.type in MIXERS, f"layer {i}: no mixer {b.type!r}: {', '.join(sorted(MIXERS))}"
         b.mlp = getattr(b, "mlp", None)
@@ -146,23 +142,15 @@ def forward(ids, places, w, c, caches, slots=None, every=False, length=None):
     return h.matmul(w["head"], dtype="fp32")
 
 
-class Caches(list):
-    """A layer's cache or state each, for sequences that share `size` places."""
-
-    def __init__(self, size, caches):
-        super().__init__(caches)
-        self.size = size
-
-
 def kv_cache(c, size, zeros, slots=1):
     make = lambda shape, dtype=c.dtype: zeros(shape, dtype)
-    return Caches(size, [MIXERS[b.type][1](b.mixer, size, make, slots) for b in c.blocks])
+    return mixers.Caches(size, [MIXERS[b.type][1](b.mixer, size, make, slots) for b in c.blocks])
 
 
 def slot(c, caches, u, slots):
     """Sequence u's part of caches made for several, in place."""
     part = caches.size // slots
-    return Caches(part, [x[:, u * part:(u + 1) * part, :] if x.rows == caches.size and x.batch == 1 and b.type == "latent_attention" else x[u:u + 1, :, :]
+    return mixers.Caches(part, [x[:, u * part:(u + 1) * part, :] if x.rows == caches.size and x.batch == 1 and b.type == "latent_attention" else x[u:u + 1, :, :]
                          for x, b in zip(caches, c.blocks)])
 
 

@@ -18,6 +18,11 @@
 // gated unit (gate and up rows alternate in runs of 16 inside a tile, so a pair is 16 lanes apart), a gate per head, and the
 // Dynamic Tanh - residual add - Dynamic Tanh between two branches, which needs no sum over the row and therefore no
 // kernel of its own.  Every wait is bounded (sm100.cuh).
+//
+// fb_dense_grouped is the same kernel over rows in tiles that each have a matrix of their own (a mixture's experts): which,
+// and how many tiles there are, it reads on the device.
+#include <math.h>
+
 #include "sm100.cuh"
 #include "tma_host.cuh"
 #include "values.cuh"
@@ -41,15 +46,22 @@ struct DenseParams {
   int out_dtype;
   int64_t ldo, out_batch;
   int settled;
+  // rows in tiles of `nt`, each with a matrix of its own (fb_dense_grouped): the tiles' matrices and how many there are, both
+  // read on the device; x_step: how far the rows move on a tile (nt, or 0: every tile the same rows)
+  const int32_t *tile_expert, *live;
+  int x_step;
+  float shift;  // GLU: added to the up half
   fb_dense_epilogue e;
 };
 
 struct DenseTile {
   int m, n, b;
 };
-__device__ __forceinline__ DenseTile tile_of(const DenseParams& p, int id) {  // tokens fastest: tiles that share weights run together
-  const int rest = id / p.tiles_m;
-  return {id % p.tiles_m, rest % p.tiles_n, rest / p.tiles_n};
+// tiles_m: the tiles of rows there are (grouped: those in use)
+__device__ __forceinline__ DenseTile tile_of(const DenseParams& p, int id, int tiles_m) {  // tokens fastest: tiles that share weights run together
+  const int rest = id / tiles_m, m = id % tiles_m;
+  if (p.tile_expert) return {m, rest, p.tile_expert[m]};
+  return {m, rest % p.tiles_n, rest / p.tiles_n};
 }
 
 // what the epilogue needs of a column, read once a tile
@@ -82,10 +94,10 @@ __device__ __forceinline__ void emit(const DenseParams& p, const Column& c, int 
   }
   if constexpr (EPI == FB_DENSE_GLU) {
     const float g = fminf(v, p.e.limit), u = fminf(fmaxf(up, -p.e.limit), p.e.limit);
-    v = g / (1.f + __expf(-p.e.slope * g)) * (u + 1.f);
+    v = g / (1.f + __expf(-p.e.slope * g)) * (u + p.shift);
   }
   if constexpr (EPI == FB_DENSE_GATE) v *= gate;
-  const int64_t at = b * p.out_batch + t * p.ldo + n;
+  const int64_t at = b * p.out_batch + t * p.ldo + n;  // (grouped: out_batch 0, the rows follow the tiles)
   if (p.out_dtype == FB_FP32) static_cast<float*>(p.out)[at] = v;
   else static_cast<uint16_t*>(p.out)[at] = (uint16_t)float_to_bf16_bits(v);
 }
@@ -114,33 +126,39 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = tmem_slot[0];
+  int tiles = p.tiles, tiles_m = p.tiles_m;
+  if (p.live) {
+    griddep_wait();
+    tiles_m = min(max(*p.live, 0), p.tiles_m), tiles = tiles_m * p.tiles_n;
+  }
+  const bool idle = p.splits > 1 && (int)blockIdx.x >= tiles;  // (a whole cluster without a tile)
 
   if (warp == D_WARP_LOAD && lane == 0) {
     prefetch_tensormap(&tw), prefetch_tensormap(&tx);
     auto weights = [&](const DenseTile& t, int k, int slot) {
       const uint32_t bar = smem_u32(full + slot), dst = smem_u32(smem + slot * stage_bytes);
       mbar_expect_tx(bar, (uint32_t)stage_bytes);
-      if (EPI == FB_DENSE_GLU) tma_load_4d(dst, &tw, 64 * k, 0, 0, 4 * t.n, bar);
+      if (EPI == FB_DENSE_GLU) tma_load_5d(dst, &tw, 64 * k, 0, 0, 4 * t.n, t.b, bar);
       else tma_load_3d(dst, &tw, 64 * k, 128 * t.n, t.b, bar);
     };
     int early = 0;
-    if (p.settled && (int)blockIdx.x < p.tiles) {
-      const DenseTile t = tile_of(p, blockIdx.x);
+    if (p.settled && !p.live && (int)blockIdx.x < p.tiles) {
+      const DenseTile t = tile_of(p, blockIdx.x, tiles_m);
       for (early = 0; early < min(S, n_steps); ++early) weights(t, s0 + early, early);
     }
     griddep_wait();  // the activations come from the kernel before
     int i = 0, slot = 0;
     uint32_t phase = 0;
     bool ok = true;
-    for (int id = blockIdx.x; id < p.tiles && ok; id += gridDim.x) {
-      const DenseTile t = tile_of(p, id);
+    for (int id = blockIdx.x; id < tiles && ok; id += gridDim.x) {
+      const DenseTile t = tile_of(p, id, tiles_m);
       for (int k = 0; k < n_steps && ok; ++k, ++i) {
         if (i >= early) {
           ok = mbar_wait(smem_u32(empty + slot), phase ^ 1, abort_flag, DW_EMPTY);
           if (!ok) break;
           weights(t, s0 + k, slot);
         }
-        tma_load_3d(smem_u32(smem + slot * stage_bytes + D_A_BYTES), &tx, 64 * (s0 + k), nt * t.m, t.b, smem_u32(full + slot));
+        tma_load_3d(smem_u32(smem + slot * stage_bytes + D_A_BYTES), &tx, 64 * (s0 + k), p.x_step * t.m, p.live ? 0 : t.b, smem_u32(full + slot));
         if (++slot == S) slot = 0, phase ^= 1;
       }
     }
@@ -156,7 +174,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
     const uint64_t d0 = umma_smem_desc(smem_u32(smem), 16, 1024);
     int slot = 0, n = 0;
     uint32_t phase = 0;
-    for (int id = blockIdx.x; id < p.tiles; id += gridDim.x, ++n) {
+    for (int id = blockIdx.x; id < tiles; id += gridDim.x, ++n) {
       const uint32_t acc = tmem + (n & 1) * nt;
       mbar_wait(smem_u32(acc_empty + (n & 1)), ((n >> 1) & 1) ^ 1, abort_flag, DW_ACC_EMPTY);
       tc_fence_after();
@@ -175,8 +193,8 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
     griddep_wait();
     const int q = warp & 3, half = nt / 2, col0 = (warp >> 2) * half, row = 32 * q + lane;
     int n = 0;
-    for (int id = blockIdx.x; id < p.tiles; id += gridDim.x, ++n) {
-      const DenseTile t = tile_of(p, id);
+    for (int id = blockIdx.x; id < tiles; id += gridDim.x, ++n) {
+      const DenseTile t = tile_of(p, id, tiles_m);
       mbar_wait(smem_u32(acc_full + (n & 1)), (n >> 1) & 1, abort_flag, DW_ACC_FULL);
       tc_fence_after();
       const uint32_t acc = tmem + ((uint32_t)(32 * q) << 16) + (n & 1) * nt + col0;
@@ -235,8 +253,8 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
 
   if (p.splits > 1) {
     cluster_barrier();  // every CTA's sums are in its shared memory
-    if (warp < D_EPI_WARPS) {
-      const DenseTile t = tile_of(p, blockIdx.x);
+    if (warp < D_EPI_WARPS && !idle) {
+      const DenseTile t = tile_of(p, blockIdx.x, tiles_m);
       const int share = (nt + p.splits - 1) / p.splits, first = blockIdx.y * share, last = min(nt, first + share);
       const int row = tid & 127;
       const int64_t col = EPI == FB_DENSE_GLU ? 64 * (int64_t)t.n + (row >> 5) * 16 + (row & 15) : 128 * (int64_t)t.n + row;
@@ -296,34 +314,15 @@ static const StatusWord g_status_reader(read_and_clear_status_word);
 
 extern "C" int fb_dense_supports(const void* x, int64_t ldx, int64_t x_batch, const void* W, int64_t ldw, int64_t w_batch, int64_t K, int64_t N, int kind) {
   return K >= 8 && K % 8 == 0 && N >= 1 && ldx % 8 == 0 && ldw % 8 == 0 && x_batch % 8 == 0 && w_batch % 8 == 0 && ldx >= K && ldw >= K && (uintptr_t)x % 16 == 0 &&
-         (uintptr_t)W % 16 == 0 && (kind != FB_DENSE_GLU || N % 32 == 0) && fb::tma_encoder() != nullptr;
+         (uintptr_t)W % 16 == 0 && ((kind != FB_DENSE_GLU && kind != FB_DENSE_SWIGLU) || N % 32 == 0) && fb::tma_encoder() != nullptr;
 }
 
-extern "C" int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_t x_batch, const void* W, int64_t N, int64_t ldw, int64_t w_batch, int64_t batch,
-                        void* out, int out_dtype, int64_t ldo, int64_t out_batch, const fb_dense_epilogue* epilogue_host, int settled, void* stream) {
+// what fb_dense and fb_dense_grouped share: the tiles' depth and the CTAs', and the launch.  p: sizes, results and the way rows
+// become tiles are filled in; x_rows, x_entries: the rows and batch entries that x has
+static int run_dense(fb::DenseParams& p, const void* x, int64_t x_rows, int64_t x_entries, int64_t K, int64_t ldx, int64_t x_batch, const void* W, int64_t ldw, int64_t w_batch,
+                     int64_t matrices, cudaStream_t s) {
   using namespace fb;
-  FB_REQUIRE(x && W && out && M >= 1 && batch >= 1 && M < (1 << 30) && N < (1 << 30), "fb_dense: null pointer or empty");
-  const fb_dense_epilogue e = epilogue_host ? *epilogue_host : fb_dense_epilogue{};
-  FB_REQUIRE(e.kind >= FB_DENSE_NONE && e.kind <= FB_DENSE_DYT_ADD, "fb_dense: unknown epilogue %d", e.kind);
-  FB_REQUIRE(K >= 8 && K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && x_batch % 8 == 0 && w_batch % 8 == 0 && ldx >= K && ldw >= K && (uintptr_t)x % 16 == 0 &&
-                 (uintptr_t)W % 16 == 0 && N >= 1,
-             "fb_dense: rows of x and W 16-byte aligned, K a multiple of 8 (K %lld, row strides %lld and %lld)", (long long)K, (long long)ldx, (long long)ldw);
-  FB_REQUIRE(out_dtype == FB_BF16 || out_dtype == FB_FP32, "fb_dense: out is bf16 or fp32");
-  FB_REQUIRE(e.kind != FB_DENSE_GLU || (N % 32 == 0 && batch == 1), "fb_dense: a gated unit takes one matrix of whole runs of 16 gate rows and as many up rows");
-  FB_REQUIRE(e.kind != FB_DENSE_GATE || e.gate, "fb_dense: no gate given");
-  FB_REQUIRE(e.kind != FB_DENSE_DYT_ADD || (e.residual && e.alpha && e.w && e.b && out_dtype == FB_FP32 && batch == 1 && (!e.h_out || (e.alpha2 && e.w2 && e.b2))),
-             "fb_dense: a Dynamic Tanh and add takes its vectors, a residual and an fp32 result");
-  FB_REQUIRE(tma_encoder() != nullptr, "fb_dense: no CUDA driver");
-  const int64_t out_cols = e.kind == FB_DENSE_GLU ? N / 2 : N;
-  FB_REQUIRE(ldo >= out_cols, "fb_dense: rows of out too close");
-  DenseParams p{};
-  p.M = M, p.N = N, p.e = e, p.out = out, p.out_dtype = out_dtype, p.ldo = ldo, p.out_batch = out_batch, p.settled = settled;
-  p.tiles_m = (int)ceil_div(M, 256);
-  p.nt = (int)ceil_div(ceil_div(M, p.tiles_m), 16) * 16;
-  p.tiles_m = (int)ceil_div(M, p.nt);
-  p.tiles_n = (int)ceil_div(out_cols, e.kind == FB_DENSE_GLU ? 64 : 128);
-  FB_REQUIRE((int64_t)p.tiles_m * p.tiles_n * batch < (1 << 30), "fb_dense: too many tiles");
-  p.tiles = (int)(p.tiles_m * p.tiles_n * batch);
+  const int kind = p.e.kind;
   p.steps = (int)ceil_div(K, 64);
   p.tmem_cols = 32;
   while (p.tmem_cols < 2 * p.nt) p.tmem_cols *= 2;
@@ -345,26 +344,84 @@ extern "C" int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_
   p.steps_per_split = (int)ceil_div(p.steps, p.splits);
   const int grid = p.splits > 1 ? p.tiles : p.tiles < sms ? p.tiles : sms;
   CUtensorMap tw, tx;
-  if (e.kind == FB_DENSE_GLU) {
-    const int64_t dims[4] = {K, 16, 2, N / 32}, strides[3] = {ldw, N / 2 * ldw, 16 * ldw};
-    const int box[4] = {64, 16, 2, 4};
-    if (int rc = tma_map_bf16(&tw, W, 4, dims, strides, box, "fb_dense (weights)")) return rc;
+  if (kind == FB_DENSE_GLU) {
+    const int64_t dims[5] = {K, 16, 2, p.N / 32, matrices}, strides[4] = {ldw, p.N / 2 * ldw, 16 * ldw, matrices > 1 ? w_batch : ldw};
+    const int box[5] = {64, 16, 2, 4, 1};
+    if (int rc = tma_map_bf16(&tw, W, 5, dims, strides, box, "fb_dense (weights)")) return rc;
   } else {
-    const int64_t dims[3] = {K, N, batch}, strides[2] = {ldw, batch > 1 ? w_batch : ldw};
+    const int64_t dims[3] = {K, p.N, matrices}, strides[2] = {ldw, matrices > 1 ? w_batch : ldw};
     const int box[3] = {64, 128, 1};
     if (int rc = tma_map_bf16(&tw, W, 3, dims, strides, box, "fb_dense (weights)")) return rc;
   }
-  const int64_t dims[3] = {K, M, batch}, strides[2] = {ldx, batch > 1 && x_batch ? x_batch : ldx};
-  FB_REQUIRE(batch == 1 || x_batch > 0, "fb_dense: a batch takes rows of its own an entry");
+  const int64_t dims[3] = {K, x_rows, x_entries}, strides[2] = {ldx, x_entries > 1 && x_batch ? x_batch : ldx};
   const int box[3] = {64, p.nt, 1};
   if (int rc = tma_map_bf16(&tx, x, 3, dims, strides, box, "fb_dense (activations)")) return rc;
   const size_t smem = 1024 + (size_t)p.stages * stage_bytes;
-  const auto s = (cudaStream_t)stream;
-  switch (e.kind) {
+  switch (kind) {
     case FB_DENSE_SILU: return launch_dense<FB_DENSE_SILU>(tw, tx, p, grid, smem, s);
     case FB_DENSE_GLU: return launch_dense<FB_DENSE_GLU>(tw, tx, p, grid, smem, s);
     case FB_DENSE_GATE: return launch_dense<FB_DENSE_GATE>(tw, tx, p, grid, smem, s);
     case FB_DENSE_DYT_ADD: return launch_dense<FB_DENSE_DYT_ADD>(tw, tx, p, grid, smem, s);
     default: return launch_dense<FB_DENSE_NONE>(tw, tx, p, grid, smem, s);
   }
+}
+
+// FB_DENSE_SWIGLU is the clamped unit without its limit, slope and shift
+static float settle_unit(fb_dense_epilogue& e) {
+  if (e.kind != FB_DENSE_SWIGLU) return 1.f;
+  e.kind = FB_DENSE_GLU, e.limit = INFINITY, e.slope = 1.f;
+  return 0.f;
+}
+
+extern "C" int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_t x_batch, const void* W, int64_t N, int64_t ldw, int64_t w_batch, int64_t batch,
+                        void* out, int out_dtype, int64_t ldo, int64_t out_batch, const fb_dense_epilogue* epilogue_host, int settled, void* stream) {
+  using namespace fb;
+  FB_REQUIRE(x && W && out && M >= 1 && batch >= 1 && M < (1 << 30) && N < (1 << 30), "fb_dense: null pointer or empty");
+  fb_dense_epilogue e = epilogue_host ? *epilogue_host : fb_dense_epilogue{};
+  FB_REQUIRE(e.kind >= FB_DENSE_NONE && e.kind <= FB_DENSE_SWIGLU, "fb_dense: unknown epilogue %d", e.kind);
+  const float shift = settle_unit(e);
+  FB_REQUIRE(K >= 8 && K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && x_batch % 8 == 0 && w_batch % 8 == 0 && ldx >= K && ldw >= K && (uintptr_t)x % 16 == 0 &&
+                 (uintptr_t)W % 16 == 0 && N >= 1,
+             "fb_dense: rows of x and W 16-byte aligned, K a multiple of 8 (K %lld, row strides %lld and %lld)", (long long)K, (long long)ldx, (long long)ldw);
+  FB_REQUIRE(out_dtype == FB_BF16 || out_dtype == FB_FP32, "fb_dense: out is bf16 or fp32");
+  FB_REQUIRE(e.kind != FB_DENSE_GLU || (N % 32 == 0 && batch == 1), "fb_dense: a gated unit takes one matrix of whole runs of 16 gate rows and as many up rows");
+  FB_REQUIRE(e.kind != FB_DENSE_GATE || e.gate, "fb_dense: no gate given");
+  FB_REQUIRE(e.kind != FB_DENSE_DYT_ADD || (e.residual && e.alpha && e.w && e.b && out_dtype == FB_FP32 && batch == 1 && (!e.h_out || (e.alpha2 && e.w2 && e.b2))),
+             "fb_dense: a Dynamic Tanh and add takes its vectors, a residual and an fp32 result");
+  FB_REQUIRE(tma_encoder() != nullptr, "fb_dense: no CUDA driver");
+  const int64_t out_cols = e.kind == FB_DENSE_GLU ? N / 2 : N;
+  FB_REQUIRE(ldo >= out_cols, "fb_dense: rows of out too close");
+  DenseParams p{};
+  p.M = M, p.N = N, p.e = e, p.out = out, p.out_dtype = out_dtype, p.ldo = ldo, p.out_batch = out_batch, p.settled = settled, p.shift = shift;
+  p.tiles_m = (int)ceil_div(M, 256);
+  p.nt = (int)ceil_div(ceil_div(M, p.tiles_m), 16) * 16;
+  p.tiles_m = (int)ceil_div(M, p.nt);
+  p.tiles_n = (int)ceil_div(out_cols, e.kind == FB_DENSE_GLU ? 64 : 128);
+  FB_REQUIRE((int64_t)p.tiles_m * p.tiles_n * batch < (1 << 30), "fb_dense: too many tiles");
+  p.tiles = (int)(p.tiles_m * p.tiles_n * batch);
+  p.x_step = p.nt;
+  FB_REQUIRE(batch == 1 || x_batch > 0, "fb_dense: a batch takes rows of its own an entry");
+  return run_dense(p, x, M, batch, K, ldx, x_batch, W, ldw, w_batch, batch, (cudaStream_t)stream);
+}
+
+extern "C" int fb_dense_grouped(const void* x, int64_t x_rows, int64_t K, int64_t ldx, int shared_rows, const void* W, int64_t N, int64_t ldw, int64_t w_batch, int n,
+                                const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, void* out, int out_dtype, int64_t ldo,
+                                const fb_dense_epilogue* epilogue_host, void* stream) {
+  using namespace fb;
+  FB_REQUIRE(x && W && out && tile_expert && live && tiles >= 1 && n >= 1 && x_rows >= 1 && tiles * tile < (1 << 30) && N < (1 << 30), "fb_dense_grouped: null pointer or empty");
+  fb_dense_epilogue e = epilogue_host ? *epilogue_host : fb_dense_epilogue{};
+  FB_REQUIRE(e.kind == FB_DENSE_NONE || e.kind == FB_DENSE_GLU || e.kind == FB_DENSE_SWIGLU, "fb_dense_grouped: plain, or a gated unit");
+  FB_REQUIRE(tile >= 16 && tile <= 256 && tile % 16 == 0 && (shared_rows ? x_rows <= tile : x_rows >= tiles * tile), "fb_dense_grouped: tiles of 16 to 256 rows, all of them there");
+  FB_REQUIRE(fb_dense_supports(x, ldx, 0, W, ldw, n > 1 ? w_batch : 0, K, N, e.kind), "fb_dense_grouped: rows of x and W 16-byte aligned, K a multiple of 8, a gated unit's halves whole runs of 16");
+  FB_REQUIRE(out_dtype == FB_BF16 || out_dtype == FB_FP32, "fb_dense_grouped: out is bf16 or fp32");
+  DenseParams p{};
+  p.shift = settle_unit(e);
+  const int64_t out_cols = e.kind == FB_DENSE_GLU ? N / 2 : N;
+  FB_REQUIRE(ldo >= out_cols, "fb_dense_grouped: rows of out too close");
+  p.M = tiles * tile, p.N = N, p.e = e, p.out = out, p.out_dtype = out_dtype, p.ldo = ldo;
+  p.nt = tile, p.tiles_m = (int)tiles, p.x_step = shared_rows ? 0 : tile, p.tile_expert = tile_expert, p.live = live;
+  p.tiles_n = (int)ceil_div(out_cols, e.kind == FB_DENSE_GLU ? 64 : 128);
+  FB_REQUIRE(tiles * p.tiles_n < (1 << 30), "fb_dense_grouped: too many tiles");
+  p.tiles = (int)tiles * p.tiles_n;
+  return run_dense(p, x, x_rows, 1, K, ldx, 0, W, ldw, w_batch, n, (cudaStream_t)stream);
 }

@@ -1,0 +1,207 @@
+// A mixture of experts around its matmuls, for weights kept as bf16 or fp32:
+//   fb_route            router logits (with a bias) -> each token's k largest, the softmax of those, and where each choice's row
+//                       goes: the touched experts' rows in whole tiles, a list of the tiles' experts, how many there are
+//   fb_grouped_matmul   rows of tiles by each tile's own matrix, any sizes, bf16 or fp32 (the tensor cores' form: fb_dense_grouped)
+//
+// Two layouts of the rows.  A few tokens: a tile a touched expert, holding all the tokens (nothing is gathered; an expert's
+// weights, not its rows, are what such a step reads).  Many: each expert's choices one after another, filled up to whole tiles.
+#include "launch.cuh"
+#include "values.cuh"
+
+namespace fb {
+
+struct RouteArgs {
+  const float* logits;  // [T, ld]
+  int64_t T, ld;
+  const float* bias;  // [n] or null
+  int n, k, tile, shared;
+  int tiles;  // entries of tile_expert
+  float* weights;       // [T, k]
+  int32_t* ids;         // [T, k]
+  int32_t* slots;       // [T, k]: the row of each choice
+  int32_t* order;       // [tiles * tile] the token each row holds, -1: none (null with shared rows)
+  int32_t* tile_expert; // [tiles], n past those used
+  int32_t* live;        // [1] tiles used
+};
+
+// the k largest of a token's logits, the lower column first among equals, and the softmax of those: a warp a token
+__device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int lane) {
+  const float* z = a.logits + t * a.ld;
+  float prev = INFINITY, mine = -INFINITY;
+  int prev_at = -1, my_id = 0;
+  float held[4];  // the first 128 columns stay in registers
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int c = 32 * i + lane;
+    held[i] = c < a.n ? z[c] + (a.bias ? a.bias[c] : 0.f) : -INFINITY;
+  }
+  for (int j = 0; j < a.k; ++j) {
+    float best = -INFINITY;
+    int at = a.n;
+    auto look = [&](int c, float v) {
+      const bool after = v < prev || (v == prev && c > prev_at);
+      if (after && (at == a.n || v > best)) best = v, at = c;  // (columns rise: the first of equals stays)
+    };
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (32 * i + lane < a.n) look(32 * i + lane, held[i]);
+    for (int c = 128 + lane; c < a.n; c += 32) look(c, z[c] + (a.bias ? a.bias[c] : 0.f));
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, at, o);
+      if (oi < a.n && (at == a.n || ov > best || (ov == best && oi < at))) best = ov, at = oi;
+    }
+    if (at == a.n) at = 0;  // (only where a logit is not a number)
+    prev = best, prev_at = at;
+    if (lane == j) mine = best, my_id = at;
+  }
+  const float top = __shfl_sync(0xffffffffu, mine, 0), e = lane < a.k ? expf(mine - top) : 0.f, sum = warp_sum(e);
+  if (lane < a.k) a.weights[t * a.k + lane] = e / sum, a.ids[t * a.k + lane] = my_id;
+}
+
+__global__ void __launch_bounds__(256) route_tokens_kernel(const RouteArgs a) {
+  griddep_launch_dependents();
+  griddep_wait();
+  const int64_t t = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (t < a.T) route_token(a, t, threadIdx.x & 31);
+}
+
+// one block: the choices' places.  `pick`: it makes the choices first
+__global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, const int pick) {
+  griddep_launch_dependents();
+  griddep_wait();
+  extern __shared__ int32_t route_smem[];  // [n] counts, then each expert's next row; [33] sums
+  int32_t *count = route_smem, *sums = route_smem + a.n;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  for (int e = tid; e < a.n; e += blockDim.x) count[e] = 0;
+  if (pick)
+    for (int64_t t = warp; t < a.T; t += 32) route_token(a, t, lane);
+  __syncthreads();
+  const int64_t choices = a.T * a.k;
+  for (int64_t i = tid; i < choices; i += blockDim.x) atomicAdd(count + a.ids[i], 1);
+  __syncthreads();
+  // tiles of each expert, scanned: a thread has a run of experts
+  const int run = (a.n + 1023) / 1024, e0 = min(a.n, tid * run), e1 = min(a.n, e0 + run);
+  auto tiles_of = [&](int e) { return a.shared ? (count[e] ? 1 : 0) : (count[e] + a.tile - 1) / a.tile; };
+  int own = 0;
+  for (int e = e0; e < e1; ++e) own += tiles_of(e);
+  int before = own;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int v = __shfl_up_sync(0xffffffffu, before, o);
+    if (lane >= o) before += v;
+  }
+  if (lane == 31) sums[warp] = before;
+  __syncthreads();
+  if (warp == 0) {
+    int v = sums[lane];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int u = __shfl_up_sync(0xffffffffu, v, o);
+      if (lane >= o) v += u;
+    }
+    sums[lane] = v;
+  }
+  __syncthreads();
+  int first = before - own + (warp ? sums[warp - 1] : 0);
+  const int used = sums[31];
+  if (tid == 0) *a.live = used;
+  for (int e = e0; e < e1; ++e) {
+    const int n = tiles_of(e);
+    for (int i = 0; i < n; ++i)
+      if (first + i < a.tiles) a.tile_expert[first + i] = e;
+    count[e] = first * a.tile;
+    first += n;
+  }
+  for (int i = used + tid; i < a.tiles; i += blockDim.x) a.tile_expert[i] = a.n;
+  if (a.order)
+    for (int64_t i = tid; i < (int64_t)a.tiles * a.tile; i += blockDim.x) a.order[i] = -1;
+  __syncthreads();
+  for (int64_t i = tid; i < choices; i += blockDim.x) {
+    const int e = a.ids[i];
+    const int64_t t = i / a.k;
+    const int slot = a.shared ? count[e] + (int)t : atomicAdd(count + e, 1);
+    a.slots[i] = slot;
+    if (a.order) a.order[slot] = (int32_t)t;
+  }
+}
+
+struct GroupedArgs {
+  const void* x;
+  int x_dtype;
+  int64_t x_row, x_rows;  // x's rows; row r of tile i is row i * tile + r, or, with shared rows, r
+  int shared;
+  const void* w;
+  int w_dtype;
+  int64_t w_s[3];  // matrix, row (K), column (N)
+  void* out;
+  int out_dtype;
+  int64_t ldo, N, K;
+  int tile, n;
+  const int32_t *tile_expert, *live;
+};
+
+__device__ __forceinline__ float typed(const void* p, int dtype, int64_t at) {
+  return dtype == FB_FP32 ? static_cast<const float*>(p)[at] : bf16_bits_to_float(static_cast<const uint16_t*>(p)[at]);
+}
+
+__global__ void __launch_bounds__(256) grouped_matmul_kernel(const GroupedArgs g) {
+  griddep_launch_dependents();
+  griddep_wait();
+  const int i = blockIdx.y * 16 / g.tile, r0 = blockIdx.y * 16 % g.tile;
+  if (i >= *g.live) return;
+  const int e = g.tile_expert[i];
+  if (e < 0 || e >= g.n) return;
+  __shared__ float sa[16][17], sb[16][17];
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const int64_t col = blockIdx.x * 16 + tx, row = (g.shared ? 0 : (int64_t)i * g.tile) + r0 + ty, x0 = row * g.x_row;
+  const bool there = row < g.x_rows;  // (a tile that holds all of a few tokens has rows to spare)
+  float acc = 0.f;
+  for (int64_t k0 = 0; k0 < g.K; k0 += 16) {
+    sa[ty][tx] = there && k0 + tx < g.K ? typed(g.x, g.x_dtype, x0 + k0 + tx) : 0.f;
+    sb[ty][tx] = col < g.N && k0 + ty < g.K ? typed(g.w, g.w_dtype, e * g.w_s[0] + (k0 + ty) * g.w_s[1] + col * g.w_s[2]) : 0.f;
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) acc = fmaf(sa[ty][k], sb[k][tx], acc);
+    __syncthreads();
+  }
+  if (col >= g.N) return;
+  const int64_t at = ((int64_t)i * g.tile + r0 + ty) * g.ldo + col;
+  if (g.out_dtype == FB_FP32) static_cast<float*>(g.out)[at] = acc;
+  else static_cast<uint16_t*>(g.out)[at] = (uint16_t)float_to_bf16_bits(acc);
+}
+
+}  // namespace fb
+
+extern "C" int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_rows) {
+  if (T < 1 || n < 1 || k < 1 || tile < 1) return 0;
+  const int64_t choices = T * k, most = choices < n ? choices : n;
+  if (shared_rows) return most;
+  return choices / tile + most;  // (each touched expert adds less than a tile)
+}
+
+extern "C" int fb_route(const float* logits, int64_t T, int64_t ld, const float* bias, int n, int k, int tile, int shared_rows, float* weights, int32_t* ids, int32_t* slots,
+                        int32_t* order, int32_t* tile_expert, int32_t* live, void* stream) {
+  FB_REQUIRE(logits && weights && ids && slots && tile_expert && live && T >= 1 && T <= (1 << 24), "fb_route: null pointer or no tokens");
+  FB_REQUIRE(n >= 1 && n <= 8192 && k >= 1 && k <= 32 && k <= n && ld >= n, "fb_route: up to 32 choices among up to 8192 experts (got %d of %d)", k, n);
+  FB_REQUIRE(tile >= 16 && tile % 16 == 0 && (shared_rows ? T <= tile : order != nullptr), "fb_route: tiles of whole runs of 16 rows; shared rows: all the tokens in one");
+  const int64_t tiles = fb_route_tiles(T, n, k, tile, shared_rows);
+  FB_REQUIRE(tiles * tile < (1ll << 31), "fb_route: too many rows");
+  const fb::RouteArgs a{logits, T, ld, bias, n, k, tile, shared_rows, (int)tiles, weights, ids, slots, shared_rows ? nullptr : order, tile_expert, live};
+  const auto s = (cudaStream_t)stream;
+  const int pick = T <= 128;
+  if (!pick)
+    if (int rc = fb::launch_after(fb::route_tokens_kernel, dim3((unsigned)fb::ceil_div(T, 8)), dim3(256), 0, s, "fb_route", a)) return rc;
+  return fb::launch_after(fb::route_places_kernel, dim3(1), dim3(1024), (size_t)(n + 33) * sizeof(int32_t), s, "fb_route", a, pick);
+}
+
+extern "C" int fb_grouped_matmul(int x_dtype, const void* x, int64_t x_rows, int64_t ldx, int shared_rows, int w_dtype, const void* W, const int64_t* w_strides_host, int n, int64_t K, int64_t N,
+                                 const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, int out_dtype, void* out, int64_t ldo, void* stream) {
+  FB_REQUIRE(x && W && w_strides_host && tile_expert && live && out && tiles >= 1 && K >= 1 && N >= 1 && n >= 1, "fb_grouped_matmul: null pointer or empty");
+  FB_REQUIRE(tile >= 16 && tile % 16 == 0 && ldx >= K && ldo >= N && tiles * (tile / 16) <= 65535, "fb_grouped_matmul: tiles of whole runs of 16 rows, at most 65535 such runs");
+  FB_REQUIRE(shared_rows ? x_rows >= 1 && x_rows <= tile : x_rows >= tiles * tile, "fb_grouped_matmul: all the tiles' rows there");
+  for (int d : {x_dtype, w_dtype, out_dtype}) FB_REQUIRE(d == FB_BF16 || d == FB_FP32, "fb_grouped_matmul: bf16 or fp32");
+  const fb::GroupedArgs g{x, x_dtype, ldx, x_rows, shared_rows, W, w_dtype, {w_strides_host[0], w_strides_host[1], w_strides_host[2]}, out, out_dtype, ldo, N, K, tile, n, tile_expert, live};
+  return fb::launch_after(fb::grouped_matmul_kernel, dim3((unsigned)fb::ceil_div(N, 16), (unsigned)(tiles * (tile / 16))), dim3(256), 0, (cudaStream_t)stream, "fb_grouped_matmul", g);
+}

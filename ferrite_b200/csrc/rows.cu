@@ -1,0 +1,244 @@
+// What stands between the matmuls of a decoder with grouped-query attention and an fp32 residual stream, a kernel each:
+//   fb_embed       the stream's start: a row of one table and, where given, a row of another, added in fp32
+//   fb_heads_put   after a joint q | k | v projection: biases, RMSNorm of each query and key head, values mixed with another
+//                  layer's, the new cache row
+//   fb_add_norm    a layer's end: the branches' results scaled by column, a mixture's chosen rows weighted and summed, all
+//                  added to the stream, and the next layer's RMSNorm of it
+#include "launch.cuh"
+#include "values.cuh"
+
+namespace fb {
+
+struct EmbedArgs {
+  const void *table, *places_table;  // [rows, cols], [place_rows, cols] or null
+  int64_t rows, place_rows, cols;
+  const int32_t *ids, *places;
+  float* out;  // [T, cols]
+};
+
+template <typename Act>
+__global__ void __launch_bounds__(256) embed_kernel(const EmbedArgs a) {
+  griddep_launch_dependents();
+  griddep_wait();
+  const int64_t t = blockIdx.x, id = min(max((int64_t)a.ids[t], (int64_t)0), a.rows - 1);
+  const Act* x = static_cast<const Act*>(a.table) + id * a.cols;
+  const Act* y = nullptr;
+  if (a.places_table) y = static_cast<const Act*>(a.places_table) + min(max((int64_t)a.places[t], (int64_t)0), a.place_rows - 1) * a.cols;
+  for (int64_t c = threadIdx.x; c < a.cols; c += blockDim.x) a.out[t * a.cols + c] = value_of(x[c]) + (y ? value_of(y[c]) : 0.f);
+}
+
+// ---- heads: a warp per token and head (the query heads, then the key heads, then the value heads)
+struct HeadsPutArgs {
+  fb_heads h;
+  const void* qkv;
+  int64_t T, ld;
+  const int32_t* rows;
+  void* q_out;
+  int64_t ld_q;
+  void* cache;  // [kv_heads, cache_rows, dim + vdim]: a key, then its value
+  int64_t cache_rows, head_stride;
+};
+
+constexpr int HEADS_WARPS = 8, HEADS_REGS = 8;  // a lane keeps up to 8 columns (heads of up to 256) between the two passes
+
+template <typename In, typename Act>
+__global__ void __launch_bounds__(32 * HEADS_WARPS) heads_put_kernel(const HeadsPutArgs a) {
+  griddep_launch_dependents();
+  griddep_wait();
+  const fb_heads& s = a.h;
+  const int lane = threadIdx.x & 31, units = s.heads + 2 * s.kv_heads;
+  const int64_t job = blockIdx.x * (int64_t)HEADS_WARPS + (threadIdx.x >> 5);
+  if (job >= a.T * units) return;
+  const int64_t t = job / units;
+  const int u = (int)(job % units);
+  const bool is_q = u < s.heads, is_v = u >= s.heads + s.kv_heads;
+  const int n = is_v ? s.vdim : s.dim, g = is_q ? u : is_v ? u - s.heads - s.kv_heads : u - s.heads;
+  const int64_t at = is_v ? (int64_t)(s.heads + s.kv_heads) * s.dim + (int64_t)g * s.vdim : (int64_t)u * s.dim;
+  const int64_t row = a.rows[t];
+  if (!is_q && (row < 0 || row >= a.cache_rows)) return;  // nothing is written outside the cache
+  const In* x = static_cast<const In*>(a.qkv) + t * a.ld + at;
+  const float* bias = s.bias ? s.bias + at : nullptr;
+  Act* out = is_q ? static_cast<Act*>(a.q_out) + t * a.ld_q + (int64_t)g * s.dim
+                  : static_cast<Act*>(a.cache) + g * a.head_stride + row * (s.dim + s.vdim) + (is_v ? s.dim : 0);
+  if (is_v) {
+    const In* first = s.first ? static_cast<const In*>(s.first) + t * s.ld_first + (int64_t)g * s.vdim : nullptr;
+    const float* first_bias = s.first && s.first_bias ? s.first_bias + (int64_t)g * s.vdim : nullptr;
+    const float share = s.first ? *s.share : 0.f;
+    for (int c = lane; c < n; c += 32) {
+      float v = value_of(x[c]) + (bias ? bias[c] : 0.f);
+      if (first) v = (1.f - share) * v + share * (value_of(first[c]) + (first_bias ? first_bias[c] : 0.f));
+      store_value(out + c, v);
+    }
+    return;
+  }
+  const float* w = is_q ? s.q_norm : s.k_norm;
+  float keep[HEADS_REGS], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < HEADS_REGS; ++i) {
+    const int c = 32 * i + lane;
+    keep[i] = c < n ? value_of(x[c]) + (bias ? bias[c] : 0.f) : 0.f;
+    ss = fmaf(keep[i], keep[i], ss);
+  }
+  for (int c = 32 * HEADS_REGS + lane; c < n; c += 32) {  // (wider heads: read twice)
+    const float v = value_of(x[c]) + (bias ? bias[c] : 0.f);
+    ss = fmaf(v, v, ss);
+  }
+  const float r = w ? 1.f / sqrtf(warp_sum(ss) / (float)n + s.eps) : 1.f;
+#pragma unroll
+  for (int i = 0; i < HEADS_REGS; ++i) {
+    const int c = 32 * i + lane;
+    if (c < n) store_value(out + c, keep[i] * r * (w ? w[c] : 1.f));
+  }
+  for (int c = 32 * HEADS_REGS + lane; c < n; c += 32) store_value(out + c, (value_of(x[c]) + (bias ? bias[c] : 0.f)) * r * (w ? w[c] : 1.f));
+}
+
+// ---- a layer's end: a block per token; the new row stays in shared memory for the norm's second pass
+template <typename In, typename Act>
+__global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, const int64_t cols) {
+  griddep_launch_dependents();
+  griddep_wait();
+  extern __shared__ float row[];  // [cols]
+  __shared__ float red[32];
+  __shared__ int64_t at[64];
+  __shared__ float weight[64];
+  const int64_t t = blockIdx.x;
+  if (a.chosen && (int)threadIdx.x < a.k) at[threadIdx.x] = a.slots[t * a.k + threadIdx.x] * a.ld_chosen, weight[threadIdx.x] = a.weights[t * a.k + threadIdx.x];
+  __syncthreads();
+  const float* x = a.x + t * a.ld_x;
+  const In* y1 = a.mixer ? static_cast<const In*>(a.mixer) + t * a.ld_mixer : nullptr;
+  const In* y2 = a.other ? static_cast<const In*>(a.other) + t * a.ld_other : nullptr;
+  float ss = 0.f;
+  for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) {
+    float v = x[c];
+    if (y1) v = fmaf(value_of(y1[c]), a.mixer_scale ? a.mixer_scale[c] : 1.f, v);
+    if (a.chosen || y2) {
+      float f = y2 ? value_of(y2[c]) : 0.f;
+      if (a.chosen)
+        for (int j = 0; j < a.k; ++j) f = fmaf(weight[j], value_of(static_cast<const Act*>(a.chosen)[at[j] + c]), f);
+      v = fmaf(f, a.other_scale ? a.other_scale[c] : 1.f, v);
+    }
+    row[c] = v;
+    if (a.x_out) a.x_out[t * a.ld_x_out + c] = v;
+    ss = fmaf(v, v, ss);
+  }
+  if (!a.h) return;
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps);
+  Act* h = static_cast<Act*>(a.h) + t * a.ld_h;
+  for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) store_value(h + c, row[c] * r * (a.w[c] + a.plus));
+}
+
+// the same for rows of whole groups of four columns, 16-byte aligned: a thread takes its groups in one go, everything it
+// reads on its way at once
+__device__ __forceinline__ float4 four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 four(const uint16_t* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16_bits_to_float(v.x & 0xffffu), bf16_bits_to_float(v.x >> 16), bf16_bits_to_float(v.y & 0xffffu), bf16_bits_to_float(v.y >> 16));
+}
+__device__ __forceinline__ void put_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put_four(uint16_t* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
+__device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) { return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w)); }
+
+template <typename In, typename Act>
+__global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, const int64_t cols) {
+  griddep_launch_dependents();
+  griddep_wait();
+  extern __shared__ float row[];  // [cols]
+  __shared__ float red[32];
+  __shared__ int64_t at[64];
+  __shared__ float weight[64];
+  const int64_t t = blockIdx.x;
+  if (a.chosen && (int)threadIdx.x < a.k) at[threadIdx.x] = a.slots[t * a.k + threadIdx.x] * a.ld_chosen, weight[threadIdx.x] = a.weights[t * a.k + threadIdx.x];
+  __syncthreads();
+  const float4 one = make_float4(1.f, 1.f, 1.f, 1.f), none = make_float4(0.f, 0.f, 0.f, 0.f);
+  float ss = 0.f;
+  for (int64_t c = 4 * threadIdx.x; c < cols; c += 4 * blockDim.x) {
+    float4 v = four(a.x + t * a.ld_x + c), f = none;
+    if (a.mixer) v = fma4(four(static_cast<const In*>(a.mixer) + t * a.ld_mixer + c), a.mixer_scale ? four(a.mixer_scale + c) : one, v);
+    if (a.other) f = four(static_cast<const In*>(a.other) + t * a.ld_other + c);
+    if (a.chosen) {
+      const Act* y = static_cast<const Act*>(a.chosen) + c;
+      for (int j = 0; j < a.k; j += 4) {
+        float4 part[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) part[i] = j + i < a.k ? four(y + at[j + i]) : none;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float s = j + i < a.k ? weight[j + i] : 0.f;
+          f = fma4(make_float4(s, s, s, s), part[i], f);
+        }
+      }
+    }
+    if (a.chosen || a.other) v = fma4(f, a.other_scale ? four(a.other_scale + c) : one, v);
+    put_four(row + c, v);
+    if (a.x_out) put_four(a.x_out + t * a.ld_x_out + c, v);
+    ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+  }
+  if (!a.h) return;
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps);
+  for (int64_t c = 4 * threadIdx.x; c < cols; c += 4 * blockDim.x) {
+    const float4 v = four(row + c), w = four(a.w + c);
+    put_four(static_cast<Act*>(a.h) + t * a.ld_h + c,
+             make_float4(v.x * r * (w.x + a.plus), v.y * r * (w.y + a.plus), v.z * r * (w.z + a.plus), v.w * r * (w.w + a.plus)));
+  }
+}
+
+template <typename In, typename Act>
+static int launch_add_norm(const fb_branches& a, int64_t T, int64_t cols, cudaStream_t s) {
+  static std::atomic<uint64_t> opted{0};
+  if (first_on_device(opted)) {
+    cudaFuncSetAttribute(add_norm_kernel<In, Act>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaFuncSetAttribute(add_norm4_kernel<In, Act>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+  }
+  auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
+  const bool fours = cols % 4 == 0 && whole(a.x, a.ld_x, 4) && whole(a.mixer, a.ld_mixer, sizeof(In)) && whole(a.mixer_scale, 0, 4) && whole(a.other, a.ld_other, sizeof(In)) &&
+                     whole(a.other_scale, 0, 4) && whole(a.chosen, a.ld_chosen, sizeof(Act)) && whole(a.x_out, a.ld_x_out, 4) && whole(a.w, 0, 4) && whole(a.h, a.ld_h, sizeof(Act));
+  const int64_t work = fours ? cols / 4 : cols;
+  const int threads = (int)(work >= 512 ? 512 : ceil_div(work, 32) * 32 < 64 ? 64 : ceil_div(work, 32) * 32);
+  auto kernel = fours ? add_norm4_kernel<In, Act> : add_norm_kernel<In, Act>;
+  return launch_after(kernel, dim3((unsigned)T), dim3(threads), (size_t)cols * sizeof(float), s, "fb_add_norm", a, cols);
+}
+
+}  // namespace fb
+
+extern "C" int fb_embed(int dtype, const void* table, int64_t rows, int64_t cols, const int32_t* ids, const void* places_table, int64_t place_rows, const int32_t* places,
+                        int64_t T, float* out, void* stream) {
+  FB_REQUIRE(table && ids && out && T >= 1 && rows >= 1 && cols >= 1, "fb_embed: null pointer or empty");
+  FB_REQUIRE(!places_table || (places && place_rows >= 1), "fb_embed: a table of places takes the places");
+  FB_REQUIRE(dtype == FB_BF16 || dtype == FB_FP32, "fb_embed: bf16 or fp32 tables");
+  const fb::EmbedArgs a{table, places_table, rows, place_rows, cols, ids, places, out};
+  const auto s = (cudaStream_t)stream;
+  if (dtype == FB_FP32) return fb::launch_after(fb::embed_kernel<float>, dim3((unsigned)T), dim3(256), 0, s, "fb_embed", a);
+  return fb::launch_after(fb::embed_kernel<uint16_t>, dim3((unsigned)T), dim3(256), 0, s, "fb_embed", a);
+}
+
+extern "C" int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void* qkv, int64_t T, int64_t ld, const int32_t* rows, int dtype, void* q_out, int64_t ld_q,
+                            void* cache, int64_t cache_rows, int64_t head_stride, void* stream) {
+  FB_REQUIRE(heads_host && qkv && rows && q_out && cache && T >= 1, "fb_heads_put: null pointer or empty");
+  const fb_heads& h = *heads_host;
+  FB_REQUIRE(h.heads >= 1 && h.kv_heads >= 1 && h.heads % h.kv_heads == 0 && h.dim >= 1 && h.vdim >= 1, "fb_heads_put: whole groups of query heads per key head (got %d / %d)", h.heads, h.kv_heads);
+  const int64_t cols = (int64_t)(h.heads + h.kv_heads) * h.dim + (int64_t)h.kv_heads * h.vdim;
+  FB_REQUIRE(ld >= cols && ld_q >= (int64_t)h.heads * h.dim && cache_rows >= 1 && head_stride >= cache_rows * (h.dim + h.vdim), "fb_heads_put: row strides too small");
+  FB_REQUIRE(!h.first || (h.share && h.ld_first >= (int64_t)h.kv_heads * h.vdim), "fb_heads_put: mixed values take the other layer's and their share");
+  FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32) && (in_dtype == FB_FP32 || dtype == FB_BF16),
+             "fb_heads_put: bf16 or fp32; fp32 results come from fp32");
+  const fb::HeadsPutArgs a{h, qkv, T, ld, rows, q_out, ld_q, cache, cache_rows, head_stride};
+  const dim3 grid((unsigned)fb::ceil_div(T * (h.heads + 2 * h.kv_heads), fb::HEADS_WARPS)), block(32 * fb::HEADS_WARPS);
+  const auto s = (cudaStream_t)stream;
+  if (in_dtype == FB_FP32 && dtype == FB_FP32) return fb::launch_after(fb::heads_put_kernel<float, float>, grid, block, 0, s, "fb_heads_put", a);
+  if (in_dtype == FB_FP32) return fb::launch_after(fb::heads_put_kernel<float, uint16_t>, grid, block, 0, s, "fb_heads_put", a);
+  return fb::launch_after(fb::heads_put_kernel<uint16_t, uint16_t>, grid, block, 0, s, "fb_heads_put", a);
+}
+
+extern "C" int fb_add_norm(const fb_branches* branches_host, int64_t T, int64_t cols, int in_dtype, int dtype, void* stream) {
+  FB_REQUIRE(branches_host && branches_host->x && T >= 1 && cols >= 1 && cols * 4 <= 200 * 1024, "fb_add_norm: null pointer, empty or rows past 51200 columns");
+  const fb_branches& a = *branches_host;
+  FB_REQUIRE(a.x_out || a.h, "fb_add_norm: no result");
+  FB_REQUIRE(!a.h || a.w, "fb_add_norm: a norm takes its weight");
+  FB_REQUIRE(!a.chosen || (a.slots && a.weights && a.k >= 1 && a.k <= 64), "fb_add_norm: chosen rows take their places and weights, up to 64 a token");
+  FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32) && (in_dtype == FB_FP32 || dtype == FB_BF16),
+             "fb_add_norm: bf16 or fp32; fp32 results come from fp32");
+  const auto s = (cudaStream_t)stream;
+  if (in_dtype == FB_FP32 && dtype == FB_FP32) return fb::launch_add_norm<float, float>(a, T, cols, s);
+  if (in_dtype == FB_FP32) return fb::launch_add_norm<float, uint16_t>(a, T, cols, s);
+  return fb::launch_add_norm<uint16_t, uint16_t>(a, T, cols, s);
+}

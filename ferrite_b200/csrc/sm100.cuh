@@ -116,6 +116,12 @@ __device__ __forceinline__ void tma_load_4d(uint32_t dst, const void* tmap, int 
                : "memory");
 }
 
+__device__ __forceinline__ void tma_load_5d(uint32_t dst, const void* tmap, int x, int y, int z, int w, int v, uint32_t bar) {
+  asm volatile("cp.async.bulk.tensor.5d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5, %6}], [%7];" ::"r"(dst),
+               "l"(tmap), "r"(x), "r"(y), "r"(z), "r"(w), "r"(v), "r"(bar)
+               : "memory");
+}
+
 // ---- thread-block clusters
 __device__ __forceinline__ void cluster_barrier() {  // every thread of every CTA of the cluster
   __syncwarp();

@@ -1,6 +1,9 @@
 """Layer parts beside the Llama block's (llama.attention, llama.mlp, llama.rms): token mixers that keep something per
-sequence - attention over cached latents, linear attention with a decaying state - a norm and a gated unit.  Every
-constant is a parameter; a design's module (binutar.py) says which parts it is made of.
+sequence, feed-forwards, a norm.  Every constant is a parameter; a design's module (binutar.py, labepel.py) says which parts
+it is made of.
+
+They are: attention over cached latents, grouped-query attention within spans of the sequence, linear attention with a
+decaying state; a clamped gated unit, a mixture of experts; Dynamic Tanh.
 
 A mixer is a pair of functions: `*_cache(m, size, zeros, slots)` makes what it keeps for `slots` sequences of size / slots
 places each, and the mixer itself maps normed rows to rows, given its weights, its sizes m and where the tokens stand
@@ -9,7 +12,16 @@ import math
 
 import torch
 
-from .tensor import Tensor
+from . import llama
+from .tensor import BFP, Tensor
+
+
+class Caches(list):
+    """A layer's cache or state each, for sequences that share `size` places."""
+
+    def __init__(self, size, caches):
+        super().__init__(caches)
+        self.size = size
 
 
 def dyt(x, p, name):
@@ -28,6 +40,29 @@ def clamped_mlp(h, p, pre, limit, slope):
     gate_up = h.matmul(p[pre + "gate_up"], dtype="fp32")
     m = gate_up.cols // 2
     return clamped_glu(gate_up[:, :m], gate_up[:, m:], limit, slope).cast(h.dtype).matmul(p[pre + "down"], dtype="fp32")
+
+
+def gated_mlp(h, p, pre):
+    """down(silu(gate(h)) * up(h)), gate and up side by side in gate_up."""
+    gate_up = p[pre + "gate_up"]
+    both = h.matmul(gate_up, dtype="bf16" if gate_up.dtype in BFP else "fp32")
+    m = gate_up.cols // 2
+    return llama.glu(both[:, :m], both[:, m:]).cast(h.dtype).matmul(p[pre + "down"], dtype=h.dtype)
+
+
+def mixture(h, logits, p, pre, k):
+    """A mixture of experts for rows h with their router logits (fp32): the k largest of each row's, weighted by their softmax.
+    p: gate_up and down as batches of experts, the router's bias if it has one (router.b), a shared expert's own pair
+    (shared.gate_up, shared.down) if there is one.  Returns (the shared expert's result or None, (the chosen experts' rows, their
+    routes)) as Tensor.add_norm adds them up."""
+    gate_up, down = p[pre + "gate_up"], p[pre + "down"]
+    routes = logits.route(gate_up.batch, k, p.get(pre + "router.b"))
+    shared = gated_mlp(h, p, pre + "shared.") if pre + "shared.gate_up" in p else None
+    if gate_up.dtype not in BFP:
+        return shared, (h.experts(routes, gate_up, down), routes)
+    of = lambda buf, dtype: Tensor(h.rt, routes.T, routes.k, dtype=dtype, buf=buf.view(1, routes.T, routes.k))
+    y = llama.experts(h, {"experts.gate_up": gate_up, "experts.down": down}, of(routes.ids, "int32"), of(routes.weights, "fp32"))
+    return (y if shared is None else shared + y), None
 
 
 # -------------------------------------------------------------------- rotation
@@ -82,6 +117,38 @@ def latent_attention(h, p, m, eps, at, cache):
     gates = down[:, :, down.cols - H:].permute(2, 1, 0)  # a number a head and token
     (o.split(H).matmul(p["mix.uv"]) * gates.sigmoid()).cast(h.dtype).realize(into=values.split(H))
     return values.matmul(p["mix.o"], dtype="fp32")
+
+
+# -------------------------------------------------------------------- grouped-query attention
+
+def heads_width(m):
+    """Columns of the joint projection: queries, keys, values, and a gate for each column of the result."""
+    return (m.heads + m.kv_heads) * m.dim + (m.kv_heads + m.heads) * m.vdim
+
+
+def heads_cache(m, size, zeros, slots):
+    """A key and its value side by side, a row a place and key head."""
+    return zeros((m.kv_heads, size, m.dim + m.vdim))
+
+
+def heads_attention(joint, p, m, eps, at, cache, sink=None):
+    """Attention of query heads that share key heads, each token within its own span of m.mask.size places.
+    joint: q | k | v | gate (| more), fp32; p: their biases side by side (mix.b), the heads' norms (mix.q.norm, mix.k.norm), the
+    output's matrix (mix.o); with m.v_mix, the values of the first such layer of the pass (at.first) are mixed in by mix.vmix.
+    sink: a number that joins every head's denominator as exp(sink)."""
+    H, n, wide = m.heads, (m.heads + m.kv_heads) * m.dim, m.kv_heads * m.vdim
+    base, last, length, _ = at.seen
+    mix = None
+    if m.v_mix:
+        mix = (*at.first, p["mix.vmix"]) if at.first else None
+        at.first = at.first or (joint[:, n:n + wide], p["mix.b"][:, n:])
+    q = joint.heads_put(H, m.dim, m.vdim, at.rows, cache, p["mix.b"], p["mix.q.norm"], p["mix.k.norm"], eps, mix)
+    key = ("sink", H, sink)
+    if sink is not None and key not in joint.rt.numbers:
+        joint.rt.numbers[key] = Tensor.of(joint.rt, [[sink] * H], "fp32")
+    gate = joint[:, n + wide:n + wide + H * m.vdim]
+    o = q.attend_heads(cache, base, last, m.vdim, m.scale, length, m.mask.size, joint.rt.numbers.get(key), gate, chunk=at.chunk)
+    return o.matmul(p["mix.o"], dtype=o.dtype)
 
 
 # -------------------------------------------------------------------- linear attention with a decaying state

@@ -2,9 +2,10 @@
 precision, forward, kv_cache, slot - and everything that drives a model (the checkpoint reader, the engine, the command
 line) finds it here: by a config's `family`, or, when a checkpoint is opened, by config.json."""
 import importlib
+from types import SimpleNamespace
 
-FAMILIES = {"llama": "llama", "binutar": "binutar"}  # a config's family -> its module of this package
-ARCHITECTURES = {"Binutar": "binutar"}  # config.json's "architecture" -> family (Hugging Face configs, which have none, are Llama-like)
+FAMILIES = {"llama": "llama", "binutar": "binutar", "labepel": "labepel"}  # a config's family -> its module of this package
+ARCHITECTURES = {"Binutar": "binutar", "Labepel": "labepel"}  # config.json's "architecture" -> family (Hugging Face configs, which have none, are Llama-like)
 
 
 def module(family):
@@ -27,3 +28,8 @@ def family_of_json(j):
 def of_json(j):
     """The family module of a parsed config.json."""
     return module(family_of_json(j))
+
+
+def sizes(x):
+    """A parsed config's object, and those inside it, with its keys as names."""
+    return SimpleNamespace(**{k: sizes(v) if isinstance(v, dict) else v for k, v in x.items()})

@@ -332,3 +332,104 @@ def dense(x, w, out, settled=False, /, kind=_lib.DENSE_NONE, **extra):
                          w.stride(0) if batch > 1 else 0, batch, out.data_ptr(), _CODES[out.dtype], out.stride(1), out.stride(0), ctypes.byref(e), int(settled), _stream()))
     count()
     return out
+
+
+def embed(table, ids, places_table, places, out):
+    """out (fp32) = table[ids] + places_table[places] (fb_embed)."""
+    check(lib().fb_embed(_CODES[table.dtype], table.data_ptr(), table.shape[0], table.shape[1], ids.data_ptr(), _ptr(places_table), places_table.shape[0] if places_table is not None else 0,
+                         _ptr(places), ids.numel(), out.data_ptr(), _stream()))
+    count()
+    return out
+
+
+def heads_put(qkv, heads, kv_heads, dim, vdim, rows, cache, q_out, bias=None, q_norm=None, k_norm=None, eps=0.0, first=None, first_bias=None, share=None):
+    """Biases, norms, mixed values and the cache write after a joint projection of heads (fb_heads_put); cache [kv_heads, rows, dim + vdim]."""
+    h = _lib.Heads(heads, kv_heads, dim, vdim, _ptr(bias), _ptr(q_norm), _ptr(k_norm), eps, _ptr(first), first.stride(0) if first is not None else 0, _ptr(first_bias), _ptr(share))
+    assert cache.shape[0] == kv_heads and cache.shape[2] == dim + vdim and cache.stride(2) == 1 and cache.stride(1) == dim + vdim and q_out.dtype == cache.dtype
+    check(lib().fb_heads_put(ctypes.byref(h), _CODES[qkv.dtype], qkv.data_ptr(), qkv.shape[0], qkv.stride(0), rows.data_ptr(), _CODES[cache.dtype], q_out.data_ptr(), q_out.stride(0),
+                             cache.data_ptr(), cache.shape[1], cache.stride(0), _stream()))
+    count()
+    return q_out
+
+
+def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, span=0, sink=None, gate=None, row0=0, out=None):
+    """q [T, heads * dim] over cache [kv_heads, rows, dim + vdim] (fb_heads_attention)."""
+    T, dim = q.shape[0], cache.shape[2] - vdim
+    assert q.shape[1] == heads * dim and q.dtype == cache.dtype and cache.stride(2) == 1 and cache.stride(1) == cache.shape[2]
+    assert last.dtype == torch.int32 and last.numel() == T and (base is None or base.numel() == T)
+    if out is None:
+        out = torch.empty(T, heads * vdim, dtype=q.dtype, device=q.device)
+    check(lib().fb_heads_attention(_CODES[q.dtype], q.data_ptr(), T, q.stride(0), heads, cache.shape[0], dim, vdim, cache.data_ptr(), cache.shape[1], cache.stride(0), _ptr(base), row0,
+                                   last.data_ptr(), max_keys, int(chunk), span, scale, _ptr(sink), _CODES[gate.dtype] if gate is not None else 0, _ptr(gate),
+                                   gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), _stream()))
+    count()
+    return out
+
+
+class Routes:
+    """Where a mixture's rows go (fb_route): tokens' weights and slots [T, k], the rows' tokens (order; None: every tile holds
+    all the tokens), the tiles' experts, how many tiles are in use, and the sizes of all that."""
+
+    def __init__(self, device, T, n, k, tile, shared):
+        self.T, self.n, self.k, self.tile, self.shared = T, n, k, tile, shared
+        self.tiles = lib().fb_route_tiles(T, n, k, tile, int(shared))
+        i32 = lambda *shape: torch.empty(*shape, dtype=torch.int32, device=device)
+        self.weights, self.ids, self.slots = torch.empty(T, k, dtype=torch.float32, device=device), i32(T, k), i32(T, k)
+        self.order, self.tile_expert, self.live = None if shared else i32(self.tiles * tile), i32(self.tiles), i32(1)
+
+
+def route_tile(T, n, k):
+    """(rows of a tile, whether each tile holds all the tokens) for T tokens with k of n experts each: a few tokens are not
+    sorted, more take tiles about as high as an expert has rows (the fuller the tiles, the fewer times its weights are read)."""
+    if T <= 64:
+        return -(-T // 16) * 16, True
+    rows = T * k / n
+    return (256 if rows >= 384 else 128 if rows >= 80 else 64 if rows >= 40 else 32), False
+
+
+def route(logits, n, k, bias=None):
+    """Router logits (fp32 [T, >= n]) to Routes."""
+    T = logits.shape[0]
+    tile, shared = route_tile(T, n, k)
+    r = Routes(logits.device, T, n, k, tile, shared)
+    check(lib().fb_route(logits.data_ptr(), T, logits.stride(0), _ptr(bias), n, k, tile, int(shared), r.weights.data_ptr(), r.ids.data_ptr(), r.slots.data_ptr(), _ptr(r.order),
+                         r.tile_expert.data_ptr(), r.live.data_ptr(), _stream()))
+    count(1 if T <= 128 else 2)
+    return r
+
+
+def grouped(x, w, routes, out, kind=_lib.DENSE_NONE, shared=False):
+    """Rows of tiles (shared: x's rows in every tile) by each tile's matrix of the batch w [n, K, N]: on the tensor cores
+    where operands allow it (with a gated unit, if asked for); False where they do not."""
+    n, K, N = w.shape
+    if not (x.dtype == w.dtype == torch.bfloat16 and x.stride(1) == 1 and w.stride(1) == 1 and lib().fb_dense_supports(
+            x.data_ptr(), x.stride(0), 0, w.data_ptr(), w.stride(2), w.stride(0) if n > 1 else 0, K, N, kind)):
+        return False
+    e = _lib.DenseEpilogue(kind=kind)
+    check(lib().fb_dense_grouped(x.data_ptr(), x.shape[0], K, x.stride(0), int(shared), w.data_ptr(), N, w.stride(2), w.stride(0), n, routes.tile_expert.data_ptr(),
+                                 routes.live.data_ptr(), routes.tiles, routes.tile, out.data_ptr(), _CODES[out.dtype], out.stride(0), ctypes.byref(e), _stream()))
+    count()
+    return True
+
+
+def grouped_matmul(x, w, routes, out, shared=False):
+    """The same without a unit for any sizes, bf16 or fp32 (fb_grouped_matmul)."""
+    n, K, N = w.shape
+    assert x.stride(1) == 1 and out.stride(1) == 1
+    check(lib().fb_grouped_matmul(_CODES[x.dtype], x.data_ptr(), x.shape[0], x.stride(0), int(shared), _CODES[w.dtype], w.data_ptr(), (ctypes.c_int64 * 3)(*w.stride()), n, K, N,
+                                  routes.tile_expert.data_ptr(), routes.live.data_ptr(), routes.tiles, routes.tile, _CODES[out.dtype], out.data_ptr(), out.stride(0), _stream()))
+    count()
+    return out
+
+
+def add_norm(x, x_out, mixer=None, mixer_scale=None, other=None, other_scale=None, chosen=None, routes=None, w=None, plus=0.0, eps=0.0, h=None):
+    """A layer's end (fb_add_norm): x [T, cols] fp32 plus its branches into x_out, and that normed by w + plus into h."""
+    ld = lambda t: t.stride(0) if t is not None else 0
+    of = lambda *ts: next((t.dtype for t in ts if t is not None), None)
+    dtype = of(h, chosen) or torch.float32
+    kind = of(mixer, other) or dtype if dtype == torch.bfloat16 else torch.float32
+    assert all(t is None or t.dtype == kind for t in (mixer, other)) and all(t is None or t.dtype == dtype for t in (h, chosen))
+    b = _lib.Branches(x.data_ptr(), ld(x), _ptr(mixer), ld(mixer), _ptr(mixer_scale), _ptr(other), ld(other), _ptr(other_scale), _ptr(chosen), ld(chosen),
+                      _ptr(routes.slots) if routes else None, _ptr(routes.weights) if routes else None, routes.k if routes else 0, _ptr(x_out), ld(x_out), _ptr(w), plus, eps, _ptr(h), ld(h))
+    check(lib().fb_add_norm(ctypes.byref(b), x.shape[0], x.shape[1], _CODES[kind], _CODES[dtype], _stream()))
+    count()

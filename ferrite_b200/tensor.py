@@ -7,7 +7,7 @@ sm_100a kernels reached through the C ABI (ferrite_b200/_lib.py), launched on to
 maps the trees a Llama block builds onto the fused kernels:
 
     x * rsqrt(mean(x*x) + eps) * w  feeding a block-float matmul   -> RMSNorm prologue of fb_linear
-    silu(mm[:, :m]) * mm[:, m:]                                      -> SwiGLU epilogue of fb_linear
+    silu(mm[:, :m]) * mm[:, m:]                                      -> SwiGLU epilogue of fb_linear (bf16 weights: fb_dense)
     x + mm                                                           -> residual epilogue of fb_linear
     any other elementwise tree                                       -> one fb_elementwise launch (postfix program)
 
@@ -607,6 +607,98 @@ class Tensor:
         self.rt.launched("gated rmsnorm")
         return out
 
+    # ---------------------------------------------------------------- an fp32 residual stream with grouped-query heads and experts
+
+    def embed(self, ids, places_table=None, places=None):
+        """Rows ids of this table, plus rows `places` of another where given, as an fp32 matrix: a residual stream's start."""
+        ids, places = ids.realize(), None if places is None else places.realize()
+        out = Tensor(self.rt, ids.cols, self.cols, dtype="fp32")
+        assert places_table is None or (places_table.cols == self.cols and places_table.dtype == self.dtype and places.cols == ids.cols)
+        ops.embed(self.realize().buf[0], ids.buf.reshape(-1), None if places_table is None else places_table.realize().buf[0], None if places is None else places.buf.reshape(-1), out.buf[0])
+        self.rt.launched("embed")
+        return out
+
+    def heads_put(self, heads, dim, vdim, rows, cache, bias=None, q_norm=None, k_norm=None, eps=0.0, mix=None):
+        """self: a joint projection [1, tokens, q (heads x dim) | k | v (| more)]; its keys and values go into `cache` ([key
+        heads, size, dim + vdim]) at `rows`, its queries come back, as the cache is stored.  bias: a number a column of q | k | v;
+        q_norm, k_norm: RMSNorm of each head; mix: (other values of the tokens, their bias or None, share): the values become
+        (1 - share) own + share other."""
+        x, rows = self.realize(), rows.realize()
+        assert x.batch == 1 and x.buf.stride(2) == 1 and rows.cols == x.rows and x.cols >= (heads + cache.batch) * dim + cache.batch * vdim, f"{self.shape} into a cache {cache.shape}"
+        assert all(t is None or t.dtype == "fp32" for t in (bias, q_norm, k_norm)) and (bias is None or bias.cols == (heads + cache.batch) * dim + cache.batch * vdim)
+        buf = lambda t: None if t is None else t.realize().buf
+        first, first_bias, share = mix or (None, None, None)
+        assert first is None or (first.dtype == x.dtype and first.shape == (1, x.rows, cache.batch * vdim) and first.buf.stride(2) == 1), "the other layer's values, a column each of this one's"
+        out = Tensor(self.rt, x.rows, heads * dim, dtype=cache.dtype)
+        ops.heads_put(x.buf[0], heads, cache.batch, dim, vdim, rows.buf.reshape(-1), cache.buf, out.buf[0], buf(bias), buf(q_norm), buf(k_norm), eps,
+                      None if first is None else first.buf[0], buf(first_bias), buf(share))
+        self.rt.launched("heads put")
+        return out
+
+    def attend_heads(self, cache, base, last, vdim, scale, length=None, span=0, sink=None, gate=None, chunk=False):
+        """self: [1, tokens, heads x dim] over such a cache.  Token t, which stands at place last[t], attends the rows from base[t]
+        on up to its own; with span, only those of its own span of that many places.  sink: a number per head that joins the
+        softmax's denominator; gate: the result is multiplied by its sigmoid, column by column; chunk: one sequence's tokens,
+        its first cache row 0.  Returns [1, tokens, heads x vdim]."""
+        q, last = self.realize(), last.realize()
+        dim = cache.cols - vdim
+        assert q.batch == 1 and q.cols % dim == 0 and q.dtype == cache.dtype and (q.cols // dim) % cache.batch == 0, f"{q.shape} over a cache {cache.shape}"
+        heads = q.cols // dim
+        out = Tensor(self.rt, q.rows, heads * vdim, dtype=q.dtype)
+        assert gate is None or gate.shape == out.shape
+        ops.heads_attention(q.buf[0], cache.buf, None if chunk else base.realize().buf.reshape(-1), last.buf.reshape(-1), heads, vdim, scale, min(length or cache.rows, cache.rows), chunk, span,
+                            None if sink is None else sink.realize().buf, None if gate is None else gate.realize().buf[0], out=out.buf[0])
+        self.rt.launched("attention")
+        return out
+
+    def route(self, n, k, bias=None):
+        """self: fp32 router logits, n a token: each token's k experts, their weights and where their rows go (ops.Routes)."""
+        x = self.realize()
+        assert x.dtype == "fp32" and x.batch == 1 and x.cols == n and x.buf.stride(2) == 1 and (bias is None or (bias.dtype == "fp32" and bias.cols == n))
+        self.rt.launched("route")
+        return ops.route(x.buf[0], n, k, None if bias is None else bias.realize().buf)
+
+    def experts(self, routes, gate_up, down):
+        """self: rows of tokens.  Every chosen expert's down(silu(gate) * up) of its tokens' rows, a row a choice where `routes`
+        puts it; gate and up side by side in gate_up [n, K, 2 m], down [n, m, N]."""
+        rt, h, m = self.rt, self.realize(), down.rows
+        assert h.batch == 1 and gate_up.cols == 2 * m and gate_up.batch == down.batch == routes.n and h.rows == routes.T
+        if not routes.shared:
+            h = h if h.buf.is_contiguous() else (h + 0).realize()
+            x = Tensor(rt, routes.tiles * routes.tile, h.cols, dtype=h.dtype)
+            ops.gather_rows(h.buf[0], routes.order, x.buf[0])
+            rt.launched("gather")
+            h = x
+        act = Tensor(rt, routes.tiles * routes.tile, m, dtype=h.dtype)
+        out = Tensor(rt, routes.tiles * routes.tile, down.cols, dtype=h.dtype)
+        if ops.grouped(h.buf[0], gate_up.buf, routes, act.buf[0], _lib.DENSE_SWIGLU, routes.shared):
+            rt.launched("experts swiglu")
+        else:
+            both = Tensor(rt, act.rows, 2 * m, dtype="fp32")
+            ops.grouped_matmul(h.buf[0], gate_up.buf, routes, both.buf[0], routes.shared)
+            rt.launched("experts matmul")
+            (both[:, :m].silu() * both[:, m:]).cast(h.dtype).realize(into=act)
+        if ops.grouped(act.buf[0], down.buf, routes, out.buf[0]):
+            rt.launched("experts")
+        else:
+            ops.grouped_matmul(act.buf[0], down.buf, routes, out.buf[0])
+            rt.launched("experts matmul")
+        return out
+
+    def add_norm(self, w, eps, plus=0.0, dtype="bf16", mixer=None, mixer_scale=None, other=None, other_scale=None, experts=None):
+        """self: an fp32 residual stream.  (self + mixer * mixer_scale + (other + the experts' rows by their weights) *
+        other_scale, and that as RMSNorm by w + plus leaves it); experts: (rows, routes).  Without branches: (self, its norm)."""
+        x = self.realize()
+        get = lambda t: None if t is None else t.realize().buf[0]
+        assert x.dtype == "fp32" and x.batch == 1 and all(t is None or (t.shape == x.shape and t.buf.stride(2) == 1) for t in (mixer and mixer.realize(), other and other.realize()))
+        bare = mixer is other is experts is None
+        out, h = x if bare else Tensor(self.rt, x.rows, x.cols, dtype="fp32"), Tensor(self.rt, x.rows, x.cols, dtype=dtype)
+        scale = lambda t: None if t is None else t.realize().buf
+        rows, routes = experts or (None, None)
+        ops.add_norm(x.buf[0], None if bare else out.buf[0], get(mixer), scale(mixer_scale), get(other), scale(other_scale), get(rows), routes, w.realize().buf, plus, eps, h.buf[0])
+        self.rt.launched("norm" if bare else "add norm")
+        return out, h
+
     def greedy(self, values=None):
         """Each row's first largest logit's column, int32 [1, 1, rows], picked on the device (the reference reads the
         logits back and takes numpy's argmax, models/llama.py:787-795): fp32 logits of one matrix."""
@@ -787,6 +879,17 @@ def _match_clamped_glu(t):
     return mm, float(limit), float(neg.srcs[0].srcs[1])
 
 
+def _match_swiglu(t):
+    """The matmul if t is silu(mm[:, :m]) * mm[:, m:] over the halves of one matmul not yet computed, else None."""
+    for g, u in (t.srcs, t.srcs[::-1]):
+        gate = _match_silu_of(g)
+        if gate is not None and isinstance(u, Tensor) and gate.op == u.op == "cols" and gate.srcs[0] is u.srcs[0]:
+            mm = gate.srcs[0]
+            if gate.args["start"] == 0 and u.args["start"] == gate.cols and 2 * gate.cols == mm.cols and mm.batch == 1:
+                return mm
+    return None
+
+
 def _match_gated(t):
     """(matmul, gate) if t is matmul * gate.sigmoid(), a number a row of each of the matmul's batch, else None."""
     if t.op != "mul" or not all(isinstance(s, Tensor) for s in t.srcs):
@@ -809,7 +912,7 @@ def _dense(t, mm, into, kind, **extra):
     a, w = mm.srcs
     if not (a.dtype == "bf16" and w.dtype == "bf16" and w.op is None and a.batch == w.batch and w.buf.stride(1) == 1 and w.rows % 8 == 0 and w.buf.stride(2) % 8 == 0):
         return False
-    if kind == _lib.DENSE_GLU and w.cols % 32:
+    if kind in (_lib.DENSE_GLU, _lib.DENSE_SWIGLU) and w.cols % 32:
         return False
     x = a.realize()
     if not ops.dense_supports(x.buf, w.buf, kind):
@@ -828,7 +931,7 @@ def _dense(t, mm, into, kind, **extra):
         elif v is not None:
             fields[name] = v
     ops.dense(x.buf, w.buf, out.buf, getattr(w, "settled", False), kind=kind, **fields)
-    t.rt.launched("dense" + ("", " silu", " glu", " gate", " dyt add")[kind])
+    t.rt.launched("dense" + ("", " silu", " glu", " gate", " dyt add", " swiglu")[kind])
     _done(t, buf=out.buf)
     if into is not None and out is not into:
         _copy(t, into)
@@ -849,6 +952,9 @@ def _fused_dense(t, into, hand_on=None):
         found = _match_gated(inner)
         if found:
             return _dense(t, found[0], into, _lib.DENSE_GATE, gate=found[1])
+        found = _match_swiglu(inner)
+        if found:
+            return _dense(t, found, into, _lib.DENSE_SWIGLU)
     if t.op == "cast" and t.dtype == "bf16" and t.batch == 1:
         found = _match_dyt(inner)
         if found and found[0].op == "add" and found[0].dtype == "fp32":

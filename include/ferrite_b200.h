@@ -149,8 +149,9 @@ enum fb_dense_epilogue_kind {
   FB_DENSE_GLU = 2,     /* W holds gate rows, then as many up rows: out = g sigmoid(slope g) (u + 1), g = min(gate, limit), u = up in -limit .. limit;
                            out is [M, N / 2] */
   FB_DENSE_GATE = 3,    /* times sigmoid(gate[t * ld_gate + batch entry]) */
-  FB_DENSE_DYT_ADD = 4  /* out (fp32) = residual + tanh(alpha acc) w + b, and, with h_out given, h_out (bf16) = tanh(alpha2 out) w2 + b2: a Dynamic
+  FB_DENSE_DYT_ADD = 4, /* out (fp32) = residual + tanh(alpha acc) w + b, and, with h_out given, h_out (bf16) = tanh(alpha2 out) w2 + b2: a Dynamic
                            Tanh on a branch, the residual add, and the Dynamic Tanh that the next branch starts with */
+  FB_DENSE_SWIGLU = 5   /* as FB_DENSE_GLU, the plain unit: out = g sigmoid(g) u */
 };
 typedef struct {
   int kind;
@@ -172,6 +173,29 @@ typedef struct {
 int fb_dense_supports(const void* x, int64_t ldx, int64_t x_batch, const void* W, int64_t ldw, int64_t w_batch, int64_t K, int64_t N, int kind);
 int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_t x_batch, const void* W, int64_t N, int64_t ldw, int64_t w_batch, int64_t batch,
              void* out, int out_dtype, int64_t ldo, int64_t out_batch, const fb_dense_epilogue* epilogue_host, int settled, void* stream);
+
+/* ---- a mixture of experts with bf16 or fp32 weights ------------------------------------------------------ */
+
+/* Each token's k largest of n router logits (fp32, + bias where given; the lower column first among equals) and the softmax of
+ * those (weights), and where each choice's row goes (slots, both [T, k]) in rows of whole tiles of `tile` (a multiple of 16):
+ *   shared_rows   a tile a touched expert, holding all the tokens (T <= tile): the choice's row is the token's in its expert's tile
+ *   otherwise     each expert's choices in tiles of their own; order[tiles * tile]: the token each row holds, -1 for none
+ * tile_expert[tiles]: each tile's expert, ascending (n past those used); live[0]: how many are used; tiles =
+ * fb_route_tiles(...), the most there can be.  ids [T, k]: the choices. */
+int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_rows);
+int fb_route(const float* logits, int64_t T, int64_t ld, const float* bias, int n, int k, int tile, int shared_rows, float* weights, int32_t* ids,
+             int32_t* slots, int32_t* order, int32_t* tile_expert, int32_t* live, void* stream);
+
+/* Rows of tiles by each tile's own matrix: rows i * tile .. of out = rows i * tile .. of x (shared_rows: x's `x_rows` rows, the
+ * same for every tile) @ W[tile_expert[i]]^T for the tiles i < live[0]; the other rows of out are left alone.
+ * fb_dense_grouped: on the tensor cores, operands as fb_dense takes them (W [n, N, K], w_batch elements apart), epilogues
+ * FB_DENSE_NONE, FB_DENSE_GLU and FB_DENSE_SWIGLU.  fb_grouped_matmul: any sizes, bf16 or fp32, W by strides (matrix, row of K, column). */
+int fb_dense_grouped(const void* x, int64_t x_rows, int64_t K, int64_t ldx, int shared_rows, const void* W, int64_t N, int64_t ldw, int64_t w_batch,
+                     int n, const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, void* out, int out_dtype, int64_t ldo,
+                     const fb_dense_epilogue* epilogue_host, void* stream);
+int fb_grouped_matmul(int x_dtype, const void* x, int64_t x_rows, int64_t ldx, int shared_rows, int w_dtype, const void* W, const int64_t* w_strides_host, int n,
+                      int64_t K, int64_t N, const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, int out_dtype, void* out,
+                      int64_t ldo, void* stream);
 
 /* Tensor.matmul(index=) (ferrite/tensor.py:450-460; ferrite/compiler.py:704-706): a mixture of experts' matmul.  W is
  * a batch of n_experts packed [K, N] matrices fb_packed_bytes(fmt, K, N) apart; index[slot] (int32, read on the
@@ -366,6 +390,61 @@ int fb_decay_scan(int dtype, const void* qkv, int64_t ld, int heads, int dim, in
 /* out = RMSNorm(x) * w * sigmoid(gate), row by row; x, w fp32, gate and out of `dtype` */
 int fb_gated_rmsnorm(const float* x, int64_t rows, int64_t cols, int64_t ldx, int dtype, const void* gate, int64_t ld_g, const float* w, float eps,
                      void* out, int64_t ldo, void* stream);
+
+/* ---- grouped-query attention over rows of a key and its value, and what stands around it ------------------- */
+
+/* out[t] = table[ids[t]] + places_table[places[t]] (or the first alone) in fp32; ids and places outside are clamped */
+int fb_embed(int dtype, const void* table, int64_t rows, int64_t cols, const int32_t* ids, const void* places_table, int64_t place_rows,
+             const int32_t* places, int64_t T, float* out, void* stream);
+
+typedef struct {
+  int heads, kv_heads, dim, vdim; /* dim: a query's and a key's columns, vdim: a value's */
+  const float* bias;              /* one a column of q | k | v, or null */
+  const float *q_norm, *k_norm;   /* [dim]: RMSNorm of each head, all heads by the same weight; null: none */
+  float eps;
+  const void* first;              /* other values of the same tokens (kv_heads * vdim columns, stored as qkv is), or null: the value
+                                     becomes (1 - share) value + share (first + first_bias) */
+  int64_t ld_first;
+  const float *first_bias, *share; /* share: one number on the device */
+} fb_heads;
+/* After a joint projection q (heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim) (| more): biases and norms in fp32, queries
+ * to q_out, and (key | value) into row rows[t] of each key head of cache [kv_heads, cache_rows, dim + vdim] (heads head_stride
+ * elements apart; a row outside is not written).  in_dtype: how qkv is stored, dtype: q_out and the cache. */
+int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void* qkv, int64_t T, int64_t ld, const int32_t* rows, int dtype, void* q_out,
+                 int64_t ld_q, void* cache, int64_t cache_rows, int64_t head_stride, void* stream);
+
+/* Attention over such a cache: query head h reads key head h / (heads / kv_heads); token t, whose place is last[t], sees the cache
+ * rows base[t] + row0 + lo .. + last[t] (base null: row0 alone), lo = 0, or, with span, the first place of its span of `span`
+ * places.  sink (fp32 [heads], or null): exp(sink[h]) joins head h's denominator.  gate (or null): the result times its sigmoid,
+ * column by column.  chunk: the tokens are consecutive ones of one sequence.  max_keys: an upper bound of last[t] + 1. */
+int fb_heads_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int kv_heads, int dim, int vdim, const void* cache,
+                       int64_t cache_rows, int64_t head_stride, const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk,
+                       int span, float scale, const float* sink, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o,
+                       void* stream);
+
+typedef struct {
+  const float* x; /* the residual stream [T, cols] */
+  int64_t ld_x;
+  const void* mixer; /* a branch's result and its scale by column (or null: 1) */
+  int64_t ld_mixer;
+  const float* mixer_scale;
+  const void* other; /* the other branch's; a mixture adds to it the rows slots[t, j] of `chosen`, times weights[t, j] */
+  int64_t ld_other;
+  const float* other_scale;
+  const void* chosen;
+  int64_t ld_chosen;
+  const int32_t* slots;
+  const float* weights;
+  int k;
+  float* x_out; /* x + mixer * mixer_scale + (other + chosen) * other_scale, or null */
+  int64_t ld_x_out;
+  const float* w; /* h = RMSNorm of that, times (w + plus); h null: none */
+  float plus, eps;
+  void* h;
+  int64_t ld_h;
+} fb_branches;
+/* A layer's end and the next one's start.  Branches null: not there.  in_dtype: mixer and other; dtype: chosen and h. */
+int fb_add_norm(const fb_branches* branches_host, int64_t T, int64_t cols, int in_dtype, int dtype, void* stream);
 
 /* ---- several GPUs -------------------------------------------------------------------------------------- */
 
