@@ -27,8 +27,8 @@ struct RouteArgs {
 // the k largest of a token's logits, the lower column first among equals, and the softmax of those: a warp a token
 __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int lane) {
   const float* z = a.logits + t * a.ld;
-  float prev = INFINITY, mine = -INFINITY;
-  int prev_at = -1, my_id = 0;
+  float prev = INFINITY, mine[2] = {-INFINITY, -INFINITY};  // lane j keeps the picks j and 32 + j
+  int prev_at = -1, my_id[2] = {0, 0};
   float held[4];  // the first 128 columns stay in registers
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
@@ -54,10 +54,13 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
     }
     if (at == a.n) at = 0;  // (only where a logit is not a number)
     prev = best, prev_at = at;
-    if (lane == j) mine = best, my_id = at;
+    if (j < 32 && lane == j) mine[0] = best, my_id[0] = at;
+    if (j >= 32 && lane == j - 32) mine[1] = best, my_id[1] = at;
   }
-  const float top = __shfl_sync(0xffffffffu, mine, 0), e = lane < a.k ? expf(mine - top) : 0.f, sum = warp_sum(e);
-  if (lane < a.k) a.weights[t * a.k + lane] = e / sum, a.ids[t * a.k + lane] = my_id;
+  const float top = __shfl_sync(0xffffffffu, mine[0], 0);
+  const float e0 = lane < a.k ? expf(mine[0] - top) : 0.f, e1 = lane + 32 < a.k ? expf(mine[1] - top) : 0.f, sum = warp_sum(e0 + e1);
+  if (lane < a.k) a.weights[t * a.k + lane] = e0 / sum, a.ids[t * a.k + lane] = my_id[0];
+  if (lane + 32 < a.k) a.weights[t * a.k + lane + 32] = e1 / sum, a.ids[t * a.k + lane + 32] = my_id[1];
 }
 
 __global__ void __launch_bounds__(256) route_tokens_kernel(const RouteArgs a) {
@@ -184,7 +187,7 @@ extern "C" int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_
 extern "C" int fb_route(const float* logits, int64_t T, int64_t ld, const float* bias, int n, int k, int tile, int shared_rows, float* weights, int32_t* ids, int32_t* slots,
                         int32_t* order, int32_t* tile_expert, int32_t* live, void* stream) {
   FB_REQUIRE(logits && weights && ids && slots && tile_expert && live && T >= 1 && T <= (1 << 24), "fb_route: null pointer or no tokens");
-  FB_REQUIRE(n >= 1 && n <= 8192 && k >= 1 && k <= 32 && k <= n && ld >= n, "fb_route: up to 32 choices among up to 8192 experts (got %d of %d)", k, n);
+  FB_REQUIRE(n >= 1 && n <= 8192 && k >= 1 && k <= 64 && k <= n && ld >= n, "fb_route: up to 64 choices among up to 8192 experts (got %d of %d)", k, n);
   FB_REQUIRE(tile >= 16 && tile % 16 == 0 && (shared_rows ? T <= tile : order != nullptr), "fb_route: tiles of whole runs of 16 rows; shared rows: all the tokens in one");
   const int64_t tiles = fb_route_tiles(T, n, k, tile, shared_rows);
   FB_REQUIRE(tiles * tile < (1ll << 31), "fb_route: too many rows");

@@ -7,6 +7,6 @@ of the benchmark), never the thing that is shipped or measured as the product.
 Parity status: PINNED.  Every function here is checked against the reference's
 own numpy code (models/gpt2.py, models/llama.py), imported unmodified in the
 build container by tests/golden/make_golden.py, and against the fixtures that
-script commits under tests/golden/.  binutar.py stands apart: that design has no reference code, and the
-file is its equations in plain numpy.
+script commits under tests/golden/.  binutar.py and labepel.py stand apart: those designs have no reference
+code, and the files are their equations in plain numpy.
 """

@@ -44,7 +44,7 @@ def project(h, w, name):
 
 def mix_values(v, first, share):
     """The layer's values and the first mixing layer's of the same token; the first such layer's are its own."""
-    return v if first is None else (1 - share) * v + share * first
+    return v if first is None else (1 - share) * v + share * first.reshape(v.shape)
 
 
 def attention(h, w, pre, m, eps, places, cache, shared):

@@ -96,3 +96,34 @@ def test_dense_latent_and_decay_entry_points_refuse_bad_arguments_without_a_gpu(
     assert rc == -1 and b"up to 512" in lib.fb_last_error()
     rc = lib.fb_gated_rmsnorm(16, 2, 64, 32, _lib.BF16, 16, 64, 16, 1e-5, 16, 64, None)
     assert rc == -1
+
+
+def test_heads_and_experts_entry_points_refuse_bad_arguments_without_a_gpu():
+    import ctypes
+    lib = _lib.lib()
+    h = _lib.Heads(heads=5, kv_heads=2, dim=8, vdim=8)
+    rc = lib.fb_heads_put(ctypes.byref(h), _lib.FP32, 16, 4, 64, 16, _lib.BF16, 16, 40, 16, 64, 64 * 16, None)
+    assert rc == -1 and b"whole groups" in lib.fb_last_error()
+    rc = lib.fb_heads_put(ctypes.byref(_lib.Heads(heads=4, kv_heads=2, dim=8, vdim=8)), _lib.BF16, 16, 4, 64, 16, _lib.FP32, 16, 32, 16, 64, 64 * 16, None)
+    assert rc == -1 and b"fp32 results come from fp32" in lib.fb_last_error()
+    attend = lambda heads, dim, span, chunk=0, base=16: lib.fb_heads_attention(_lib.BF16, 16, 2, heads * dim, heads, 2, dim, 64, 16, 64, 64 * (dim + 64), base, 0, 16, 64, chunk, span, 1.0, None, 0,
+                                                                               None, 0, 16, heads * 64, None)
+    assert attend(3, 64, 0) == -1 and b"whole groups" in lib.fb_last_error()
+    assert attend(4, 2048, 0) == -1 and b"up to 1024" in lib.fb_last_error()
+    assert attend(4, 64, -1) == -1 and attend(4, 64, 8, chunk=1) == -1 and b"one sequence's" in lib.fb_last_error()
+    assert lib.fb_route_tiles(5, 12, 4, 16, 1) == 12 and lib.fb_route_tiles(1, 12, 4, 16, 1) == 4 and lib.fb_route_tiles(100, 12, 4, 32, 0) == 400 // 32 + 12
+    rc = lib.fb_route(16, 100, 12, None, 12, 4, 64, 1, 16, 16, 16, None, 16, 16, None)
+    assert rc == -1 and b"all the tokens in one" in lib.fb_last_error()
+    rc = lib.fb_route(16, 4, 70, None, 70, 65, 16, 1, 16, 16, 16, None, 16, 16, None)
+    assert rc == -1 and b"up to 64 choices" in lib.fb_last_error()
+    e = _lib.DenseEpilogue(kind=_lib.DENSE_DYT_ADD)
+    rc = lib.fb_dense_grouped(16, 64, 64, 64, 0, 16, 64, 64, 4096, 2, 16, 16, 2, 32, 16, _lib.BF16, 64, ctypes.byref(e), None)
+    assert rc == -1 and b"a gated unit" in lib.fb_last_error()
+    rc = lib.fb_dense_grouped(16, 64, 64, 64, 0, 16, 64, 64, 4096, 2, 16, 16, 3, 32, 16, _lib.BF16, 64, None, None)
+    assert rc == -1 and b"all of them there" in lib.fb_last_error()
+    rc = lib.fb_grouped_matmul(_lib.FP32, 16, 8, 64, 0, _lib.FP32, 16, (ctypes.c_int64 * 3)(4096, 1, 64), 2, 64, 64, 16, 16, 1, 16, _lib.FP32, 16, 64, None)
+    assert rc == -1 and b"rows there" in lib.fb_last_error()
+    rc = lib.fb_add_norm(ctypes.byref(_lib.Branches(x=16, h=16)), 2, 64, _lib.BF16, _lib.BF16, None)
+    assert rc == -1 and b"takes its weight" in lib.fb_last_error()
+    rc = lib.fb_embed(_lib.BF16, 16, 8, 64, 16, 16, 0, None, 2, 16, None)
+    assert rc == -1 and b"takes the places" in lib.fb_last_error()
