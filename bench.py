@@ -3,7 +3,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--workload llama8b|smollm] [--layers L] [--impl reference]
     python bench.py --matmul 32,4096,14336,bfp8,6      (one isolated matmul, a few calls: what the ncu captures run)
     python bench.py --attend 32,32,8,128,2048,6        (the decode attention alone, likewise)
-    python bench.py --design binutar                   (prefill, decode and kernels of that design beside the Llama decoder)
+    python bench.py --design binutar|labepel           (prefill, decode and kernels of that design beside the Llama decoder)
 
 The default workload is the Llama-3.1-8B-shape batched decode (32 sequences, 2048 tokens of context each, bfp8 weights,
 bf16 KV cache), tensor-parallel over N GPUs with an NCCL all-reduce after o_proj and down_proj.  A step is one decode
@@ -64,7 +64,7 @@ def parse():
     ap.add_argument("--sweep", type=int, default=1, help="0: leave the isolated matmul sweep out of the line (a profiling run)")
     ap.add_argument("--attend", default="", help="T,H,KV,hd,context[,calls]: only the decode attention, e.g. 32,32,8,128,2048,6")
     ap.add_argument("--matmul", default="", help="M,K,N,fmt[,calls]: only that isolated matmul (RMSNorm + SwiGLU fused), e.g. 32,4096,14336,bfp8,6")
-    ap.add_argument("--design", default="", help="binutar[:SIZE]: instead of the workload, prefill and decode of that design at sizes like a real model's layers, "
+    ap.add_argument("--design", default="", help="binutar[:SIZE] or labepel[:SIZE]: instead of the workload, prefill and decode of that design at sizes like a real model's layers, "
                                                  "and each of its kernels, beside the Llama decoder at equal size (one GPU)")
     return ap.parse_args()
 
@@ -417,6 +417,23 @@ DESIGN_SIZES = {
     "2560": dict(width=2560, layers=8, ff=6400, vocab=32000, heads=32, dim=64, rot_dim=32, vdim=64, kv_rank=256, q_rank=768, kv=8),
 }
 
+# grouped-query attention within spans and a mixture of experts with a shared one, at a Mixtral-like and a Qwen3-30B-A3B-like size, a
+# Llama-like mixture of the same heads, experts and depth beside each
+LABEPEL_SIZES = {
+    "4096": dict(width=4096, layers=6, vocab=32000, heads=32, kv=8, dim=128, vdim=128, span=8192, experts=8, top=2, ff=14336, shared=14336),
+    "2048": dict(width=2048, layers=8, vocab=32000, heads=32, kv=4, dim=128, vdim=128, span=8192, experts=128, top=8, ff=768, shared=768),
+}
+
+
+def labepel_models(s, places):
+    """(Labepel config, Llama config of a mixture) of one size."""
+    from ferrite_b200 import labepel, llama
+    block = dict(type="attention", mixer=dict(heads=s["heads"], kv_heads=s["kv"], dim=s["dim"], vdim=s["vdim"], mask=dict(size=s["span"]), scale=s["dim"] ** -0.5, v_mix=True),
+                 mlp=dict(kind="moe", router=dict(experts=s["experts"], top=s["top"]), expert=dict(ff=s["ff"]), shared=dict(ff=s["shared"])))
+    return (labepel.model(vocab=s["vocab"], dim=s["width"], eps=1e-5, blocks=[block] * s["layers"], positions=places, places=places),
+            llama.model(dim=s["width"], heads=s["heads"], kv=s["kv"], head_dim=s["dim"], layers=s["layers"], vocab=s["vocab"], ffn=0, experts=s["experts"], k=s["top"], moe=s["ff"], theta=10000.0,
+                        eps=1e-5, places=places))
+
 
 def design_models(s, places):
     """(Binutar config, Llama config) of one size."""
@@ -453,7 +470,7 @@ def timed(calls, copies, call):
 
 
 def design_steps(rt, c, prec, S, ctx, prompt, steps):
-    """Decode of S sequences at ctx tokens each (a recorded step, picks fed back on the device) and one sequence's prompt."""
+    """Decode of S sequences at ctx tokens each (a recorded step of distinct tokens) and one sequence's prompt."""
     import torch
     from ferrite_b200 import llama, models
     from ferrite_b200.tensor import Tensor, jit
@@ -467,13 +484,12 @@ def design_steps(rt, c, prec, S, ctx, prompt, steps):
         t.buf.normal_(0, 1, generator=gen)
     on = lambda row: Tensor.of(rt, [row], "int32")
     step = jit(lambda ids, at: llama.next_tokens(family.forward(ids, at, w, c, kv, S), c))
-    ids, one = on([1] * S), Tensor.of(rt, [[1] * S], "int32")
+    ids, one = on([(37 * i + 1) % c.vocab for i in range(S)]), Tensor.of(rt, [[1] * S], "int32")  # (the same every step: a mixture's sequences would else fall into step)
     bump = jit(lambda p: p + one)
     at = on([ctx] * S)
     before = rt.launches
     for i in range(4):
         out = step(ids, at)
-        ids.buf.copy_(out.buf)
         at = bump(at)
         if i == 0:
             names = rt.profile(before)
@@ -482,7 +498,6 @@ def design_steps(rt, c, prec, S, ctx, prompt, steps):
     e0.record()
     for _ in range(steps):
         out = step(ids, at)
-        ids.buf.copy_(out.buf)
         at = bump(at)
     e1.record()
     torch.cuda.synchronize()
@@ -638,26 +653,144 @@ def llama_kernels(rt, s, T, ctx, peaks):
     return rows
 
 
+def labepel_kernels(rt, s, T, ctx, peaks):
+    """Each kernel of a Labepel layer, as design_kernels does it."""
+    import torch
+    from ferrite_b200 import _lib, ops
+    dev, gen = rt.device, torch.Generator(device=rt.device).manual_seed(0)
+    f32 = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.float32).normal_(0, 1, generator=gen)
+    bf = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.bfloat16).normal_(0, 1, generator=gen)
+    rows, prompt = [], ctx == 0
+    d, H, G, dim, vd, E, k, ff, sff = (s[n] for n in ("width", "heads", "kv", "dim", "vdim", "experts", "top", "ff", "shared"))
+
+    def row(name, us, nbytes, flops=0.0, like=None):
+        floor = max(nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6)
+        rows.append({"kernel": name, "us": round(us, 2), "roofline_us": round(floor, 2), "frac": round(floor / us, 3)} | ({"like": like} if like else {}))
+
+    def dense(name, K, N, kind=_lib.DENSE_NONE, out_dtype=torch.bfloat16, like="fb_linear"):
+        copies = max(1, min(16, int(3e8 // (2 * K * N))))
+        ws, x, cols = [bf(1, N, K) for _ in range(copies)], bf(1, T, K), N // 2 if kind == _lib.DENSE_SWIGLU else N
+        out = torch.empty(1, T, cols, device=dev, dtype=out_dtype)
+        us = timed(40, copies, lambda i: ops.dense(x, ws[i].transpose(1, 2), out, True, kind))
+        row(f"fb_dense {name} [{K}, {N}]", us, 2 * K * N + 2 * T * K + out.element_size() * T * cols, 2.0 * T * K * N, like)
+
+    n = (H + G) * dim + G * vd
+    dense("in", d, n + H * vd + E, out_dtype=torch.float32)
+    dense("o", H * vd, d)
+    dense("shared gate_up, swiglu", d, 2 * sff, _lib.DENSE_SWIGLU)
+    dense("shared down", sff, d)
+    dense("head", d, s["vocab"], out_dtype=torch.float32)
+
+    joint, keys = f32(T, n + H * vd + E), T if prompt else ctx
+    part = keys + -keys % 64
+    caches = [bf(G, (1 if prompt else T) * part, dim + vd) for _ in range(4)]
+    last = torch.arange(T, device=dev, dtype=torch.int32) if prompt else torch.full((T,), ctx - 1, device=dev, dtype=torch.int32)
+    base = torch.arange(T, device=dev, dtype=torch.int32) * part
+    at, q, o = (last if prompt else base + last), bf(T, H * dim), bf(T, H * vd)
+    us = timed(40, 1, lambda i: ops.heads_put(joint, H, G, dim, vd, at, caches[0], q, f32_ones(dev, n), f32_ones(dev, dim), f32_ones(dev, dim), 1e-5, joint[:, n:n + G * vd], f32_ones(dev, G * vd),
+                                              f32_ones(dev, 1)))
+    row("fb_heads_put", us, T * (4 * (n + G * vd) + 2 * n), like="fb_rope_kv_write")
+    sink, gate, pairs = f32(H), joint[:, n:n + H * vd], T * (T + 1) / 2 if prompt else T * ctx
+    us = timed(20, 4, lambda i: ops.heads_attention(q, caches[i], None if prompt else base, last, H, vd, 0.1, keys, prompt, s["span"], sink, gate, out=o))
+    row("fb_heads_attention", us, 2 * ((1 if prompt else T) * keys * G * (dim + vd) + T * H * (dim + vd)) + 4 * T * H * vd, 2.0 * pairs * H * (dim + vd), "attention")
+
+    logits = f32(T, E)
+    us = timed(40, 1, lambda i: ops.route(logits, E, k, f32_ones(dev, E)))
+    row("fb_route", us, T * (4 * E + 12 * k), like="fb_topk and fb_touched (fb_group)")
+    r = ops.route(logits, E, k)
+    touched, live = len(set(r.ids.cpu().reshape(-1).tolist())), int(r.live)
+    copies = max(1, min(4, int(3e8 // (6 * touched * d * ff)) + 1))
+    gate_up, down, h = [bf(E, 2 * ff, d).transpose(1, 2) for _ in range(copies)], [bf(E, d, ff).transpose(1, 2) for _ in range(copies)], bf(T, d)
+    x, act, y = bf(r.tiles * r.tile, d), bf(r.tiles * r.tile, ff), bf(r.tiles * r.tile, d)
+    if not r.shared:
+        us = timed(20, 1, lambda i: ops.gather_rows(h, r.order, x))
+        row("fb_gather_rows", us, 4 * T * k * d, like="fb_gather_rows")
+    us = timed(20, copies, lambda i: ops.grouped(h if r.shared else x, gate_up[i], r, act, _lib.DENSE_SWIGLU, r.shared))
+    row(f"fb_dense_grouped gate_up, swiglu ({touched} experts, {live} tiles of {r.tile})", us, 4 * touched * d * ff + T * k * 2 * (d + ff), 4.0 * T * k * d * ff, "fb_linear_indexed")
+    us = timed(20, copies, lambda i: ops.grouped(act, down[i], r, y))
+    row("fb_dense_grouped down", us, 2 * touched * d * ff + T * k * 2 * (d + ff), 2.0 * T * k * d * ff, "fb_linear_indexed")
+    res, out, one = f32(T, d), f32(T, d), f32_ones(dev, d)
+    us = timed(40, 1, lambda i: ops.add_norm(res, out, h, one, h, one, y, r, one, 1.0, 1e-5, x[:T]))
+    row("fb_add_norm", us, T * d * (8 + 6 + 2 * k), like="fb_rmsnorm")
+    table, ids = bf(s["vocab"], d), torch.arange(T, device=dev, dtype=torch.int32)
+    us = timed(40, 1, lambda i: ops.embed(table, ids, table, ids, out))
+    row("fb_embed", us, T * d * 8, like="fb_gather_rows")
+    return rows
+
+
+def llama_expert_kernels(rt, s, T, peaks):
+    """The Llama mixture's own kernels at the same size (bfp8 experts): its router's and its experts', decode or prompt."""
+    import torch
+    from ferrite_b200 import ops
+    from ferrite_b200.llama import glu
+    from ferrite_b200.tensor import Tensor
+    dev, gen = rt.device, torch.Generator(device=rt.device).manual_seed(0)
+    d, E, k, ff, rows = s["width"], s["experts"], s["top"], s["ff"], []
+    bf = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.bfloat16).normal_(0, 1, generator=gen)
+
+    def row(name, us, nbytes, flops=0.0):
+        floor = max(nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6)
+        rows.append({"kernel": name, "us": round(us, 2), "roofline_us": round(floor, 2), "frac": round(floor / us, 3)})
+
+    logits = Tensor(rt, T, E, dtype="fp32", buf=torch.empty(1, T, E, device=dev).normal_(0, 1, generator=gen))
+    values, ids = logits.topk(k)
+    w = values.softmax().bfloat16().realize()
+    touched = len(set(ids.numpy().reshape(-1).tolist()))
+
+    def picks():
+        v, i = logits.topk(k)
+        u = v.softmax().bfloat16().realize()
+        return i.touched(E, u) if T <= 128 else i.group(E)
+    row("fb_topk, softmax and " + ("fb_touched" if T <= 128 else "fb_group"), timed(20, 1, lambda i: picks()), T * (4 * E + 12 * k))
+    pack = lambda K, N: Tensor(rt, K, N, batch=E, dtype="bfp8", packed=ops.quantize(bf(E, K, N), "bfp8"))
+    gate_up, down, h = pack(d, 2 * ff), pack(ff, d), Tensor(rt, T, d, buf=bf(1, T, d))
+    up_bytes, down_bytes = 1.0625 * touched * 2 * d * ff, 1.0625 * touched * d * ff
+    if T <= 128:
+        index, weights = ids.touched(E, w)
+        act, n = bf(T, index.rows * ff), index.rows
+        idx, out = index.buf.reshape(-1), bf(T, d)
+        us = timed(20, 1, lambda i: ops.linear_indexed(h.buf[0], gate_up.packed, idx, act, out_slot_stride=ff, epilogue="swiglu", row_scale=weights.buf))
+        row(f"fb_linear_indexed gate_up, swiglu ({touched} experts)", us, up_bytes + T * k * 2 * (d + ff), 4.0 * T * k * d * ff)
+        us = timed(20, 1, lambda i: ops.linear_indexed(act, down.packed, idx, out, sum_slots=True))
+        row("fb_linear_indexed down, summed", us, down_bytes + T * k * 2 * (d + ff), 2.0 * T * k * d * ff)
+    else:
+        order, tiles, _ = ids.group(E)
+        x = Tensor(rt, 32, d, batch=tiles.rows, buf=bf(tiles.rows, 32, d))
+        us = timed(4, 1, lambda i: x.matmul(gate_up, index=tiles).realize())
+        row(f"fb_linear_indexed gate_up ({touched} experts, tiles of 32)", us, up_bytes + T * k * 2 * (d + 2 * ff), 4.0 * T * k * d * ff)
+        y = x.matmul(gate_up, index=tiles).realize()
+        us = timed(4, 1, lambda i: glu(y[:, :, :ff], y[:, :, ff:]).realize())
+        row("fb_elementwise silu, times", us, T * k * 6 * ff)
+        z = glu(y[:, :, :ff], y[:, :, ff:]).realize()
+        us = timed(4, 1, lambda i: z.matmul(down, index=tiles).realize())
+        row("fb_linear_indexed down", us, down_bytes + T * k * 2 * (d + ff), 2.0 * T * k * d * ff)
+    return rows
+
+
 def run_design(args):
     """--design: one JSON line a size."""
     import torch
-    from ferrite_b200 import binutar, llama
+    from ferrite_b200 import llama, models
     from ferrite_b200.tensor import Runtime
     name, _, size = args.design.partition(":")
-    assert name == "binutar" and args.gpus == 1, "--design binutar[:SIZE], one GPU"
-    rt, (peaks, kind) = Runtime(0), measured_peaks()
+    assert name in ("binutar", "labepel") and args.gpus == 1, "--design binutar[:SIZE] or labepel[:SIZE], one GPU"
+    sizes, make, kernels = (DESIGN_SIZES, design_models, design_kernels) if name == "binutar" else (LABEPEL_SIZES, labepel_models, labepel_kernels)
+    rt, (peaks, kind), family = Runtime(0), measured_peaks(), models.module(name)
     S, ctx, prompt = 32, 2048, 2048
-    for key in [size] if size else DESIGN_SIZES:
-        s = DESIGN_SIZES[key]
+    for key in [size] if size else sizes:
+        s = sizes[key]
         clocks = Clocks(0)
         clocks.start()
         line = {"design": name, "size": key, "shape": s, "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "source": kind}, "weights": "random"}
-        b, l = design_models(s, ctx + 256)
-        line["binutar bf16"] = design_steps(rt, b, binutar.precision(b, "bf16"), S, ctx, prompt, args.steps)
-        line["binutar bfp8"] = design_steps(rt, b, binutar.precision(b, "bfp8"), S, ctx, prompt, args.steps)
-        line["llama bfp8"] = design_steps(rt, l, llama.precision(l, "bfp8"), S, ctx, prompt, args.steps)
+        b, l = make(s, ctx + 256)
+        for c, module, mode in ((b, family, "bf16"), (b, family, "bfp8"), (l, llama, "bfp8")):
+            line[f"{c.family} {mode}"] = design_steps(rt, c, module.precision(c, mode), S, ctx, prompt, args.steps)
+            torch.cuda.empty_cache()
         for what, T, at in (("decode", S, ctx), ("prefill", prompt, 0)):
-            line["kernels " + what] = {"binutar": design_kernels(rt, s, T, at, peaks), "llama": llama_kernels(rt, s, T, at, peaks)}
+            own = kernels(rt, s, T, at, peaks)
+            torch.cuda.empty_cache()
+            like = llama_kernels(rt, s, T, at, peaks) + (llama_expert_kernels(rt, s, T, peaks) if name == "labepel" else [])
+            line["kernels " + what] = {name: own, "llama": like}
             torch.cuda.empty_cache()
         line["clocks"] = clocks.summary()
         print(json.dumps(line), flush=True)

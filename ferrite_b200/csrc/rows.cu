@@ -47,10 +47,9 @@ __global__ void __launch_bounds__(32 * HEADS_WARPS) heads_put_kernel(const Heads
   griddep_wait();
   const fb_heads& s = a.h;
   const int lane = threadIdx.x & 31, units = s.heads + 2 * s.kv_heads;
-  const int64_t job = blockIdx.x * (int64_t)HEADS_WARPS + (threadIdx.x >> 5);
-  if (job >= a.T * units) return;
-  const int64_t t = job / units;
-  const int u = (int)(job % units);
+  const int64_t t = blockIdx.x;
+  const int u = blockIdx.y * HEADS_WARPS + (threadIdx.x >> 5);
+  if (u >= units) return;
   const bool is_q = u < s.heads, is_v = u >= s.heads + s.kv_heads;
   const int n = is_v ? s.vdim : s.dim, g = is_q ? u : is_v ? u - s.heads - s.kv_heads : u - s.heads;
   const int64_t at = is_v ? (int64_t)(s.heads + s.kv_heads) * s.dim + (int64_t)g * s.vdim : (int64_t)u * s.dim;
@@ -215,14 +214,14 @@ extern "C" int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void
                             void* cache, int64_t cache_rows, int64_t head_stride, void* stream) {
   FB_REQUIRE(heads_host && qkv && rows && q_out && cache && T >= 1, "fb_heads_put: null pointer or empty");
   const fb_heads& h = *heads_host;
-  FB_REQUIRE(h.heads >= 1 && h.kv_heads >= 1 && h.heads % h.kv_heads == 0 && h.dim >= 1 && h.vdim >= 1, "fb_heads_put: whole groups of query heads per key head (got %d / %d)", h.heads, h.kv_heads);
+  FB_REQUIRE(h.heads >= 1 && h.kv_heads >= 1 && h.heads % h.kv_heads == 0 && h.heads <= 100000 && h.dim >= 1 && h.vdim >= 1, "fb_heads_put: whole groups of query heads per key head (got %d / %d)", h.heads, h.kv_heads);
   const int64_t cols = (int64_t)(h.heads + h.kv_heads) * h.dim + (int64_t)h.kv_heads * h.vdim;
   FB_REQUIRE(ld >= cols && ld_q >= (int64_t)h.heads * h.dim && cache_rows >= 1 && head_stride >= cache_rows * (h.dim + h.vdim), "fb_heads_put: row strides too small");
   FB_REQUIRE(!h.first || (h.share && h.ld_first >= (int64_t)h.kv_heads * h.vdim), "fb_heads_put: mixed values take the other layer's and their share");
   FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32) && (in_dtype == FB_FP32 || dtype == FB_BF16),
              "fb_heads_put: bf16 or fp32; fp32 results come from fp32");
   const fb::HeadsPutArgs a{h, qkv, T, ld, rows, q_out, ld_q, cache, cache_rows, head_stride};
-  const dim3 grid((unsigned)fb::ceil_div(T * (h.heads + 2 * h.kv_heads), fb::HEADS_WARPS)), block(32 * fb::HEADS_WARPS);
+  const dim3 grid((unsigned)T, (unsigned)fb::ceil_div(h.heads + 2 * h.kv_heads, fb::HEADS_WARPS)), block(32 * fb::HEADS_WARPS);
   const auto s = (cudaStream_t)stream;
   if (in_dtype == FB_FP32 && dtype == FB_FP32) return fb::launch_after(fb::heads_put_kernel<float, float>, grid, block, 0, s, "fb_heads_put", a);
   if (in_dtype == FB_FP32) return fb::launch_after(fb::heads_put_kernel<float, uint16_t>, grid, block, 0, s, "fb_heads_put", a);

@@ -162,8 +162,10 @@ def experts(h, p, ids, w, c=None):
     run = places.cols // k
     terms = [y.gather(places[:, :, j * run:j * run + n]) * w[:, :, j:j + 1] for j in range(k)]
     out = terms[0]
-    for term in terms[1:]:
+    for j, term in enumerate(terms[1:]):
         out = out + term
+        if j % 3 == 2:  # (an expression has only so many inputs)
+            out = out.realize()
     return out
 
 

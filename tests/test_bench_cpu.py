@@ -46,3 +46,11 @@ def test_design_models_are_of_equal_size():
         b, l = bench.design_models(s, 512)
         assert (b.dim, b.vocab, b.layers) == (l.dim, l.vocab, l.layers) and all(e.mlp.ff == l.ffn for e in b.blocks)
         assert [e.type for e in b.blocks[:2]] == ["latent_attention", "lightning"] and b.blocks[0].mixer.heads == l.heads
+
+
+def test_labepel_models_are_of_equal_size():
+    for s in bench.LABEPEL_SIZES.values():
+        b, l = bench.labepel_models(s, 512)
+        assert (b.dim, b.vocab, b.layers, b.positions) == (l.dim, l.vocab, l.layers, 512)
+        e = b.blocks[0]
+        assert (e.mixer.heads, e.mixer.kv_heads, e.mixer.dim, e.mlp.router.experts, e.mlp.router.top, e.mlp.expert.ff) == (l.heads, l.kv, l.head_dim, l.experts, l.k, l.moe)
