@@ -1,0 +1,48 @@
+// Arguments of fb_heads_attention as its kernels see them.
+#pragma once
+#include "values.cuh"
+
+namespace fb {
+
+struct HeadsArgs {
+  const void* q;  // [T, ld_q]: head h at h * dim
+  int64_t T, ld_q;
+  int heads, kv_heads, dim, vdim, rep;  // rep: query heads per key head
+  const void* cache;  // [kv_heads, cache_rows, dim + vdim]
+  int64_t cache_rows, head_stride;
+  const int32_t *base, *last;  // token t sees cache rows base[t] + row0 + lo .. + last[t]; lo: where last[t]'s span begins
+  int64_t row0;
+  int chunk;  // the tokens are one sequence's, their places rising
+  int span;   // 0: no spans
+  float scale;
+  const float* sink;  // [heads] or null
+  int gate_dtype;
+  const void* gate;  // [T, ld_g]: head h at h * vdim; the output times its sigmoid
+  int64_t ld_g;
+  void* out;  // [T, ld_o]: head h at h * vdim
+  int64_t ld_o;
+  int64_t seen;  // an upper bound of the keys a token sees
+  int entries, pairs, tiles;  // entries of `pairs` pairs each (a token's, or the chunk's), cut into tiles
+};
+
+__device__ __forceinline__ int span_start(int place, int span) { return span > 0 ? place - place % span : 0; }
+
+// 2^x, the hardware's (x far below: 0)
+__device__ __forceinline__ float exp2_of(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+__device__ __forceinline__ float gate_value(const HeadsArgs& a, int64_t at) {
+  return a.gate_dtype == FB_FP32 ? static_cast<const float*>(a.gate)[at] : bf16_bits_to_float(static_cast<const uint16_t*>(a.gate)[at]);
+}
+__device__ __forceinline__ float gate_of(const HeadsArgs& a, int64_t t, int64_t col) {
+  return a.gate ? sigmoid_f(gate_value(a, t * a.ld_g + col)) : 1.f;
+}
+
+// heads_prompt.cu: a prompt's chunk on the 5th-generation tensor cores
+bool heads_prompt_supports(const HeadsArgs& a);
+int heads_prompt(const HeadsArgs& a, cudaStream_t s);
+
+}  // namespace fb

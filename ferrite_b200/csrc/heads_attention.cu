@@ -12,48 +12,12 @@
 //
 // bf16 rows of whole 16-byte pieces, heads of up to 256 columns; everything else (fp32, odd or wider heads) takes a plain
 // kernel at the end of the file.
+#include "heads.cuh"
 #include "launch.cuh"
 #include "mma_sync.cuh"
 #include "sm100.cuh"
-#include "values.cuh"
 
 namespace fb {
-
-struct HeadsArgs {
-  const void* q;  // [T, ld_q]: head h at h * dim
-  int64_t T, ld_q;
-  int heads, kv_heads, dim, vdim, rep;  // rep: query heads per key head
-  const void* cache;  // [kv_heads, cache_rows, dim + vdim]
-  int64_t cache_rows, head_stride;
-  const int32_t *base, *last;  // token t sees cache rows base[t] + row0 + lo .. + last[t]; lo: where last[t]'s span begins
-  int64_t row0;
-  int chunk;  // the tokens are one sequence's, their places rising
-  int span;   // 0: no spans
-  float scale;
-  const float* sink;  // [heads] or null
-  int gate_dtype;
-  const void* gate;  // [T, ld_g]: head h at h * vdim; the output times its sigmoid
-  int64_t ld_g;
-  void* out;  // [T, ld_o]: head h at h * vdim
-  int64_t ld_o;
-  int64_t seen;  // an upper bound of the keys a token sees
-  int entries, pairs, tiles;  // entries of `pairs` pairs each (a token's, or the chunk's), cut into tiles
-};
-
-__device__ __forceinline__ int span_start(int place, int span) { return span > 0 ? place - place % span : 0; }
-
-// 2^x, the hardware's (x far below: 0)
-__device__ __forceinline__ float exp2_of(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
-__device__ __forceinline__ float gate_of(const HeadsArgs& a, int64_t t, int64_t col) {
-  if (!a.gate) return 1.f;
-  const int64_t at = t * a.ld_g + col;
-  return sigmoid_f(a.gate_dtype == FB_FP32 ? static_cast<const float*>(a.gate)[at] : bf16_bits_to_float(static_cast<const uint16_t*>(a.gate)[at]));
-}
 
 constexpr int HA_KEYS = 64;
 constexpr float LOG2E = 1.4426950408889634f;
@@ -449,7 +413,8 @@ extern "C" int fb_heads_attention(int dtype, const void* q, int64_t T, int64_t l
   const auto s = (cudaStream_t)stream;
   const bool pieces = dim % 8 == 0 && vdim % 8 == 0 && ld_q % 8 == 0 && head_stride % 8 == 0 && ld_o % 2 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)cache % 16 == 0 && (uintptr_t)out % 4 == 0;
   if (dtype == FB_FP32) return vdim <= 256 ? launch_plain<float, 8>(a, s) : launch_plain<float, PLAIN_COLS>(a, s);
+  if (pieces && scale > 0.f && heads_prompt_supports(a)) return heads_prompt(a, s);
   const int64_t most = chunk ? ceil_div(T * a.rep, 64) : T * ceil_div(a.rep, 16);  // (of tiles: a grid's limit)
-  if (!pieces || dim > 256 || vdim > 256 || most > 65535) return vdim <= 256 ? launch_plain<uint16_t, 8>(a, s) : launch_plain<uint16_t, PLAIN_COLS>(a, s);
+  if (!pieces || !(scale > 0.f) || dim > 256 || vdim > 256 || most > 65535) return vdim <= 256 ? launch_plain<uint16_t, 8>(a, s) : launch_plain<uint16_t, PLAIN_COLS>(a, s);
   return dim <= 64 ? launch_values<64>(a, s) : dim <= 96 ? launch_values<96>(a, s) : dim <= 128 ? launch_values<128>(a, s) : dim <= 192 ? launch_values<192>(a, s) : launch_values<256>(a, s);
 }

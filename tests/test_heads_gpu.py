@@ -54,6 +54,7 @@ def attention_case(torch, shape, bf16, T, places, span, rng, sink=True, gate=Tru
     q, cache = rounded(rng.normal(0, 1, (T, H, dim)), bf16), rounded(rng.normal(0, 1, (G, S * part, dim + vdim)), bf16)
     if keys is not None:
         keys(q, cache, part)
+        q, cache = rounded(q, bf16), rounded(cache, bf16)
     zero = rng.normal(0.5, 1, H).astype(np.float32)
     g = rng.normal(0, 1.5, (T, H * vdim)).astype(np.float32)
     scale = 1.3 / np.sqrt(dim)
@@ -63,12 +64,13 @@ def attention_case(torch, shape, bf16, T, places, span, rng, sink=True, gate=Tru
     want = np.zeros((T, H, vdim))
     for t, p in enumerate(places):
         lo, first = oracle.chunk_of(p, span) if span else 0, base[t] if seqs else 0
-        for h in range(H):
-            rows = cache[h // (H // G), first + lo:first + p + 1]
-            s = rows[:, :dim] @ q[t, h] * scale
-            m = max(s.max(), zero[h]) if sink else s.max()
+        for kv in range(G):
+            mine = slice(kv * (H // G), (kv + 1) * (H // G))
+            rows = cache[kv, first + lo:first + p + 1]
+            s = q[t, mine] @ rows[:, :dim].T * scale
+            m = np.maximum(s.max(-1), zero[mine] if sink else -np.inf)[:, None]
             e = np.exp(s - m)
-            want[t, h] = e @ rows[:, dim:] / (e.sum() + (np.exp(zero[h] - m) if sink else 0))
+            want[t, mine] = e @ rows[:, dim:] / (e.sum(-1, keepdims=True) + (np.exp(zero[mine, None] - m) if sink else 0))
     want = want.reshape(T, H * vdim)
     return to_numpy(got), want * oracle.sigmoid(np.float64(g)) if gate else want
 
@@ -87,6 +89,30 @@ def test_attention_of_a_prompt(torch, shape, bf16):
     close(got, want, bf16)
 
 
+# prompts with tiles enough for the tcgen05 kernel: one group of pairs a CTA and two; pairs that fill a group's 128 rows and
+# pairs that do not; keys and values of whole 64-column pieces, of 16-column steps and of neither; spans that begin inside tiles
+@pytest.mark.parametrize("shape,cases", [((64, 32, 96, 48), ((0, 150, 48), (37, 200, 64), (190, 161, 0))), ((40, 40, 64, 64), ((0, 300, 100), (95, 257, 96))), ((90, 30, 40, 24), ((0, 130, 0), (60, 127, 33))),
+                                         ((37, 37, 256, 128), ((0, 200, 77),)), ((48, 24, 136, 72), ((5, 260, 130),)), ((200, 2, 64, 32), ((0, 40, 0), (50, 40, 17))), ((74, 74, 8, 8), ((0, 70, 20), (3, 2, 1))),
+                                         ((64, 32, 128, 128), ((0, 600, 0), (100, 640, 200))), ((32, 32, 192, 128), ((0, 640, 300),))])
+def test_attention_of_a_long_prompt(torch, shape, cases):
+    rng = np.random.default_rng(8)
+    for first, T, span in cases:
+        got, want = attention_case(torch, shape, True, T, list(range(first, first + T)), span, rng)
+        close(got, want, True, (first, T, span))
+    got, want = attention_case(torch, shape, True, T, list(range(first, first + T)), span, rng, sink=False, gate=False)
+    close(got, want, True, (first, T, span))
+
+
+def test_scores_that_grow_along_the_keys(torch):
+    # each key outdoes the ones before, so the reference maximum moves at every tile, by different steps in different rows
+    def plant(q, cache, part):
+        cache[:, :, :64] = cache[:, :1, :64] * (1 + np.arange(part)[None, :, None] / 16)
+        q[:] = cache[0, 0, :64] * np.linspace(0.2, 3, q.shape[0])[:, None, None]
+    for T, shape in ((300, (32, 32, 64, 64)), (40, (4, 2, 64, 64))):
+        got, want = attention_case(torch, shape, True, T, list(range(T)), 0, np.random.default_rng(9), keys=plant)
+        close(got, want, True, T)
+
+
 @pytest.mark.parametrize("shape,bf16", [(s, True) for s in SHAPES + PLAIN] + [(s, False) for s in SHAPES[:2] + PLAIN[:2]])
 def test_attention_of_a_decode_step(torch, shape, bf16):
     rng = np.random.default_rng(1)
@@ -95,10 +121,10 @@ def test_attention_of_a_decode_step(torch, shape, bf16):
         close(got, want, bf16, (places, span))
 
 
-@pytest.mark.parametrize("prompt", [True, False])
-def test_a_key_at_the_edge_of_a_span(torch, prompt):
+@pytest.mark.parametrize("prompt,shape", [(True, (4, 2, 64, 32)), (False, (4, 2, 64, 32)), (True, (74, 74, 64, 32))])
+def test_a_key_at_the_edge_of_a_span(torch, prompt, shape):
     # the first key of a span, and the last of the one before, scored far above all others: the one decides, the other is unseen
-    shape, span = (4, 2, 64, 32), 40
+    span = 40
     rng = np.random.default_rng(2)
     for first in (80, 160):
         for key, seen in ((first, True), (first - 1, False)):
