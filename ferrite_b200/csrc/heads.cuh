@@ -22,6 +22,7 @@ struct HeadsArgs {
   void* out;  // [T, ld_o]: head h at h * vdim
   int64_t ld_o;
   int64_t seen;  // an upper bound of the keys a token sees
+  int stages;  // tiles of keys in the ring
   int entries, pairs, tiles;  // entries of `pairs` pairs each (a token's, or the chunk's), cut into tiles
 };
 
