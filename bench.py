@@ -703,8 +703,8 @@ def labepel_kernels(rt, s, T, ctx, peaks):
     gate_up, down, h = [bf(E, 2 * ff, d).transpose(1, 2) for _ in range(copies)], [bf(E, d, ff).transpose(1, 2) for _ in range(copies)], bf(T, d)
     x, act, y = bf(r.tiles * r.tile, d), bf(r.tiles * r.tile, ff), bf(r.tiles * r.tile, d)
     if not r.shared:
-        us = timed(20, 1, lambda i: ops.gather_rows(h, r.order, x))
-        row("fb_gather_rows", us, 4 * T * k * d, like="fb_gather_rows")
+        us = timed(20, 1, lambda i: ops.spread_rows(h, r, x))
+        row("fb_spread_rows", us, 2 * T * (k + 1) * d, like="fb_gather_rows")
     us = timed(20, copies, lambda i: ops.grouped(h if r.shared else x, gate_up[i], r, act, _lib.DENSE_SWIGLU, r.shared))
     row(f"fb_dense_grouped gate_up, swiglu ({touched} experts, {live} tiles of {r.tile})", us, 4 * touched * d * ff + T * k * 2 * (d + ff), 4.0 * T * k * d * ff, "fb_linear_indexed")
     us = timed(20, copies, lambda i: ops.grouped(act, down[i], r, y))

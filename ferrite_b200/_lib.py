@@ -83,7 +83,8 @@ SIGNATURES = {
     "fb_gated_rmsnorm": (_i, [_p, _i64, _i64, _i64, _i, _p, _i64, _p, _f, _p, _i64, _p]),
     "fb_dense_grouped": (_i, [_p, _i64, _i64, _i64, _i, _p, _i64, _i64, _i64, _i, _p, _p, _i64, _i, _p, _i, _i64, _p, _p]),
     "fb_route_tiles": (_i64, [_i64, _i, _i, _i, _i]),
-    "fb_route": (_i, [_p, _i64, _i64, _p, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p, _p]),
+    "fb_route": (_i, [_p, _i64, _i64, _p, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p]),
+    "fb_spread_rows": (_i, [_p, _i64, _i64, _i64, _p, _i, _p, _i64, _p]),
     "fb_grouped_matmul": (_i, [_i, _p, _i64, _i64, _i, _i, _p, _p, _i, _i64, _i64, _p, _p, _i64, _i, _i, _p, _i64, _p]),
     "fb_embed": (_i, [_i, _p, _i64, _i64, _p, _p, _i64, _p, _i64, _p, _p]),
     "fb_heads_put": (_i, [_p, _i, _p, _i64, _i64, _p, _i, _p, _i64, _p, _i64, _i64, _p]),

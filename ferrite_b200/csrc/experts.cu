@@ -1,6 +1,7 @@
 // A mixture of experts around its matmuls, for weights kept as bf16 or fp32:
 //   fb_route            router logits (with a bias) -> each token's k largest, the softmax of those, and where each choice's row
 //                       goes: the touched experts' rows in whole tiles, a list of the tiles' experts, how many there are
+//   fb_spread_rows      the tokens' rows to their choices' places
 //   fb_grouped_matmul   rows of tiles by each tile's own matrix, any sizes, bf16 or fp32 (the tensor cores' form: fb_dense_grouped)
 //
 // Two layouts of the rows.  A few tokens: a tile a touched expert, holding all the tokens (nothing is gathered; an expert's
@@ -19,43 +20,67 @@ struct RouteArgs {
   float* weights;       // [T, k]
   int32_t* ids;         // [T, k]
   int32_t* slots;       // [T, k]: the row of each choice
-  int32_t* order;       // [tiles * tile] the token each row holds, -1: none (null with shared rows)
   int32_t* tile_expert; // [tiles], n past those used
   int32_t* live;        // [1] tiles used
 };
 
-// the k largest of a token's logits, the lower column first among equals, and the softmax of those: a warp a token
+// a float as a number that orders like it (-0 as 0), above 0 for all of them
+__device__ __forceinline__ uint32_t ordered(float v) {
+  const uint32_t b = __float_as_uint(v + 0.f);
+  return b & 0x80000000u ? ~b : b | 0x80000000u;
+}
+__device__ __forceinline__ float from_ordered(uint32_t b) { return __uint_as_float(b & 0x80000000u ? b & 0x7fffffffu : ~b); }
+
+// the k largest of a token's logits, the lower column first among equals, and the softmax of those: a warp a token.  Up to 128
+// experts: the lanes hold the logits as ordered numbers, 0 once picked
 __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int lane) {
   const float* z = a.logits + t * a.ld;
-  float prev = INFINITY, mine[2] = {-INFINITY, -INFINITY};  // lane j keeps the picks j and 32 + j
-  int prev_at = -1, my_id[2] = {0, 0};
-  float held[4];  // the first 128 columns stay in registers
+  float mine[2] = {-INFINITY, -INFINITY};  // lane j keeps the picks j and 32 + j
+  int my_id[2] = {0, 0};
+  auto keep = [&](int j, float v, int at) {
+    if (j < 32 && lane == j) mine[0] = v, my_id[0] = at;
+    if (j >= 32 && lane == j - 32) mine[1] = v, my_id[1] = at;
+  };
+  if (a.n <= 128) {
+    uint32_t held[4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int c = 32 * i + lane;
-    held[i] = c < a.n ? z[c] + (a.bias ? a.bias[c] : 0.f) : -INFINITY;
-  }
-  for (int j = 0; j < a.k; ++j) {
-    float best = -INFINITY;
-    int at = a.n;
-    auto look = [&](int c, float v) {
-      const bool after = v < prev || (v == prev && c > prev_at);
-      if (after && (at == a.n || v > best)) best = v, at = c;  // (columns rise: the first of equals stays)
-    };
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-      if (32 * i + lane < a.n) look(32 * i + lane, held[i]);
-    for (int c = 128 + lane; c < a.n; c += 32) look(c, z[c] + (a.bias ? a.bias[c] : 0.f));
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, at, o);
-      if (oi < a.n && (at == a.n || ov > best || (ov == best && oi < at))) best = ov, at = oi;
+    for (int i = 0; i < 4; ++i) {
+      const int c = 32 * i + lane;
+      held[i] = c < a.n ? ordered(z[c] + (a.bias ? a.bias[c] : 0.f)) : 0;
     }
-    if (at == a.n) at = 0;  // (only where a logit is not a number)
-    prev = best, prev_at = at;
-    if (j < 32 && lane == j) mine[0] = best, my_id[0] = at;
-    if (j >= 32 && lane == j - 32) mine[1] = best, my_id[1] = at;
+    for (int j = 0; j < a.k; ++j) {
+      uint32_t best = held[0];
+      int at = lane;
+#pragma unroll
+      for (int i = 1; i < 4; ++i)
+        if (held[i] > best) best = held[i], at = 32 * i + lane;
+      const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+      at = __reduce_min_sync(0xffffffffu, best == top ? at : a.n);
+      keep(j, from_ordered(top), at);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (at == 32 * i + lane) held[i] = 0;
+    }
+  } else {
+    float prev = INFINITY;
+    int prev_at = -1;
+    for (int j = 0; j < a.k; ++j) {
+      float best = -INFINITY;
+      int at = a.n;
+      for (int c = lane; c < a.n; c += 32) {  // (what comes after the pick before in the order of the picks; columns rise: the first of equals stays)
+        const float v = z[c] + (a.bias ? a.bias[c] : 0.f);
+        if ((v < prev || (v == prev && c > prev_at)) && (at == a.n || v > best)) best = v, at = c;
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, at, o);
+        if (oi < a.n && (at == a.n || ov > best || (ov == best && oi < at))) best = ov, at = oi;
+      }
+      if (at == a.n) at = 0;  // (only where a logit is not a number)
+      prev = best, prev_at = at;
+      keep(j, best, at);
+    }
   }
   const float top = __shfl_sync(0xffffffffu, mine[0], 0);
   const float e0 = lane < a.k ? expf(mine[0] - top) : 0.f, e1 = lane + 32 < a.k ? expf(mine[1] - top) : 0.f, sum = warp_sum(e0 + e1);
@@ -82,7 +107,15 @@ __global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, c
     for (int64_t t = warp; t < a.T; t += 32) route_token(a, t, lane);
   __syncthreads();
   const int64_t choices = a.T * a.k;
-  for (int64_t i = tid; i < choices; i += blockDim.x) atomicAdd(count + a.ids[i], 1);
+  constexpr int BATCH = 8;  // a thread's choices on their way at once
+  for (int64_t i0 = tid; i0 < choices; i0 += BATCH * 1024) {
+    int e[BATCH];
+#pragma unroll
+    for (int b = 0; b < BATCH; ++b) e[b] = i0 + b * 1024 < choices ? a.ids[i0 + b * 1024] : -1;
+#pragma unroll
+    for (int b = 0; b < BATCH; ++b)
+      if (e[b] >= 0) atomicAdd(count + e[b], 1);
+  }
   __syncthreads();
   // tiles of each expert, scanned: a thread has a run of experts
   const int run = (a.n + 1023) / 1024, e0 = min(a.n, tid * run), e1 = min(a.n, e0 + run);
@@ -118,15 +151,29 @@ __global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, c
     first += n;
   }
   for (int i = used + tid; i < a.tiles; i += blockDim.x) a.tile_expert[i] = a.n;
-  if (a.order)
-    for (int64_t i = tid; i < (int64_t)a.tiles * a.tile; i += blockDim.x) a.order[i] = -1;
   __syncthreads();
-  for (int64_t i = tid; i < choices; i += blockDim.x) {
-    const int e = a.ids[i];
-    const int64_t t = i / a.k;
-    const int slot = a.shared ? count[e] + (int)t : atomicAdd(count + e, 1);
-    a.slots[i] = slot;
-    if (a.order) a.order[slot] = (int32_t)t;
+  for (int64_t i0 = tid; i0 < choices; i0 += BATCH * 1024) {
+    int e[BATCH];
+#pragma unroll
+    for (int b = 0; b < BATCH; ++b) e[b] = i0 + b * 1024 < choices ? a.ids[i0 + b * 1024] : -1;
+#pragma unroll
+    for (int b = 0; b < BATCH; ++b)
+      if (e[b] >= 0) a.slots[i0 + b * 1024] = a.shared ? count[e[b]] + (int)((i0 + b * 1024) / a.k) : atomicAdd(count + e[b], 1);
+  }
+}
+
+// row t of x into the rows slots[t, 0 .. k) of out
+template <typename Piece>
+__global__ void __launch_bounds__(128) spread_rows_kernel(const Piece* __restrict__ x, int64_t row_x, const int32_t* __restrict__ slots, int k, int64_t pieces, Piece* __restrict__ out, int64_t out_rows) {
+  griddep_launch_dependents();
+  griddep_wait();
+  const int64_t t = blockIdx.x;
+  for (int64_t c = blockIdx.y * (int64_t)blockDim.x + threadIdx.x; c < pieces; c += (int64_t)gridDim.y * blockDim.x) {
+    const Piece v = x[t * row_x + c];
+    for (int j = 0; j < k; ++j) {
+      const int64_t to = slots[t * k + j];
+      if (to >= 0 && to < out_rows) out[to * pieces + c] = v;
+    }
   }
 }
 
@@ -185,18 +232,28 @@ extern "C" int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_
 }
 
 extern "C" int fb_route(const float* logits, int64_t T, int64_t ld, const float* bias, int n, int k, int tile, int shared_rows, float* weights, int32_t* ids, int32_t* slots,
-                        int32_t* order, int32_t* tile_expert, int32_t* live, void* stream) {
+                        int32_t* tile_expert, int32_t* live, void* stream) {
   FB_REQUIRE(logits && weights && ids && slots && tile_expert && live && T >= 1 && T <= (1 << 24), "fb_route: null pointer or no tokens");
   FB_REQUIRE(n >= 1 && n <= 8192 && k >= 1 && k <= 64 && k <= n && ld >= n, "fb_route: up to 64 choices among up to 8192 experts (got %d of %d)", k, n);
-  FB_REQUIRE(tile >= 16 && tile % 16 == 0 && (shared_rows ? T <= tile : order != nullptr), "fb_route: tiles of whole runs of 16 rows; shared rows: all the tokens in one");
+  FB_REQUIRE(tile >= 16 && tile % 16 == 0 && (!shared_rows || T <= tile), "fb_route: tiles of whole runs of 16 rows; shared rows: all the tokens in one");
   const int64_t tiles = fb_route_tiles(T, n, k, tile, shared_rows);
   FB_REQUIRE(tiles * tile < (1ll << 31), "fb_route: too many rows");
-  const fb::RouteArgs a{logits, T, ld, bias, n, k, tile, shared_rows, (int)tiles, weights, ids, slots, shared_rows ? nullptr : order, tile_expert, live};
+  const fb::RouteArgs a{logits, T, ld, bias, n, k, tile, shared_rows, (int)tiles, weights, ids, slots, tile_expert, live};
   const auto s = (cudaStream_t)stream;
-  const int pick = T <= 128;
+  const int pick = T <= 32;
   if (!pick)
     if (int rc = fb::launch_after(fb::route_tokens_kernel, dim3((unsigned)fb::ceil_div(T, 8)), dim3(256), 0, s, "fb_route", a)) return rc;
   return fb::launch_after(fb::route_places_kernel, dim3(1), dim3(1024), (size_t)(n + 33) * sizeof(int32_t), s, "fb_route", a, pick);
+}
+
+extern "C" int fb_spread_rows(const void* x, int64_t T, int64_t row_bytes, int64_t ldx_bytes, const int32_t* slots, int k, void* out, int64_t out_rows, void* stream) {
+  FB_REQUIRE(x && slots && out && T >= 1 && k >= 1 && out_rows >= 1 && row_bytes >= 2 && row_bytes % 2 == 0 && ldx_bytes >= row_bytes && ldx_bytes % 2 == 0, "fb_spread_rows: null pointer, or rows of no whole 2-byte values");
+  const auto s = (cudaStream_t)stream;
+  if (row_bytes % 16 == 0 && ldx_bytes % 16 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)out % 16 == 0) {
+    const dim3 grid((unsigned)T, (unsigned)(fb::ceil_div(row_bytes / 16, 128) < 4 ? fb::ceil_div(row_bytes / 16, 128) : 4));
+    return fb::launch_after(fb::spread_rows_kernel<uint4>, grid, dim3(128), 0, s, "fb_spread_rows", (const uint4*)x, ldx_bytes / 16, slots, k, row_bytes / 16, (uint4*)out, out_rows);
+  }
+  return fb::launch_after(fb::spread_rows_kernel<uint16_t>, dim3((unsigned)T, 4), dim3(128), 0, s, "fb_spread_rows", (const uint16_t*)x, ldx_bytes / 2, slots, k, row_bytes / 2, (uint16_t*)out, out_rows);
 }
 
 extern "C" int fb_grouped_matmul(int x_dtype, const void* x, int64_t x_rows, int64_t ldx, int shared_rows, int w_dtype, const void* W, const int64_t* w_strides_host, int n, int64_t K, int64_t N,

@@ -9,6 +9,16 @@
 
 namespace fb {
 
+// four columns at a time
+__device__ __forceinline__ float4 four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 four(const uint16_t* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16_bits_to_float(v.x & 0xffffu), bf16_bits_to_float(v.x >> 16), bf16_bits_to_float(v.y & 0xffffu), bf16_bits_to_float(v.y >> 16));
+}
+__device__ __forceinline__ void put_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put_four(uint16_t* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
+__device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) { return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w)); }
+
 struct EmbedArgs {
   const void *table, *places_table;  // [rows, cols], [place_rows, cols] or null
   int64_t rows, place_rows, cols;
@@ -91,6 +101,83 @@ __global__ void __launch_bounds__(32 * HEADS_WARPS) heads_put_kernel(const Heads
   for (int c = 32 * HEADS_REGS + lane; c < n; c += 32) store_value(out + c, (value_of(x[c]) + (bias ? bias[c] : 0.f)) * r * (w ? w[c] : 1.f));
 }
 
+// the same for heads of whole groups of four columns, 16-byte aligned, up to 256 wide: a warp has four heads, everything it
+// reads on its way at once
+template <typename In, typename Act, int GROUPS>
+__global__ void __launch_bounds__(128) heads_put4_kernel(const HeadsPutArgs a) {
+  griddep_launch_dependents();
+  griddep_wait();
+  constexpr int UNITS = 4;
+  const fb_heads& s = a.h;
+  const int lane = threadIdx.x & 31, keys = s.heads + s.kv_heads, units = keys + s.kv_heads;
+  const int64_t t = blockIdx.x, row = a.rows[t];
+  const bool inside = row >= 0 && row < a.cache_rows;  // nothing is written outside the cache
+  const int u0 = (blockIdx.y * 4 + (threadIdx.x >> 5)) * UNITS;
+  const In* x = static_cast<const In*>(a.qkv) + t * a.ld;
+  float4 v[UNITS][GROUPS], f[UNITS][GROUPS];
+#pragma unroll
+  for (int i = 0; i < UNITS; ++i)
+#pragma unroll
+    for (int j = 0; j < GROUPS; ++j) {
+      const int u = u0 + i, c = 4 * (32 * j + lane);
+      v[i][j] = f[i][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (u >= units || c >= (u < keys ? s.dim : s.vdim)) continue;
+      const int64_t at = u < keys ? (int64_t)u * s.dim : (int64_t)keys * s.dim + (int64_t)(u - keys) * s.vdim;
+      v[i][j] = four(x + at + c);
+      if (u >= keys && s.first) f[i][j] = four(static_cast<const In*>(s.first) + t * s.ld_first + (int64_t)(u - keys) * s.vdim + c);
+    }
+  const float share = s.first ? *s.share : 0.f;
+#pragma unroll
+  for (int i = 0; i < UNITS; ++i) {
+    const int u = u0 + i, n = u < keys ? s.dim : s.vdim;
+    if (u >= units) break;
+    const int64_t at = u < keys ? (int64_t)u * s.dim : (int64_t)keys * s.dim + (int64_t)(u - keys) * s.vdim;
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < GROUPS; ++j) {
+      const int c = 4 * (32 * j + lane);
+      if (c < n && s.bias) {
+        const float4 b = four(s.bias + at + c);
+        v[i][j].x += b.x, v[i][j].y += b.y, v[i][j].z += b.z, v[i][j].w += b.w;
+      }
+      if (u >= keys && s.first && c < n) {
+        float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (s.first_bias) b = four(s.first_bias + (int64_t)(u - keys) * s.vdim + c);
+        v[i][j].x = (1.f - share) * v[i][j].x + share * (f[i][j].x + b.x), v[i][j].y = (1.f - share) * v[i][j].y + share * (f[i][j].y + b.y);
+        v[i][j].z = (1.f - share) * v[i][j].z + share * (f[i][j].z + b.z), v[i][j].w = (1.f - share) * v[i][j].w + share * (f[i][j].w + b.w);
+      }
+      ss = fmaf(v[i][j].x, v[i][j].x, fmaf(v[i][j].y, v[i][j].y, fmaf(v[i][j].z, v[i][j].z, fmaf(v[i][j].w, v[i][j].w, ss))));
+    }
+    const float* w = u < s.heads ? s.q_norm : u < keys ? s.k_norm : nullptr;
+    const float r = w ? 1.f / sqrtf(warp_sum(ss) / (float)n + s.eps) : 1.f;
+    if (u >= s.heads && !inside) continue;
+    Act* out = u < s.heads ? static_cast<Act*>(a.q_out) + t * a.ld_q + (int64_t)u * s.dim
+                           : static_cast<Act*>(a.cache) + (u < keys ? u - s.heads : u - keys) * a.head_stride + row * (s.dim + s.vdim) + (u < keys ? 0 : s.dim);
+#pragma unroll
+    for (int j = 0; j < GROUPS; ++j) {
+      const int c = 4 * (32 * j + lane);
+      if (c >= n) continue;
+      const float4 g = w ? four(w + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+      put_four(out + c, make_float4(v[i][j].x * r * g.x, v[i][j].y * r * g.y, v[i][j].z * r * g.z, v[i][j].w * r * g.w));
+    }
+  }
+}
+
+template <typename In, typename Act>
+static int launch_heads_put(const HeadsPutArgs& a, cudaStream_t s) {
+  const fb_heads& h = a.h;
+  const int units = h.heads + 2 * h.kv_heads;
+  auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
+  const bool fours = h.dim % 4 == 0 && h.vdim % 4 == 0 && h.dim <= 256 && h.vdim <= 256 && whole(a.qkv, a.ld, sizeof(In)) && whole(h.first, h.ld_first, sizeof(In)) && whole(h.bias, 0, 4) &&
+                     whole(h.first_bias, 0, 4) && whole(h.q_norm, 0, 4) && whole(h.k_norm, 0, 4) && whole(a.q_out, a.ld_q, sizeof(Act)) && whole(a.cache, a.head_stride, sizeof(Act));
+  if (fours) {
+    const dim3 grid((unsigned)a.T, (unsigned)ceil_div(units, 16));
+    if (h.dim <= 128 && h.vdim <= 128) return launch_after(heads_put4_kernel<In, Act, 1>, grid, dim3(128), 0, s, "fb_heads_put", a);
+    return launch_after(heads_put4_kernel<In, Act, 2>, grid, dim3(128), 0, s, "fb_heads_put", a);
+  }
+  return launch_after(heads_put_kernel<In, Act>, dim3((unsigned)a.T, (unsigned)ceil_div(units, HEADS_WARPS)), dim3(32 * HEADS_WARPS), 0, s, "fb_heads_put", a);
+}
+
 // ---- a layer's end: a block per token; the new row stays in shared memory for the norm's second pass
 template <typename In, typename Act>
 __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, const int64_t cols) {
@@ -101,7 +188,8 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, cons
   __shared__ int64_t at[64];
   __shared__ float weight[64];
   const int64_t t = blockIdx.x;
-  if (a.chosen && (int)threadIdx.x < a.k) at[threadIdx.x] = a.slots[t * a.k + threadIdx.x] * a.ld_chosen, weight[threadIdx.x] = a.weights[t * a.k + threadIdx.x];
+  if (a.chosen)
+    for (int j = threadIdx.x; j < a.k; j += blockDim.x) at[j] = a.slots[t * a.k + j] * a.ld_chosen, weight[j] = a.weights[t * a.k + j];
   __syncthreads();
   const float* x = a.x + t * a.ld_x;
   const In* y1 = a.mixer ? static_cast<const In*>(a.mixer) + t * a.ld_mixer : nullptr;
@@ -126,75 +214,87 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, cons
   for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) store_value(h + c, row[c] * r * (a.w[c] + a.plus));
 }
 
-// the same for rows of whole groups of four columns, 16-byte aligned: a thread takes its groups in one go, everything it
+// the same for rows of whole groups of four columns, 16-byte aligned: a thread keeps its groups in registers, everything it
 // reads on its way at once
-__device__ __forceinline__ float4 four(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 four(const uint16_t* p) {
-  const uint2 v = *reinterpret_cast<const uint2*>(p);
-  return make_float4(bf16_bits_to_float(v.x & 0xffffu), bf16_bits_to_float(v.x >> 16), bf16_bits_to_float(v.y & 0xffffu), bf16_bits_to_float(v.y >> 16));
-}
-__device__ __forceinline__ void put_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void put_four(uint16_t* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
-__device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) { return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w)); }
-
-template <typename In, typename Act>
+template <typename In, typename Act, int GROUPS>
 __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, const int64_t cols) {
   griddep_launch_dependents();
   griddep_wait();
-  extern __shared__ float row[];  // [cols]
   __shared__ float red[32];
   __shared__ int64_t at[64];
   __shared__ float weight[64];
   const int64_t t = blockIdx.x;
-  if (a.chosen && (int)threadIdx.x < a.k) at[threadIdx.x] = a.slots[t * a.k + threadIdx.x] * a.ld_chosen, weight[threadIdx.x] = a.weights[t * a.k + threadIdx.x];
-  __syncthreads();
+  if (a.chosen) {
+    for (int j = threadIdx.x; j < a.k; j += blockDim.x) at[j] = a.slots[t * a.k + j] * a.ld_chosen, weight[j] = a.weights[t * a.k + j];
+    __syncthreads();
+  }
   const float4 one = make_float4(1.f, 1.f, 1.f, 1.f), none = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 v[GROUPS], f[GROUPS];
   float ss = 0.f;
-  for (int64_t c = 4 * threadIdx.x; c < cols; c += 4 * blockDim.x) {
-    float4 v = four(a.x + t * a.ld_x + c), f = none;
-    if (a.mixer) v = fma4(four(static_cast<const In*>(a.mixer) + t * a.ld_mixer + c), a.mixer_scale ? four(a.mixer_scale + c) : one, v);
-    if (a.other) f = four(static_cast<const In*>(a.other) + t * a.ld_other + c);
-    if (a.chosen) {
-      const Act* y = static_cast<const Act*>(a.chosen) + c;
-      for (int j = 0; j < a.k; j += 4) {
-        float4 part[4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) part[i] = j + i < a.k ? four(y + at[j + i]) : none;
+  for (int i = 0; i < GROUPS; ++i) {
+    const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
+    v[i] = f[i] = none;
+    if (c >= cols) continue;
+    v[i] = four(a.x + t * a.ld_x + c);
+    if (a.mixer) v[i] = fma4(four(static_cast<const In*>(a.mixer) + t * a.ld_mixer + c), a.mixer_scale ? four(a.mixer_scale + c) : one, v[i]);
+    if (a.other) f[i] = four(static_cast<const In*>(a.other) + t * a.ld_other + c);
+  }
+  if (a.chosen)
+    for (int j = 0; j < a.k; j += 4) {
+      float4 part[GROUPS][4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float s = j + i < a.k ? weight[j + i] : 0.f;
-          f = fma4(make_float4(s, s, s, s), part[i], f);
+      for (int i = 0; i < GROUPS; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
+          part[i][e] = j + e < a.k && c < cols ? four(static_cast<const Act*>(a.chosen) + at[j + e] + c) : none;
         }
-      }
+#pragma unroll
+      for (int i = 0; i < GROUPS; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float s = j + e < a.k ? weight[j + e] : 0.f;
+          f[i] = fma4(make_float4(s, s, s, s), part[i][e], f[i]);
+        }
     }
-    if (a.chosen || a.other) v = fma4(f, a.other_scale ? four(a.other_scale + c) : one, v);
-    put_four(row + c, v);
-    if (a.x_out) put_four(a.x_out + t * a.ld_x_out + c, v);
-    ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+#pragma unroll
+  for (int i = 0; i < GROUPS; ++i) {
+    const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
+    if (c >= cols) continue;
+    if (a.chosen || a.other) v[i] = fma4(f[i], a.other_scale ? four(a.other_scale + c) : one, v[i]);
+    if (a.x_out) put_four(a.x_out + t * a.ld_x_out + c, v[i]);
+    ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
   }
   if (!a.h) return;
   const float r = 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps);
-  for (int64_t c = 4 * threadIdx.x; c < cols; c += 4 * blockDim.x) {
-    const float4 v = four(row + c), w = four(a.w + c);
+#pragma unroll
+  for (int i = 0; i < GROUPS; ++i) {
+    const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
+    if (c >= cols) continue;
+    const float4 w = four(a.w + c);
     put_four(static_cast<Act*>(a.h) + t * a.ld_h + c,
-             make_float4(v.x * r * (w.x + a.plus), v.y * r * (w.y + a.plus), v.z * r * (w.z + a.plus), v.w * r * (w.w + a.plus)));
+             make_float4(v[i].x * r * (w.x + a.plus), v[i].y * r * (w.y + a.plus), v[i].z * r * (w.z + a.plus), v[i].w * r * (w.w + a.plus)));
   }
 }
 
 template <typename In, typename Act>
 static int launch_add_norm(const fb_branches& a, int64_t T, int64_t cols, cudaStream_t s) {
   static std::atomic<uint64_t> opted{0};
-  if (first_on_device(opted)) {
-    cudaFuncSetAttribute(add_norm_kernel<In, Act>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-    cudaFuncSetAttribute(add_norm4_kernel<In, Act>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
-  }
+  if (first_on_device(opted)) cudaFuncSetAttribute(add_norm_kernel<In, Act>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
-  const bool fours = cols % 4 == 0 && whole(a.x, a.ld_x, 4) && whole(a.mixer, a.ld_mixer, sizeof(In)) && whole(a.mixer_scale, 0, 4) && whole(a.other, a.ld_other, sizeof(In)) &&
-                     whole(a.other_scale, 0, 4) && whole(a.chosen, a.ld_chosen, sizeof(Act)) && whole(a.x_out, a.ld_x_out, 4) && whole(a.w, 0, 4) && whole(a.h, a.ld_h, sizeof(Act));
-  const int64_t work = fours ? cols / 4 : cols;
-  const int threads = (int)(work >= 512 ? 512 : ceil_div(work, 32) * 32 < 64 ? 64 : ceil_div(work, 32) * 32);
-  auto kernel = fours ? add_norm4_kernel<In, Act> : add_norm_kernel<In, Act>;
-  return launch_after(kernel, dim3((unsigned)T), dim3(threads), (size_t)cols * sizeof(float), s, "fb_add_norm", a, cols);
+  const bool fours = cols % 4 == 0 && cols <= 4 * 4 * 512 && whole(a.x, a.ld_x, 4) && whole(a.mixer, a.ld_mixer, sizeof(In)) && whole(a.mixer_scale, 0, 4) &&
+                     whole(a.other, a.ld_other, sizeof(In)) && whole(a.other_scale, 0, 4) && whole(a.chosen, a.ld_chosen, sizeof(Act)) && whole(a.x_out, a.ld_x_out, 4) && whole(a.w, 0, 4) &&
+                     whole(a.h, a.ld_h, sizeof(Act));
+  const dim3 grid((unsigned)T);
+  auto warps = [](int64_t work) { return dim3((unsigned)(work >= 512 ? 512 : ceil_div(work, 32) * 32)); };
+  if (!fours) return launch_after(add_norm_kernel<In, Act>, grid, warps(cols), (size_t)cols * sizeof(float), s, "fb_add_norm", a, cols);
+  // few rows: a thread a group of four columns; many: fewer threads with more on their way each
+  const int groups = cols > 4 * 1024 ? 4 : cols > 4 * 512 || T >= 512 ? 2 : 1;
+  const dim3 block = warps(ceil_div(cols / 4, groups));
+  if (groups == 4) return launch_after(add_norm4_kernel<In, Act, 4>, grid, block, 0, s, "fb_add_norm", a, cols);
+  if (groups == 2) return launch_after(add_norm4_kernel<In, Act, 2>, grid, block, 0, s, "fb_add_norm", a, cols);
+  return launch_after(add_norm4_kernel<In, Act, 1>, grid, block, 0, s, "fb_add_norm", a, cols);
 }
 
 }  // namespace fb
@@ -221,11 +321,10 @@ extern "C" int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void
   FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32) && (in_dtype == FB_FP32 || dtype == FB_BF16),
              "fb_heads_put: bf16 or fp32; fp32 results come from fp32");
   const fb::HeadsPutArgs a{h, qkv, T, ld, rows, q_out, ld_q, cache, cache_rows, head_stride};
-  const dim3 grid((unsigned)T, (unsigned)fb::ceil_div(h.heads + 2 * h.kv_heads, fb::HEADS_WARPS)), block(32 * fb::HEADS_WARPS);
   const auto s = (cudaStream_t)stream;
-  if (in_dtype == FB_FP32 && dtype == FB_FP32) return fb::launch_after(fb::heads_put_kernel<float, float>, grid, block, 0, s, "fb_heads_put", a);
-  if (in_dtype == FB_FP32) return fb::launch_after(fb::heads_put_kernel<float, uint16_t>, grid, block, 0, s, "fb_heads_put", a);
-  return fb::launch_after(fb::heads_put_kernel<uint16_t, uint16_t>, grid, block, 0, s, "fb_heads_put", a);
+  if (in_dtype == FB_FP32 && dtype == FB_FP32) return fb::launch_heads_put<float, float>(a, s);
+  if (in_dtype == FB_FP32) return fb::launch_heads_put<float, uint16_t>(a, s);
+  return fb::launch_heads_put<uint16_t, uint16_t>(a, s);
 }
 
 extern "C" int fb_add_norm(const fb_branches* branches_host, int64_t T, int64_t cols, int in_dtype, int dtype, void* stream) {

@@ -1,6 +1,8 @@
 """Thin typed wrappers over the C ABI: torch tensors own the device memory, every call is one or two
 kernel launches on torch's current CUDA stream.  No arithmetic happens in Python or in torch here."""
 import ctypes
+import functools
+import math
 
 import torch
 
@@ -367,24 +369,29 @@ def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, s
 
 
 class Routes:
-    """Where a mixture's rows go (fb_route): tokens' weights and slots [T, k], the rows' tokens (order; None: every tile holds
-    all the tokens), the tiles' experts, how many tiles are in use, and the sizes of all that."""
+    """Where a mixture's rows go (fb_route): tokens' weights, choices and slots [T, k], the tiles' experts, how many tiles are in
+    use, and the sizes of all that; shared: every tile holds all the tokens."""
 
     def __init__(self, device, T, n, k, tile, shared):
         self.T, self.n, self.k, self.tile, self.shared = T, n, k, tile, shared
         self.tiles = lib().fb_route_tiles(T, n, k, tile, int(shared))
         i32 = lambda *shape: torch.empty(*shape, dtype=torch.int32, device=device)
         self.weights, self.ids, self.slots = torch.empty(T, k, dtype=torch.float32, device=device), i32(T, k), i32(T, k)
-        self.order, self.tile_expert, self.live = None if shared else i32(self.tiles * tile), i32(self.tiles), i32(1)
+        self.tile_expert, self.live = i32(self.tiles), i32(1)
 
 
+@functools.lru_cache
 def route_tile(T, n, k):
     """(rows of a tile, whether each tile holds all the tokens) for T tokens with k of n experts each: a few tokens are not
-    sorted, more take tiles about as high as an expert has rows (the fuller the tiles, the fewer times its weights are read)."""
+    sorted.  More: the height at which evenly drawn choices make for the least work, a tile costing what its weights' way
+    through a CTA does (about 60 rows' products) or its products."""
     if T <= 64:
         return -(-T // 16) * 16, True
-    rows = T * k / n
-    return (256 if rows >= 384 else 128 if rows >= 80 else 64 if rows >= 40 else 32), False
+    m = T * k / n
+    spread = (m * (1 - k / n)) ** 0.5 + 1e-9
+    above = lambda x: 0.5 * math.erfc((x - m) / (spread * 2 ** 0.5))  # how likely an expert has more than x rows
+    work = lambda tile: sum(above(j * tile) for j in range(int((m + 5 * spread) / tile) + 2)) * max(62 + 0.1 * tile, tile)
+    return min(range(32, 257, 16), key=work), False
 
 
 def route(logits, n, k, bias=None):
@@ -392,10 +399,19 @@ def route(logits, n, k, bias=None):
     T = logits.shape[0]
     tile, shared = route_tile(T, n, k)
     r = Routes(logits.device, T, n, k, tile, shared)
-    check(lib().fb_route(logits.data_ptr(), T, logits.stride(0), _ptr(bias), n, k, tile, int(shared), r.weights.data_ptr(), r.ids.data_ptr(), r.slots.data_ptr(), _ptr(r.order),
+    check(lib().fb_route(logits.data_ptr(), T, logits.stride(0), _ptr(bias), n, k, tile, int(shared), r.weights.data_ptr(), r.ids.data_ptr(), r.slots.data_ptr(),
                          r.tile_expert.data_ptr(), r.live.data_ptr(), _stream()))
-    count(1 if T <= 128 else 2)
+    count(1 if T <= 32 else 2)
     return r
+
+
+def spread_rows(x, routes, out):
+    """Each token's row of x into its choices' rows of out (fb_spread_rows)."""
+    assert x.stride(1) == 1 and out.is_contiguous() and x.dtype == out.dtype
+    size = x.element_size()
+    check(lib().fb_spread_rows(x.data_ptr(), x.shape[0], x.shape[1] * size, x.stride(0) * size, routes.slots.data_ptr(), routes.k, out.data_ptr(), out.shape[0], _stream()))
+    count()
+    return out
 
 
 def grouped(x, w, routes, out, kind=_lib.DENSE_NONE, shared=False):

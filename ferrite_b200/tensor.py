@@ -664,10 +664,9 @@ class Tensor:
         rt, h, m = self.rt, self.realize(), down.rows
         assert h.batch == 1 and gate_up.cols == 2 * m and gate_up.batch == down.batch == routes.n and h.rows == routes.T
         if not routes.shared:
-            h = h if h.buf.is_contiguous() else (h + 0).realize()
             x = Tensor(rt, routes.tiles * routes.tile, h.cols, dtype=h.dtype)
-            ops.gather_rows(h.buf[0], routes.order, x.buf[0])
-            rt.launched("gather")
+            ops.spread_rows(h.buf[0], routes, x.buf[0])
+            rt.launched("spread rows")
             h = x
         act = Tensor(rt, routes.tiles * routes.tile, m, dtype=h.dtype)
         out = Tensor(rt, routes.tiles * routes.tile, down.cols, dtype=h.dtype)

@@ -179,12 +179,17 @@ int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_t x_batch, 
 /* Each token's k largest of n router logits (fp32, + bias where given; the lower column first among equals) and the softmax of
  * those (weights), and where each choice's row goes (slots, both [T, k]) in rows of whole tiles of `tile` (a multiple of 16):
  *   shared_rows   a tile a touched expert, holding all the tokens (T <= tile): the choice's row is the token's in its expert's tile
- *   otherwise     each expert's choices in tiles of their own; order[tiles * tile]: the token each row holds, -1 for none
+ *   otherwise     each expert's choices in tiles of their own
  * tile_expert[tiles]: each tile's expert, ascending (n past those used); live[0]: how many are used; tiles =
  * fb_route_tiles(...), the most there can be.  ids [T, k]: the choices. */
 int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_rows);
 int fb_route(const float* logits, int64_t T, int64_t ld, const float* bias, int n, int k, int tile, int shared_rows, float* weights, int32_t* ids,
-             int32_t* slots, int32_t* order, int32_t* tile_expert, int32_t* live, void* stream);
+             int32_t* slots, int32_t* tile_expert, int32_t* live, void* stream);
+
+/* Row t of x (row_bytes bytes, rows ldx_bytes apart) into the rows slots[t, 0 .. k) of out (rows one after another): the
+ * tokens' rows to their choices' places. */
+int fb_spread_rows(const void* x, int64_t T, int64_t row_bytes, int64_t ldx_bytes, const int32_t* slots, int k, void* out, int64_t out_rows,
+                   void* stream);
 
 /* Rows of tiles by each tile's own matrix: rows i * tile .. of out = rows i * tile .. of x (shared_rows: x's `x_rows` rows, the
  * same for every tile) @ W[tile_expert[i]]^T for the tiles i < live[0]; the other rows of out are left alone.

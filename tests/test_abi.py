@@ -112,9 +112,9 @@ def test_heads_and_experts_entry_points_refuse_bad_arguments_without_a_gpu():
     assert attend(4, 2048, 0) == -1 and b"up to 1024" in lib.fb_last_error()
     assert attend(4, 64, -1) == -1 and attend(4, 64, 8, chunk=1) == -1 and b"one sequence's" in lib.fb_last_error()
     assert lib.fb_route_tiles(5, 12, 4, 16, 1) == 12 and lib.fb_route_tiles(1, 12, 4, 16, 1) == 4 and lib.fb_route_tiles(100, 12, 4, 32, 0) == 400 // 32 + 12
-    rc = lib.fb_route(16, 100, 12, None, 12, 4, 64, 1, 16, 16, 16, None, 16, 16, None)
+    rc = lib.fb_route(16, 100, 12, None, 12, 4, 64, 1, 16, 16, 16, 16, 16, None)
     assert rc == -1 and b"all the tokens in one" in lib.fb_last_error()
-    rc = lib.fb_route(16, 4, 70, None, 70, 65, 16, 1, 16, 16, 16, None, 16, 16, None)
+    rc = lib.fb_route(16, 4, 70, None, 70, 65, 16, 1, 16, 16, 16, 16, 16, None)
     assert rc == -1 and b"up to 64 choices" in lib.fb_last_error()
     e = _lib.DenseEpilogue(kind=_lib.DENSE_DYT_ADD)
     rc = lib.fb_dense_grouped(16, 64, 64, 64, 0, 16, 64, 64, 4096, 2, 16, 16, 2, 32, 16, _lib.BF16, 64, ctypes.byref(e), None)

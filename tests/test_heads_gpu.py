@@ -190,8 +190,11 @@ def test_routes(torch, T, n, k):
     if r.shared:
         assert np.array_equal(slots % r.tile, np.repeat(np.arange(T)[:, None], k, 1))
     else:
-        order = to_numpy(r.order)
-        assert len(set(slots.reshape(-1).tolist())) == T * k and np.array_equal(order[slots], np.repeat(np.arange(T)[:, None], k, 1)) and (order >= 0).sum() == T * k
+        assert len(set(slots.reshape(-1).tolist())) == T * k
+        for dtype, cols in ((torch.bfloat16, 24), (torch.float32, 7), (torch.bfloat16, 9)):
+            x = on(rng.integers(-99, 99, (T, cols + 8)), dtype)[:, :cols]
+            out = ops.spread_rows(x, r, torch.zeros(r.tiles * r.tile, cols, dtype=dtype, device="cuda"))
+            assert np.array_equal(to_numpy(out)[slots], np.repeat(to_numpy(x)[:, None], k, 1))
 
 
 @pytest.mark.parametrize("T,n,k,K,m,N,bf16", [(1, 6, 2, 64, 32, 96, True), (32, 12, 4, 256, 64, 200, True), (17, 40, 8, 72, 48, 40, True), (64, 3, 1, 1024, 512, 512, True), (300, 12, 4, 256, 64, 264, True),
@@ -218,11 +221,12 @@ def test_experts(torch, T, n, k, K, m, N, bf16):
             assert np.abs(rows[slots[t, j]] - want).max() < (2e-2 if bf16 else 3e-6) * max(np.abs(want).max(), 0.5), (t, j)
 
 
-@pytest.mark.parametrize("cols,source,bf16", [(256, "bf16", True), (260, "fp32", True), (61, "fp32", False), (61, "bf16", True), (4096, "bf16", True), (5120, "fp32", False)])
-def test_the_end_of_a_layer(torch, cols, source, bf16):
+@pytest.mark.parametrize("cols,source,bf16,T,k", [(256, "bf16", True, 9, 5), (260, "fp32", True, 9, 5), (61, "fp32", False, 9, 40), (61, "bf16", True, 9, 5), (128, "bf16", True, 3, 50), (4096, "bf16", True, 9, 5),
+                                                  (2048, "bf16", True, 600, 2), (5120, "fp32", False, 9, 8), (9000, "bf16", True, 3, 2)])
+def test_the_end_of_a_layer(torch, cols, source, bf16, T, k):
     from types import SimpleNamespace as NS
     from ferrite_b200 import ops
-    rng, on, src, T, k = np.random.default_rng(6), Device(torch, bf16), Device(torch, source == "bf16"), 9, 5
+    rng, on, src = np.random.default_rng(6), Device(torch, bf16), Device(torch, source == "bf16")
     x, s1, s2, w = (np.float64(np.float32(rng.normal(0, 1, shape))) for shape in ((T, cols), cols, cols, cols))
     y, f = (rounded(rng.normal(0, 1, (T, cols)), source == "bf16") for _ in range(2))
     rows, slots, weights = rounded(rng.normal(0, 1, (T * k + 3, cols)), bf16), rng.permutation(T * k + 3)[:T * k].reshape(T, k), np.float64(np.float32(rng.uniform(0, 1, (T, k))))
@@ -232,7 +236,7 @@ def test_the_end_of_a_layer(torch, cols, source, bf16):
         out, h = on.f32(np.zeros((T, cols))), on(np.zeros((T, cols)))
         ops.add_norm(on.f32(x), out, src(y) if mixer else None, on.f32(s1), src(f) if other else None, on.f32(s2), on(rows) if experts else None, routes if experts else None, on.f32(w), 1.0, 1e-3, h)
         want = x + mixer * y * s1 + (other * f + experts * chosen) * s2
-        np.testing.assert_allclose(to_numpy(out), want, rtol=1e-5, atol=1e-5)
+        np.testing.assert_allclose(to_numpy(out), want, rtol=1e-5, atol=2e-5)
         tol = 6e-3 if bf16 else 1e-5
         np.testing.assert_allclose(to_numpy(h), oracle.rms(want, 1 + w, 1e-3), rtol=tol, atol=tol)
 
