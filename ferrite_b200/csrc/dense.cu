@@ -46,8 +46,8 @@ struct DenseParams {
   int out_dtype;
   int64_t ldo, out_batch;
   int settled;
-  // rows in tiles of `nt`, each with a matrix of its own (fb_dense_grouped): the tiles' matrices and how many there are, both
-  // read on the device; x_step: how far the rows move on a tile (nt, or 0: every tile the same rows)
+  // rows in tiles of `nt`, each with a matrix of its own (fb_dense_grouped): the tiles' matrices (and which tiles share one) and
+  // how many there are, both read on the device; x_step: how far the rows move on a tile (nt, or 0: every tile the same rows)
   const int32_t *tile_expert, *live;
   int x_step;
   float shift;  // GLU: added to the up half
@@ -59,9 +59,13 @@ struct DenseTile {
 };
 // tiles_m: the tiles of rows there are (grouped: those in use)
 __device__ __forceinline__ DenseTile tile_of(const DenseParams& p, int id, int tiles_m) {  // tokens fastest: tiles that share weights run together
-  const int rest = id / tiles_m, m = id % tiles_m;
-  if (p.tile_expert) return {m, rest, p.tile_expert[m]};
-  return {m, rest % p.tiles_n, rest / p.tiles_n};
+  if (p.tile_expert) {  // (a matrix after the other, so that its rows are read again from L2: the tiles id / tiles_n has them side by side)
+    const int32_t* run = p.tile_expert + 3 * (id / p.tiles_n);
+    const int at = id - run[1] * p.tiles_n;
+    return {run[1] + at % run[2], at / run[2], run[0]};
+  }
+  const int rest = id / tiles_m;
+  return {id % tiles_m, rest % p.tiles_n, rest / p.tiles_n};
 }
 
 // what the epilogue needs of a column, read once a tile

@@ -20,7 +20,7 @@ struct RouteArgs {
   float* weights;       // [T, k]
   int32_t* ids;         // [T, k]
   int32_t* slots;       // [T, k]: the row of each choice
-  int32_t* tile_expert; // [tiles], n past those used
+  int32_t* tile_expert; // [tiles, 3]: a tile's expert (n past those used), its expert's first tile and how many it has
   int32_t* live;        // [1] tiles used
 };
 
@@ -145,12 +145,11 @@ __global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, c
   if (tid == 0) *a.live = used;
   for (int e = e0; e < e1; ++e) {
     const int n = tiles_of(e);
-    for (int i = 0; i < n; ++i)
-      if (first + i < a.tiles) a.tile_expert[first + i] = e;
+    for (int i = first; i < first + n && i < a.tiles; ++i) a.tile_expert[3 * i] = e, a.tile_expert[3 * i + 1] = first, a.tile_expert[3 * i + 2] = n;
     count[e] = first * a.tile;
     first += n;
   }
-  for (int i = used + tid; i < a.tiles; i += blockDim.x) a.tile_expert[i] = a.n;
+  for (int i = used + tid; i < a.tiles; i += blockDim.x) a.tile_expert[3 * i] = a.n, a.tile_expert[3 * i + 1] = a.tile_expert[3 * i + 2] = 0;
   __syncthreads();
   for (int64_t i0 = tid; i0 < choices; i0 += BATCH * 1024) {
     int e[BATCH];
@@ -201,7 +200,7 @@ __global__ void __launch_bounds__(256) grouped_matmul_kernel(const GroupedArgs g
   griddep_wait();
   const int i = blockIdx.y * 16 / g.tile, r0 = blockIdx.y * 16 % g.tile;
   if (i >= *g.live) return;
-  const int e = g.tile_expert[i];
+  const int e = g.tile_expert[3 * i];
   if (e < 0 || e >= g.n) return;
   __shared__ float sa[16][17], sb[16][17];
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;

@@ -377,20 +377,20 @@ class Routes:
         self.tiles = lib().fb_route_tiles(T, n, k, tile, int(shared))
         i32 = lambda *shape: torch.empty(*shape, dtype=torch.int32, device=device)
         self.weights, self.ids, self.slots = torch.empty(T, k, dtype=torch.float32, device=device), i32(T, k), i32(T, k)
-        self.tile_expert, self.live = i32(self.tiles), i32(1)
+        self.tile_expert, self.live = i32(self.tiles, 3), i32(1)
 
 
 @functools.lru_cache
 def route_tile(T, n, k):
     """(rows of a tile, whether each tile holds all the tokens) for T tokens with k of n experts each: a few tokens are not
     sorted.  More: the height at which evenly drawn choices make for the least work, a tile costing what its weights' way
-    through a CTA does (about 60 rows' products) or its products."""
+    through a CTA does (as much as 110 rows' products, measured) or its products."""
     if T <= 64:
         return -(-T // 16) * 16, True
     m = T * k / n
     spread = (m * (1 - k / n)) ** 0.5 + 1e-9
     above = lambda x: 0.5 * math.erfc((x - m) / (spread * 2 ** 0.5))  # how likely an expert has more than x rows
-    work = lambda tile: sum(above(j * tile) for j in range(int((m + 5 * spread) / tile) + 2)) * max(62 + 0.1 * tile, tile)
+    work = lambda tile: sum(above(j * tile) for j in range(int((m + 5 * spread) / tile) + 2)) * max(110 + 0.1 * tile, tile)
     return min(range(32, 257, 16), key=work), False
 
 

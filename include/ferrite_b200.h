@@ -180,7 +180,7 @@ int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_t x_batch, 
  * those (weights), and where each choice's row goes (slots, both [T, k]) in rows of whole tiles of `tile` (a multiple of 16):
  *   shared_rows   a tile a touched expert, holding all the tokens (T <= tile): the choice's row is the token's in its expert's tile
  *   otherwise     each expert's choices in tiles of their own
- * tile_expert[tiles]: each tile's expert, ascending (n past those used); live[0]: how many are used; tiles =
+ * tile_expert[tiles, 3]: each tile's expert, ascending (n past those used), that expert's first tile and its number of tiles; live[0]: how many are used; tiles =
  * fb_route_tiles(...), the most there can be.  ids [T, k]: the choices. */
 int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_rows);
 int fb_route(const float* logits, int64_t T, int64_t ld, const float* bias, int n, int k, int tile, int shared_rows, float* weights, int32_t* ids,
@@ -192,7 +192,7 @@ int fb_spread_rows(const void* x, int64_t T, int64_t row_bytes, int64_t ldx_byte
                    void* stream);
 
 /* Rows of tiles by each tile's own matrix: rows i * tile .. of out = rows i * tile .. of x (shared_rows: x's `x_rows` rows, the
- * same for every tile) @ W[tile_expert[i]]^T for the tiles i < live[0]; the other rows of out are left alone.
+ * same for every tile) @ W[tile_expert[i, 0]]^T for the tiles i < live[0]; the other rows of out are left alone.
  * fb_dense_grouped: on the tensor cores, operands as fb_dense takes them (W [n, N, K], w_batch elements apart), epilogues
  * FB_DENSE_NONE, FB_DENSE_GLU and FB_DENSE_SWIGLU.  fb_grouped_matmul: any sizes, bf16 or fp32, W by strides (matrix, row of K, column). */
 int fb_dense_grouped(const void* x, int64_t x_rows, int64_t K, int64_t ldx, int shared_rows, const void* W, int64_t N, int64_t ldw, int64_t w_batch,

@@ -182,10 +182,14 @@ def test_routes(torch, T, n, k):
     e = np.exp(np.take_along_axis(z, picks, -1) - z.max(-1, keepdims=True))
     assert np.array_equal(to_numpy(r.ids), picks)
     np.testing.assert_allclose(to_numpy(r.weights), e / e.sum(-1, keepdims=True), rtol=1e-5, atol=1e-7)
-    live, experts, slots = int(to_numpy(r.live)[0]), to_numpy(r.tile_expert), to_numpy(r.slots)
+    live, runs, slots = int(to_numpy(r.live)[0]), to_numpy(r.tile_expert), to_numpy(r.slots)
+    experts = runs[:, 0]
     count = np.bincount(picks.reshape(-1), minlength=n)
     assert r.shared == (T <= 64) and live == ((count > 0) if r.shared else -(-count // r.tile)).sum() <= r.tiles
     assert (experts[live:] == n).all() and (np.diff(experts[:live]) >= 0).all()
+    for i in range(live):
+        mine = np.flatnonzero(experts[:live] == experts[i])
+        assert runs[i, 1] == mine[0] and runs[i, 2] == len(mine)
     assert np.array_equal(experts[slots // r.tile], picks)
     if r.shared:
         assert np.array_equal(slots % r.tile, np.repeat(np.arange(T)[:, None], k, 1))
