@@ -34,8 +34,12 @@ enum PromptWait { PW_Q = 501, PW_EMPTY, PW_FULL, PW_S, PW_P, PW_PV, PW_PV_MMA, P
 struct PromptParams {
   HeadsArgs a;
   int groups, tokens;  // tokens of a group
+  int fours;           // gates and results are whole, aligned groups of four columns
   int ck, cv, nv, stages, q_bytes, tmem_cols;  // 64-column pieces of a query / key and of a value; columns of the sums; bytes from one group's queries to the next's
 };
+
+// v times the sigmoid of g
+__device__ __forceinline__ float gated(float v, float g) { return __fdividef(v, 1.f + __expf(-g)); }
 
 template <int GROUPS>
 __global__ void __launch_bounds__(HP_THREADS, 1) heads_prompt_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tkv, const PromptParams p) {
@@ -240,6 +244,29 @@ __global__ void __launch_bounds__(HP_THREADS, 1) heads_prompt_kernel(const __gri
 #pragma unroll
       for (int e = 0; e < 32; ++e) stage[lane * 33 + e] = n_tiles && c + e < p.nv ? v[e] * f : 0.f;
       __syncwarp();
+      if (p.fours) {  // eight lanes a row, four columns each: all of a block's gates on their way at once
+        const int c4 = 4 * (lane & 7);
+        const bool mine = c + c4 < a.vdim;
+        float4 gate[8];
+        int64_t to[8];
+#pragma unroll
+        for (int r = 0; r < 8; ++r) {
+          const int64_t from = __shfl_sync(0xffffffffu, gate_at, 4 * r + (lane >> 3)) + c + c4;
+          to[r] = __shfl_sync(0xffffffffu, out_at, 4 * r + (lane >> 3));
+          gate[r] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (a.gate && mine && to[r] >= 0) gate[r] = a.gate_dtype == FB_FP32 ? four(static_cast<const float*>(a.gate) + from) : four(static_cast<const uint16_t*>(a.gate) + from);
+        }
+#pragma unroll
+        for (int r = 0; r < 8; ++r)
+          if (mine && to[r] >= 0) {
+            const float* v = stage + (4 * r + (lane >> 3)) * 33 + c4;
+            float4 y = make_float4(v[0], v[1], v[2], v[3]);
+            if (a.gate) y = make_float4(gated(y.x, gate[r].x), gated(y.y, gate[r].y), gated(y.z, gate[r].z), gated(y.w, gate[r].w));
+            put_four(static_cast<uint16_t*>(a.out) + to[r] + c + c4, y);
+          }
+        __syncwarp();
+        continue;
+      }
       const bool mine = c + lane < a.vdim;
 #pragma unroll 1
       for (int r0 = 0; r0 < 32; r0 += 8) {
@@ -255,7 +282,7 @@ __global__ void __launch_bounds__(HP_THREADS, 1) heads_prompt_kernel(const __gri
         for (int r = 0; r < 8; ++r)
           if (mine && to[r] >= 0) {
             const float v = stage[(r0 + r) * 33 + lane];
-            static_cast<uint16_t*>(a.out)[to[r] + c + lane] = (uint16_t)float_to_bf16_bits(a.gate ? __fdividef(v, 1.f + __expf(-gate[r])) : v);
+            static_cast<uint16_t*>(a.out)[to[r] + c + lane] = (uint16_t)float_to_bf16_bits(a.gate ? gated(v, gate[r]) : v);
           }
       }
       __syncwarp();
@@ -314,6 +341,7 @@ int heads_prompt(const HeadsArgs& a, cudaStream_t s) {
   p.a = a;
   const bool two = ceil_div(a.T, 2 * (HP_ROWS / a.rep)) * a.kv_heads >= sm_count_of_device() && prompt_sizes(p, 2);
   if (!two) prompt_sizes(p, 1);
+  p.fours = a.ld_o % 4 == 0 && (uintptr_t)a.out % 8 == 0 && (!a.gate || (a.ld_g % 4 == 0 && (uintptr_t)a.gate % (a.gate_dtype == FB_FP32 ? 16 : 8) == 0));
   CUtensorMap tq, tkv;
   const int64_t qd[4] = {a.dim, a.rep, a.kv_heads, a.T}, qs[3] = {a.dim, (int64_t)a.rep * a.dim, a.ld_q};
   const int qb[4] = {64, a.rep, 1, p.tokens};

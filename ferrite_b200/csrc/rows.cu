@@ -9,16 +9,6 @@
 
 namespace fb {
 
-// four columns at a time
-__device__ __forceinline__ float4 four(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 four(const uint16_t* p) {
-  const uint2 v = *reinterpret_cast<const uint2*>(p);
-  return make_float4(bf16_bits_to_float(v.x & 0xffffu), bf16_bits_to_float(v.x >> 16), bf16_bits_to_float(v.y & 0xffffu), bf16_bits_to_float(v.y >> 16));
-}
-__device__ __forceinline__ void put_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void put_four(uint16_t* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
-__device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) { return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w)); }
-
 struct EmbedArgs {
   const void *table, *places_table;  // [rows, cols], [place_rows, cols] or null
   int64_t rows, place_rows, cols;

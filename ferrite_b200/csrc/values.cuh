@@ -10,6 +10,16 @@ __device__ __forceinline__ float value_of(uint16_t x) { return bf16_bits_to_floa
 __device__ __forceinline__ void store_value(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store_value(uint16_t* p, float v) { *p = (uint16_t)float_to_bf16_bits(v); }
 
+// four columns at a time
+__device__ __forceinline__ float4 four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 four(const uint16_t* p) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16_bits_to_float(v.x & 0xffffu), bf16_bits_to_float(v.x >> 16), bf16_bits_to_float(v.y & 0xffffu), bf16_bits_to_float(v.y >> 16));
+}
+__device__ __forceinline__ void put_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put_four(uint16_t* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
+__device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) { return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w)); }
+
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
 // tanh by one exponential, and by its power series where that would cancel: about 2e-7 of the result either way
