@@ -22,8 +22,8 @@ namespace fb {
 
 namespace {
 
-constexpr int HP_KEYS = 64, HP_WARP_LOAD = 8, HP_WARP_MMA = 9, HP_THREADS = 10 * 32, HP_MAX_STAGES = 6, HP_ROWS = 128;
-constexpr size_t HP_SMEM = 224 * 1024;
+constexpr int HP_KEYS = 64, HP_MAX_STAGES = 6, HP_ROWS = 128;
+constexpr size_t HP_SMEM = 224 * 1024, HP_SMEM_HALF = 112 * 1024;  // a CTA's alone on its SM, one of two
 constexpr int HP_Q_CHUNK = HP_ROWS * 128, HP_K_CHUNK = HP_KEYS * 128;  // 64 columns of a group's queries, of a tile's keys or values
 constexpr int HP_COLS = 2 * HP_KEYS + 128;                             // tensor memory of a group: two tiles of scores, the sums
 constexpr float HP_SLACK = 8.f;                                        // log2 of how far scores may outgrow the reference maximum
@@ -35,14 +35,15 @@ struct PromptParams {
   HeadsArgs a;
   int groups, tokens;  // tokens of a group
   int fours;           // gates and results are whole, aligned groups of four columns
-  int ck, cv, nv, stages, q_bytes, tmem_cols;  // 64-column pieces of a query / key and of a value; columns of the sums; bytes from one group's queries to the next's
+  int ck, cv, nv, stages, q_bytes, tmem_cols, smem;  // 64-column pieces of a query / key and of a value; columns of the sums; bytes from one group's queries to the next's
 };
 
 // v times the sigmoid of g
 __device__ __forceinline__ float gated(float v, float g) { return __fdividef(v, 1.f + __expf(-g)); }
 
 template <int GROUPS>
-__global__ void __launch_bounds__(HP_THREADS, 1) heads_prompt_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tkv, const PromptParams p) {
+__global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) heads_prompt_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tkv, const PromptParams p) {
+  constexpr int HP_WARP_LOAD = 4 * GROUPS, HP_WARP_MMA = HP_WARP_LOAD + 1;
   extern __shared__ uint8_t prompt_smem[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(prompt_smem) + 1023) & ~uintptr_t(1023));
   __shared__ uint64_t bars[2 * HP_MAX_STAGES + 10];
@@ -50,8 +51,8 @@ __global__ void __launch_bounds__(HP_THREADS, 1) heads_prompt_kernel(const __gri
   uint64_t *full = bars, *empty = bars + HP_MAX_STAGES, *q_full = bars + 2 * HP_MAX_STAGES, *s_full = q_full + 2, *p_full = s_full + 4, *pv_done = p_full + 2;
   const uint32_t abort_flag = smem_u32(tmem_slot + 1);
   const HeadsArgs& a = p.a;
-  const int tid = threadIdx.x, warp = uniform_warp(), lane = tid & 31, g = blockIdx.y, S = p.stages;
-  const int tile = gridDim.x - 1 - blockIdx.x;  // (the last see the most keys: they start first)
+  const int tid = threadIdx.x, warp = uniform_warp(), lane = tid & 31, g = blockIdx.x, S = p.stages;
+  const int tile = gridDim.y - 1 - blockIdx.y;  // (the last see the most keys: they start first)
   const uint32_t sQ = smem_u32(smem), sKV = sQ + GROUPS * p.q_bytes, stage_bytes = (p.ck + p.cv) * HP_K_CHUNK;
 
   griddep_launch_dependents();
@@ -248,17 +249,26 @@ __global__ void __launch_bounds__(HP_THREADS, 1) heads_prompt_kernel(const __gri
         const int c4 = 4 * (lane & 7);
         const bool mine = c + c4 < a.vdim;
         float4 gate[8];
-        int64_t to[8];
+        int64_t from[8], to[8];
 #pragma unroll
         for (int r = 0; r < 8; ++r) {
-          const int64_t from = __shfl_sync(0xffffffffu, gate_at, 4 * r + (lane >> 3)) + c + c4;
+          from[r] = __shfl_sync(0xffffffffu, gate_at, 4 * r + (lane >> 3)) + c + c4;
           to[r] = __shfl_sync(0xffffffffu, out_at, 4 * r + (lane >> 3));
+          if (!mine) to[r] = -1;
           gate[r] = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (a.gate && mine && to[r] >= 0) gate[r] = a.gate_dtype == FB_FP32 ? four(static_cast<const float*>(a.gate) + from) : four(static_cast<const uint16_t*>(a.gate) + from);
+        }
+        if (a.gate && a.gate_dtype == FB_FP32) {
+#pragma unroll
+          for (int r = 0; r < 8; ++r)
+            if (to[r] >= 0) gate[r] = four(static_cast<const float*>(a.gate) + from[r]);
+        } else if (a.gate) {
+#pragma unroll
+          for (int r = 0; r < 8; ++r)
+            if (to[r] >= 0) gate[r] = four(static_cast<const uint16_t*>(a.gate) + from[r]);
         }
 #pragma unroll
         for (int r = 0; r < 8; ++r)
-          if (mine && to[r] >= 0) {
+          if (to[r] >= 0) {
             const float* v = stage + (4 * r + (lane >> 3)) * 33 + c4;
             float4 y = make_float4(v[0], v[1], v[2], v[3]);
             if (a.gate) y = make_float4(gated(y.x, gate[r].x), gated(y.y, gate[r].y), gated(y.z, gate[r].z), gated(y.w, gate[r].w));
@@ -303,9 +313,11 @@ bool prompt_sizes(PromptParams& p, int groups) {
   p.groups = groups, p.tokens = HP_ROWS / a.rep, p.ck = (a.dim + 63) / 64, p.cv = (a.vdim + 63) / 64, p.nv = (a.vdim + 15) / 16 * 16;
   p.q_bytes = p.ck * HP_Q_CHUNK > 17 * 1024 ? p.ck * HP_Q_CHUNK : 17 * 1024;  // (17 KB: what the result takes on its way out)
   p.tmem_cols = groups * HP_COLS;
-  const int64_t room = (int64_t)HP_SMEM - 1024 - groups * p.q_bytes, stage = (p.ck + p.cv) * HP_K_CHUNK;
-  p.stages = (int)(room / stage < HP_MAX_STAGES ? room / stage : HP_MAX_STAGES);
-  return room > 0 && p.stages >= 2;
+  const int64_t stage = (p.ck + p.cv) * HP_K_CHUNK, rest = 1024 + groups * p.q_bytes;
+  p.smem = groups == 1 && rest + 2 * stage <= (int64_t)HP_SMEM_HALF ? HP_SMEM_HALF : HP_SMEM;
+  const int64_t room = ((int64_t)p.smem - rest) / stage;
+  p.stages = (int)(room < HP_MAX_STAGES ? room : HP_MAX_STAGES);
+  return p.stages >= 2;
 }
 
 template <int GROUPS>
@@ -313,8 +325,8 @@ int launch_prompt(const PromptParams& p, const CUtensorMap& tq, const CUtensorMa
   static std::atomic<uint64_t> opted{0};
   if (first_on_device(opted)) cudaFuncSetAttribute(heads_prompt_kernel<GROUPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)HP_SMEM);
   cudaLaunchConfig_t cfg{};
-  cfg.gridDim = dim3((unsigned)ceil_div(p.a.T, GROUPS * p.tokens), (unsigned)p.a.kv_heads), cfg.blockDim = dim3(HP_THREADS);
-  cfg.dynamicSmemBytes = HP_SMEM, cfg.stream = s;
+  cfg.gridDim = dim3((unsigned)p.a.kv_heads, (unsigned)ceil_div(p.a.T, GROUPS * p.tokens)), cfg.blockDim = dim3((4 * GROUPS + 2) * 32);
+  cfg.dynamicSmemBytes = p.smem, cfg.stream = s;
   cudaLaunchAttribute attr[1];
   attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   attr[0].val.programmaticStreamSerializationAllowed = 1;
@@ -330,7 +342,7 @@ static const StatusWord g_status_reader(read_and_clear_status_word);
 // a chunk of one sequence with tiles enough for half the SMs (fewer: heads_attention.cu splits the keys), heads that tensor
 // memory takes, rows that TMA takes (the caller has checked that q and the cache are whole 16-byte pieces)
 bool heads_prompt_supports(const HeadsArgs& a) {
-  if (!a.chunk || a.rep > HP_ROWS || a.dim > 256 || a.vdim > 128 || a.ld_o % 2 || a.T >= (1 << 30) || a.cache_rows >= (1ll << 31)) return false;
+  if (!a.chunk || a.rep > HP_ROWS || a.dim > 256 || a.vdim > 128 || a.ld_o % 2 || ceil_div(a.T, HP_ROWS / a.rep) > 65535 || a.cache_rows >= (1ll << 31)) return false;
   PromptParams p{};
   p.a = a;
   return ceil_div(a.T, HP_ROWS / a.rep) * a.kv_heads >= 74 && prompt_sizes(p, 1) && tma_encoder() != nullptr;
@@ -339,7 +351,8 @@ bool heads_prompt_supports(const HeadsArgs& a) {
 int heads_prompt(const HeadsArgs& a, cudaStream_t s) {
   PromptParams p{};
   p.a = a;
-  const bool two = ceil_div(a.T, 2 * (HP_ROWS / a.rep)) * a.kv_heads >= sm_count_of_device() && prompt_sizes(p, 2);
+  // two groups a CTA share the tiles of wide heads; CTAs of narrow ones stand side by side on an SM instead
+  const bool two = a.dim + a.vdim > 192 && ceil_div(a.T, 2 * (HP_ROWS / a.rep)) * a.kv_heads >= sm_count_of_device() && prompt_sizes(p, 2);
   if (!two) prompt_sizes(p, 1);
   p.fours = a.ld_o % 4 == 0 && (uintptr_t)a.out % 8 == 0 && (!a.gate || (a.ld_g % 4 == 0 && (uintptr_t)a.gate % (a.gate_dtype == FB_FP32 ? 16 : 8) == 0));
   CUtensorMap tq, tkv;
