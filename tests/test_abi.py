@@ -111,8 +111,8 @@ def test_heads_and_experts_entry_points_refuse_bad_arguments_without_a_gpu():
     assert attend(3, 64, 0) == -1 and b"whole groups" in lib.fb_last_error()
     assert attend(4, 2048, 0) == -1 and b"up to 1024" in lib.fb_last_error()
     assert attend(4, 64, -1) == -1 and attend(4, 64, 8, chunk=1) == -1 and b"one sequence's" in lib.fb_last_error()
-    assert lib.fb_route_tiles(5, 12, 4, 16, 1) == 12 and lib.fb_route_tiles(1, 12, 4, 16, 1) == 4 and lib.fb_route_tiles(100, 12, 4, 32, 0) == 400 // 32 + 12
-    rc = lib.fb_route(16, 100, 12, None, 12, 4, 64, 1, 16, 16, 16, 16, 16, None)
+    assert lib.fb_route_tiles(5, 10, 3, 16, 1) == 10 and lib.fb_route_tiles(1, 10, 3, 16, 1) == 3 and lib.fb_route_tiles(100, 10, 3, 32, 0) == 300 // 32 + 10
+    rc = lib.fb_route(16, 100, 10, None, 10, 3, 64, 1, 16, 16, 16, 16, 16, None)
     assert rc == -1 and b"all the tokens in one" in lib.fb_last_error()
     rc = lib.fb_route(16, 4, 70, None, 70, 65, 16, 1, 16, 16, 16, 16, 16, None)
     assert rc == -1 and b"up to 64 choices" in lib.fb_last_error()
