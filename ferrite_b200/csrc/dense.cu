@@ -15,7 +15,7 @@
 // memory, each then takes a share of the tokens and adds the others' sums to its own in rank order (the same every run).
 //
 // What follows a matmul in its model runs on the accumulators (fb_dense_epilogue): SiLU on the first columns, a clamped
-// gated unit (gate and up rows alternate in runs of 16 inside a tile, so a pair is 16 lanes apart), a gate per head, and the
+// or a GELU-gated unit (gate and up rows alternate in runs of 16 inside a tile, so a pair is 16 lanes apart), a gate per head, and the
 // Dynamic Tanh - residual add - Dynamic Tanh between two branches, which needs no sum over the row and therefore no
 // kernel of its own.  Every wait is bounded (sm100.cuh).
 //
@@ -28,6 +28,9 @@
 #include "values.cuh"
 
 namespace fb {
+
+// whether W holds gate rows, then as many up rows, that meet in the epilogue
+__host__ __device__ constexpr bool paired(int kind) { return kind == FB_DENSE_GLU || kind == FB_DENSE_GEGLU; }
 
 namespace {
 
@@ -81,6 +84,9 @@ __device__ __forceinline__ Column column_of(const DenseParams& p, int64_t n, boo
       if (p.e.h_out) c.alpha2 = *p.e.alpha2, c.w2 = p.e.w2[n], c.b2 = p.e.b2[n];
     }
   }
+  if constexpr (EPI == FB_DENSE_GEGLU) {
+    if (live) c.w = p.e.gate_bias ? p.e.gate_bias[n] : 0.f, c.b = p.e.up_bias ? p.e.up_bias[n] : 0.f;
+  }
   return c;
 }
 
@@ -99,6 +105,10 @@ __device__ __forceinline__ void emit(const DenseParams& p, const Column& c, int 
   if constexpr (EPI == FB_DENSE_GLU) {
     const float g = fminf(v, p.e.limit), u = fminf(fmaxf(up, -p.e.limit), p.e.limit);
     v = g / (1.f + __expf(-p.e.slope * g)) * (u + p.shift);
+  }
+  if constexpr (EPI == FB_DENSE_GEGLU) {
+    const float g = v + c.w;
+    v = 0.5f * g * (1.f + tanh_of(0.7978845608028654f * fmaf(0.044715f * g * g, g, g))) * (up + c.b);
   }
   if constexpr (EPI == FB_DENSE_GATE) v *= gate;
   const int64_t at = b * p.out_batch + t * p.ldo + n;  // (grouped: out_batch 0, the rows follow the tiles)
@@ -142,7 +152,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
     auto weights = [&](const DenseTile& t, int k, int slot) {
       const uint32_t bar = smem_u32(full + slot), dst = smem_u32(smem + slot * stage_bytes);
       mbar_expect_tx(bar, (uint32_t)stage_bytes);
-      if (EPI == FB_DENSE_GLU) tma_load_5d(dst, &tw, 64 * k, 0, 0, 4 * t.n, t.b, bar);
+      if (paired(EPI)) tma_load_5d(dst, &tw, 64 * k, 0, 0, 4 * t.n, t.b, bar);
       else tma_load_3d(dst, &tw, 64 * k, 128 * t.n, t.b, bar);
     };
     int early = 0;
@@ -212,8 +222,8 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
           for (int e = 0; e < 8; ++e) ex[(col0 + c + e) * 128 + row] = v[e];
         }
       } else {
-        const int64_t col = EPI == FB_DENSE_GLU ? 64 * (int64_t)t.n + 16 * q + (lane & 15) : 128 * (int64_t)t.n + row;
-        const bool live = col < (EPI == FB_DENSE_GLU ? p.N / 2 : p.N);
+        const int64_t col = paired(EPI) ? 64 * (int64_t)t.n + 16 * q + (lane & 15) : 128 * (int64_t)t.n + row;
+        const bool live = col < (paired(EPI) ? p.N / 2 : p.N);
         const Column mine = column_of<EPI>(p, col, live);
         for (int c = 0; c < half && t0 + c < p.M; c += 8) {
           float v[8], extra[8];
@@ -227,7 +237,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
             }
           }
           tmem_ld_wait();
-          if constexpr (EPI == FB_DENSE_GLU) {
+          if constexpr (paired(EPI)) {
             // lanes 0-15 hold gates, 16-31 their ups: the low half takes the first four tokens, the high half the others
             const bool high = lane >= 16;
 #pragma unroll
@@ -261,8 +271,8 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
       const DenseTile t = tile_of(p, blockIdx.x, tiles_m);
       const int share = (nt + p.splits - 1) / p.splits, first = blockIdx.y * share, last = min(nt, first + share);
       const int row = tid & 127;
-      const int64_t col = EPI == FB_DENSE_GLU ? 64 * (int64_t)t.n + (row >> 5) * 16 + (row & 15) : 128 * (int64_t)t.n + row;
-      const bool live = col < (EPI == FB_DENSE_GLU ? p.N / 2 : p.N) && (EPI != FB_DENSE_GLU || !(row & 16));
+      const int64_t col = paired(EPI) ? 64 * (int64_t)t.n + (row >> 5) * 16 + (row & 15) : 128 * (int64_t)t.n + row;
+      const bool live = col < (paired(EPI) ? p.N / 2 : p.N) && (!paired(EPI) || !(row & 16));
       const Column mine = column_of<EPI>(p, col, live);
       for (int c = first + (tid >> 7); c < last; c += 2) {
         const int64_t tt = (int64_t)nt * t.m + c;
@@ -277,7 +287,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) dense_kernel(const __grid_consta
           part[s] = upper[s] = 0.f;
           if (s < p.splits) {
             part[s] = load_cluster_f32(at, s);
-            if constexpr (EPI == FB_DENSE_GLU) upper[s] = load_cluster_f32(at + 64, s);
+            if constexpr (paired(EPI)) upper[s] = load_cluster_f32(at + 64, s);
           }
         }
 #pragma unroll
@@ -318,7 +328,7 @@ static const StatusWord g_status_reader(read_and_clear_status_word);
 
 extern "C" int fb_dense_supports(const void* x, int64_t ldx, int64_t x_batch, const void* W, int64_t ldw, int64_t w_batch, int64_t K, int64_t N, int kind) {
   return K >= 8 && K % 8 == 0 && N >= 1 && ldx % 8 == 0 && ldw % 8 == 0 && x_batch % 8 == 0 && w_batch % 8 == 0 && ldx >= K && ldw >= K && (uintptr_t)x % 16 == 0 &&
-         (uintptr_t)W % 16 == 0 && ((kind != FB_DENSE_GLU && kind != FB_DENSE_SWIGLU) || N % 32 == 0) && fb::tma_encoder() != nullptr;
+         (uintptr_t)W % 16 == 0 && ((!fb::paired(kind) && kind != FB_DENSE_SWIGLU) || N % 32 == 0) && fb::tma_encoder() != nullptr;
 }
 
 // what fb_dense and fb_dense_grouped share: the tiles' depth and the CTAs', and the launch.  p: sizes, results and the way rows
@@ -348,7 +358,7 @@ static int run_dense(fb::DenseParams& p, const void* x, int64_t x_rows, int64_t 
   p.steps_per_split = (int)ceil_div(p.steps, p.splits);
   const int grid = p.splits > 1 ? p.tiles : p.tiles < sms ? p.tiles : sms;
   CUtensorMap tw, tx;
-  if (kind == FB_DENSE_GLU) {
+  if (paired(kind)) {
     const int64_t dims[5] = {K, 16, 2, p.N / 32, matrices}, strides[4] = {ldw, p.N / 2 * ldw, 16 * ldw, matrices > 1 ? w_batch : ldw};
     const int box[5] = {64, 16, 2, 4, 1};
     if (int rc = tma_map_bf16(&tw, W, 5, dims, strides, box, "fb_dense (weights)")) return rc;
@@ -364,6 +374,7 @@ static int run_dense(fb::DenseParams& p, const void* x, int64_t x_rows, int64_t 
   switch (kind) {
     case FB_DENSE_SILU: return launch_dense<FB_DENSE_SILU>(tw, tx, p, grid, smem, s);
     case FB_DENSE_GLU: return launch_dense<FB_DENSE_GLU>(tw, tx, p, grid, smem, s);
+    case FB_DENSE_GEGLU: return launch_dense<FB_DENSE_GEGLU>(tw, tx, p, grid, smem, s);
     case FB_DENSE_GATE: return launch_dense<FB_DENSE_GATE>(tw, tx, p, grid, smem, s);
     case FB_DENSE_DYT_ADD: return launch_dense<FB_DENSE_DYT_ADD>(tw, tx, p, grid, smem, s);
     default: return launch_dense<FB_DENSE_NONE>(tw, tx, p, grid, smem, s);
@@ -382,25 +393,25 @@ extern "C" int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_
   using namespace fb;
   FB_REQUIRE(x && W && out && M >= 1 && batch >= 1 && M < (1 << 30) && N < (1 << 30), "fb_dense: null pointer or empty");
   fb_dense_epilogue e = epilogue_host ? *epilogue_host : fb_dense_epilogue{};
-  FB_REQUIRE(e.kind >= FB_DENSE_NONE && e.kind <= FB_DENSE_SWIGLU, "fb_dense: unknown epilogue %d", e.kind);
+  FB_REQUIRE(e.kind >= FB_DENSE_NONE && e.kind <= FB_DENSE_GEGLU, "fb_dense: unknown epilogue %d", e.kind);
   const float shift = settle_unit(e);
   FB_REQUIRE(K >= 8 && K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && x_batch % 8 == 0 && w_batch % 8 == 0 && ldx >= K && ldw >= K && (uintptr_t)x % 16 == 0 &&
                  (uintptr_t)W % 16 == 0 && N >= 1,
              "fb_dense: rows of x and W 16-byte aligned, K a multiple of 8 (K %lld, row strides %lld and %lld)", (long long)K, (long long)ldx, (long long)ldw);
   FB_REQUIRE(out_dtype == FB_BF16 || out_dtype == FB_FP32, "fb_dense: out is bf16 or fp32");
-  FB_REQUIRE(e.kind != FB_DENSE_GLU || (N % 32 == 0 && batch == 1), "fb_dense: a gated unit takes one matrix of whole runs of 16 gate rows and as many up rows");
+  FB_REQUIRE(!paired(e.kind) || (N % 32 == 0 && batch == 1), "fb_dense: a gated unit takes one matrix of whole runs of 16 gate rows and as many up rows");
   FB_REQUIRE(e.kind != FB_DENSE_GATE || e.gate, "fb_dense: no gate given");
   FB_REQUIRE(e.kind != FB_DENSE_DYT_ADD || (e.residual && e.alpha && e.w && e.b && out_dtype == FB_FP32 && batch == 1 && (!e.h_out || (e.alpha2 && e.w2 && e.b2))),
              "fb_dense: a Dynamic Tanh and add takes its vectors, a residual and an fp32 result");
   FB_REQUIRE(tma_encoder() != nullptr, "fb_dense: no CUDA driver");
-  const int64_t out_cols = e.kind == FB_DENSE_GLU ? N / 2 : N;
+  const int64_t out_cols = fb::paired(e.kind) ? N / 2 : N;
   FB_REQUIRE(ldo >= out_cols, "fb_dense: rows of out too close");
   DenseParams p{};
   p.M = M, p.N = N, p.e = e, p.out = out, p.out_dtype = out_dtype, p.ldo = ldo, p.out_batch = out_batch, p.settled = settled, p.shift = shift;
   p.tiles_m = (int)ceil_div(M, 256);
   p.nt = (int)ceil_div(ceil_div(M, p.tiles_m), 16) * 16;
   p.tiles_m = (int)ceil_div(M, p.nt);
-  p.tiles_n = (int)ceil_div(out_cols, e.kind == FB_DENSE_GLU ? 64 : 128);
+  p.tiles_n = (int)ceil_div(out_cols, fb::paired(e.kind) ? 64 : 128);
   FB_REQUIRE((int64_t)p.tiles_m * p.tiles_n * batch < (1 << 30), "fb_dense: too many tiles");
   p.tiles = (int)(p.tiles_m * p.tiles_n * batch);
   p.x_step = p.nt;
@@ -420,11 +431,11 @@ extern "C" int fb_dense_grouped(const void* x, int64_t x_rows, int64_t K, int64_
   FB_REQUIRE(out_dtype == FB_BF16 || out_dtype == FB_FP32, "fb_dense_grouped: out is bf16 or fp32");
   DenseParams p{};
   p.shift = settle_unit(e);
-  const int64_t out_cols = e.kind == FB_DENSE_GLU ? N / 2 : N;
+  const int64_t out_cols = fb::paired(e.kind) ? N / 2 : N;
   FB_REQUIRE(ldo >= out_cols, "fb_dense_grouped: rows of out too close");
   p.M = tiles * tile, p.N = N, p.e = e, p.out = out, p.out_dtype = out_dtype, p.ldo = ldo;
   p.nt = tile, p.tiles_m = (int)tiles, p.x_step = shared_rows ? 0 : tile, p.tile_expert = tile_expert, p.live = live;
-  p.tiles_n = (int)ceil_div(out_cols, e.kind == FB_DENSE_GLU ? 64 : 128);
+  p.tiles_n = (int)ceil_div(out_cols, fb::paired(e.kind) ? 64 : 128);
   FB_REQUIRE(tiles * p.tiles_n < (1 << 30), "fb_dense_grouped: too many tiles");
   p.tiles = (int)tiles * p.tiles_n;
   return run_dense(p, x, x_rows, 1, K, ldx, 0, W, ldw, w_batch, n, (cudaStream_t)stream);

@@ -1,6 +1,6 @@
 // A mixture of experts around its matmuls, for weights kept as bf16 or fp32:
-//   fb_route            router logits (with a bias) -> each token's k largest, the softmax of those, and where each choice's row
-//                       goes: the touched experts' rows in whole tiles, a list of the tiles' experts, how many there are
+//   fb_route            router logits -> each token's k largest (by logit, or by corrected score), their weights, and where each
+//                       choice's row goes (an identity expert's: nowhere): the touched experts' rows in whole tiles, a list of the tiles' experts, how many there are
 //   fb_spread_rows      the tokens' rows to their choices' places
 //   fb_grouped_matmul   rows of tiles by each tile's own matrix, any sizes, bf16 or fp32 (the tensor cores' form: fb_dense_grouped)
 //
@@ -16,6 +16,8 @@ struct RouteArgs {
   int64_t T, ld;
   const float* bias;  // [n] or null
   int n, k, tile, shared;
+  int real, scored;  // outputs 0 .. real - 1 are experts with rows
+  float scale;
   int tiles;  // entries of tile_expert
   float* weights;       // [T, k]
   int32_t* ids;         // [T, k]
@@ -31,12 +33,22 @@ __device__ __forceinline__ uint32_t ordered(float v) {
 }
 __device__ __forceinline__ float from_ordered(uint32_t b) { return __uint_as_float(b & 0x80000000u ? b & 0x7fffffffu : ~b); }
 
-// the k largest of a token's logits, the lower column first among equals, and the softmax of those: a warp a token.  Up to 128
-// experts: the lanes hold the logits as ordered numbers, 0 once picked
+// the k largest of a token's logits or scores, the lower column first among equals, and their weights: a warp a token.  Up to 128
+// outputs: the lanes hold the logits as ordered numbers, 0 once picked
 __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int lane) {
   const float* z = a.logits + t * a.ld;
   float mine[2] = {-INFINITY, -INFINITY};  // lane j keeps the picks j and 32 + j
   int my_id[2] = {0, 0};
+  float most = 0.f, norm = 1.f;  // scored: a score is exp(z - most) * norm
+  if (a.scored) {
+    most = -INFINITY;
+    for (int c = lane; c < a.n; c += 32) most = fmaxf(most, z[c]);
+    most = warp_max(most);
+    float sum = 0.f;
+    for (int c = lane; c < a.n; c += 32) sum += expf(z[c] - most);
+    norm = 1.f / warp_sum(sum);
+  }
+  auto chosen_by = [&](int c) { return (a.scored ? expf(z[c] - most) * norm : z[c]) + (a.bias ? a.bias[c] : 0.f); };
   auto keep = [&](int j, float v, int at) {
     if (j < 32 && lane == j) mine[0] = v, my_id[0] = at;
     if (j >= 32 && lane == j - 32) mine[1] = v, my_id[1] = at;
@@ -46,7 +58,7 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int c = 32 * i + lane;
-      held[i] = c < a.n ? ordered(z[c] + (a.bias ? a.bias[c] : 0.f)) : 0;
+      held[i] = c < a.n ? ordered(chosen_by(c)) : 0;
     }
     for (int j = 0; j < a.k; ++j) {
       uint32_t best = held[0];
@@ -68,7 +80,7 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
       float best = -INFINITY;
       int at = a.n;
       for (int c = lane; c < a.n; c += 32) {  // (what comes after the pick before in the order of the picks; columns rise: the first of equals stays)
-        const float v = z[c] + (a.bias ? a.bias[c] : 0.f);
+        const float v = chosen_by(c);
         if ((v < prev || (v == prev && c > prev_at)) && (at == a.n || v > best)) best = v, at = c;
       }
 #pragma unroll
@@ -83,9 +95,10 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
     }
   }
   const float top = __shfl_sync(0xffffffffu, mine[0], 0);
-  const float e0 = lane < a.k ? expf(mine[0] - top) : 0.f, e1 = lane + 32 < a.k ? expf(mine[1] - top) : 0.f, sum = warp_sum(e0 + e1);
-  if (lane < a.k) a.weights[t * a.k + lane] = e0 / sum, a.ids[t * a.k + lane] = my_id[0];
-  if (lane + 32 < a.k) a.weights[t * a.k + lane + 32] = e1 / sum, a.ids[t * a.k + lane + 32] = my_id[1];
+  auto weight = [&](int i) { return lane + 32 * i >= a.k ? 0.f : a.scored ? expf(z[min(my_id[i], a.n - 1)] - most) * norm : expf(mine[i] - top); };
+  const float e0 = weight(0), e1 = weight(1), sum = warp_sum(e0 + e1) + (a.scored ? 1e-20f : 0.f);
+  if (lane < a.k) a.weights[t * a.k + lane] = e0 / sum * a.scale, a.ids[t * a.k + lane] = my_id[0];
+  if (lane + 32 < a.k) a.weights[t * a.k + lane + 32] = e1 / sum * a.scale, a.ids[t * a.k + lane + 32] = my_id[1];
 }
 
 __global__ void __launch_bounds__(256) route_tokens_kernel(const RouteArgs a) {
@@ -99,10 +112,10 @@ __global__ void __launch_bounds__(256) route_tokens_kernel(const RouteArgs a) {
 __global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, const int pick) {
   griddep_launch_dependents();
   griddep_wait();
-  extern __shared__ int32_t route_smem[];  // [n] counts, then each expert's next row; [33] sums
-  int32_t *count = route_smem, *sums = route_smem + a.n;
+  extern __shared__ int32_t route_smem[];  // [real] counts, then each expert's next row; [33] sums
+  int32_t *count = route_smem, *sums = route_smem + a.real;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  for (int e = tid; e < a.n; e += blockDim.x) count[e] = 0;
+  for (int e = tid; e < a.real; e += blockDim.x) count[e] = 0;
   if (pick)
     for (int64_t t = warp; t < a.T; t += 32) route_token(a, t, lane);
   __syncthreads();
@@ -114,11 +127,11 @@ __global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, c
     for (int b = 0; b < BATCH; ++b) e[b] = i0 + b * 1024 < choices ? a.ids[i0 + b * 1024] : -1;
 #pragma unroll
     for (int b = 0; b < BATCH; ++b)
-      if (e[b] >= 0) atomicAdd(count + e[b], 1);
+      if (e[b] >= 0 && e[b] < a.real) atomicAdd(count + e[b], 1);
   }
   __syncthreads();
   // tiles of each expert, scanned: a thread has a run of experts
-  const int run = (a.n + 1023) / 1024, e0 = min(a.n, tid * run), e1 = min(a.n, e0 + run);
+  const int run = (a.real + 1023) / 1024, e0 = min(a.real, tid * run), e1 = min(a.real, e0 + run);
   auto tiles_of = [&](int e) { return a.shared ? (count[e] ? 1 : 0) : (count[e] + a.tile - 1) / a.tile; };
   int own = 0;
   for (int e = e0; e < e1; ++e) own += tiles_of(e);
@@ -149,7 +162,7 @@ __global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, c
     count[e] = first * a.tile;
     first += n;
   }
-  for (int i = used + tid; i < a.tiles; i += blockDim.x) a.tile_expert[3 * i] = a.n, a.tile_expert[3 * i + 1] = a.tile_expert[3 * i + 2] = 0;
+  for (int i = used + tid; i < a.tiles; i += blockDim.x) a.tile_expert[3 * i] = a.real, a.tile_expert[3 * i + 1] = a.tile_expert[3 * i + 2] = 0;
   __syncthreads();
   for (int64_t i0 = tid; i0 < choices; i0 += BATCH * 1024) {
     int e[BATCH];
@@ -157,7 +170,7 @@ __global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, c
     for (int b = 0; b < BATCH; ++b) e[b] = i0 + b * 1024 < choices ? a.ids[i0 + b * 1024] : -1;
 #pragma unroll
     for (int b = 0; b < BATCH; ++b)
-      if (e[b] >= 0) a.slots[i0 + b * 1024] = a.shared ? count[e[b]] + (int)((i0 + b * 1024) / a.k) : atomicAdd(count + e[b], 1);
+      if (e[b] >= 0) a.slots[i0 + b * 1024] = e[b] >= a.real ? -1 : a.shared ? count[e[b]] + (int)((i0 + b * 1024) / a.k) : atomicAdd(count + e[b], 1);
   }
 }
 
@@ -230,19 +243,21 @@ extern "C" int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_
   return choices / tile + most;  // (each touched expert adds less than a tile)
 }
 
-extern "C" int fb_route(const float* logits, int64_t T, int64_t ld, const float* bias, int n, int k, int tile, int shared_rows, float* weights, int32_t* ids, int32_t* slots,
+extern "C" int fb_route(const fb_router* router_host, const float* logits, int64_t T, int64_t ld, int tile, int shared_rows, float* weights, int32_t* ids, int32_t* slots,
                         int32_t* tile_expert, int32_t* live, void* stream) {
-  FB_REQUIRE(logits && weights && ids && slots && tile_expert && live && T >= 1 && T <= (1 << 24), "fb_route: null pointer or no tokens");
+  FB_REQUIRE(router_host && logits && weights && ids && slots && tile_expert && live && T >= 1 && T <= (1 << 24), "fb_route: null pointer or no tokens");
+  const int n = router_host->n, k = router_host->k, real = n - router_host->identity;
+  FB_REQUIRE(router_host->identity >= 0 && real >= 1, "fb_route: at least one expert with rows");
   FB_REQUIRE(n >= 1 && n <= 8192 && k >= 1 && k <= 64 && k <= n && ld >= n, "fb_route: up to 64 choices among up to 8192 experts (got %d of %d)", k, n);
   FB_REQUIRE(tile >= 16 && tile % 16 == 0 && (!shared_rows || T <= tile), "fb_route: tiles of whole runs of 16 rows; shared rows: all the tokens in one");
-  const int64_t tiles = fb_route_tiles(T, n, k, tile, shared_rows);
+  const int64_t tiles = fb_route_tiles(T, real, k, tile, shared_rows);
   FB_REQUIRE(tiles * tile < (1ll << 31), "fb_route: too many rows");
-  const fb::RouteArgs a{logits, T, ld, bias, n, k, tile, shared_rows, (int)tiles, weights, ids, slots, tile_expert, live};
+  const fb::RouteArgs a{logits, T, ld, router_host->bias, n, k, tile, shared_rows, real, router_host->scored, router_host->scale, (int)tiles, weights, ids, slots, tile_expert, live};
   const auto s = (cudaStream_t)stream;
   const int pick = T <= 32;
   if (!pick)
     if (int rc = fb::launch_after(fb::route_tokens_kernel, dim3((unsigned)fb::ceil_div(T, 8)), dim3(256), 0, s, "fb_route", a)) return rc;
-  return fb::launch_after(fb::route_places_kernel, dim3(1), dim3(1024), (size_t)(n + 33) * sizeof(int32_t), s, "fb_route", a, pick);
+  return fb::launch_after(fb::route_places_kernel, dim3(1), dim3(1024), (size_t)(real + 33) * sizeof(int32_t), s, "fb_route", a, pick);
 }
 
 extern "C" int fb_spread_rows(const void* x, int64_t T, int64_t row_bytes, int64_t ldx_bytes, const int32_t* slots, int k, void* out, int64_t out_rows, void* stream) {

@@ -14,7 +14,8 @@ struct HeadsArgs {
   int64_t row0;
   int chunk;  // the tokens are one sequence's, their places rising
   int span;   // 0: no spans
-  float scale;
+  int window; // 0: none; else a token sees the last `window` places only
+  float scale, softcap;  // softcap > 0: a scaled score s becomes softcap tanh(s / softcap)
   const float* sink;  // [heads] or null
   int gate_dtype;
   const void* gate;  // [T, ld_g]: head h at h * vdim; the output times its sigmoid
@@ -26,7 +27,11 @@ struct HeadsArgs {
   int entries, pairs, tiles;  // entries of `pairs` pairs each (a token's, or the chunk's), cut into tiles
 };
 
-__device__ __forceinline__ int span_start(int place, int span) { return span > 0 ? place - place % span : 0; }
+// the first place that a token at `place` sees
+__device__ __forceinline__ int first_seen(const HeadsArgs& a, int place) {
+  const int lo = a.span > 0 ? place - place % a.span : 0;
+  return a.window > 0 ? max(lo, place - a.window + 1) : lo;
+}
 
 // 2^x, the hardware's (x far below: 0)
 __device__ __forceinline__ float exp2_of(float x) {
@@ -34,6 +39,14 @@ __device__ __forceinline__ float exp2_of(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+
+// an unscaled score s as the unscaled score that the cap leaves: (softcap / scale) tanh(s scale / softcap), tanh by one exponential
+// (to about 2e-7 of 1)
+struct SoftCap {
+  float in, out;
+};
+__device__ __forceinline__ SoftCap soft_cap(const HeadsArgs& a) { return {a.softcap > 0.f ? 2.8853900817779268f * a.scale / a.softcap : 0.f, a.softcap > 0.f ? a.softcap / a.scale : 0.f}; }
+__device__ __forceinline__ float capped(const SoftCap& c, float s) { return fmaf(-2.f * c.out, __fdividef(1.f, 1.f + exp2_of(fminf(s * c.in, 80.f))), c.out); }
 
 __device__ __forceinline__ float gate_value(const HeadsArgs& a, int64_t at) {
   return a.gate_dtype == FB_FP32 ? static_cast<const float*>(a.gate)[at] : bf16_bits_to_float(static_cast<const uint16_t*>(a.gate)[at]);

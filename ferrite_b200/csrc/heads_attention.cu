@@ -1,6 +1,7 @@
 // Attention with grouped key heads over a cache whose rows are a key and then its value: the two may differ in width, the
-// keys a token sees may be confined to its own span of the sequence (spans of `span` places, counted from its start), a
-// number per head may join the softmax's denominator, and the output may be gated column by column.
+// keys a token sees may be confined to its own span of the sequence (spans of `span` places, counted from its start) or to the
+// last `window` places, scores may be capped, a number per head may join the softmax's denominator, and the output may be gated
+// column by column.
 //
 // A CTA has one key head, a tile of (token, query head) pairs that share it - the pairs of one token in a decode step, those
 // of consecutive tokens in a prompt's chunk - and a run of the keys that they see; tiles of 64 keys and their values come in by
@@ -37,7 +38,7 @@ __global__ void __launch_bounds__(32 * PLAIN_HEADS) heads_attention_plain_kernel
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y * PLAIN_HEADS + warp, W = a.dim + a.vdim;
   if (h >= a.heads) return;
   const int64_t seq = (a.base ? a.base[t] : 0) + a.row0, room = seq < 0 ? 0 : a.cache_rows - seq;
-  const int place = a.last[t], keys = (int)max((int64_t)0, min((int64_t)place + 1, room)), lo = span_start(place, a.span);
+  const int place = a.last[t], keys = (int)max((int64_t)0, min((int64_t)place + 1, room)), lo = first_seen(a, place);
   const Act* cache = static_cast<const Act*>(a.cache) + (h / a.rep) * a.head_stride;
   float* q = plain_q + warp * a.dim;
   for (int c = lane; c < a.dim; c += 32) q[c] = value_of(static_cast<const Act*>(a.q)[t * a.ld_q + (int64_t)h * a.dim + c]);
@@ -54,6 +55,7 @@ __global__ void __launch_bounds__(32 * PLAIN_HEADS) heads_attention_plain_kernel
       s = 0.f;
       for (int c = 0; c < a.dim; ++c) s = fmaf(q[c], value_of(rows[(int64_t)lane * W + c]), s);
       s *= a.scale;
+      if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
     }
     const float m_new = fmaxf(m, warp_max(s)), corr = expf(m - m_new), p = lane < n ? expf(s - m_new) : 0.f;
     m = m_new, l = l * corr + warp_sum(p);
@@ -84,17 +86,20 @@ static int launch_plain(const HeadsArgs& a, cudaStream_t s) {
 }  // namespace fb
 
 extern "C" int fb_heads_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int kv_heads, int dim, int vdim, const void* cache, int64_t cache_rows,
-                                  int64_t head_stride, const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk, int span, float scale,
-                                  const float* sink, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o, void* stream) {
+                                  int64_t head_stride, const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk, int span, int window, float scale,
+                                  float softcap, const float* sink, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o, void* stream) {
   using namespace fb;
   FB_REQUIRE(q && cache && last && out && T >= 1 && max_keys >= 1 && cache_rows >= 1, "fb_heads_attention: null pointer or empty");
   FB_REQUIRE(heads >= 1 && kv_heads >= 1 && heads % kv_heads == 0 && dim >= 1 && vdim >= 1 && kv_heads <= 65535, "fb_heads_attention: whole groups of query heads per key head (got %d / %d)", heads, kv_heads);
   FB_REQUIRE(dtype == FB_BF16 || dtype == FB_FP32, "fb_heads_attention: bf16 or fp32 rows");
   FB_REQUIRE(dim <= 1024 && vdim <= 32 * PLAIN_COLS, "fb_heads_attention: heads of up to 1024 columns (got %d and %d)", dim, vdim);
-  FB_REQUIRE(ld_q >= (int64_t)heads * dim && ld_o >= (int64_t)heads * vdim && head_stride >= cache_rows * (dim + vdim) && row0 >= 0 && span >= 0, "fb_heads_attention: row strides too small");
+  FB_REQUIRE(ld_q >= (int64_t)heads * dim && ld_o >= (int64_t)heads * vdim && head_stride >= cache_rows * (dim + vdim) && row0 >= 0 && span >= 0 && window >= 0, "fb_heads_attention: row strides too small");
   FB_REQUIRE(!gate || ((gate_dtype == FB_BF16 || gate_dtype == FB_FP32) && ld_g >= (int64_t)heads * vdim), "fb_heads_attention: gates, bf16 or fp32, one a column of the result");
   FB_REQUIRE(!chunk || !base, "fb_heads_attention: a chunk is one sequence's (no base)");
-  HeadsArgs a{q, T, ld_q, heads, kv_heads, dim, vdim, heads / kv_heads, cache, cache_rows, head_stride, base, last, row0, chunk, span, scale, sink, gate_dtype, gate, ld_g, out, ld_o, span > 0 && span < max_keys ? span : max_keys, 0, 0, 0, 0};
+  FB_REQUIRE(softcap >= 0.f, "fb_heads_attention: a cap of scores is positive (0: none)");
+  HeadsArgs a{q, T, ld_q, heads, kv_heads, dim, vdim, heads / kv_heads, cache, cache_rows, head_stride, base, last, row0, chunk, span, window, scale, softcap, sink, gate_dtype, gate, ld_g, out, ld_o, max_keys, 0, 0, 0, 0};
+  if (span > 0 && span < a.seen) a.seen = span;
+  if (window > 0 && window + (chunk ? ceil_div(128, a.rep) : 0) < a.seen) a.seen = window + (chunk ? ceil_div(128, a.rep) : 0);  // (a tile's tokens' windows together)
   const auto s = (cudaStream_t)stream;
   const bool pieces = dim % 8 == 0 && vdim % 8 == 0 && ld_q % 8 == 0 && head_stride % 8 == 0 && ld_o % 2 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)cache % 16 == 0 && (uintptr_t)out % 4 == 0;
   if (dtype == FB_FP32) return vdim <= 256 ? launch_plain<float, 8>(a, s) : launch_plain<float, PLAIN_COLS>(a, s);

@@ -57,7 +57,7 @@ __global__ void __launch_bounds__(32 * WR * WK + 32) heads_attention_kernel(cons
   int len = 0, lo = 0x7fffffff;
   for (int t = tok_a + lane; t <= tok_b; t += 32) {
     const int p = a.last[token0 + t];
-    len = max(len, p + 1), lo = min(lo, span_start(p, a.span));
+    len = max(len, p + 1), lo = min(lo, first_seen(a, p));
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) len = max(len, __shfl_xor_sync(0xffffffffu, len, o)), lo = min(lo, __shfl_xor_sync(0xffffffffu, lo, o));
@@ -102,7 +102,7 @@ __global__ void __launch_bounds__(32 * WR * WK + 32) heads_attention_kernel(cons
     for (int h = 0; h < 2; ++h) {
       const int r = 16 * (WR * mt + wr) + (lane >> 2) + 8 * h;
       place_r[mt][h] = r < rows ? a.last[token0 + (pair0 + r) / a.rep] : -1;
-      lo_r[mt][h] = r < rows ? span_start(place_r[mt][h], a.span) : 0;
+      lo_r[mt][h] = r < rows ? first_seen(a, place_r[mt][h]) : 0;
     }
   // the queries; past a key's columns zeros, so that what a tile holds there (its values' first) does not count
   for (int c = tid; c < ROWS * (DK / 8); c += THREADS) {
@@ -132,6 +132,7 @@ __global__ void __launch_bounds__(32 * WR * WK + 32) heads_attention_kernel(cons
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) m_run[mt][0] = m_run[mt][1] = -INFINITY, l_run[mt][0] = l_run[mt][1] = 0.f;
   const float scale_log2 = a.scale * LOG2E;
+  const SoftCap cap = soft_cap(a);
 
   // where a lane's 16 bytes stand within a swizzled row, for the four steps of 16 columns that a row has
   uint32_t k_off[4], v_off[4];
@@ -171,6 +172,12 @@ __global__ void __launch_bounds__(32 * WR * WK + 32) heads_attention_kernel(cons
     uint32_t pf[MT][NT / 2][4];
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
+      if (cap.in > 0.f) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[mt][n][e] = capped(cap, s[mt][n][e]);
+      }
       // (a whole tile that every pair of the warp sees needs no mask)
       if (!__all_sync(0xffffffffu, key_end <= k1 && min(place_r[mt][0], place_r[mt][1]) >= key_end - 1 && max(lo_r[mt][0], lo_r[mt][1]) <= key0)) {
 #pragma unroll

@@ -75,7 +75,7 @@ __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) he
   int len = 0, lo = 0x7fffffff;
   for (int t = t0 + lane; t < t1; t += 32) {
     const int at = a.last[t];
-    len = max(len, at + 1), lo = min(lo, span_start(at, a.span));
+    len = max(len, at + 1), lo = min(lo, first_seen(a, at));
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) len = max(len, __shfl_xor_sync(0xffffffffu, len, o)), lo = min(lo, __shfl_xor_sync(0xffffffffu, lo, o));
@@ -161,9 +161,10 @@ __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) he
     const int64_t token = t0 + gr * p.tokens + row / a.rep;
     const bool live = row < p.tokens * a.rep && token < a.T;
     // (a row past the last runs along and is never looked at)
-    const int place = live ? min(a.last[token], len - 1) : 0x3fffffff, first = live ? span_start(a.last[token], a.span) : 0;
+    const int place = live ? min(a.last[token], len - 1) : 0x3fffffff, first = live ? first_seen(a, a.last[token]) : 0;
     const uint32_t lanes = (uint32_t)(32 * (warp & 3)) << 16, tS = tmem + lanes + gr * HP_COLS, tO = tS + 2 * HP_KEYS;
     const float scale_log2 = a.scale * HP_LOG2E;
+    const SoftCap cap = soft_cap(a);
     float m = -INFINITY, l = 0.f;  // the reference maximum of the unscaled scores, and the sum under it
     for (int t = 0; t < n_tiles; ++t) {
       mbar_wait(smem_u32(s_full + 2 * gr + (t & 1)), (t >> 1) & 1, abort_flag, PW_S);
@@ -172,6 +173,10 @@ __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) he
       tmem_ld32_nowait(tS + (t & 1) * HP_KEYS, s);
       tmem_ld32_nowait(tS + (t & 1) * HP_KEYS + 32, s + 32);
       tmem_ld_wait();
+      if (cap.in > 0.f) {
+#pragma unroll
+        for (int j = 0; j < HP_KEYS; ++j) s[j] = capped(cap, s[j]);
+      }
       const int key0 = k0 + t * HP_KEYS, seen = place + 1 - key0, hidden = first - key0;  // of these keys, from `hidden` on and before `seen`
       if (!__all_sync(0xffffffffu, seen >= HP_KEYS && hidden <= 0)) {
 #pragma unroll

@@ -3,12 +3,14 @@
 // dot product with the whole row and its output the weighted sum of the rows' latents; the values' matrix follows after.
 // Every head reads the same row, so a row is read once for all of them.
 //
-//   fb_latent_put        what follows the joint down-projection: RMSNorm of the query latent and of the key-value latent,
-//                        rotation of the shared key part, the new row into the cache
+//   fb_latent_put        what follows the joint down-projection: RMSNorm of the query latent (or, of a design without one, the
+//                        queries taken apart and turned) and of the key-value latent, rotation of the shared key part, the new
+//                        row into the cache
 //   fb_rotate_pairs      neighbouring columns (2i, 2i + 1) of each head turned by the token's angle
-//   fb_latent_attention  softmax with an optional sink per head (one more term of the denominator); bf16 rows of suitable
+//   fb_latent_attention  softmax, within a window if there is one, with an optional sink per head (one more term of the denominator); bf16 rows of suitable
 //                        sizes on the tensor cores (latent_tcgen05.cu), everything else - fp32, odd sizes - here
 #include "latent.cuh"
+#include "launch.cuh"
 #include "values.cuh"
 
 namespace fb {
@@ -24,6 +26,9 @@ struct LatentPutArgs {
   const int32_t *places, *rows;
   void* q_out;  // [T, ld_q]
   int64_t ld_q;
+  int heads, dim;  // heads > 0: the row begins with heads x (dim | rot) instead of a query latent
+  void* q_turned;  // head h of token t at t * ld_turned + h * turned_head
+  int64_t ld_turned, turned_head;
   void* cache;  // [cache_rows, kv_rank + rot]
   int64_t cache_rows;
 };
@@ -35,6 +40,25 @@ __global__ void __launch_bounds__(256) latent_put_kernel(const LatentPutArgs a) 
   __shared__ float red[32];
   const int64_t t = blockIdx.x;
   const In* x = static_cast<const In*>(a.down) + t * a.ld;
+  extern __shared__ float put_turns[];  // [dims / 2] cos, [dims / 2] sin
+  const int half = a.dims / 2;
+  if (blockIdx.y == 0 && a.heads) {  // queries: the plain parts side by side, the others turned
+    for (int i = threadIdx.x; i < half; i += blockDim.x) turn_of(a.places[t], a.freq[i], a.mag, put_turns[i], put_turns[half + i]);
+    __syncthreads();
+    const int W = a.dim + a.rot, pairs = (a.rot + 1) / 2;
+    Act* plain = static_cast<Act*>(a.q_out) + t * a.ld_q;
+    for (int i = threadIdx.x; i < a.heads * a.dim; i += blockDim.x) store_value(plain + i, value_of(x[i / a.dim * W + i % a.dim]));
+    for (int j = threadIdx.x; j < a.heads * pairs; j += blockDim.x) {
+      const int h = j / pairs, i = j % pairs;
+      const bool two = 2 * i + 1 < a.rot;
+      const In* from = x + h * W + a.dim + 2 * i;
+      Act* out = static_cast<Act*>(a.q_turned) + t * a.ld_turned + h * a.turned_head + 2 * i;
+      const float u = value_of(from[0]), v = two ? value_of(from[1]) : 0.f;
+      store_value(out, i < half ? u * put_turns[i] - v * put_turns[half + i] : u);
+      if (two) store_value(out + 1, i < half ? v * put_turns[i] + u * put_turns[half + i] : v);
+    }
+    return;
+  }
   if (blockIdx.y == 0) {  // the query latent
     float ss = 0.f;
     for (int c = threadIdx.x; c < a.q_rank; c += blockDim.x) ss = fmaf(value_of(x[c]), value_of(x[c]), ss);
@@ -45,7 +69,7 @@ __global__ void __launch_bounds__(256) latent_put_kernel(const LatentPutArgs a) 
   }
   const int64_t row = a.rows[t];
   if (row < 0 || row >= a.cache_rows) return;  // (the whole block: nothing is written outside the cache)
-  x += a.q_rank;
+  x += a.heads ? a.heads * (a.dim + a.rot) : a.q_rank;
   float ss = 0.f;
   for (int c = threadIdx.x; c < a.kv_rank; c += blockDim.x) ss = fmaf(value_of(x[c]), value_of(x[c]), ss);
   const float r = 1.f / sqrtf(block_sum(ss, red) / (float)a.kv_rank + a.eps);
@@ -116,7 +140,7 @@ __global__ void __launch_bounds__(32 * LAT_HEADS) latent_attention_kernel(const 
   const Act* cache = static_cast<const Act*>(a.cache);
   const int64_t first = (a.base ? a.base[t] : 0) + a.row0;
   const int64_t room = first < 0 ? 0 : a.cache_rows - first;
-  const int keys = (int)max((int64_t)0, min((int64_t)a.last[t] + 1, room));
+  const int keys = (int)max((int64_t)0, min((int64_t)a.last[t] + 1, room)), lo = a.window > 0 ? max(0, a.last[t] - a.window + 1) : 0;
   if (on) {
     const Act* q = static_cast<const Act*>(a.q) + t * a.ld_q + (int64_t)h * W;
     for (int c = lane; c < W; c += 32) sq[warp * W + c] = value_of(q[c]);
@@ -125,7 +149,7 @@ __global__ void __launch_bounds__(32 * LAT_HEADS) latent_attention_kernel(const 
 #pragma unroll
   for (int i = 0; i < COLS; ++i) acc[i] = 0.f;
   float m = a.sink && on ? a.sink[h] : -INFINITY, l = a.sink ? 1.f : 0.f;  // the sink: a key of its own with no value
-  for (int k0 = 0; k0 < keys; k0 += LAT_KEYS) {
+  for (int k0 = lo; k0 < keys; k0 += LAT_KEYS) {
     const int n = min(LAT_KEYS, keys - k0);
     __syncthreads();
     for (int i = threadIdx.x; i < n * W; i += blockDim.x) sk[(i / W) * pitch + i % W] = value_of(cache[(first + k0 + i / W) * W + i % W]);
@@ -173,19 +197,20 @@ static int launch_latent(const LatentArgs& a, cudaStream_t s) {
 
 extern "C" int fb_latent_put(int in_dtype, const void* down, int64_t T, int64_t ld, int q_rank, int kv_rank, int rot, int dims, const float* q_norm,
                              const float* kv_norm, float eps, const double* freq, float mag, const int32_t* places, const int32_t* rows, int dtype,
-                             void* q_out, int64_t ld_q, void* cache, int64_t cache_rows, void* stream) {
+                             void* q_out, int64_t ld_q, int heads, int dim, void* q_turned, int64_t ld_turned, int64_t turned_head, void* cache, int64_t cache_rows, void* stream) {
   FB_REQUIRE(down && kv_norm && freq && places && rows && cache && T >= 1 && kv_rank >= 1, "fb_latent_put: null pointer or empty");
   FB_REQUIRE(q_rank >= 0 && (q_rank == 0 || (q_norm && q_out && ld_q >= q_rank)), "fb_latent_put: a query latent takes its norm and somewhere to go");
-  FB_REQUIRE(rot >= 0 && dims >= 0 && dims % 2 == 0 && dims <= rot && ld >= q_rank + kv_rank + rot && cache_rows >= 1, "fb_latent_put: the turned columns are an even number within the key part");
+  FB_REQUIRE(heads >= 0 && (heads == 0 || (q_rank == 0 && dim >= 1 && q_out && ld_q >= (int64_t)heads * dim && (rot == 0 || q_turned))), "fb_latent_put: queries take somewhere for both their parts, and no query latent");
+  FB_REQUIRE(rot >= 0 && dims >= 0 && dims % 2 == 0 && dims <= rot && dims <= 8192 && ld >= q_rank + (int64_t)heads * (dim + rot) + kv_rank + rot && cache_rows >= 1, "fb_latent_put: the turned columns are an even number within the key part");
   FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32), "fb_latent_put: bf16 or fp32");
-  fb::LatentPutArgs a{down, ld, q_rank, kv_rank, rot, dims, q_norm, kv_norm, eps, freq, mag, places, rows, q_out, ld_q, cache, cache_rows};
+  fb::LatentPutArgs a{down, ld, q_rank, kv_rank, rot, dims, q_norm, kv_norm, eps, freq, mag, places, rows, q_out, ld_q, heads, dim, q_turned, ld_turned, turned_head, cache, cache_rows};
   const auto s = (cudaStream_t)stream;
   FB_REQUIRE(in_dtype == FB_FP32 || dtype == FB_BF16, "fb_latent_put: fp32 results come from fp32");
-  const dim3 grid((unsigned)T, 2);
-  if (in_dtype == FB_FP32 && dtype == FB_FP32) fb::latent_put_kernel<float, float><<<grid, 256, 0, s>>>(a);
-  else if (in_dtype == FB_FP32) fb::latent_put_kernel<float, uint16_t><<<grid, 256, 0, s>>>(a);
-  else fb::latent_put_kernel<uint16_t, uint16_t><<<grid, 256, 0, s>>>(a);
-  return fb::launch_status("fb_latent_put");
+  const dim3 grid((unsigned)T, 2), block(256);
+  const size_t smem = heads ? dims * sizeof(float) : 0;
+  if (in_dtype == FB_FP32 && dtype == FB_FP32) return fb::launch_after(fb::latent_put_kernel<float, float>, grid, block, smem, s, "fb_latent_put", a);
+  if (in_dtype == FB_FP32) return fb::launch_after(fb::latent_put_kernel<float, uint16_t>, grid, block, smem, s, "fb_latent_put", a);
+  return fb::launch_after(fb::latent_put_kernel<uint16_t, uint16_t>, grid, block, smem, s, "fb_latent_put", a);
 }
 
 extern "C" int fb_rotate_pairs(int dtype, const void* x, int64_t T, int heads, int64_t x_row, int64_t x_head, int width, int dims, const double* freq,
@@ -199,18 +224,18 @@ extern "C" int fb_rotate_pairs(int dtype, const void* x, int64_t T, int heads, i
   return fb::launch_status("fb_rotate_pairs");
 }
 
-extern "C" size_t fb_latent_attention_workspace_bytes(int dtype, int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk) {
-  return dtype == FB_BF16 && heads >= 1 && rank >= 1 && rot >= 0 ? fb::latent_tcgen05_workspace(T, heads, rank, rot, max_keys, chunk) : 0;
+extern "C" size_t fb_latent_attention_workspace_bytes(int dtype, int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk, int window) {
+  return dtype == FB_BF16 && heads >= 1 && rank >= 1 && rot >= 0 ? fb::latent_tcgen05_workspace(T, heads, rank, rot, max_keys, chunk, window) : 0;
 }
 
 extern "C" int fb_latent_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int rank, int rot, const void* cache, int64_t cache_rows,
-                                   const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk, float scale, const float* sink,
+                                   const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk, int window, float scale, const float* sink,
                                    void* out, int64_t ld_o, void* workspace, size_t workspace_bytes, void* stream) {
   FB_REQUIRE(q && cache && last && out && T >= 1 && heads >= 1 && rank >= 1 && rot >= 0 && max_keys >= 1, "fb_latent_attention: null pointer or empty");
   FB_REQUIRE(dtype == FB_BF16 || dtype == FB_FP32, "fb_latent_attention: bf16 or fp32 rows");
-  FB_REQUIRE(ld_q >= (int64_t)heads * (rank + rot) && ld_o >= (int64_t)heads * rank && cache_rows >= 1 && row0 >= 0, "fb_latent_attention: row strides too small");
+  FB_REQUIRE(ld_q >= (int64_t)heads * (rank + rot) && ld_o >= (int64_t)heads * rank && cache_rows >= 1 && row0 >= 0 && window >= 0, "fb_latent_attention: row strides too small");
   FB_REQUIRE(rank <= 32 * fb::LAT_COLS, "fb_latent_attention: latents of up to %d columns", 32 * fb::LAT_COLS);
-  fb::LatentArgs a{q, T, ld_q, heads, rank, rot, cache, cache_rows, base, row0, last, max_keys, chunk, scale, sink, out, ld_o, workspace, workspace_bytes};
+  fb::LatentArgs a{q, T, ld_q, heads, rank, rot, cache, cache_rows, base, row0, last, max_keys, window, chunk, scale, sink, out, ld_o, workspace, workspace_bytes};
   const auto s = (cudaStream_t)stream;
   if (dtype == FB_BF16 && fb::latent_tcgen05_supports(a)) return fb::latent_tcgen05(a, s);
   if (dtype == FB_FP32) return rank <= 256 ? fb::launch_latent<float, 8>(a, s) : fb::launch_latent<float, fb::LAT_COLS>(a, s);

@@ -14,6 +14,7 @@ struct LatentArgs {
   int64_t row0;         // added to it
   const int32_t* last;  // [T] token t sees the rows 0 .. last[t] of its sequence
   int64_t max_keys;     // an upper bound of last[t] + 1
+  int window;           // 0: none; else only the last `window` of those
   int chunk;            // the tokens are one sequence's, in order (base null): they may share the rows read
   float scale;
   const float* sink;  // [heads] or null
@@ -25,7 +26,7 @@ struct LatentArgs {
 
 // latent_tcgen05.cu: bf16 rows on the tensor cores
 bool latent_tcgen05_supports(const LatentArgs& a);
-size_t latent_tcgen05_workspace(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk);
+size_t latent_tcgen05_workspace(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk, int window);
 int latent_tcgen05(const LatentArgs& a, cudaStream_t s);
 
 }  // namespace fb

@@ -64,8 +64,9 @@ struct LatentMaps {
 // where a row tile stands: its first (token, head) pair, how many, and the keys it reads
 struct RowTile {
   int64_t first_row, seq_first;
-  int rows, keys;
+  int rows, first_key, keys;  // keys first_key .. keys - 1
 };
+__device__ __forceinline__ int first_seen(const LatentArgs& a, int place) { return a.window > 0 ? max(0, place - a.window + 1) : 0; }
 __device__ __forceinline__ RowTile row_tile(const LatentParams& p, int tile) {
   const LatentArgs& a = p.a;
   RowTile r;
@@ -79,10 +80,10 @@ __device__ __forceinline__ RowTile row_tile(const LatentParams& p, int tile) {
     t0 = (int)r.first_row / a.heads, t1 = ((int)r.first_row + r.rows - 1) / a.heads;
   }
   r.seq_first = (a.base ? a.base[t0] : 0) + a.row0;
-  int last = -1;
-  for (int t = t0; t <= t1; ++t) last = max(last, a.last[t]);
+  int last = -1, lo = 0x7fffffff;
+  for (int t = t0; t <= t1; ++t) last = max(last, a.last[t]), lo = min(lo, first_seen(a, a.last[t]));
   const int64_t room = r.seq_first < 0 ? 0 : a.cache_rows - r.seq_first;
-  r.keys = (int)max((int64_t)0, min((int64_t)last + 1, room));
+  r.keys = (int)max((int64_t)0, min((int64_t)last + 1, room)), r.first_key = max(0, min(lo, r.keys));
   return r;
 }
 
@@ -119,7 +120,7 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
 
   const RowTile r = row_tile(p, tile);
   // this CTA's run of whole tiles of keys
-  const int all = (r.keys + L_KEYS - 1) / L_KEYS, per = (all + p.splits - 1) / p.splits;
+  const int all = (r.keys - r.first_key + L_KEYS - 1) / L_KEYS, per = (all + p.splits - 1) / p.splits;
   const int first_tile = split * per, n_tiles = max(0, min(all, first_tile + per) - first_tile);
 
   if (warp == L_WARP_LOAD && lane == 0) {
@@ -136,7 +137,7 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
       ok = mbar_wait(smem_u32(k_empty + buf), phase ^ 1, abort_flag, LW_K_EMPTY);
       if (!ok) break;
       mbar_expect_tx(smem_u32(k_full + buf), tile_bytes);
-      const int at = (int)(r.seq_first + (int64_t)(first_tile + i) * L_KEYS);
+      const int at = (int)(r.seq_first + r.first_key + (int64_t)(first_tile + i) * L_KEYS);
       if (whole) tma_load_3d(sK + buf * tile_bytes, &maps.k, 0, at, 0, smem_u32(k_full + buf));
       if (whole < C) tma_load_2d(sK + buf * tile_bytes + whole * L_CHUNK, &maps.k_tail, 64 * whole, at, smem_u32(k_full + buf));
       if (++buf == NB) buf = 0, phase ^= 1;
@@ -189,7 +190,7 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
   } else if (warp < L_SOFTMAX / 32) {
     const int half = warp >> 2, row = 32 * (warp & 3) + lane;  // lane `row` of the scores, half of a tile's keys (a lane past the last row runs along)
     const bool live = row < r.rows;
-    const int place = live ? a.last[(r.first_row + row) / a.heads] : 0x3fffffff;
+    const int place = live ? a.last[(r.first_row + row) / a.heads] : 0x3fffffff, first = live ? first_seen(a, place) : 0;
     const uint32_t lanes = (uint32_t)(32 * (warp & 3)) << 16;
     float m = -INFINITY, l = 0.f;  // the reference maximum (in units of log2) and this half's sum under it
     for (int t = 0; t < n_tiles; ++t) {
@@ -201,14 +202,15 @@ __global__ void __launch_bounds__(L_THREADS, 1) latent_tcgen05_kernel(const __gr
 #pragma unroll
         for (int c = 0; c < MINE; c += 8) tmem_ld8_nowait(tS + lanes + (t & 1) * KT + MINE * half + c, s + c);
         tmem_ld_wait();
-        const int seen = (live ? min(place, r.keys - 1) + 1 : place) - (first_tile + t) * KT - MINE * half;  // the first `seen` of these keys
+        const int key0 = r.first_key + (first_tile + t) * KT + MINE * half;
+        const int seen = (live ? min(place, r.keys - 1) + 1 : place) - key0, hidden = first - key0;  // of these keys, from `hidden` on and before `seen`
         float tops[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-        if (__all_sync(0xffffffffu, seen >= MINE)) {
+        if (__all_sync(0xffffffffu, seen >= MINE && hidden <= 0)) {
 #pragma unroll
           for (int j = 0; j < MINE; ++j) s[j] *= p.scale_log2, tops[j & 3] = fmaxf(tops[j & 3], s[j]);
         } else {
 #pragma unroll
-          for (int j = 0; j < MINE; ++j) s[j] = j < seen ? s[j] * p.scale_log2 : -INFINITY, tops[j & 3] = fmaxf(tops[j & 3], s[j]);
+          for (int j = 0; j < MINE; ++j) s[j] = j < seen && j >= hidden ? s[j] * p.scale_log2 : -INFINITY, tops[j & 3] = fmaxf(tops[j & 3], s[j]);
         }
         top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
         if (row < L_ROWS) row_top[t & 1][half][row] = top;
@@ -419,7 +421,11 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentParams 
 }
 
 // sizes and launch shape; false: not for this kernel
-bool make_latent_plan(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk, LatentParams& p) {
+bool make_latent_plan(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk, int window, LatentParams& p) {
+  if (window > 0) {  // (a tile of a chunk's pairs sees the windows of all its tokens)
+    const int64_t most = window + (chunk ? ceil_div(L_ROWS, heads) : 0);
+    max_keys = most < max_keys ? most : max_keys;
+  }
   const int W = rank + rot;
   if (W % 8 || rank % 8 || W > 64 * L_MAX_CHUNKS || rank > 128 * L_MAX_BLOCKS || max_keys < 1) return false;
   const int64_t rows = chunk ? T * heads : heads;
@@ -457,26 +463,26 @@ int64_t latent_tiles(const LatentParams& p, int64_t T, int heads) { return p.til
 
 }  // namespace
 
-size_t latent_tcgen05_workspace(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk) {
+size_t latent_tcgen05_workspace(int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk, int window) {
   LatentParams p{};
-  if (T < 1 || !make_latent_plan(T, heads, rank, rot, max_keys, chunk, p) || p.splits == 1 || p.clustered) return 0;
+  if (T < 1 || !make_latent_plan(T, heads, rank, rot, max_keys, chunk, window, p) || p.splits == 1 || p.clustered) return 0;
   return (size_t)latent_tiles(p, T, heads) * p.splits * L_ROWS * (rank + 2) * sizeof(float);
 }
 
 bool latent_tcgen05_supports(const LatentArgs& a) {
   LatentParams p{};
   return tma_encoder() != nullptr && a.ld_q == (int64_t)a.heads * (a.rank + a.rot) && a.ld_o == (int64_t)a.heads * a.rank && (uintptr_t)a.q % 16 == 0 &&
-         (uintptr_t)a.cache % 16 == 0 && (uintptr_t)a.out % 16 == 0 && a.cache_rows < (1ll << 31) && a.T * a.heads < (1ll << 31) && make_latent_plan(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, p);
+         (uintptr_t)a.cache % 16 == 0 && (uintptr_t)a.out % 16 == 0 && a.cache_rows < (1ll << 31) && a.T * a.heads < (1ll << 31) && make_latent_plan(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, a.window, p);
 }
 
 int latent_tcgen05(const LatentArgs& a, cudaStream_t s) {
   LatentParams p{};
   p.a = a;
-  make_latent_plan(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, p);
+  make_latent_plan(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, a.window, p);
   p.scale_log2 = a.scale * 1.4426950408889634f;
   const int64_t tiles = latent_tiles(p, a.T, a.heads);
   if (p.splits > 1 && !p.clustered) {
-    const size_t need = latent_tcgen05_workspace(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk);
+    const size_t need = latent_tcgen05_workspace(a.T, a.heads, a.rank, a.rot, a.max_keys, a.chunk, a.window);
     if (!a.workspace || a.workspace_bytes < need) {
       set_error("fb_latent_attention: workspace of %zu bytes needed, %zu given", need, a.workspace_bytes);
       return FB_ERR_MEMORY;

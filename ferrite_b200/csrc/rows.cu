@@ -1,7 +1,8 @@
 // What stands between the matmuls of a decoder with grouped-query attention and an fp32 residual stream, a kernel each:
-//   fb_embed       the stream's start: a row of one table and, where given, a row of another, added in fp32
-//   fb_heads_put   after a joint q | k | v projection: biases, RMSNorm of each query and key head, values mixed with another
-//                  layer's, the new cache row
+//   fb_embed       the stream's start: a row of one table, scaled, and, where given, a row of another, added in fp32
+//   fb_heads_put   after a joint q | k | v projection: biases, a short convolution over time, RMSNorm of each query and key head or
+//                  of all of them together, the turn by the token's place, values mixed with another layer's or the keys
+//                  themselves, the new cache row
 //   fb_add_norm    a layer's end: the branches' results scaled by column, a mixture's chosen rows weighted and summed, all
 //                  added to the stream, and the next layer's RMSNorm of it
 #include "launch.cuh"
@@ -13,6 +14,7 @@ struct EmbedArgs {
   const void *table, *places_table;  // [rows, cols], [place_rows, cols] or null
   int64_t rows, place_rows, cols;
   const int32_t *ids, *places;
+  float scale;
   float* out;  // [T, cols]
 };
 
@@ -24,7 +26,7 @@ __global__ void __launch_bounds__(256) embed_kernel(const EmbedArgs a) {
   const Act* x = static_cast<const Act*>(a.table) + id * a.cols;
   const Act* y = nullptr;
   if (a.places_table) y = static_cast<const Act*>(a.places_table) + min(max((int64_t)a.places[t], (int64_t)0), a.place_rows - 1) * a.cols;
-  for (int64_t c = threadIdx.x; c < a.cols; c += blockDim.x) a.out[t * a.cols + c] = value_of(x[c]) + (y ? value_of(y[c]) : 0.f);
+  for (int64_t c = threadIdx.x; c < a.cols; c += blockDim.x) a.out[t * a.cols + c] = value_of(x[c]) * a.scale + (y ? value_of(y[c]) : 0.f);
 }
 
 // ---- heads: a warp per token and head (the query heads, then the key heads, then the value heads)
@@ -153,9 +155,162 @@ __global__ void __launch_bounds__(128) heads_put4_kernel(const HeadsPutArgs a) {
   }
 }
 
+// ---- the same with a convolution, joint norms, turned heads or keys that are the values too: a block has a token's units - all
+// query heads, or the others, where a norm goes over them together; else some of them - and keeps their columns in shared memory.
+// The tokens whose convolution reaches into the state are one block's, one after the other, which then leaves the new state: no
+// other block reads or writes it.
+struct HeadsTurnArgs {
+  HeadsPutArgs p;
+  int per, tokens, first;  // units a block (joint norms: 0); tokens of a sequence, and how many of them its first block has
+};
+
+template <typename In, typename Act, int N>  // N: columns a thread handles at a time, 4 (whole aligned groups) or 1
+__global__ void __launch_bounds__(256) heads_turn_kernel(const HeadsTurnArgs args) {
+  griddep_launch_dependents();
+  griddep_wait();
+  extern __shared__ __align__(16) float turn_row[];  // the block's columns, then [turned / 2] cos and sin
+  __shared__ float red[32];
+  const HeadsPutArgs& a = args.p;
+  const fb_heads& s = a.h;
+  const int keys = s.heads + s.kv_heads, units = s.keys_are_values ? keys : keys + s.kv_heads;
+  const int u0 = args.per ? blockIdx.y * args.per : blockIdx.y ? s.heads : 0, u1 = args.per ? min(units, u0 + args.per) : blockIdx.y ? units : s.heads;
+  auto column = [&](int u) { return (int64_t)min(u, keys) * s.dim + (int64_t)max(u - keys, 0) * s.vdim; };
+  const int64_t c0 = column(u0), all = column(units);
+  const int cols = (int)(column(u1) - c0);
+  float *turns = turn_row + (cols + 3) / 4 * 4;
+  const int half = s.turned / 2, blocks = args.tokens - args.first + 1;
+  const int seq = blockIdx.x / blocks, b = blockIdx.x % blocks, begin = b ? args.first + b - 1 : 0, count = b ? 1 : args.first;
+  const int64_t row0 = (int64_t)seq * args.tokens;
+  const int start = s.places ? s.places[row0] : 0;  // where the sequence's first token of this call stands
+  const bool dead = s.conv && start == s.dead, held = s.conv && start != 0 && !dead;
+  const int back = s.conv ? s.taps - 1 : 0;
+  const In* x = static_cast<const In*>(a.qkv) + row0 * a.ld + c0;
+  float* state = s.conv ? s.state + seq * s.state_stride + c0 : nullptr;
+  // N columns of the sequence's token i as projected, from the state where i < 0
+  auto projected = [&](int i, int c, float v[N]) {
+    if (i >= 0) {
+      if constexpr (N == 4) {
+        const float4 f = four(x + (int64_t)i * a.ld + c);
+        v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
+      } else {
+        v[0] = value_of(x[(int64_t)i * a.ld + c]);
+      }
+      if (s.bias) {
+#pragma unroll
+        for (int e = 0; e < N; ++e) v[e] += s.bias[c0 + c + e];
+      }
+    } else {
+#pragma unroll
+      for (int e = 0; e < N; ++e) v[e] = held ? state[(int64_t)(back + i) * all + c + e] : 0.f;
+    }
+  };
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int i = begin; i < begin + count; ++i) {
+    const int64_t t = row0 + i, row = a.rows[t];
+    if (s.turned) {
+      const int place = s.places[t];
+      for (int j = threadIdx.x; j < half; j += blockDim.x) turn_of(place, s.freq[j], s.mag, turns[j], turns[half + j]);
+    }
+    float ss = 0.f;
+    for (int c = N * threadIdx.x; c < cols; c += N * blockDim.x) {
+      float v[N];
+      if (s.conv) {
+#pragma unroll
+        for (int e = 0; e < N; ++e) v[e] = 0.f;
+        for (int j = 0; j < s.taps; ++j) {
+          float u[N];
+          projected(i - back + j, c, u);
+#pragma unroll
+          for (int e = 0; e < N; ++e) v[e] = fmaf(s.conv[j * all + c0 + c + e], u[e], v[e]);
+        }
+      } else {
+        projected(i, c, v);
+      }
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        turn_row[c + e] = v[e];
+        if (c0 + c + e < column(keys)) ss = fmaf(v[e], v[e], ss);  // (joint norms: a block's query heads, or its key heads)
+      }
+    }
+    const float joint = s.norm_all ? 1.f / sqrtf(block_sum(ss, red) / (float)((blockIdx.y ? s.kv_heads : s.heads) * s.dim) + s.eps) : 1.f;
+    __syncthreads();
+    const bool inside = row >= 0 && row < a.cache_rows;  // nothing is written outside the cache
+    for (int u = u0 + warp; u < u1; u += 8) {
+      const bool is_q = u < s.heads, is_v = u >= keys;
+      const int n = is_v ? s.vdim : s.dim, g = is_q ? u : is_v ? u - keys : u - s.heads;
+      if (!is_q && !inside) continue;
+      const float* mine = turn_row + (column(u) - c0);
+      const float* w = is_v ? nullptr : is_q ? s.q_norm : s.k_norm;
+      if (w && s.norm_all) w += g * s.dim;
+      float r = joint;
+      if (w && !s.norm_all) {
+        float own = 0.f;
+        for (int c = lane; c < n; c += 32) own = fmaf(mine[c], mine[c], own);
+        r = 1.f / sqrtf(warp_sum(own) / (float)n + s.eps);
+      }
+      Act* cached = static_cast<Act*>(a.cache) + g * a.head_stride + row * (s.dim + s.vdim);
+      Act* out = is_q ? static_cast<Act*>(a.q_out) + t * a.ld_q + (int64_t)g * s.dim : is_v ? cached + s.dim : cached;
+      auto normed = [&](int c) { return w ? mine[c] * r * w[c] : mine[c]; };
+      auto result = [&](int c) {
+        if (is_v || c >= s.turned) return normed(c);
+        const float own = normed(c), other = normed(c ^ 1), cs = turns[c >> 1], sn = turns[half + (c >> 1)];
+        return c & 1 ? own * cs + other * sn : own * cs - other * sn;
+      };
+      for (int c = N * lane; c < n; c += 32 * N) {
+        if constexpr (N == 4) {
+          put_four(out + c, make_float4(result(c), result(c + 1), result(c + 2), result(c + 3)));
+          if (s.keys_are_values && !is_q) put_four(cached + s.dim + c, make_float4(mine[c], mine[c + 1], mine[c + 2], mine[c + 3]));
+        } else {
+          store_value(out + c, result(c));
+          if (s.keys_are_values && !is_q) store_value(cached + s.dim + c, mine[c]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+  if (s.conv && b == 0 && !dead)  // (a thread's own columns, rows rising: what a row is made of is read before it is overwritten)
+    for (int c = N * threadIdx.x; c < cols; c += N * blockDim.x)
+      for (int r = 0; r < back; ++r) {
+        float v[N];
+        projected(args.tokens + r - back, c, v);
+#pragma unroll
+        for (int e = 0; e < N; ++e) state[r * all + c + e] = v[e];
+      }
+}
+
+template <typename In, typename Act>
+static int launch_heads_turn(const HeadsPutArgs& a, cudaStream_t s) {
+  const fb_heads& h = a.h;
+  HeadsTurnArgs t{a, 0, 1, 1};
+  const int units = h.heads + (h.keys_are_values ? 1 : 2) * h.kv_heads, wide = h.dim > h.vdim ? h.dim : h.vdim;
+  unsigned parts = 2;
+  int64_t most = (int64_t)(h.heads > 2 * h.kv_heads ? h.heads : 2 * h.kv_heads) * wide;
+  if (!h.norm_all) {
+    t.per = 1024 / wide < 1 ? 1 : 1024 / wide;
+    parts = (unsigned)ceil_div(units, t.per), most = (int64_t)t.per * wide;
+  }
+  const size_t smem = (size_t)((most + 3) / 4 * 4 + h.turned) * sizeof(float);
+  FB_REQUIRE(smem <= 200 * 1024, "fb_heads_put: too many columns for a norm over all heads");
+  int64_t grid = a.T;
+  if (h.conv) {
+    t.tokens = (int)(a.T / h.sequences), t.first = h.taps - 1 < 1 ? 1 : h.taps - 1 < t.tokens ? h.taps - 1 : t.tokens;
+    grid = (int64_t)h.sequences * (t.tokens - t.first + 1);
+  }
+  auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
+  const bool fours = h.dim % 4 == 0 && h.vdim % 4 == 0 && whole(a.qkv, a.ld, sizeof(In)) && whole(a.q_out, a.ld_q, sizeof(Act)) && whole(a.cache, a.head_stride, sizeof(Act));
+  static std::atomic<uint64_t> opted{0};
+  if (first_on_device(opted)) {
+    cudaFuncSetAttribute(heads_turn_kernel<In, Act, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    cudaFuncSetAttribute(heads_turn_kernel<In, Act, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+  }
+  const dim3 g((unsigned)grid, parts);
+  return fours ? launch_after(heads_turn_kernel<In, Act, 4>, g, dim3(256), smem, s, "fb_heads_put", t) : launch_after(heads_turn_kernel<In, Act, 1>, g, dim3(256), smem, s, "fb_heads_put", t);
+}
+
 template <typename In, typename Act>
 static int launch_heads_put(const HeadsPutArgs& a, cudaStream_t s) {
   const fb_heads& h = a.h;
+  if (h.turned || h.conv || h.norm_all || h.keys_are_values) return launch_heads_turn<In, Act>(a, s);
   const int units = h.heads + 2 * h.kv_heads;
   auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
   const bool fours = h.dim % 4 == 0 && h.vdim % 4 == 0 && h.dim <= 256 && h.vdim <= 256 && whole(a.qkv, a.ld, sizeof(In)) && whole(h.first, h.ld_first, sizeof(In)) && whole(h.bias, 0, 4) &&
@@ -168,6 +323,17 @@ static int launch_heads_put(const HeadsPutArgs& a, cudaStream_t s) {
   return launch_after(heads_put_kernel<In, Act>, dim3((unsigned)a.T, (unsigned)ceil_div(units, HEADS_WARPS)), dim3(32 * HEADS_WARPS), 0, s, "fb_heads_put", a);
 }
 
+// where a token's chosen rows are: one with slot -1 is the token's own (or, where there are none, counts for nothing)
+template <typename Act>
+__device__ __forceinline__ void chosen_rows(const fb_branches& a, int64_t t, const Act** from, float* weight) {
+  for (int j = threadIdx.x; j < a.k; j += blockDim.x) {
+    const int64_t slot = a.slots[t * a.k + j];
+    const bool own = slot < 0 && a.own;
+    from[j] = own ? static_cast<const Act*>(a.own) + t * a.ld_own : static_cast<const Act*>(a.chosen) + (slot < 0 ? 0 : slot) * a.ld_chosen;
+    weight[j] = slot < 0 && !own ? 0.f : a.weights[t * a.k + j];
+  }
+}
+
 // ---- a layer's end: a block per token; the new row stays in shared memory for the norm's second pass
 template <typename In, typename Act>
 __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, const int64_t cols) {
@@ -175,11 +341,10 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, cons
   griddep_wait();
   extern __shared__ float row[];  // [cols]
   __shared__ float red[32];
-  __shared__ int64_t at[64];
+  __shared__ const Act* from[64];
   __shared__ float weight[64];
   const int64_t t = blockIdx.x;
-  if (a.chosen)
-    for (int j = threadIdx.x; j < a.k; j += blockDim.x) at[j] = a.slots[t * a.k + j] * a.ld_chosen, weight[j] = a.weights[t * a.k + j];
+  if (a.chosen) chosen_rows(a, t, from, weight);
   __syncthreads();
   const float* x = a.x + t * a.ld_x;
   const In* y1 = a.mixer ? static_cast<const In*>(a.mixer) + t * a.ld_mixer : nullptr;
@@ -187,11 +352,11 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, cons
   float ss = 0.f;
   for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) {
     float v = x[c];
-    if (y1) v = fmaf(value_of(y1[c]), a.mixer_scale ? a.mixer_scale[c] : 1.f, v);
+    if (y1 || a.mixer_bias) v = fmaf((y1 ? value_of(y1[c]) : 0.f) + (a.mixer_bias ? a.mixer_bias[c] : 0.f), a.mixer_scale ? a.mixer_scale[c] : 1.f, v);
     if (a.chosen || y2) {
       float f = y2 ? value_of(y2[c]) : 0.f;
       if (a.chosen)
-        for (int j = 0; j < a.k; ++j) f = fmaf(weight[j], value_of(static_cast<const Act*>(a.chosen)[at[j] + c]), f);
+        for (int j = 0; j < a.k; ++j) f = fmaf(weight[j], value_of(from[j][c]), f);
       v = fmaf(f, a.other_scale ? a.other_scale[c] : 1.f, v);
     }
     row[c] = v;
@@ -199,9 +364,9 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, cons
     ss = fmaf(v, v, ss);
   }
   if (!a.h) return;
-  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps);
+  const float r = a.w ? 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps) : 1.f;
   Act* h = static_cast<Act*>(a.h) + t * a.ld_h;
-  for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) store_value(h + c, row[c] * r * (a.w[c] + a.plus));
+  for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) store_value(h + c, a.w ? row[c] * r * (a.w[c] + a.plus) : row[c]);
 }
 
 // the same for rows of whole groups of four columns, 16-byte aligned: a thread keeps its groups in registers, everything it
@@ -211,11 +376,11 @@ __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, con
   griddep_launch_dependents();
   griddep_wait();
   __shared__ float red[32];
-  __shared__ int64_t at[64];
+  __shared__ const Act* from[64];
   __shared__ float weight[64];
   const int64_t t = blockIdx.x;
   if (a.chosen) {
-    for (int j = threadIdx.x; j < a.k; j += blockDim.x) at[j] = a.slots[t * a.k + j] * a.ld_chosen, weight[j] = a.weights[t * a.k + j];
+    chosen_rows(a, t, from, weight);
     __syncthreads();
   }
   const float4 one = make_float4(1.f, 1.f, 1.f, 1.f), none = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -228,6 +393,7 @@ __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, con
     if (c >= cols) continue;
     v[i] = four(a.x + t * a.ld_x + c);
     if (a.mixer) v[i] = fma4(four(static_cast<const In*>(a.mixer) + t * a.ld_mixer + c), a.mixer_scale ? four(a.mixer_scale + c) : one, v[i]);
+    if (a.mixer_bias) v[i] = fma4(four(a.mixer_bias + c), a.mixer_scale ? four(a.mixer_scale + c) : one, v[i]);
     if (a.other) f[i] = four(static_cast<const In*>(a.other) + t * a.ld_other + c);
   }
   if (a.chosen)
@@ -238,7 +404,7 @@ __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, con
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
-          part[i][e] = j + e < a.k && c < cols ? four(static_cast<const Act*>(a.chosen) + at[j + e] + c) : none;
+          part[i][e] = j + e < a.k && c < cols ? four(from[j + e] + c) : none;
         }
 #pragma unroll
       for (int i = 0; i < GROUPS; ++i)
@@ -257,11 +423,15 @@ __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, con
     ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
   }
   if (!a.h) return;
-  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps);
+  const float r = a.w ? 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps) : 1.f;
 #pragma unroll
   for (int i = 0; i < GROUPS; ++i) {
     const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
     if (c >= cols) continue;
+    if (!a.w) {
+      put_four(static_cast<Act*>(a.h) + t * a.ld_h + c, v[i]);
+      continue;
+    }
     const float4 w = four(a.w + c);
     put_four(static_cast<Act*>(a.h) + t * a.ld_h + c,
              make_float4(v[i].x * r * (w.x + a.plus), v[i].y * r * (w.y + a.plus), v[i].z * r * (w.z + a.plus), v[i].w * r * (w.w + a.plus)));
@@ -274,7 +444,7 @@ static int launch_add_norm(const fb_branches& a, int64_t T, int64_t cols, cudaSt
   if (first_on_device(opted)) cudaFuncSetAttribute(add_norm_kernel<In, Act>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
   const bool fours = cols % 4 == 0 && cols <= 4 * 4 * 512 && whole(a.x, a.ld_x, 4) && whole(a.mixer, a.ld_mixer, sizeof(In)) && whole(a.mixer_scale, 0, 4) &&
-                     whole(a.other, a.ld_other, sizeof(In)) && whole(a.other_scale, 0, 4) && whole(a.chosen, a.ld_chosen, sizeof(Act)) && whole(a.x_out, a.ld_x_out, 4) && whole(a.w, 0, 4) &&
+                     whole(a.other, a.ld_other, sizeof(In)) && whole(a.other_scale, 0, 4) && whole(a.chosen, a.ld_chosen, sizeof(Act)) && whole(a.x_out, a.ld_x_out, 4) && whole(a.w, 0, 4) && whole(a.mixer_bias, 0, 4) && whole(a.own, a.ld_own, sizeof(Act)) &&
                      whole(a.h, a.ld_h, sizeof(Act));
   const dim3 grid((unsigned)T);
   auto warps = [](int64_t work) { return dim3((unsigned)(work >= 512 ? 512 : ceil_div(work, 32) * 32)); };
@@ -290,11 +460,11 @@ static int launch_add_norm(const fb_branches& a, int64_t T, int64_t cols, cudaSt
 }  // namespace fb
 
 extern "C" int fb_embed(int dtype, const void* table, int64_t rows, int64_t cols, const int32_t* ids, const void* places_table, int64_t place_rows, const int32_t* places,
-                        int64_t T, float* out, void* stream) {
+                        int64_t T, float scale, float* out, void* stream) {
   FB_REQUIRE(table && ids && out && T >= 1 && rows >= 1 && cols >= 1, "fb_embed: null pointer or empty");
   FB_REQUIRE(!places_table || (places && place_rows >= 1), "fb_embed: a table of places takes the places");
   FB_REQUIRE(dtype == FB_BF16 || dtype == FB_FP32, "fb_embed: bf16 or fp32 tables");
-  const fb::EmbedArgs a{table, places_table, rows, place_rows, cols, ids, places, out};
+  const fb::EmbedArgs a{table, places_table, rows, place_rows, cols, ids, places, scale, out};
   const auto s = (cudaStream_t)stream;
   if (dtype == FB_FP32) return fb::launch_after(fb::embed_kernel<float>, dim3((unsigned)T), dim3(256), 0, s, "fb_embed", a);
   return fb::launch_after(fb::embed_kernel<uint16_t>, dim3((unsigned)T), dim3(256), 0, s, "fb_embed", a);
@@ -305,7 +475,13 @@ extern "C" int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void
   FB_REQUIRE(heads_host && qkv && rows && q_out && cache && T >= 1, "fb_heads_put: null pointer or empty");
   const fb_heads& h = *heads_host;
   FB_REQUIRE(h.heads >= 1 && h.kv_heads >= 1 && h.heads % h.kv_heads == 0 && h.heads <= 100000 && h.dim >= 1 && h.vdim >= 1, "fb_heads_put: whole groups of query heads per key head (got %d / %d)", h.heads, h.kv_heads);
-  const int64_t cols = (int64_t)(h.heads + h.kv_heads) * h.dim + (int64_t)h.kv_heads * h.vdim;
+  const int64_t cols = (int64_t)(h.heads + h.kv_heads) * h.dim + (h.keys_are_values ? 0 : (int64_t)h.kv_heads * h.vdim);
+  FB_REQUIRE(!h.keys_are_values || h.vdim == h.dim, "fb_heads_put: values that are keys are as wide");
+  FB_REQUIRE(h.turned >= 0 && h.turned % 2 == 0 && h.turned <= h.dim && (!h.turned || (h.freq && h.places)), "fb_heads_put: an even number of a head's columns turn, by frequencies and places");
+  FB_REQUIRE(!h.conv || (h.taps >= 1 && h.state && h.places && h.sequences >= 1 && T % h.sequences == 0 && (h.sequences == 1 || h.state_stride >= (h.taps - 1) * cols)),
+             "fb_heads_put: a convolution takes its state, the places, and as many rows of each sequence");
+  FB_REQUIRE(!h.norm_all || (h.q_norm && h.k_norm), "fb_heads_put: a norm over all heads takes its weights");
+  FB_REQUIRE(!h.first || !(h.turned || h.conv || h.norm_all || h.keys_are_values), "fb_heads_put: mixed values go with plain heads");
   FB_REQUIRE(ld >= cols && ld_q >= (int64_t)h.heads * h.dim && cache_rows >= 1 && head_stride >= cache_rows * (h.dim + h.vdim), "fb_heads_put: row strides too small");
   FB_REQUIRE(!h.first || (h.share && h.ld_first >= (int64_t)h.kv_heads * h.vdim), "fb_heads_put: mixed values take the other layer's and their share");
   FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32) && (in_dtype == FB_FP32 || dtype == FB_BF16),
@@ -321,7 +497,6 @@ extern "C" int fb_add_norm(const fb_branches* branches_host, int64_t T, int64_t 
   FB_REQUIRE(branches_host && branches_host->x && T >= 1 && cols >= 1 && cols * 4 <= 200 * 1024, "fb_add_norm: null pointer, empty or rows past 51200 columns");
   const fb_branches& a = *branches_host;
   FB_REQUIRE(a.x_out || a.h, "fb_add_norm: no result");
-  FB_REQUIRE(!a.h || a.w, "fb_add_norm: a norm takes its weight");
   FB_REQUIRE(!a.chosen || (a.slots && a.weights && a.k >= 1 && a.k <= 64), "fb_add_norm: chosen rows take their places and weights, up to 64 a token");
   FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32) && (in_dtype == FB_FP32 || dtype == FB_BF16),
              "fb_add_norm: bf16 or fp32; fp32 results come from fp32");

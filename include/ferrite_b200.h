@@ -151,7 +151,8 @@ enum fb_dense_epilogue_kind {
   FB_DENSE_GATE = 3,    /* times sigmoid(gate[t * ld_gate + batch entry]) */
   FB_DENSE_DYT_ADD = 4, /* out (fp32) = residual + tanh(alpha acc) w + b, and, with h_out given, h_out (bf16) = tanh(alpha2 out) w2 + b2: a Dynamic
                            Tanh on a branch, the residual add, and the Dynamic Tanh that the next branch starts with */
-  FB_DENSE_SWIGLU = 5   /* as FB_DENSE_GLU, the plain unit: out = g sigmoid(g) u */
+  FB_DENSE_SWIGLU = 5,  /* as FB_DENSE_GLU, the plain unit: out = g sigmoid(g) u */
+  FB_DENSE_GEGLU = 6    /* as FB_DENSE_GLU: out = gelu(gate + gate_bias) (up + up_bias), GELU's tanh form */
 };
 typedef struct {
   int kind;
@@ -165,6 +166,7 @@ typedef struct {
   void* h_out;
   int64_t ld_h;
   const float *alpha2, *w2, *b2;
+  const float *gate_bias, *up_bias; /* GEGLU: [N / 2] each, or null */
 } fb_dense_epilogue;
 /* batch independent matmuls: x, W and out move on by x_batch, w_batch and out_batch elements an entry (x_batch 0: all take the
  * same rows).  ldx, ldw, x_batch, w_batch multiples of 8 elements, x and W 16-byte aligned, K a multiple of 8 (GLU: N / 2 a
@@ -176,14 +178,22 @@ int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_t x_batch, 
 
 /* ---- a mixture of experts with bf16 or fp32 weights ------------------------------------------------------ */
 
-/* Each token's k largest of n router logits (fp32, + bias where given; the lower column first among equals) and the softmax of
- * those (weights), and where each choice's row goes (slots, both [T, k]) in rows of whole tiles of `tile` (a multiple of 16):
+typedef struct {
+  int n, k;          /* router outputs, choices a token */
+  int identity;      /* the last so many outputs stand for experts that give back their input: they have no rows */
+  const float* bias; /* [n] or null: joins what the choice goes by and, unless scored, the weights */
+  int scored;        /* 0: choices by logit + bias, weights the softmax of the chosen; 1: scores = softmax of all logits, choices by
+                        score + bias, weights the chosen scores over their sum (+ 1e-20) */
+  float scale;       /* the weights times this */
+} fb_router;
+/* Each token's k largest of its router's n outputs (fp32 logits; the lower column first among equals), their weights, and
+ * where each choice's row goes (slots, both [T, k]; -1: an identity expert's) in rows of whole tiles of `tile` (a multiple of 16):
  *   shared_rows   a tile a touched expert, holding all the tokens (T <= tile): the choice's row is the token's in its expert's tile
  *   otherwise     each expert's choices in tiles of their own
- * tile_expert[tiles, 3]: each tile's expert, ascending (n past those used), that expert's first tile and its number of tiles; live[0]: how many are used; tiles =
- * fb_route_tiles(...), the most there can be.  ids [T, k]: the choices. */
+ * tile_expert[tiles, 3]: each tile's expert, ascending (past those used: the number of experts with rows), that expert's first tile and its number
+ * of tiles; live[0]: how many are used; tiles = fb_route_tiles(...) of the experts with rows, the most there can be.  ids [T, k]: the choices. */
 int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_rows);
-int fb_route(const float* logits, int64_t T, int64_t ld, const float* bias, int n, int k, int tile, int shared_rows, float* weights, int32_t* ids,
+int fb_route(const fb_router* router_host, const float* logits, int64_t T, int64_t ld, int tile, int shared_rows, float* weights, int32_t* ids,
              int32_t* slots, int32_t* tile_expert, int32_t* live, void* stream);
 
 /* Row t of x (row_bytes bytes, rows ldx_bytes apart) into the rows slots[t, 0 .. k) of out (rows one after another): the
@@ -363,10 +373,13 @@ int fb_matmul(const void* a, const int64_t* a_strides_host, int a_dtype, const v
  * of the key part that all heads share): q_out[t] = RMSNorm(query latent) * q_norm (q_rank 0: a design without one), and
  * cache row rows[t] = RMSNorm(key-value latent) * kv_norm | the key part, its first `dims` columns turned pair by pair (2i,
  * 2i + 1) by places[t] * freq[i] with cos and sin times `mag`.  Norms and angles in fp32 or better; in_dtype: how `down`
- * is stored, dtype: q_out and the cache.  A row outside the cache is not written. */
+ * is stored, dtype: q_out and the cache.  A row outside the cache is not written.
+ * heads >= 1 (then q_rank is 0): the row begins with the queries instead, heads x (dim | rot): their first parts side by side to
+ * q_out [T, heads * dim], the others, turned, to q_turned + t * ld_turned + h * turned_head. */
 int fb_latent_put(int in_dtype, const void* down, int64_t T, int64_t ld, int q_rank, int kv_rank, int rot, int dims, const float* q_norm,
                   const float* kv_norm, float eps, const double* freq, float mag, const int32_t* places, const int32_t* rows, int dtype,
-                  void* q_out, int64_t ld_q, void* cache, int64_t cache_rows, void* stream);
+                  void* q_out, int64_t ld_q, int heads, int dim, void* q_turned, int64_t ld_turned, int64_t turned_head, void* cache,
+                  int64_t cache_rows, void* stream);
 
 /* The same turn for each head of x (head h of token t at x + t * x_row + h * x_head, `width` columns, the first `dims` of
  * them turned, the rest copied) into out (strides alike). */
@@ -376,12 +389,13 @@ int fb_rotate_pairs(int dtype, const void* x, int64_t T, int heads, int64_t x_ro
 /* Attention whose keys and values are one row of cache [cache_rows, rank + rot] a token, shared by all heads: head h of token t
  * has its query at q + t * ld_q + h * (rank + rot), scores are scale * (query . row), the output (out + t * ld_o + h * rank) is
  * the softmax-weighted sum of the rows' first `rank` columns.  Token t sees the rows base[t] + row0 + 0 .. last[t] (base null:
- * row0 alone).  sink (fp32 [heads], or null): exp(sink[h]) joins head h's denominator once, unscaled and without a value.
+ * row0 alone), with window only the last `window` of them.  sink (fp32 [heads], or null): exp(sink[h]) joins head h's denominator
+ * once, unscaled and without a value.
  * chunk: the tokens are consecutive ones of one sequence (they may share the rows they read).  max_keys: an upper bound of
  * last[t] + 1.  workspace: fb_latent_attention_workspace_bytes bytes. */
-size_t fb_latent_attention_workspace_bytes(int dtype, int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk);
+size_t fb_latent_attention_workspace_bytes(int dtype, int64_t T, int heads, int rank, int rot, int64_t max_keys, int chunk, int window);
 int fb_latent_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int rank, int rot, const void* cache, int64_t cache_rows,
-                        const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk, float scale, const float* sink,
+                        const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk, int window, float scale, const float* sink,
                         void* out, int64_t ld_o, void* workspace, size_t workspace_bytes, void* stream);
 
 /* Linear attention with a decay per head, token after token: S = decay[h] * S + k v^T, out = S^T q, over `sequences`
@@ -398,9 +412,9 @@ int fb_gated_rmsnorm(const float* x, int64_t rows, int64_t cols, int64_t ldx, in
 
 /* ---- grouped-query attention over rows of a key and its value, and what stands around it ------------------- */
 
-/* out[t] = table[ids[t]] + places_table[places[t]] (or the first alone) in fp32; ids and places outside are clamped */
+/* out[t] = table[ids[t]] * scale + places_table[places[t]] (or the first alone) in fp32; ids and places outside are clamped */
 int fb_embed(int dtype, const void* table, int64_t rows, int64_t cols, const int32_t* ids, const void* places_table, int64_t place_rows,
-             const int32_t* places, int64_t T, float* out, void* stream);
+             const int32_t* places, int64_t T, float scale, float* out, void* stream);
 
 typedef struct {
   int heads, kv_heads, dim, vdim; /* dim: a query's and a key's columns, vdim: a value's */
@@ -411,6 +425,18 @@ typedef struct {
                                      becomes (1 - share) value + share (first + first_bias) */
   int64_t ld_first;
   const float *first_bias, *share; /* share: one number on the device */
+  int norm_all;                    /* the norms go over all query (key) heads together; q_norm [heads * dim], k_norm [kv_heads * dim] */
+  int keys_are_values;             /* qkv has no v: the values are the keys as projected, before norm and turn (vdim = dim) */
+  int turned;                      /* of each query and key head the first so many columns turn pair by pair (2i, 2i + 1) by */
+  const double* freq;              /* places[t] * freq[i], cos and sin times mag */
+  float mag;
+  const int32_t* places;
+  int taps;                        /* a short convolution over time, before norm, turn and cache: each column becomes the sum over j of */
+  const float* conv;               /* conv[j, column] times its value (with its bias) taps - 1 - j tokens ago, zeros before the */
+  float* state;                    /* sequence's start; conv [taps, columns of q | k | v], null: none.  state: the last taps - 1 rows of */
+  int64_t state_stride;            /* each sequence, read and left for the next call, state_stride elements a sequence.  The T rows are */
+  int sequences, dead;             /* `sequences` sequences' in turn; one whose first token stands at place 0 starts from zeros, one whose
+                                      first token stands at place `dead` (-1: none) leaves its state alone */
 } fb_heads;
 /* After a joint projection q (heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim) (| more): biases and norms in fp32, queries
  * to q_out, and (key | value) into row rows[t] of each key head of cache [kv_heads, cache_rows, dim + vdim] (heads head_stride
@@ -420,11 +446,11 @@ int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void* qkv, int6
 
 /* Attention over such a cache: query head h reads key head h / (heads / kv_heads); token t, whose place is last[t], sees the cache
  * rows base[t] + row0 + lo .. + last[t] (base null: row0 alone), lo = 0, or, with span, the first place of its span of `span`
- * places.  sink (fp32 [heads], or null): exp(sink[h]) joins head h's denominator.  gate (or null): the result times its sigmoid,
+ * places; with window, only the last `window` of them.  softcap c > 0: a scaled score s becomes c tanh(s / c).  sink (fp32 [heads], or null): exp(sink[h]) joins head h's denominator.  gate (or null): the result times its sigmoid,
  * column by column.  chunk: the tokens are consecutive ones of one sequence.  max_keys: an upper bound of last[t] + 1. */
 int fb_heads_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int kv_heads, int dim, int vdim, const void* cache,
                        int64_t cache_rows, int64_t head_stride, const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk,
-                       int span, float scale, const float* sink, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o,
+                       int span, int window, float scale, float softcap, const float* sink, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o,
                        void* stream);
 
 typedef struct {
@@ -447,8 +473,12 @@ typedef struct {
   float plus, eps;
   void* h;
   int64_t ld_h;
+  const float* mixer_bias; /* added to the mixer's result (where there is none, in its place), one a column */
+  const void* own;         /* the row of a choice with slot -1: token t's is row t */
+  int64_t ld_own;
 } fb_branches;
-/* A layer's end and the next one's start.  Branches null: not there.  in_dtype: mixer and other; dtype: chosen and h. */
+/* A layer's end and the next one's start.  Branches null: not there; h without w: the sum itself.  in_dtype: mixer and other; dtype:
+ * chosen, own and h. */
 int fb_add_norm(const fb_branches* branches_host, int64_t T, int64_t cols, int in_dtype, int dtype, void* stream);
 
 /* ---- several GPUs -------------------------------------------------------------------------------------- */

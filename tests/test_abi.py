@@ -123,7 +123,7 @@ def test_heads_and_experts_entry_points_refuse_bad_arguments_without_a_gpu():
     assert rc == -1 and b"all of them there" in lib.fb_last_error()
     rc = lib.fb_grouped_matmul(_lib.FP32, 16, 8, 64, 0, _lib.FP32, 16, (ctypes.c_int64 * 3)(4096, 1, 64), 2, 64, 64, 16, 16, 1, 16, _lib.FP32, 16, 64, None)
     assert rc == -1 and b"rows there" in lib.fb_last_error()
-    rc = lib.fb_add_norm(ctypes.byref(_lib.Branches(x=16, h=16)), 2, 64, _lib.BF16, _lib.BF16, None)
-    assert rc == -1 and b"takes its weight" in lib.fb_last_error()
+    rc = lib.fb_add_norm(ctypes.byref(_lib.Branches(x=16)), 2, 64, _lib.BF16, _lib.BF16, None)
+    assert rc == -1 and b"no result" in lib.fb_last_error()
     rc = lib.fb_embed(_lib.BF16, 16, 8, 64, 16, 16, 0, None, 2, 16, None)
     assert rc == -1 and b"takes the places" in lib.fb_last_error()
