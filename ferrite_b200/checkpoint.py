@@ -106,6 +106,11 @@ def turned(w):
     return Weight(lambda: np.ascontiguousarray(np.swapaxes(w.bits(), -1, -2)), lambda rt: w.device(rt).T)
 
 
+def scaled(w, s):
+    """A weight times a number: exact in fp32 on the device, rounded again on the host."""
+    return Weight(lambda: bf16_bits(w.values() * np.float32(s)), lambda rt: (w.device(rt).float() * s).realize())
+
+
 def columns_together(w):
     """A matrix that x @ w takes as it is, laid out on the device as `turned` leaves one: each output column's weights together."""
     return Weight(w.bits, lambda rt: (w.device(rt).T + 0).realize().T)

@@ -269,10 +269,11 @@ def linear_indexed(x, w, index, out, sum_slots=False, x_slot_rows=0, out_slot_st
     return out
 
 
-def latent_put(down, q_rank, kv_rank, rot, dims, q_norm, kv_norm, eps, freq, mag, places, rows, cache, q_out):
-    """The norms, the turn and the cache write after a joint down-projection (fb_latent_put)."""
+def latent_put(down, q_rank, kv_rank, rot, dims, q_norm, kv_norm, eps, freq, mag, places, rows, cache, q_out, heads=0, dim=0, q_turned=None):
+    """The norms, the turn and the cache write after a joint down-projection (fb_latent_put); q_turned: [heads, T, rot]."""
     check(lib().fb_latent_put(_CODES[down.dtype], down.data_ptr(), down.shape[0], down.stride(0), q_rank, kv_rank, rot, dims, _ptr(q_norm), kv_norm.data_ptr(), eps,
                               freq.data_ptr(), mag, places.data_ptr(), rows.data_ptr(), _CODES[cache.dtype], _ptr(q_out), q_out.stride(0) if q_out is not None else 0,
+                              heads, dim, _ptr(q_turned), q_turned.stride(1) if q_turned is not None else 0, q_turned.stride(0) if q_turned is not None else 0,
                               cache.data_ptr(), cache.shape[0], _stream()))
     count()
 
@@ -286,17 +287,17 @@ def rotate_pairs(x, rotation, places, out):
     return out
 
 
-def latent_attention(q, cache, base, last, heads, rank, scale, sink, max_keys, chunk, row0=0, out=None):
+def latent_attention(q, cache, base, last, heads, rank, scale, sink, max_keys, chunk, row0=0, out=None, window=0):
     """q [T, heads * (rank + rot)] over cache [rows, rank + rot] (fb_latent_attention)."""
     T, rot = q.shape[0], cache.shape[1] - rank
     if out is None:
         out = torch.empty(T, heads * rank, dtype=q.dtype, device=q.device)
     assert cache.is_contiguous() and last.numel() == T and (base is None or base.numel() == T) and last.dtype == torch.int32
     code = _CODES[q.dtype]
-    need = lib().fb_latent_attention_workspace_bytes(code, T, heads, rank, rot, max_keys, int(chunk))
+    need = lib().fb_latent_attention_workspace_bytes(code, T, heads, rank, rot, max_keys, int(chunk), window)
     ws = attention_workspace(q.device, need)
     check(lib().fb_latent_attention(code, q.data_ptr(), T, q.stride(0), heads, rank, rot, cache.data_ptr(), cache.shape[0], _ptr(base), row0, last.data_ptr(), max_keys,
-                                    int(chunk), scale, _ptr(sink), out.data_ptr(), out.stride(0), _ptr(ws) if need else None, ws.numel() if need else 0, _stream()))
+                                    int(chunk), window, scale, _ptr(sink), out.data_ptr(), out.stride(0), _ptr(ws) if need else None, ws.numel() if need else 0, _stream()))
     count(2 if need else 1)
     return out
 
@@ -336,17 +337,23 @@ def dense(x, w, out, settled=False, /, kind=_lib.DENSE_NONE, **extra):
     return out
 
 
-def embed(table, ids, places_table, places, out):
-    """out (fp32) = table[ids] + places_table[places] (fb_embed)."""
+def embed(table, ids, places_table, places, out, scale=1.0):
+    """out (fp32) = table[ids] * scale + places_table[places] (fb_embed)."""
     check(lib().fb_embed(_CODES[table.dtype], table.data_ptr(), table.shape[0], table.shape[1], ids.data_ptr(), _ptr(places_table), places_table.shape[0] if places_table is not None else 0,
-                         _ptr(places), ids.numel(), out.data_ptr(), _stream()))
+                         _ptr(places), ids.numel(), scale, out.data_ptr(), _stream()))
     count()
     return out
 
 
-def heads_put(qkv, heads, kv_heads, dim, vdim, rows, cache, q_out, bias=None, q_norm=None, k_norm=None, eps=0.0, first=None, first_bias=None, share=None):
-    """Biases, norms, mixed values and the cache write after a joint projection of heads (fb_heads_put); cache [kv_heads, rows, dim + vdim]."""
-    h = _lib.Heads(heads, kv_heads, dim, vdim, _ptr(bias), _ptr(q_norm), _ptr(k_norm), eps, _ptr(first), first.stride(0) if first is not None else 0, _ptr(first_bias), _ptr(share))
+def heads_put(qkv, heads, kv_heads, dim, vdim, rows, cache, q_out, bias=None, q_norm=None, k_norm=None, eps=0.0, first=None, first_bias=None, share=None,
+              norm_all=False, keys_are_values=False, rotation=None, places=None, conv=None, state=None, dead=-1):
+    """Biases, convolution, norms, turn, values and the cache write after a joint projection of heads (fb_heads_put); cache [kv_heads,
+    rows, dim + vdim]; rotation: (frequencies, columns that turn, factor); conv [taps, columns] and state [sequences, taps - 1, columns]."""
+    freq, dims, mag = rotation or (None, 0, 1.0)
+    h = _lib.Heads(heads, kv_heads, dim, vdim, _ptr(bias), _ptr(q_norm), _ptr(k_norm), eps, _ptr(first), first.stride(0) if first is not None else 0, _ptr(first_bias), _ptr(share),
+                   int(norm_all), int(keys_are_values), dims, _ptr(freq) if dims else None, mag, _ptr(places), conv.shape[0] if conv is not None else 0, _ptr(conv), _ptr(state),
+                   state.stride(0) if state is not None else 0, state.shape[0] if state is not None else 1, dead)
+    assert conv is None or (conv.is_contiguous() and state.dtype == conv.dtype == torch.float32 and state.shape[2] == state.stride(1) == conv.shape[1] and state.stride(2) == 1 and state.shape[1] >= conv.shape[0] - 1)
     assert cache.shape[0] == kv_heads and cache.shape[2] == dim + vdim and cache.stride(2) == 1 and cache.stride(1) == dim + vdim and q_out.dtype == cache.dtype
     check(lib().fb_heads_put(ctypes.byref(h), _CODES[qkv.dtype], qkv.data_ptr(), qkv.shape[0], qkv.stride(0), rows.data_ptr(), _CODES[cache.dtype], q_out.data_ptr(), q_out.stride(0),
                              cache.data_ptr(), cache.shape[1], cache.stride(0), _stream()))
@@ -354,7 +361,7 @@ def heads_put(qkv, heads, kv_heads, dim, vdim, rows, cache, q_out, bias=None, q_
     return q_out
 
 
-def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, span=0, sink=None, gate=None, row0=0, out=None):
+def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, span=0, sink=None, gate=None, row0=0, out=None, window=0, softcap=0.0):
     """q [T, heads * dim] over cache [kv_heads, rows, dim + vdim] (fb_heads_attention)."""
     T, dim = q.shape[0], cache.shape[2] - vdim
     assert q.shape[1] == heads * dim and q.dtype == cache.dtype and cache.stride(2) == 1 and cache.stride(1) == cache.shape[2]
@@ -362,7 +369,7 @@ def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, s
     if out is None:
         out = torch.empty(T, heads * vdim, dtype=q.dtype, device=q.device)
     check(lib().fb_heads_attention(_CODES[q.dtype], q.data_ptr(), T, q.stride(0), heads, cache.shape[0], dim, vdim, cache.data_ptr(), cache.shape[1], cache.stride(0), _ptr(base), row0,
-                                   last.data_ptr(), max_keys, int(chunk), span, scale, _ptr(sink), _CODES[gate.dtype] if gate is not None else 0, _ptr(gate),
+                                   last.data_ptr(), max_keys, int(chunk), span, window, scale, softcap, _ptr(sink), _CODES[gate.dtype] if gate is not None else 0, _ptr(gate),
                                    gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), _stream()))
     count()
     return out
@@ -370,7 +377,7 @@ def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, s
 
 class Routes:
     """Where a mixture's rows go (fb_route): tokens' weights, choices and slots [T, k], the tiles' experts, how many tiles are in
-    use, and the sizes of all that; shared: every tile holds all the tokens."""
+    use, and the sizes of all that (n: the experts that have rows); shared: every tile holds all the tokens."""
 
     def __init__(self, device, T, n, k, tile, shared):
         self.T, self.n, self.k, self.tile, self.shared = T, n, k, tile, shared
@@ -394,12 +401,13 @@ def route_tile(T, n, k):
     return min(range(32, 257, 16), key=work), False
 
 
-def route(logits, n, k, bias=None):
-    """Router logits (fp32 [T, >= n]) to Routes."""
+def route(logits, n, k, bias=None, scored=False, identity=0, scale=1.0):
+    """Router logits (fp32 [T, >= n]) to Routes; scored, identity, scale: fb_router's."""
     T = logits.shape[0]
     tile, shared = route_tile(T, n, k)
-    r = Routes(logits.device, T, n, k, tile, shared)
-    check(lib().fb_route(logits.data_ptr(), T, logits.stride(0), _ptr(bias), n, k, tile, int(shared), r.weights.data_ptr(), r.ids.data_ptr(), r.slots.data_ptr(),
+    r = Routes(logits.device, T, n - identity, k, tile, shared)
+    router = _lib.Router(n, k, identity, _ptr(bias), int(scored), scale)
+    check(lib().fb_route(ctypes.byref(router), logits.data_ptr(), T, logits.stride(0), tile, int(shared), r.weights.data_ptr(), r.ids.data_ptr(), r.slots.data_ptr(),
                          r.tile_expert.data_ptr(), r.live.data_ptr(), _stream()))
     count(1 if T <= 32 else 2)
     return r
@@ -414,14 +422,14 @@ def spread_rows(x, routes, out):
     return out
 
 
-def grouped(x, w, routes, out, kind=_lib.DENSE_NONE, shared=False):
+def grouped(x, w, routes, out, kind=_lib.DENSE_NONE, shared=False, **extra):
     """Rows of tiles (shared: x's rows in every tile) by each tile's matrix of the batch w [n, K, N]: on the tensor cores
-    where operands allow it (with a gated unit, if asked for); False where they do not."""
+    where operands allow it (with a gated unit, if asked for; extra: its numbers); False where they do not."""
     n, K, N = w.shape
     if not (x.dtype == w.dtype == torch.bfloat16 and x.stride(1) == 1 and w.stride(1) == 1 and lib().fb_dense_supports(
             x.data_ptr(), x.stride(0), 0, w.data_ptr(), w.stride(2), w.stride(0) if n > 1 else 0, K, N, kind)):
         return False
-    e = _lib.DenseEpilogue(kind=kind)
+    e = _lib.DenseEpilogue(kind=kind, **extra)
     check(lib().fb_dense_grouped(x.data_ptr(), x.shape[0], K, x.stride(0), int(shared), w.data_ptr(), N, w.stride(2), w.stride(0), n, routes.tile_expert.data_ptr(),
                                  routes.live.data_ptr(), routes.tiles, routes.tile, out.data_ptr(), _CODES[out.dtype], out.stride(0), ctypes.byref(e), _stream()))
     count()
@@ -438,14 +446,16 @@ def grouped_matmul(x, w, routes, out, shared=False):
     return out
 
 
-def add_norm(x, x_out, mixer=None, mixer_scale=None, other=None, other_scale=None, chosen=None, routes=None, w=None, plus=0.0, eps=0.0, h=None):
-    """A layer's end (fb_add_norm): x [T, cols] fp32 plus its branches into x_out, and that normed by w + plus into h."""
+def add_norm(x, x_out, mixer=None, mixer_scale=None, other=None, other_scale=None, chosen=None, routes=None, w=None, plus=0.0, eps=0.0, h=None,
+             mixer_bias=None, own=None):
+    """A layer's end (fb_add_norm): x [T, cols] fp32 plus its branches into x_out, and that normed by w + plus (w None: as it is) into h."""
     ld = lambda t: t.stride(0) if t is not None else 0
     of = lambda *ts: next((t.dtype for t in ts if t is not None), None)
     dtype = of(h, chosen) or torch.float32
     kind = of(mixer, other) or dtype if dtype == torch.bfloat16 else torch.float32
-    assert all(t is None or t.dtype == kind for t in (mixer, other)) and all(t is None or t.dtype == dtype for t in (h, chosen))
+    assert all(t is None or t.dtype == kind for t in (mixer, other)) and all(t is None or t.dtype == dtype for t in (h, chosen, own))
     b = _lib.Branches(x.data_ptr(), ld(x), _ptr(mixer), ld(mixer), _ptr(mixer_scale), _ptr(other), ld(other), _ptr(other_scale), _ptr(chosen), ld(chosen),
-                      _ptr(routes.slots) if routes else None, _ptr(routes.weights) if routes else None, routes.k if routes else 0, _ptr(x_out), ld(x_out), _ptr(w), plus, eps, _ptr(h), ld(h))
+                      _ptr(routes.slots) if routes else None, _ptr(routes.weights) if routes else None, routes.k if routes else 0, _ptr(x_out), ld(x_out), _ptr(w), plus, eps, _ptr(h), ld(h),
+                      _ptr(mixer_bias), _ptr(own), ld(own))
     check(lib().fb_add_norm(ctypes.byref(b), x.shape[0], x.shape[1], _CODES[kind], _CODES[dtype], _stream()))
     count()

@@ -496,6 +496,11 @@ class Tensor:
         self.rt.launched("touched", 1)
         return experts, out
 
+    def gelu_gated(self, bias=None, dtype=None):
+        """gelu(gate) * up of self's two halves, bias (fp32, a number a column of self) added before; fuses into a matmul."""
+        assert self.cols % 2 == 0 and (bias is None or (bias.dtype == "fp32" and bias.shape == (1, 1, self.cols)))
+        return self._lazy("gelu_gated", (self,) if bias is None else (self, bias), (self.batch, self.rows, self.cols // 2), dtype or self.dtype)
+
     def silu_columns(self, n):
         """self with its first n columns through SiLU (a joint projection of activated and plain parts); fuses into a matmul."""
         return self._lazy("silu_columns", (self,), self.shape, self.dtype, n=n)
@@ -547,6 +552,21 @@ class Tensor:
 
     # ---------------------------------------------------------------- latent attention and decaying linear attention
 
+    def latent_heads_put(self, rotation, places, rows, cache, heads, dim, turned, kv_norm, eps):
+        """self: a joint projection [1, tokens, queries (heads x (dim | rot)) | key-value latent | shared key part].  As latent_put for a
+        design without a query latent: the queries' first parts come back side by side, as the cache is stored, the others go,
+        turned, into `turned` (a view [heads, tokens, rot])."""
+        x, places, rows = self.realize(), places.realize(), rows.realize()
+        rank = kv_norm.cols
+        rot = cache.cols - rank
+        assert x.batch == 1 and x.buf.stride(2) == 1 and x.cols >= heads * (dim + rot) + cache.cols and cache.buf.is_contiguous(), f"{self.shape} into a cache {cache.shape}"
+        assert turned.shape == (heads, x.rows, rot) and turned.dtype == cache.dtype and turned.buf.stride(2) == 1 and kv_norm.dtype == "fp32" and places.cols == rows.cols == x.rows
+        freq, dims, mag = rotation
+        out = Tensor(self.rt, x.rows, heads * dim, dtype=cache.dtype)
+        ops.latent_put(x.buf[0], 0, rank, rot, dims, None, kv_norm.buf, eps, freq, mag, places.buf.reshape(-1), rows.buf.reshape(-1), cache.buf[0], out.buf[0], heads, dim, turned.buf)
+        self.rt.launched("latent put")
+        return out
+
     def latent_put(self, rotation, places, rows, cache, q_rank, q_norm, kv_norm, eps):
         """self: a joint down-projection [1, tokens, query latent | key-value latent | shared key part | ...].  One kernel norms
         both latents, turns the key part and puts (key-value latent | key part) into `cache` ([1, size, kv_rank + rot]) at
@@ -574,17 +594,17 @@ class Tensor:
         self.rt.launched("rotate pairs")
         return into
 
-    def attend_latent(self, cache, base, last, rank, scale, sink=None, length=None, chunk=False):
+    def attend_latent(self, cache, base, last, rank, scale, sink=None, length=None, chunk=False, window=0):
         """self: [1, tokens, heads (rank + rot)], each head's query in the latents' space and its turned part.  Token t attends
-        the cache rows base[t] .. base[t] + last[t]: one row is key (all of it) and value (its first `rank` columns) of every
-        head.  sink: a number per head that joins the softmax's denominator.  chunk: the tokens are one sequence's, its first
+        the cache rows base[t] .. base[t] + last[t] (the last `window` of them, if any): one row is key (all of it) and value (its
+        first `rank` columns) of every head.  sink: a number per head that joins the softmax's denominator.  chunk: the tokens are one sequence's, its first
         cache row 0.  Returns [1, tokens, heads rank]: weighted sums of latents."""
         q, last = self.realize(), last.realize()
         heads = q.cols // cache.cols
         assert q.batch == cache.batch == 1 and q.cols % cache.cols == 0 and q.dtype == cache.dtype and q.buf.stride(2) == 1, f"{q.shape} over a cache {cache.shape}"
         out = Tensor(self.rt, q.rows, heads * rank, dtype=q.dtype)
         ops.latent_attention(q.buf[0], cache.buf[0], None if chunk else base.realize().buf.reshape(-1), last.buf.reshape(-1), heads, rank, scale,
-                             None if sink is None else sink.buf, min(length or cache.rows, cache.rows), chunk, out=out.buf[0])
+                             None if sink is None else sink.buf, min(length or cache.rows, cache.rows), chunk, out=out.buf[0], window=window)
         self.rt.launched("latent attention")
         return out
 
@@ -609,35 +629,43 @@ class Tensor:
 
     # ---------------------------------------------------------------- an fp32 residual stream with grouped-query heads and experts
 
-    def embed(self, ids, places_table=None, places=None):
-        """Rows ids of this table, plus rows `places` of another where given, as an fp32 matrix: a residual stream's start."""
+    def embed(self, ids, places_table=None, places=None, scale=1.0):
+        """Rows ids of this table times scale, plus rows `places` of another where given, as an fp32 matrix: a residual stream's start."""
         ids, places = ids.realize(), None if places is None else places.realize()
         out = Tensor(self.rt, ids.cols, self.cols, dtype="fp32")
         assert places_table is None or (places_table.cols == self.cols and places_table.dtype == self.dtype and places.cols == ids.cols)
-        ops.embed(self.realize().buf[0], ids.buf.reshape(-1), None if places_table is None else places_table.realize().buf[0], None if places is None else places.buf.reshape(-1), out.buf[0])
+        ops.embed(self.realize().buf[0], ids.buf.reshape(-1), None if places_table is None else places_table.realize().buf[0], None if places is None else places.buf.reshape(-1), out.buf[0], scale)
         self.rt.launched("embed")
         return out
 
-    def heads_put(self, heads, dim, vdim, rows, cache, bias=None, q_norm=None, k_norm=None, eps=0.0, mix=None):
+    def heads_put(self, heads, dim, vdim, rows, cache, bias=None, q_norm=None, k_norm=None, eps=0.0, mix=None, norm_all=False,
+                  keys_are_values=False, rotation=None, places=None, conv=None, state=None, dead=-1):
         """self: a joint projection [1, tokens, q (heads x dim) | k | v (| more)]; its keys and values go into `cache` ([key
         heads, size, dim + vdim]) at `rows`, its queries come back, as the cache is stored.  bias: a number a column of q | k | v;
-        q_norm, k_norm: RMSNorm of each head; mix: (other values of the tokens, their bias or None, share): the values become
-        (1 - share) own + share other."""
+        q_norm, k_norm: RMSNorm of each head (norm_all: of all of them together); mix: (other values of the tokens, their bias or
+        None, share): the values become (1 - share) own + share other; keys_are_values: there is no v, the keys as projected are the
+        values; rotation: mixers.rotation's, by `places`; conv ([taps, columns]): a short convolution over time of every column, state
+        ([sequences, taps - 1, columns], fp32, read and written) what it needs of earlier tokens - nothing at place 0, and a sequence
+        at place `dead` leaves it alone."""
         x, rows = self.realize(), rows.realize()
-        assert x.batch == 1 and x.buf.stride(2) == 1 and rows.cols == x.rows and x.cols >= (heads + cache.batch) * dim + cache.batch * vdim, f"{self.shape} into a cache {cache.shape}"
-        assert all(t is None or t.dtype == "fp32" for t in (bias, q_norm, k_norm)) and (bias is None or bias.cols == (heads + cache.batch) * dim + cache.batch * vdim)
+        wide = (heads + cache.batch) * dim + (0 if keys_are_values else cache.batch * vdim)
+        assert x.batch == 1 and x.buf.stride(2) == 1 and rows.cols == x.rows and x.cols >= wide, f"{self.shape} into a cache {cache.shape}"
+        assert all(t is None or t.dtype == "fp32" for t in (bias, q_norm, k_norm, conv, state)) and all(t is None or t.cols == wide for t in (bias, conv, state))
+        assert q_norm is None or (q_norm.cols, k_norm.cols) == ((heads * dim, cache.batch * dim) if norm_all else (dim, dim))
         buf = lambda t: None if t is None else t.realize().buf
         first, first_bias, share = mix or (None, None, None)
         assert first is None or (first.dtype == x.dtype and first.shape == (1, x.rows, cache.batch * vdim) and first.buf.stride(2) == 1), "the other layer's values, a column each of this one's"
         out = Tensor(self.rt, x.rows, heads * dim, dtype=cache.dtype)
         ops.heads_put(x.buf[0], heads, cache.batch, dim, vdim, rows.buf.reshape(-1), cache.buf, out.buf[0], buf(bias), buf(q_norm), buf(k_norm), eps,
-                      None if first is None else first.buf[0], buf(first_bias), buf(share))
+                      None if first is None else first.buf[0], buf(first_bias), buf(share), norm_all, keys_are_values, rotation, None if places is None else places.realize().buf.reshape(-1),
+                      None if conv is None else conv.realize().buf[0], buf(state), dead)
         self.rt.launched("heads put")
         return out
 
-    def attend_heads(self, cache, base, last, vdim, scale, length=None, span=0, sink=None, gate=None, chunk=False):
+    def attend_heads(self, cache, base, last, vdim, scale, length=None, span=0, sink=None, gate=None, chunk=False, window=0, softcap=0.0):
         """self: [1, tokens, heads x dim] over such a cache.  Token t, which stands at place last[t], attends the rows from base[t]
-        on up to its own; with span, only those of its own span of that many places.  sink: a number per head that joins the
+        on up to its own; with span, only those of its own span of that many places, with window, only the last so many.  softcap: c
+        > 0 makes a scaled score s c tanh(s / c).  sink: a number per head that joins the
         softmax's denominator; gate: the result is multiplied by its sigmoid, column by column; chunk: one sequence's tokens,
         its first cache row 0.  Returns [1, tokens, heads x vdim]."""
         q, last = self.realize(), last.realize()
@@ -647,20 +675,22 @@ class Tensor:
         out = Tensor(self.rt, q.rows, heads * vdim, dtype=q.dtype)
         assert gate is None or gate.shape == out.shape
         ops.heads_attention(q.buf[0], cache.buf, None if chunk else base.realize().buf.reshape(-1), last.buf.reshape(-1), heads, vdim, scale, min(length or cache.rows, cache.rows), chunk, span,
-                            None if sink is None else sink.realize().buf, None if gate is None else gate.realize().buf[0], out=out.buf[0])
+                            None if sink is None else sink.realize().buf, None if gate is None else gate.realize().buf[0], out=out.buf[0], window=window, softcap=softcap)
         self.rt.launched("attention")
         return out
 
-    def route(self, n, k, bias=None):
-        """self: fp32 router logits, n a token: each token's k experts, their weights and where their rows go (ops.Routes)."""
+    def route(self, n, k, bias=None, scored=False, identity=0, scale=1.0):
+        """self: fp32 router logits, n a token: each token's k experts, their weights and where their rows go (ops.Routes).  scored: chosen
+        by softmax + bias, weighted by the softmax; identity: the last so many give back their input; scale: of the weights."""
         x = self.realize()
         assert x.dtype == "fp32" and x.batch == 1 and x.cols == n and x.buf.stride(2) == 1 and (bias is None or (bias.dtype == "fp32" and bias.cols == n))
         self.rt.launched("route")
-        return ops.route(x.buf[0], n, k, None if bias is None else bias.realize().buf)
+        return ops.route(x.buf[0], n, k, None if bias is None else bias.realize().buf, scored, identity, scale)
 
-    def experts(self, routes, gate_up, down):
+    def experts(self, routes, gate_up, down, clamp=None):
         """self: rows of tokens.  Every chosen expert's down(silu(gate) * up) of its tokens' rows, a row a choice where `routes`
-        puts it; gate and up side by side in gate_up [n, K, 2 m], down [n, m, N]."""
+        puts it; gate and up side by side in gate_up [n, K, 2 m], down [n, m, N].  clamp: (limit, slope) of clamped_glu in the
+        unit's place."""
         rt, h, m = self.rt, self.realize(), down.rows
         assert h.batch == 1 and gate_up.cols == 2 * m and gate_up.batch == down.batch == routes.n and h.rows == routes.T
         if not routes.shared:
@@ -670,13 +700,15 @@ class Tensor:
             h = x
         act = Tensor(rt, routes.tiles * routes.tile, m, dtype=h.dtype)
         out = Tensor(rt, routes.tiles * routes.tile, down.cols, dtype=h.dtype)
-        if ops.grouped(h.buf[0], gate_up.buf, routes, act.buf[0], _lib.DENSE_SWIGLU, routes.shared):
-            rt.launched("experts swiglu")
+        unit = dict(kind=_lib.DENSE_GLU, limit=clamp[0], slope=clamp[1]) if clamp else dict(kind=_lib.DENSE_SWIGLU)
+        if ops.grouped(h.buf[0], gate_up.buf, routes, act.buf[0], shared=routes.shared, **unit):
+            rt.launched("experts glu" if clamp else "experts swiglu")
         else:
             both = Tensor(rt, act.rows, 2 * m, dtype="fp32")
             ops.grouped_matmul(h.buf[0], gate_up.buf, routes, both.buf[0], routes.shared)
             rt.launched("experts matmul")
-            (both[:, :m].silu() * both[:, m:]).cast(h.dtype).realize(into=act)
+            gate, up = both[:, :m], both[:, m:]
+            (clamped_glu(gate, up, *clamp) if clamp else gate.silu() * up).cast(h.dtype).realize(into=act)
         if ops.grouped(act.buf[0], down.buf, routes, out.buf[0]):
             rt.launched("experts")
         else:
@@ -684,17 +716,20 @@ class Tensor:
             rt.launched("experts matmul")
         return out
 
-    def add_norm(self, w, eps, plus=0.0, dtype="bf16", mixer=None, mixer_scale=None, other=None, other_scale=None, experts=None):
-        """self: an fp32 residual stream.  (self + mixer * mixer_scale + (other + the experts' rows by their weights) *
-        other_scale, and that as RMSNorm by w + plus leaves it); experts: (rows, routes).  Without branches: (self, its norm)."""
+    def add_norm(self, w, eps, plus=0.0, dtype="bf16", mixer=None, mixer_scale=None, other=None, other_scale=None, experts=None,
+                 mixer_bias=None, own=None, into=None):
+        """self: an fp32 residual stream.  (self + (mixer + mixer_bias) * mixer_scale + (other + the experts' rows by their weights) *
+        other_scale, and that as RMSNorm by w + plus leaves it, or, w None, as it is); experts: (rows, routes), own: the row that an
+        identity expert gives back.  Without branches: (self, its norm).  into: where the second goes."""
         x = self.realize()
         get = lambda t: None if t is None else t.realize().buf[0]
         assert x.dtype == "fp32" and x.batch == 1 and all(t is None or (t.shape == x.shape and t.buf.stride(2) == 1) for t in (mixer and mixer.realize(), other and other.realize()))
-        bare = mixer is other is experts is None
-        out, h = x if bare else Tensor(self.rt, x.rows, x.cols, dtype="fp32"), Tensor(self.rt, x.rows, x.cols, dtype=dtype)
+        bare = mixer is other is experts is mixer_bias is None
+        out, h = x if bare else Tensor(self.rt, x.rows, x.cols, dtype="fp32"), into if into is not None else Tensor(self.rt, x.rows, x.cols, dtype=dtype)
+        assert h.shape == x.shape and h.dtype == dtype and h.buf.stride(2) == 1
         scale = lambda t: None if t is None else t.realize().buf
         rows, routes = experts or (None, None)
-        ops.add_norm(x.buf[0], None if bare else out.buf[0], get(mixer), scale(mixer_scale), get(other), scale(other_scale), get(rows), routes, w.realize().buf, plus, eps, h.buf[0])
+        ops.add_norm(x.buf[0], None if bare else out.buf[0], get(mixer), scale(mixer_scale), get(other), scale(other_scale), get(rows), routes, scale(w), plus, eps, h.buf[0], scale(mixer_bias), get(own))
         self.rt.launched("norm" if bare else "add norm")
         return out, h
 
@@ -718,6 +753,12 @@ class Tensor:
             return self
         _realize(self, into)
         return self
+
+
+def clamped_glu(gate, up, limit, slope):
+    """g sigmoid(slope g) (u + 1) with the gate's half cut at limit and the other within -limit .. limit."""
+    g, u = gate.minimum(limit), up.maximum(-limit).minimum(limit)
+    return g * (g * slope).sigmoid() * (u + 1)
 
 
 # -------------------------------------------------------------------- the planner
@@ -776,6 +817,16 @@ def _realize(t, into=None):
         part = out[:, :, :t.args["n"]]
         part.assign(part.silu())
         _done(t, buf=out.buf)
+    elif op == "gelu_gated":
+        mm, m = t.srcs[0], t.cols
+        bias = t.srcs[1].realize() if len(t.srcs) > 1 else None
+        half = lambda x, i: x[:, :, i * m:(i + 1) * m]
+        if mm.batch == 1 and _dense(t, mm, into, _lib.DENSE_GEGLU, gate_bias=bias and half(bias, 0), up_bias=bias and half(bias, 1)):
+            return
+        mm = mm.realize()
+        gate, up = (half(mm, i) + half(bias, i) if bias is not None else half(mm, i) for i in (0, 1))
+        out = (gate.gelu() * up).cast(t.dtype).realize(into=into)
+        return _done(t, buf=out.buf)
     elif op == "repeat":
         src, n = t.srcs[0].realize(), t.args["n"]
         out = Tensor(t.rt, t.rows, t.cols, batch=t.batch, dtype=t.dtype)
@@ -854,7 +905,7 @@ def _match_dyt(t):
 
 
 def _match_clamped_glu(t):
-    """(matmul, limit, slope) if t is mixers.clamped_glu over the halves of one matmul not yet computed, else None."""
+    """(matmul, limit, slope) if t is clamped_glu over the halves of one matmul not yet computed, else None."""
     if not (t.op == "mul" and all(isinstance(s, Tensor) for s in t.srcs)):
         return None
     act, plus = t.srcs
@@ -911,7 +962,7 @@ def _dense(t, mm, into, kind, **extra):
     a, w = mm.srcs
     if not (a.dtype == "bf16" and w.dtype == "bf16" and w.op is None and a.batch == w.batch and w.buf.stride(1) == 1 and w.rows % 8 == 0 and w.buf.stride(2) % 8 == 0):
         return False
-    if kind in (_lib.DENSE_GLU, _lib.DENSE_SWIGLU) and w.cols % 32:
+    if kind in (_lib.DENSE_GLU, _lib.DENSE_SWIGLU, _lib.DENSE_GEGLU) and w.cols % 32:
         return False
     x = a.realize()
     if not ops.dense_supports(x.buf, w.buf, kind):
@@ -930,7 +981,7 @@ def _dense(t, mm, into, kind, **extra):
         elif v is not None:
             fields[name] = v
     ops.dense(x.buf, w.buf, out.buf, getattr(w, "settled", False), kind=kind, **fields)
-    t.rt.launched("dense" + ("", " silu", " glu", " gate", " dyt add", " swiglu")[kind])
+    t.rt.launched("dense" + ("", " silu", " glu", " gate", " dyt add", " swiglu", " geglu")[kind])
     _done(t, buf=out.buf)
     if into is not None and out is not into:
         _copy(t, into)
