@@ -86,11 +86,11 @@ def test_dense_latent_and_decay_entry_points_refuse_bad_arguments_without_a_gpu(
     rc = lib.fb_dense(16, 4, 64, 64, 0, 16, 32, 64, 0, 1, 16, _lib.FP32, 32, 0, ctypes.byref(e), 0, None)
     assert rc == -1 and b"its vectors" in lib.fb_last_error()
     assert lib.fb_dense_supports(8, 64, 0, 16, 64, 0, 64, 32, _lib.DENSE_NONE) == 0, "a row of x that is not 16-byte aligned"
-    rc = lib.fb_latent_put(_lib.FP32, 16, 2, 100, 40, 40, 21, 8, 16, 16, 1e-5, 16, 1.0, 16, 16, _lib.BF16, 16, 40, 16, 64, None)
+    rc = lib.fb_latent_put(_lib.FP32, 16, 2, 100, 40, 40, 21, 8, 16, 16, 1e-5, 16, 1.0, 16, 16, _lib.BF16, 16, 40, 0, 0, None, 0, 0, 16, 64, None)
     assert rc == -1 and b"within the key part" in lib.fb_last_error()
     rc = lib.fb_rotate_pairs(_lib.BF16, 16, 2, 4, 64, 16, 16, 5, 16, 1.0, 16, 16, 64, 16, None)
     assert rc == -1 and b"even number" in lib.fb_last_error()
-    rc = lib.fb_latent_attention(_lib.BF16, 16, 2, 100, 4, 32, 8, 16, 64, 16, 0, 16, 64, 0, 1.0, None, 16, 128, None, 0, None)
+    rc = lib.fb_latent_attention(_lib.BF16, 16, 2, 100, 4, 32, 8, 16, 64, 16, 0, 16, 64, 0, 0, 1.0, None, 16, 128, None, 0, None)
     assert rc == -1 and b"row strides too small" in lib.fb_last_error()
     rc = lib.fb_decay_scan(_lib.BF16, 16, 4096, 2, 600, 64, 16, 16, -1, 1, 4, 16, 2 * 600 * 64, 16, 128, None)
     assert rc == -1 and b"up to 512" in lib.fb_last_error()
@@ -106,15 +106,15 @@ def test_heads_and_experts_entry_points_refuse_bad_arguments_without_a_gpu():
     assert rc == -1 and b"whole groups" in lib.fb_last_error()
     rc = lib.fb_heads_put(ctypes.byref(_lib.Heads(heads=4, kv_heads=2, dim=8, vdim=8)), _lib.BF16, 16, 4, 64, 16, _lib.FP32, 16, 32, 16, 64, 64 * 16, None)
     assert rc == -1 and b"fp32 results come from fp32" in lib.fb_last_error()
-    attend = lambda heads, dim, span, chunk=0, base=16: lib.fb_heads_attention(_lib.BF16, 16, 2, heads * dim, heads, 2, dim, 64, 16, 64, 64 * (dim + 64), base, 0, 16, 64, chunk, span, 1.0, None, 0,
+    attend = lambda heads, dim, span, chunk=0, base=16: lib.fb_heads_attention(_lib.BF16, 16, 2, heads * dim, heads, 2, dim, 64, 16, 64, 64 * (dim + 64), base, 0, 16, 64, chunk, span, 0, 1.0, 0.0, None, 0,
                                                                                None, 0, 16, heads * 64, None)
     assert attend(3, 64, 0) == -1 and b"whole groups" in lib.fb_last_error()
     assert attend(4, 2048, 0) == -1 and b"up to 1024" in lib.fb_last_error()
     assert attend(4, 64, -1) == -1 and attend(4, 64, 8, chunk=1) == -1 and b"one sequence's" in lib.fb_last_error()
     assert lib.fb_route_tiles(5, 10, 3, 16, 1) == 10 and lib.fb_route_tiles(1, 10, 3, 16, 1) == 3 and lib.fb_route_tiles(100, 10, 3, 32, 0) == 300 // 32 + 10
-    rc = lib.fb_route(16, 100, 10, None, 10, 3, 64, 1, 16, 16, 16, 16, 16, None)
+    rc = lib.fb_route(ctypes.byref(_lib.Router(10, 3, 0, None, 0, 1.0)), 16, 100, 10, 64, 1, 16, 16, 16, 16, 16, None)
     assert rc == -1 and b"all the tokens in one" in lib.fb_last_error()
-    rc = lib.fb_route(16, 4, 70, None, 70, 65, 16, 1, 16, 16, 16, 16, 16, None)
+    rc = lib.fb_route(ctypes.byref(_lib.Router(70, 65, 0, None, 0, 1.0)), 16, 4, 70, 16, 1, 16, 16, 16, 16, 16, None)
     assert rc == -1 and b"up to 64 choices" in lib.fb_last_error()
     e = _lib.DenseEpilogue(kind=_lib.DENSE_DYT_ADD)
     rc = lib.fb_dense_grouped(16, 64, 64, 64, 0, 16, 64, 64, 4096, 2, 16, 16, 2, 32, 16, _lib.BF16, 64, ctypes.byref(e), None)
@@ -125,5 +125,27 @@ def test_heads_and_experts_entry_points_refuse_bad_arguments_without_a_gpu():
     assert rc == -1 and b"rows there" in lib.fb_last_error()
     rc = lib.fb_add_norm(ctypes.byref(_lib.Branches(x=16)), 2, 64, _lib.BF16, _lib.BF16, None)
     assert rc == -1 and b"no result" in lib.fb_last_error()
-    rc = lib.fb_embed(_lib.BF16, 16, 8, 64, 16, 16, 0, None, 2, 16, None)
+    rc = lib.fb_embed(_lib.BF16, 16, 8, 64, 16, 16, 0, None, 2, 1.0, 16, None)
     assert rc == -1 and b"takes the places" in lib.fb_last_error()
+
+
+def test_turned_heads_windows_and_scored_routes_refuse_bad_arguments_without_a_gpu():
+    import ctypes
+    lib = _lib.lib()
+    put = lambda **h: lib.fb_heads_put(ctypes.byref(_lib.Heads(**dict(heads=4, kv_heads=2, dim=8, vdim=8) | h)), _lib.FP32, 16, 6, 64, 16, _lib.BF16, 16, 32, 16, 64, 64 * 16, None)
+    for h, what in ((dict(turned=10, freq=16, places=16), b"even number"), (dict(turned=4, freq=16), b"even number"), (dict(keys_are_values=1, vdim=4), b"as wide"), (dict(norm_all=1, q_norm=16), b"its weights"),
+                    (dict(conv=16, taps=3, places=16, sequences=1), b"its state"), (dict(conv=16, taps=3, state=16, places=16, sequences=4, state_stride=999), b"as many rows"),
+                    (dict(conv=16, taps=3, state=16, places=16, sequences=2, state_stride=64), b"as many rows"), (dict(norm_all=1, q_norm=16, k_norm=16, first=16, ld_first=16, share=16), b"plain heads")):
+        assert put(**h) == -1 and what in lib.fb_last_error(), h
+    put = lambda **a: lib.fb_latent_put(_lib.FP32, 16, 2, 200, a.get("q_rank", 0), 40, 8, 8, None, 16, 1e-5, 16, 1.0, 16, 16, _lib.BF16, 16, a.get("ld_q", 40), 5, 8, a.get("turned", 16), 240, 48, 16, 64, None)
+    assert put(turned=None) == -1 and b"both their parts" in lib.fb_last_error()
+    assert put(ld_q=39) == -1 and put(q_rank=8) == -1
+    attend = lambda window, cap: lib.fb_heads_attention(_lib.BF16, 16, 2, 128, 2, 2, 64, 64, 16, 64, 64 * 128, 16, 0, 16, 64, 0, 0, window, 1.0, cap, None, 0, None, 0, 16, 128, None)
+    assert attend(-1, 0.0) == -1 and attend(4, -1.0) == -1 and b"a cap of scores" in lib.fb_last_error()
+    rc = lib.fb_route(ctypes.byref(_lib.Router(10, 3, 10, None, 1, 1.0)), 16, 4, 10, 16, 1, 16, 16, 16, 16, 16, None)
+    assert rc == -1 and b"at least one expert" in lib.fb_last_error()
+    e = _lib.DenseEpilogue(kind=_lib.DENSE_GEGLU)
+    rc = lib.fb_dense(16, 4, 64, 64, 0, 16, 40, 64, 0, 1, 16, _lib.BF16, 32, 0, ctypes.byref(e), 0, None)
+    assert rc == -1 and b"whole runs of 16" in lib.fb_last_error()
+    rc = lib.fb_dense_grouped(16, 64, 64, 64, 0, 16, 64, 64, 4096, 2, 16, 16, 2, 32, 16, _lib.BF16, 64, ctypes.byref(e), None)
+    assert rc == -1 and b"a gated unit" in lib.fb_last_error()
