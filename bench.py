@@ -3,7 +3,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--workload llama8b|smollm] [--layers L] [--impl reference]
     python bench.py --matmul 32,4096,14336,bfp8,6      (one isolated matmul, a few calls: what the ncu captures run)
     python bench.py --attend 32,32,8,128,2048,6        (the decode attention alone, likewise)
-    python bench.py --design binutar|labepel           (prefill, decode and kernels of that design beside the Llama decoder)
+    python bench.py --design binutar|labepel|vunadra   (prefill, decode and kernels of that design beside the Llama decoder)
 
 The default workload is the Llama-3.1-8B-shape batched decode (32 sequences, 2048 tokens of context each, bfp8 weights,
 bf16 KV cache), tensor-parallel over N GPUs with an NCCL all-reduce after o_proj and down_proj.  A step is one decode
@@ -64,7 +64,7 @@ def parse():
     ap.add_argument("--sweep", type=int, default=1, help="0: leave the isolated matmul sweep out of the line (a profiling run)")
     ap.add_argument("--attend", default="", help="T,H,KV,hd,context[,calls]: only the decode attention, e.g. 32,32,8,128,2048,6")
     ap.add_argument("--matmul", default="", help="M,K,N,fmt[,calls]: only that isolated matmul (RMSNorm + SwiGLU fused), e.g. 32,4096,14336,bfp8,6")
-    ap.add_argument("--design", default="", help="binutar[:SIZE] or labepel[:SIZE]: instead of the workload, prefill and decode of that design at sizes like a real model's layers, "
+    ap.add_argument("--design", default="", help="binutar[:SIZE], labepel[:SIZE] or vunadra[:SIZE]: instead of the workload, prefill and decode of that design at sizes like a real model's layers, "
                                                  "and each of its kernels, beside the Llama decoder at equal size (one GPU)")
     return ap.parse_args()
 
@@ -425,6 +425,30 @@ LABEPEL_SIZES = {
 }
 
 
+# a layer of each kind - attention with a short convolution before a dense feed-forward, attention whose values are its keys and
+# attention over latents, both within a window, before a mixture - run twice in a loop; a Llama-like mixture of the same heads,
+# experts and layer runs beside it
+VUNADRA_SIZES = {
+    "4096": dict(width=4096, layers=6, vocab=32000, heads=32, kv=8, dim=128, vdim=128, conv=4, window=1024, rot_dim=64, kv_rank=512, experts=8, identity=1, top=2, ff=14336, dense=14336),
+    "2048": dict(width=2048, layers=6, vocab=32000, heads=32, kv=4, dim=128, vdim=128, conv=4, window=1024, rot_dim=64, kv_rank=512, experts=128, identity=8, top=8, ff=768, dense=6144),
+}
+
+
+def vunadra_models(s, places):
+    """(Vunadra config, Llama config of a mixture) of one size."""
+    from ferrite_b200 import llama, vunadra
+    heads, d = dict(heads=s["heads"], kv_heads=s["kv"], dim=s["dim"], vdim=s["vdim"], scale=s["dim"] ** -0.5), s["dim"]
+    mixture = dict(kind="moe", router=dict(experts=s["experts"], identity=s["identity"], top=s["top"], scale=1.0), expert=dict(ff=s["ff"], limit=7.0))
+    yarn, waves = dict(factor=4.0, original=4096, fast=32.0, slow=1.0), dict(factor=8.0, low=1.0, high=4.0, original=8192)
+    blocks = [dict(type="attention", mixer=heads | dict(conv=s["conv"], rot=dict(base=500000.0, dims=d, scaling=yarn)), mlp=dict(kind="dense", ff=s["dense"])),
+              dict(type="attention_2", mixer=heads | dict(mask=dict(size=s["window"]), softcap=30.0, rot=dict(base=500000.0, dims=d, scaling=waves)), mlp=mixture),
+              dict(type="latent_attention", mixer=dict(heads=s["heads"], dim=d, rot_dim=s["rot_dim"], vdim=s["vdim"], kv_rank=s["kv_rank"], mask=dict(size=s["window"]), scale=(d + s["rot_dim"]) ** -0.5,
+                                                       rot=dict(base=500000.0, dims=s["rot_dim"])), mlp=mixture)]
+    return (vunadra.model(vocab=s["vocab"], dim=s["width"], eps=1e-5, blocks=blocks, loop=dict(start=0, stop=3, times=s["layers"] // 3), places=places),
+            llama.model(dim=s["width"], heads=s["heads"], kv=s["kv"], head_dim=d, layers=s["layers"], vocab=s["vocab"], ffn=0, experts=s["experts"], k=s["top"], moe=s["ff"], theta=10000.0,
+                        eps=1e-5, places=places))
+
+
 def labepel_models(s, places):
     """(Labepel config, Llama config of a mixture) of one size."""
     from ferrite_b200 import labepel, llama
@@ -480,7 +504,7 @@ def design_steps(rt, c, prec, S, ctx, prompt, steps):
     part += -part % 64
     kv = family.kv_cache(c, S * part, llama.zeros(rt), S)
     gen = torch.Generator(device=rt.device).manual_seed(1)
-    for t in kv:  # (what the prompts would have left)
+    for t in [t for x in kv for t in (x if isinstance(x, tuple) else (x,))]:  # (what the prompts would have left)
         t.buf.normal_(0, 1, generator=gen)
     on = lambda row: Tensor.of(rt, [row], "int32")
     step = jit(lambda ids, at: llama.next_tokens(family.forward(ids, at, w, c, kv, S), c))
@@ -718,6 +742,99 @@ def labepel_kernels(rt, s, T, ctx, peaks):
     return rows
 
 
+def vunadra_kernels(rt, s, T, ctx, peaks):
+    """Each kernel of the Vunadra layers, as design_kernels does it."""
+    import torch
+    from ferrite_b200 import _lib, ops
+    dev, gen = rt.device, torch.Generator(device=rt.device).manual_seed(0)
+    f32 = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.float32).normal_(0, 1, generator=gen)
+    bf = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.bfloat16).normal_(0, 1, generator=gen)
+    ones = lambda n: f32_ones(dev, n)
+    rows, prompt = [], ctx == 0
+    d, H, G, dim, vd, E, k, ff, dff, rank, rd, window, taps = (s[n] for n in ("width", "heads", "kv", "dim", "vdim", "experts", "top", "ff", "dense", "kv_rank", "rot_dim", "window", "conv"))
+
+    def row(name, us, nbytes, flops=0.0, like=None):
+        floor = max(nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6)
+        rows.append({"kernel": name, "us": round(us, 2), "roofline_us": round(floor, 2), "frac": round(floor / us, 3)} | ({"like": like} if like else {}))
+
+    def dense(name, K, N, batch=1, kind=_lib.DENSE_NONE, out_dtype=torch.bfloat16, like="fb_linear"):
+        copies = max(1, min(16, int(3e8 // (2 * batch * K * N))))
+        ws, x, cols = [bf(batch, N, K) for _ in range(copies)], bf(T, batch, K).permute(1, 0, 2), N // 2 if kind == _lib.DENSE_GEGLU else N
+        out, b = torch.empty(T, batch, cols, device=dev, dtype=out_dtype).permute(1, 0, 2), ones(N)
+        extra = dict(gate_bias=b.data_ptr(), up_bias=b.data_ptr()) if kind == _lib.DENSE_GEGLU else {}
+        us = timed(40, copies, lambda i: ops.dense(x, ws[i].transpose(1, 2), out, True, kind, **extra))
+        row(f"fb_dense {name} {batch}x[{K}, {N}]" if batch > 1 else f"fb_dense {name} [{K}, {N}]", us, 2 * batch * K * N + 2 * T * batch * K + out.element_size() * T * batch * cols,
+            2.0 * T * batch * K * N, like)
+
+    qkv, qk, W = (H + G) * dim + G * vd, (H + G) * dim, rank + rd
+    dense("pass start", 2 * d, d, out_dtype=torch.float32)
+    dense("q, k, v", d, qkv, out_dtype=torch.float32)
+    dense("q, k", d, qk, out_dtype=torch.float32)
+    dense("q, dkv", d, H * (dim + rd) + W, out_dtype=torch.float32)
+    dense("uk by head", dim, rank, H)
+    dense("uv by head", rank, vd, H)
+    dense("o", H * vd, d)
+    dense("gate_up, gelu", d, 2 * dff, 1, _lib.DENSE_GEGLU)
+    dense("down", dff, d)
+    dense("router", d, E + s["identity"], out_dtype=torch.float32, like="router")
+    dense("head", d, s["vocab"], out_dtype=torch.float32)
+
+    keys = T if prompt else ctx
+    part, seqs = keys + -keys % 64, 1 if prompt else T
+    caches = [bf(G, seqs * part, dim + vd) for _ in range(4)]
+    last = torch.arange(T, device=dev, dtype=torch.int32) if prompt else torch.full((T,), ctx - 1, device=dev, dtype=torch.int32)
+    base = torch.arange(T, device=dev, dtype=torch.int32) * part
+    at, q, o, first = (last if prompt else base + last), bf(T, H * dim), bf(T, H * vd), None if prompt else base
+    joint, state, turn = f32(T, qkv), f32(seqs, taps - 1, qkv), (torch.ones(dim // 2, device=dev, dtype=torch.float64), dim, 1.0)
+    conv = f32(taps, qkv)
+    us = timed(40, 1, lambda i: ops.heads_put(joint, H, G, dim, vd, at, caches[0], q, rotation=turn, places=last, conv=conv, state=state, dead=-1))
+    row("fb_heads_put, convolution, turn", us, T * 6 * qkv + (seqs * 2 * (taps - 1) + taps) * qkv * 4, like="fb_rope_kv_write")
+    us = timed(40, 1, lambda i: ops.heads_put(joint, H, G, dim, dim, at, caches[0], q, ones(qk), ones(H * dim), ones(G * dim), 1e-5, norm_all=True, keys_are_values=True, rotation=turn, places=last))
+    row("fb_heads_put, joint norms, turn, keys as values", us, T * (4 * qk + 2 * (qk + G * dim)), like="fb_rope_kv_write")
+    within = min(window, keys)
+    seen = within * (within + 1) / 2 + max(0, T - within) * within if prompt else T * within
+    pairs = T * (T + 1) / 2 if prompt else T * ctx
+    us = timed(20, 4, lambda i: ops.heads_attention(q, caches[i], first, last, H, vd, 0.1, keys, prompt, out=o))
+    row("fb_heads_attention", us, 2 * (seqs * keys * G * (dim + vd) + T * H * (dim + vd)), 2.0 * pairs * H * (dim + vd), "attention")
+    us = timed(20, 4, lambda i: ops.heads_attention(q, caches[i], first, last, H, vd, 0.1, keys, prompt, out=o, window=window, softcap=30.0))
+    row(f"fb_heads_attention, window of {window}, capped", us, 2 * (seqs * (keys if prompt else within) * G * (dim + vd) + T * H * (dim + vd)), 2.0 * seen * H * (dim + vd), "attention")
+    us = timed(20, 4, lambda i: ops.heads_attention(q, caches[i], first, last, H, vd, 0.1, keys, prompt, out=o, softcap=30.0))
+    row("fb_heads_attention, no window, capped", us, 2 * (seqs * keys * G * (dim + vd) + T * H * (dim + vd)), 2.0 * pairs * H * (dim + vd), "attention")
+    lcaches, lq, lo = [bf(seqs * part, W) for _ in range(4)], bf(T, H * W), bf(T, H * rank)
+    down, plain, freq = f32(T, H * (dim + rd) + W), bf(T, H * dim), torch.ones(rd // 2, device=dev, dtype=torch.float64)
+    turned = lq.view(T, H, W).permute(1, 0, 2)[:, :, rank:]
+    us = timed(40, 1, lambda i: ops.latent_put(down, 0, rank, rd, rd, None, ones(rank), 1e-5, freq, 1.0, last, at, lcaches[0], plain, H, dim, turned))
+    row("fb_latent_put, queries", us, T * (H * (dim + rd) + W) * 6, like="fb_rope_kv_write")
+    us = timed(20, 4, lambda i: ops.latent_attention(lq, lcaches[i], first, last, H, rank, 0.1, None, keys, prompt, out=lo, window=window))
+    row(f"fb_latent_attention, window of {window}", us, 2 * (seqs * (keys if prompt else within) * W + T * H * (W + rank)), 2.0 * seen * H * (W + rank), "attention")
+    if prompt:  # (the same attention with keys and values made first)
+        row("fb_latent_attention, counted as keys and values of a head", us, 0, 2.0 * seen * H * (dim + rd + vd), "attention")
+
+    n = E + s["identity"]
+    logits = f32(T, n)
+    us = timed(40, 1, lambda i: ops.route(logits, n, k, ones(n), True, s["identity"], 1.0))
+    row("fb_route", us, T * (4 * n + 12 * k), like="fb_topk and fb_touched (fb_group)")
+    r = ops.route(logits, n, k, None, True, s["identity"], 1.0)
+    ids = [e for e in r.ids.cpu().reshape(-1).tolist() if e < E]
+    touched, live, choices = len(set(ids)), int(r.live), len(ids)
+    copies = max(1, min(4, int(3e8 // (6 * touched * d * ff)) + 1))
+    gate_up, down, h = [bf(E, 2 * ff, d).transpose(1, 2) for _ in range(copies)], [bf(E, d, ff).transpose(1, 2) for _ in range(copies)], bf(T, d)
+    x, act, y = bf(r.tiles * r.tile, d), bf(r.tiles * r.tile, ff), bf(r.tiles * r.tile, d)
+    if not r.shared:
+        us = timed(20, 1, lambda i: ops.spread_rows(h, r, x))
+        row("fb_spread_rows", us, 2 * (T + choices) * d, like="fb_gather_rows")
+    us = timed(20, copies, lambda i: ops.grouped(h if r.shared else x, gate_up[i], r, act, _lib.DENSE_GLU, r.shared, limit=7.0, slope=1.702))
+    row(f"fb_dense_grouped gate_up, clamped unit ({touched} experts, {live} tiles of {r.tile})", us, 4 * touched * d * ff + choices * 2 * (d + ff), 4.0 * choices * d * ff, "fb_linear_indexed")
+    us = timed(20, copies, lambda i: ops.grouped(act, down[i], r, y))
+    row("fb_dense_grouped down", us, 2 * touched * d * ff + choices * 2 * (d + ff), 2.0 * choices * d * ff, "fb_linear_indexed")
+    res, out, one = f32(T, d), f32(T, d), ones(d)
+    us = timed(40, 1, lambda i: ops.add_norm(res, out, chosen=y, routes=r, w=one, eps=1e-5, h=h, own=h))
+    row("fb_add_norm, chosen rows", us, T * d * (8 + 2 + 2 * k), like="fb_rmsnorm")
+    us = timed(40, 1, lambda i: ops.add_norm(res, out, o[:, :d] if H * vd >= d else h, w=one, eps=1e-5, h=h, mixer_bias=one))
+    row("fb_add_norm, bias", us, T * d * (8 + 2 + 2), like="fb_rmsnorm")
+    return rows
+
+
 def llama_expert_kernels(rt, s, T, peaks):
     """The Llama mixture's own kernels at the same size (bfp8 experts): its router's and its experts', decode or prompt."""
     import torch
@@ -773,8 +890,9 @@ def run_design(args):
     from ferrite_b200 import llama, models
     from ferrite_b200.tensor import Runtime
     name, _, size = args.design.partition(":")
-    assert name in ("binutar", "labepel") and args.gpus == 1, "--design binutar[:SIZE] or labepel[:SIZE], one GPU"
-    sizes, make, kernels = (DESIGN_SIZES, design_models, design_kernels) if name == "binutar" else (LABEPEL_SIZES, labepel_models, labepel_kernels)
+    designs = {"binutar": (DESIGN_SIZES, design_models, design_kernels), "labepel": (LABEPEL_SIZES, labepel_models, labepel_kernels), "vunadra": (VUNADRA_SIZES, vunadra_models, vunadra_kernels)}
+    assert name in designs and args.gpus == 1, "--design " + " or ".join(f"{n}[:SIZE]" for n in designs) + ", one GPU"
+    sizes, make, kernels = designs[name]
     rt, (peaks, kind), family = Runtime(0), measured_peaks(), models.module(name)
     S, ctx, prompt = 32, 2048, 2048
     for key in [size] if size else sizes:
@@ -789,7 +907,7 @@ def run_design(args):
         for what, T, at in (("decode", S, ctx), ("prefill", prompt, 0)):
             own = kernels(rt, s, T, at, peaks)
             torch.cuda.empty_cache()
-            like = llama_kernels(rt, s, T, at, peaks) + (llama_expert_kernels(rt, s, T, peaks) if name == "labepel" else [])
+            like = llama_kernels(rt, s, T, at, peaks) + (llama_expert_kernels(rt, s, T, peaks) if "experts" in s else [])
             line["kernels " + what] = {name: own, "llama": like}
             torch.cuda.empty_cache()
         line["clocks"] = clocks.summary()

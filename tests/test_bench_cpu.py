@@ -54,3 +54,12 @@ def test_labepel_models_are_of_equal_size():
         assert (b.dim, b.vocab, b.layers, b.positions) == (l.dim, l.vocab, l.layers, 512)
         e = b.blocks[0]
         assert (e.mixer.heads, e.mixer.kv_heads, e.mixer.dim, e.mlp.router.experts, e.mlp.router.top, e.mlp.expert.ff) == (l.heads, l.kv, l.head_dim, l.experts, l.k, l.moe)
+
+
+def test_vunadra_models_are_of_equal_size():
+    for s in bench.VUNADRA_SIZES.values():
+        b, l = bench.vunadra_models(s, 512)
+        assert (b.dim, b.vocab, len(b.runs)) == (l.dim, l.vocab, l.layers)
+        e = b.blocks[1]
+        assert (e.mixer.heads, e.mixer.kv_heads, e.mixer.dim, e.mlp.router.experts, e.mlp.router.top, e.mlp.expert.ff) == (l.heads, l.kv, l.head_dim, l.experts, l.k, l.moe)
+        assert [e.type for e in b.blocks] == ["attention", "attention_2", "latent_attention"]
