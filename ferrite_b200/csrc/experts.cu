@@ -33,7 +33,7 @@ __device__ __forceinline__ uint32_t ordered(float v) {
 }
 __device__ __forceinline__ float from_ordered(uint32_t b) { return __uint_as_float(b & 0x80000000u ? b & 0x7fffffffu : ~b); }
 
-// the k largest of a token's logits or scores, the lower column first among equals, and their weights: a warp a token.  Up to 128
+// the k largest of a token's logits or scores, the lower column first among equals, and their weights: a warp a token.  Up to 256
 // outputs: the lanes hold the logits as ordered numbers, 0 once picked
 __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int lane) {
   const float* z = a.logits + t * a.ld;
@@ -53,10 +53,10 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
     if (j < 32 && lane == j) mine[0] = v, my_id[0] = at;
     if (j >= 32 && lane == j - 32) mine[1] = v, my_id[1] = at;
   };
-  if (a.n <= 128) {
-    uint32_t held[4];
+  if (a.n <= 256) {
+    uint32_t held[8];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < 8; ++i) {
       const int c = 32 * i + lane;
       held[i] = c < a.n ? ordered(chosen_by(c)) : 0;
     }
@@ -64,13 +64,13 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
       uint32_t best = held[0];
       int at = lane;
 #pragma unroll
-      for (int i = 1; i < 4; ++i)
+      for (int i = 1; i < 8; ++i)
         if (held[i] > best) best = held[i], at = 32 * i + lane;
       const uint32_t top = __reduce_max_sync(0xffffffffu, best);
       at = __reduce_min_sync(0xffffffffu, best == top ? at : a.n);
       keep(j, from_ordered(top), at);
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+      for (int i = 0; i < 8; ++i)
         if (at == 32 * i + lane) held[i] = 0;
     }
   } else {

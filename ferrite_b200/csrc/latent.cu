@@ -29,6 +29,7 @@ struct LatentPutArgs {
   int heads, dim;  // heads > 0: the row begins with heads x (dim | rot) instead of a query latent
   void* q_turned;  // head h of token t at t * ld_turned + h * turned_head
   int64_t ld_turned, turned_head;
+  int per, fours;  // heads a block; all of that in whole, aligned groups of four columns
   void* cache;  // [cache_rows, kv_rank + rot]
   int64_t cache_rows;
 };
@@ -42,14 +43,37 @@ __global__ void __launch_bounds__(256) latent_put_kernel(const LatentPutArgs a) 
   const In* x = static_cast<const In*>(a.down) + t * a.ld;
   extern __shared__ float put_turns[];  // [dims / 2] cos, [dims / 2] sin
   const int half = a.dims / 2;
-  if (blockIdx.y == 0 && a.heads) {  // queries: the plain parts side by side, the others turned
-    for (int i = threadIdx.x; i < half; i += blockDim.x) turn_of(a.places[t], a.freq[i], a.mag, put_turns[i], put_turns[half + i]);
-    __syncthreads();
-    const int W = a.dim + a.rot, pairs = (a.rot + 1) / 2;
+  if (a.heads && blockIdx.y + 1 < gridDim.y) {  // queries: the plain parts side by side, the others turned
+    const int h0 = blockIdx.y * a.per, h1 = min(a.heads, h0 + a.per), W = a.dim + a.rot, pairs = (a.rot + 1) / 2, place = a.places[t];
     Act* plain = static_cast<Act*>(a.q_out) + t * a.ld_q;
-    for (int i = threadIdx.x; i < a.heads * a.dim; i += blockDim.x) store_value(plain + i, value_of(x[i / a.dim * W + i % a.dim]));
-    for (int j = threadIdx.x; j < a.heads * pairs; j += blockDim.x) {
-      const int h = j / pairs, i = j % pairs;
+    if (a.fours) {  // (a thread makes the turn of its own columns)
+      const int groups = W / 4;
+      for (int j = threadIdx.x; j < (h1 - h0) * groups; j += blockDim.x) {
+        const int h = h0 + j / groups, c = 4 * (j % groups);
+        float4 v = four(x + h * W + c);
+        if (c < a.dim) {
+          put_four(plain + h * a.dim + c, v);
+          continue;
+        }
+        const int r = c - a.dim;
+        float cs, sn;
+        if (r < a.dims) {
+          turn_of(place, a.freq[r / 2], a.mag, cs, sn);
+          v = make_float4(v.x * cs - v.y * sn, v.y * cs + v.x * sn, v.z, v.w);
+        }
+        if (r + 2 < a.dims) {
+          turn_of(place, a.freq[r / 2 + 1], a.mag, cs, sn);
+          v = make_float4(v.x, v.y, v.z * cs - v.w * sn, v.w * cs + v.z * sn);
+        }
+        put_four(static_cast<Act*>(a.q_turned) + t * a.ld_turned + h * a.turned_head + r, v);
+      }
+      return;
+    }
+    for (int i = threadIdx.x; i < half; i += blockDim.x) turn_of(place, a.freq[i], a.mag, put_turns[i], put_turns[half + i]);
+    __syncthreads();
+    for (int i = h0 * a.dim + threadIdx.x; i < h1 * a.dim; i += blockDim.x) store_value(plain + i, value_of(x[i / a.dim * W + i % a.dim]));
+    for (int j = threadIdx.x; j < (h1 - h0) * pairs; j += blockDim.x) {
+      const int h = h0 + j / pairs, i = j % pairs;
       const bool two = 2 * i + 1 < a.rot;
       const In* from = x + h * W + a.dim + 2 * i;
       Act* out = static_cast<Act*>(a.q_turned) + t * a.ld_turned + h * a.turned_head + 2 * i;
@@ -59,7 +83,7 @@ __global__ void __launch_bounds__(256) latent_put_kernel(const LatentPutArgs a) 
     }
     return;
   }
-  if (blockIdx.y == 0) {  // the query latent
+  if (blockIdx.y == 0 && !a.heads) {  // the query latent
     float ss = 0.f;
     for (int c = threadIdx.x; c < a.q_rank; c += blockDim.x) ss = fmaf(value_of(x[c]), value_of(x[c]), ss);
     const float r = 1.f / sqrtf(block_sum(ss, red) / (float)a.q_rank + a.eps);
@@ -203,10 +227,14 @@ extern "C" int fb_latent_put(int in_dtype, const void* down, int64_t T, int64_t 
   FB_REQUIRE(heads >= 0 && (heads == 0 || (q_rank == 0 && dim >= 1 && q_out && ld_q >= (int64_t)heads * dim && (rot == 0 || q_turned))), "fb_latent_put: queries take somewhere for both their parts, and no query latent");
   FB_REQUIRE(rot >= 0 && dims >= 0 && dims % 2 == 0 && dims <= rot && dims <= 8192 && ld >= q_rank + (int64_t)heads * (dim + rot) + kv_rank + rot && cache_rows >= 1, "fb_latent_put: the turned columns are an even number within the key part");
   FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32), "fb_latent_put: bf16 or fp32");
-  fb::LatentPutArgs a{down, ld, q_rank, kv_rank, rot, dims, q_norm, kv_norm, eps, freq, mag, places, rows, q_out, ld_q, heads, dim, q_turned, ld_turned, turned_head, cache, cache_rows};
+  fb::LatentPutArgs a{down, ld, q_rank, kv_rank, rot, dims, q_norm, kv_norm, eps, freq, mag, places, rows, q_out, ld_q, heads, dim, q_turned, ld_turned, turned_head, 0, 0, cache, cache_rows};
   const auto s = (cudaStream_t)stream;
   FB_REQUIRE(in_dtype == FB_FP32 || dtype == FB_BF16, "fb_latent_put: fp32 results come from fp32");
-  const dim3 grid((unsigned)T, 2), block(256);
+  auto whole = [](const void* p, int64_t ld, int64_t step, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0 && step % 4 == 0; };
+  const int in_bytes = in_dtype == FB_FP32 ? 4 : 2, bytes = dtype == FB_FP32 ? 4 : 2;
+  a.per = heads && 1024 / (dim + rot) > 1 ? 1024 / (dim + rot) : 1;
+  a.fours = dim % 4 == 0 && rot % 4 == 0 && whole(down, ld, 0, in_bytes) && whole(q_out, ld_q, 0, bytes) && whole(q_turned, ld_turned, turned_head, bytes);
+  const dim3 grid((unsigned)T, 1u + (heads ? (unsigned)fb::ceil_div(heads, a.per) : 1u)), block(256);
   const size_t smem = heads ? dims * sizeof(float) : 0;
   if (in_dtype == FB_FP32 && dtype == FB_FP32) return fb::launch_after(fb::latent_put_kernel<float, float>, grid, block, smem, s, "fb_latent_put", a);
   if (in_dtype == FB_FP32) return fb::launch_after(fb::latent_put_kernel<float, uint16_t>, grid, block, smem, s, "fb_latent_put", a);

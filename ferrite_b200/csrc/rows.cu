@@ -161,11 +161,27 @@ __global__ void __launch_bounds__(128) heads_put4_kernel(const HeadsPutArgs a) {
 // other block reads or writes it.
 struct HeadsTurnArgs {
   HeadsPutArgs p;
-  int per, tokens, first;  // units a block (joint norms: 0); tokens of a sequence, and how many of them its first block has
+  int per, tokens, first, group;  // units a block (joint norms: 0); tokens of a sequence, how many of them its first block has, and each other
 };
 
+// N values at p
+template <int N, typename T>
+__device__ __forceinline__ void read_some(const T* p, float v[N]) {
+  if constexpr (N == 4) {
+    const float4 f = four(p);
+    v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
+  } else {
+    v[0] = value_of(p[0]);
+  }
+}
+template <int N, typename T>
+__device__ __forceinline__ void put_some(T* p, const float v[N]) {
+  if constexpr (N == 4) put_four(p, make_float4(v[0], v[1], v[2], v[3]));
+  else store_value(p, v[0]);
+}
+
 template <typename In, typename Act, int N>  // N: columns a thread handles at a time, 4 (whole aligned groups) or 1
-__global__ void __launch_bounds__(256) heads_turn_kernel(const HeadsTurnArgs args) {
+__global__ void __launch_bounds__(512) heads_turn_kernel(const HeadsTurnArgs args) {
   griddep_launch_dependents();
   griddep_wait();
   extern __shared__ __align__(16) float turn_row[];  // the block's columns, then [turned / 2] cos and sin
@@ -178,8 +194,8 @@ __global__ void __launch_bounds__(256) heads_turn_kernel(const HeadsTurnArgs arg
   const int64_t c0 = column(u0), all = column(units);
   const int cols = (int)(column(u1) - c0);
   float *turns = turn_row + (cols + 3) / 4 * 4;
-  const int half = s.turned / 2, blocks = args.tokens - args.first + 1;
-  const int seq = blockIdx.x / blocks, b = blockIdx.x % blocks, begin = b ? args.first + b - 1 : 0, count = b ? 1 : args.first;
+  const int half = s.turned / 2, blocks = 1 + (args.tokens - args.first + args.group - 1) / args.group;
+  const int seq = blockIdx.x / blocks, b = blockIdx.x % blocks, begin = b ? args.first + (b - 1) * args.group : 0, count = b ? min(args.group, args.tokens - begin) : args.first;
   const int64_t row0 = (int64_t)seq * args.tokens;
   const int start = s.places ? s.places[row0] : 0;  // where the sequence's first token of this call stands
   const bool dead = s.conv && start == s.dead, held = s.conv && start != 0 && !dead;
@@ -189,15 +205,12 @@ __global__ void __launch_bounds__(256) heads_turn_kernel(const HeadsTurnArgs arg
   // N columns of the sequence's token i as projected, from the state where i < 0
   auto projected = [&](int i, int c, float v[N]) {
     if (i >= 0) {
-      if constexpr (N == 4) {
-        const float4 f = four(x + (int64_t)i * a.ld + c);
-        v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
-      } else {
-        v[0] = value_of(x[(int64_t)i * a.ld + c]);
-      }
+      read_some<N>(x + (int64_t)i * a.ld + c, v);
       if (s.bias) {
+        float bias[N];
+        read_some<N>(s.bias + c0 + c, bias);
 #pragma unroll
-        for (int e = 0; e < N; ++e) v[e] += s.bias[c0 + c + e];
+        for (int e = 0; e < N; ++e) v[e] += bias[e];
       }
     } else {
 #pragma unroll
@@ -217,11 +230,13 @@ __global__ void __launch_bounds__(256) heads_turn_kernel(const HeadsTurnArgs arg
       if (s.conv) {
 #pragma unroll
         for (int e = 0; e < N; ++e) v[e] = 0.f;
+#pragma unroll 4
         for (int j = 0; j < s.taps; ++j) {
-          float u[N];
+          float u[N], weight[N];
           projected(i - back + j, c, u);
+          read_some<N>(s.conv + j * all + c0 + c, weight);
 #pragma unroll
-          for (int e = 0; e < N; ++e) v[e] = fmaf(s.conv[j * all + c0 + c + e], u[e], v[e]);
+          for (int e = 0; e < N; ++e) v[e] = fmaf(weight[e], u[e], v[e]);
         }
       } else {
         projected(i, c, v);
@@ -235,7 +250,7 @@ __global__ void __launch_bounds__(256) heads_turn_kernel(const HeadsTurnArgs arg
     const float joint = s.norm_all ? 1.f / sqrtf(block_sum(ss, red) / (float)((blockIdx.y ? s.kv_heads : s.heads) * s.dim) + s.eps) : 1.f;
     __syncthreads();
     const bool inside = row >= 0 && row < a.cache_rows;  // nothing is written outside the cache
-    for (int u = u0 + warp; u < u1; u += 8) {
+    for (int u = u0 + warp; u < u1; u += blockDim.x / 32) {
       const bool is_q = u < s.heads, is_v = u >= keys;
       const int n = is_v ? s.vdim : s.dim, g = is_q ? u : is_v ? u - keys : u - s.heads;
       if (!is_q && !inside) continue;
@@ -250,20 +265,30 @@ __global__ void __launch_bounds__(256) heads_turn_kernel(const HeadsTurnArgs arg
       }
       Act* cached = static_cast<Act*>(a.cache) + g * a.head_stride + row * (s.dim + s.vdim);
       Act* out = is_q ? static_cast<Act*>(a.q_out) + t * a.ld_q + (int64_t)g * s.dim : is_v ? cached + s.dim : cached;
-      auto normed = [&](int c) { return w ? mine[c] * r * w[c] : mine[c]; };
-      auto result = [&](int c) {
-        if (is_v || c >= s.turned) return normed(c);
-        const float own = normed(c), other = normed(c ^ 1), cs = turns[c >> 1], sn = turns[half + (c >> 1)];
-        return c & 1 ? own * cs + other * sn : own * cs - other * sn;
-      };
       for (int c = N * lane; c < n; c += 32 * N) {
-        if constexpr (N == 4) {
-          put_four(out + c, make_float4(result(c), result(c + 1), result(c + 2), result(c + 3)));
-          if (s.keys_are_values && !is_q) put_four(cached + s.dim + c, make_float4(mine[c], mine[c + 1], mine[c + 2], mine[c + 3]));
-        } else {
-          store_value(out + c, result(c));
-          if (s.keys_are_values && !is_q) store_value(cached + s.dim + c, mine[c]);
+        float v[N];
+        read_some<N>(mine + c, v);
+        if (s.keys_are_values && !is_q) put_some<N>(cached + s.dim + c, v);
+        if (w) {
+          float g4[N];
+          read_some<N>(w + c, g4);
+#pragma unroll
+          for (int e = 0; e < N; ++e) v[e] *= r * g4[e];
         }
+        if (!is_v && c < s.turned) {
+          if constexpr (N == 4) {
+#pragma unroll
+            for (int e = 0; e < 4; e += 2)
+              if (c + e < s.turned) {
+                const float cs = turns[(c + e) / 2], sn = turns[half + (c + e) / 2], x0 = v[e], x1 = v[e + 1];
+                v[e] = x0 * cs - x1 * sn, v[e + 1] = x1 * cs + x0 * sn;
+              }
+          } else {
+            const float other = mine[c ^ 1] * (w ? r * w[c ^ 1] : 1.f), cs = turns[c >> 1], sn = turns[half + (c >> 1)];
+            v[0] = c & 1 ? v[0] * cs + other * sn : v[0] * cs - other * sn;
+          }
+        }
+        put_some<N>(out + c, v);
       }
     }
     __syncthreads();
@@ -281,7 +306,7 @@ __global__ void __launch_bounds__(256) heads_turn_kernel(const HeadsTurnArgs arg
 template <typename In, typename Act>
 static int launch_heads_turn(const HeadsPutArgs& a, cudaStream_t s) {
   const fb_heads& h = a.h;
-  HeadsTurnArgs t{a, 0, 1, 1};
+  HeadsTurnArgs t{a, 0, 1, 1, 1};
   const int units = h.heads + (h.keys_are_values ? 1 : 2) * h.kv_heads, wide = h.dim > h.vdim ? h.dim : h.vdim;
   unsigned parts = 2;
   int64_t most = (int64_t)(h.heads > 2 * h.kv_heads ? h.heads : 2 * h.kv_heads) * wide;
@@ -294,17 +319,19 @@ static int launch_heads_turn(const HeadsPutArgs& a, cudaStream_t s) {
   int64_t grid = a.T;
   if (h.conv) {
     t.tokens = (int)(a.T / h.sequences), t.first = h.taps - 1 < 1 ? 1 : h.taps - 1 < t.tokens ? h.taps - 1 : t.tokens;
-    grid = (int64_t)h.sequences * (t.tokens - t.first + 1);
+    while (t.group < 8 && ceil_div(a.T, 2 * t.group) * parts >= 8 * 148) t.group *= 2;  // (a block's next token finds the weights and the rows before it near)
+    grid = (int64_t)h.sequences * (1 + ceil_div(t.tokens - t.first, t.group));
   }
   auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
-  const bool fours = h.dim % 4 == 0 && h.vdim % 4 == 0 && whole(a.qkv, a.ld, sizeof(In)) && whole(a.q_out, a.ld_q, sizeof(Act)) && whole(a.cache, a.head_stride, sizeof(Act));
+  const bool fours = h.dim % 4 == 0 && h.vdim % 4 == 0 && whole(a.qkv, a.ld, sizeof(In)) && whole(a.q_out, a.ld_q, sizeof(Act)) && whole(a.cache, a.head_stride, sizeof(Act)) &&
+                     whole(h.bias, 0, 4) && whole(h.conv, 0, 4) && whole(h.q_norm, 0, 4) && whole(h.k_norm, 0, 4);
   static std::atomic<uint64_t> opted{0};
   if (first_on_device(opted)) {
     cudaFuncSetAttribute(heads_turn_kernel<In, Act, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     cudaFuncSetAttribute(heads_turn_kernel<In, Act, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   }
-  const dim3 g((unsigned)grid, parts);
-  return fours ? launch_after(heads_turn_kernel<In, Act, 4>, g, dim3(256), smem, s, "fb_heads_put", t) : launch_after(heads_turn_kernel<In, Act, 1>, g, dim3(256), smem, s, "fb_heads_put", t);
+  const dim3 g((unsigned)grid, parts), block(most > 1024 && h.norm_all ? 512 : 256);
+  return fours ? launch_after(heads_turn_kernel<In, Act, 4>, g, block, smem, s, "fb_heads_put", t) : launch_after(heads_turn_kernel<In, Act, 1>, g, block, smem, s, "fb_heads_put", t);
 }
 
 template <typename In, typename Act>
