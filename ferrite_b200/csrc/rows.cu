@@ -190,9 +190,8 @@ __global__ void __launch_bounds__(512) heads_turn_kernel(const HeadsTurnArgs arg
   const fb_heads& s = a.h;
   const int keys = s.heads + s.kv_heads, units = s.keys_are_values ? keys : keys + s.kv_heads;
   const int u0 = args.per ? blockIdx.y * args.per : blockIdx.y ? s.heads : 0, u1 = args.per ? min(units, u0 + args.per) : blockIdx.y ? units : s.heads;
-  auto column = [&](int u) { return (int64_t)min(u, keys) * s.dim + (int64_t)max(u - keys, 0) * s.vdim; };
-  const int64_t c0 = column(u0), all = column(units);
-  const int cols = (int)(column(u1) - c0);
+  auto column = [&](int u) { return min(u, keys) * s.dim + max(u - keys, 0) * s.vdim; };  // (fewer than 2^30 columns, the caller has seen to it)
+  const int c0 = column(u0), all = column(units), cols = column(u1) - c0, key_cols = column(keys) - c0;
   float *turns = turn_row + (cols + 3) / 4 * 4;
   const int half = s.turned / 2, blocks = 1 + (args.tokens - args.first + args.group - 1) / args.group;
   const int seq = blockIdx.x / blocks, b = blockIdx.x % blocks, begin = b ? args.first + (b - 1) * args.group : 0, count = b ? min(args.group, args.tokens - begin) : args.first;
@@ -242,10 +241,9 @@ __global__ void __launch_bounds__(512) heads_turn_kernel(const HeadsTurnArgs arg
         projected(i, c, v);
       }
 #pragma unroll
-      for (int e = 0; e < N; ++e) {
-        turn_row[c + e] = v[e];
-        if (c0 + c + e < column(keys)) ss = fmaf(v[e], v[e], ss);  // (joint norms: a block's query heads, or its key heads)
-      }
+      for (int e = 0; e < N; ++e)
+        if (s.norm_all && c + e < key_cols) ss = fmaf(v[e], v[e], ss);  // (a block's query heads, or its key heads)
+      put_some<N>(turn_row + c, v);
     }
     const float joint = s.norm_all ? 1.f / sqrtf(block_sum(ss, red) / (float)((blockIdx.y ? s.kv_heads : s.heads) * s.dim) + s.eps) : 1.f;
     __syncthreads();
@@ -503,6 +501,7 @@ extern "C" int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void
   const fb_heads& h = *heads_host;
   FB_REQUIRE(h.heads >= 1 && h.kv_heads >= 1 && h.heads % h.kv_heads == 0 && h.heads <= 100000 && h.dim >= 1 && h.vdim >= 1, "fb_heads_put: whole groups of query heads per key head (got %d / %d)", h.heads, h.kv_heads);
   const int64_t cols = (int64_t)(h.heads + h.kv_heads) * h.dim + (h.keys_are_values ? 0 : (int64_t)h.kv_heads * h.vdim);
+  FB_REQUIRE(cols < (1 << 30), "fb_heads_put: too many columns");
   FB_REQUIRE(!h.keys_are_values || h.vdim == h.dim, "fb_heads_put: values that are keys are as wide");
   FB_REQUIRE(h.turned >= 0 && h.turned % 2 == 0 && h.turned <= h.dim && (!h.turned || (h.freq && h.places)), "fb_heads_put: an even number of a head's columns turn, by frequencies and places");
   FB_REQUIRE(!h.conv || (h.taps >= 1 && h.state && h.places && h.sequences >= 1 && T % h.sequences == 0 && (h.sequences == 1 || h.state_stride >= (h.taps - 1) * cols)),
