@@ -152,8 +152,8 @@ def test_a_token_is_felt_to_the_end_of_its_window_and_no_further(rt, loaded, l, 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_a_convolution_reaches_back_over_portions(rt, loaded, dtype):
-    # keys, queries and values of one layer without attention to tell: what a token's convolution reads of the tokens before it,
-    # wherever a portion begins, and nothing of the sequence that had the slot before
+    # a portion's first tokens are convolved with the last ones of the portion before, wherever it begins, and a sequence's first
+    # tokens with nothing of the sequence that had the slot before
     cfg, raw, run = replay(rt, loaded, "mixed", dtype)
     ids, other = tokens(cfg, 30, 21), tokens(cfg, 30, 22)
     want = models.Alone(cfg, raw)(ids)
