@@ -16,32 +16,44 @@ LINEAR_AUTO, LINEAR_TCGEN05, LINEAR_GEMV, LINEAR_MMA, LINEAR_PERSISTENT, LINEAR_
 
 _p, _i, _i64, _f, _sz = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_float, ctypes.c_size_t
 
-DENSE_NONE, DENSE_SILU, DENSE_GLU, DENSE_GATE, DENSE_DYT_ADD, DENSE_SWIGLU, DENSE_GEGLU = 0, 1, 2, 3, 4, 5, 6  # fb_dense_epilogue_kind
+DENSE_NONE, DENSE_SILU, DENSE_GLU, DENSE_GATE, DENSE_DYT_ADD, DENSE_SWIGLU, DENSE_GEGLU, DENSE_RELU2 = 0, 1, 2, 3, 4, 5, 6, 7  # fb_dense_epilogue_kind
 
 
 class DenseEpilogue(ctypes.Structure):
     """fb_dense_epilogue of include/ferrite_b200.h, field by field."""
     _fields_ = [("kind", _i), ("act_cols", _i64), ("limit", _f), ("slope", _f), ("gate", _p), ("ld_gate", _i64), ("residual", _p), ("ld_residual", _i64),
-                ("alpha", _p), ("w", _p), ("b", _p), ("h_out", _p), ("ld_h", _i64), ("alpha2", _p), ("w2", _p), ("b2", _p), ("gate_bias", _p), ("up_bias", _p)]
+                ("alpha", _p), ("w", _p), ("b", _p), ("h_out", _p), ("ld_h", _i64), ("alpha2", _p), ("w2", _p), ("b2", _p), ("gate_bias", _p), ("up_bias", _p), ("row_scale", _p)]
 
 
 class Heads(ctypes.Structure):
     """fb_heads, likewise."""
     _fields_ = [("heads", _i), ("kv_heads", _i), ("dim", _i), ("vdim", _i), ("bias", _p), ("q_norm", _p), ("k_norm", _p), ("eps", _f), ("first", _p), ("ld_first", _i64),
                 ("first_bias", _p), ("share", _p), ("norm_all", _i), ("keys_are_values", _i), ("turned", _i), ("freq", _p), ("mag", _f), ("places", _p), ("taps", _i), ("conv", _p),
-                ("state", _p), ("state_stride", _i64), ("sequences", _i), ("dead", _i)]
+                ("state", _p), ("state_stride", _i64), ("sequences", _i), ("dead", _i), ("temp_coef", _f), ("temp_every", _f)]
 
 
 class Router(ctypes.Structure):
     """fb_router, likewise."""
-    _fields_ = [("n", _i), ("k", _i), ("identity", _i), ("bias", _p), ("scored", _i), ("scale", _f)]
+    _fields_ = [("n", _i), ("k", _i), ("identity", _i), ("bias", _p), ("scored", _i), ("scale", _f), ("as_scored", _i)]
 
 
 class Branches(ctypes.Structure):
     """fb_branches, likewise."""
     _fields_ = [("x", _p), ("ld_x", _i64), ("mixer", _p), ("ld_mixer", _i64), ("mixer_scale", _p), ("other", _p), ("ld_other", _i64), ("other_scale", _p), ("chosen", _p),
                 ("ld_chosen", _i64), ("slots", _p), ("weights", _p), ("k", _i), ("x_out", _p), ("ld_x_out", _i64), ("w", _p), ("plus", _f), ("eps", _f), ("h", _p), ("ld_h", _i64),
-                ("mixer_bias", _p), ("own", _p), ("ld_own", _i64)]
+                ("mixer_bias", _p), ("own", _p), ("ld_own", _i64), ("gate", _p), ("ld_gate", _i64), ("gate_bias", _p), ("post", _p)]
+
+
+class Conv(ctypes.Structure):
+    """fb_conv, likewise."""
+    _fields_ = [("cols", _i64), ("taps", _i), ("w", _p), ("bias", _p), ("in_bias", _p), ("silu", _i), ("places", _p), ("dead", _i), ("sequences", _i64), ("tokens", _i64), ("state", _p),
+                ("state_stride", _i64)]
+
+
+class Lru(ctypes.Structure):
+    """fb_lru, likewise."""
+    _fields_ = [("width", _i64), ("blocks", _i), ("lam", _p), ("rate", _f), ("gate_bias", _p), ("y_bias", _p), ("scale", _f), ("places", _p), ("dead", _i), ("sequences", _i64), ("tokens", _i64),
+                ("state", _p), ("state_stride", _i64)]
 
 
 # name -> (restype, argtypes); one entry per declaration in include/ferrite_b200.h
@@ -87,15 +99,18 @@ SIGNATURES = {
     "fb_latent_attention_workspace_bytes": (_sz, [_i, _i64, _i, _i, _i, _i64, _i, _i]),
     "fb_latent_attention": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _p, _i64, _p, _i64, _p, _i64, _i, _i, _f, _p, _p, _i64, _p, _sz, _p]),
     "fb_decay_scan": (_i, [_i, _p, _i64, _i, _i, _i, _p, _p, _i, _i64, _i64, _p, _i64, _p, _i64, _p]),
-    "fb_gated_rmsnorm": (_i, [_p, _i64, _i64, _i64, _i, _p, _i64, _p, _f, _p, _i64, _p]),
+    "fb_selective_scan": (_i, [_i, _p, _i64, _i, _i, _i, _i, _p, _i64, _p, _p, _p, _p, _i, _i64, _i64, _p, _i64, _p, _i64, _p]),
+    "fb_gated_rmsnorm": (_i, [_p, _i64, _i64, _i64, _i, _p, _i64, _i, _p, _f, _i, _i, _p, _i64, _p]),
+    "fb_short_conv": (_i, [_p, _i, _p, _i64, _i, _p, _i64, _p]),
+    "fb_lru_scan": (_i, [_p, _i, _p, _i64, _p, _i64, _i, _p, _i64, _p, _i64, _p]),
     "fb_dense_grouped": (_i, [_p, _i64, _i64, _i64, _i, _p, _i64, _i64, _i64, _i, _p, _p, _i64, _i, _p, _i, _i64, _p, _p]),
     "fb_route_tiles": (_i64, [_i64, _i, _i, _i, _i]),
-    "fb_route": (_i, [_p, _p, _i64, _i64, _i, _i, _p, _p, _p, _p, _p, _p]),
+    "fb_route": (_i, [_p, _p, _i64, _i64, _i, _i, _p, _p, _p, _p, _p, _p, _p]),
     "fb_spread_rows": (_i, [_p, _i64, _i64, _i64, _p, _i, _p, _i64, _p]),
-    "fb_grouped_matmul": (_i, [_i, _p, _i64, _i64, _i, _i, _p, _p, _i, _i64, _i64, _p, _p, _i64, _i, _i, _p, _i64, _p]),
+    "fb_grouped_matmul": (_i, [_i, _p, _i64, _i64, _i, _i, _p, _p, _i, _i64, _i64, _p, _p, _i64, _i, _p, _i, _p, _i64, _p]),
     "fb_embed": (_i, [_i, _p, _i64, _i64, _p, _p, _i64, _p, _i64, _f, _p, _p]),
     "fb_heads_put": (_i, [_p, _i, _p, _i64, _i64, _p, _i, _p, _i64, _p, _i64, _i64, _p]),
-    "fb_heads_attention": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _i, _p, _i64, _i64, _p, _i64, _p, _i64, _i, _i, _i, _f, _f, _p, _i, _p, _i64, _p, _i64, _p]),
+    "fb_heads_attention": (_i, [_i, _p, _i64, _i64, _i, _i, _i, _i, _p, _i64, _i64, _p, _i64, _p, _i64, _i, _i, _i, _f, _f, _p, _p, _f, _i, _p, _i64, _p, _i64, _p]),
     "fb_add_norm": (_i, [_p, _i64, _i64, _i, _i, _p]),
     "fb_peer_reduce_add": (_i, [_p, _p, _i, _i, _p, _i64, _p, _p, _p]),
 }

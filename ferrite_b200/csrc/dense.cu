@@ -14,8 +14,8 @@
 // the tiles are too few to fill the GPU, K is split over the CTAs of a cluster (2, 4 or 8): each leaves its sums in shared
 // memory, each then takes a share of the tokens and adds the others' sums to its own in rank order (the same every run).
 //
-// What follows a matmul in its model runs on the accumulators (fb_dense_epilogue): SiLU on the first columns, a clamped
-// or a GELU-gated unit (gate and up rows alternate in runs of 16 inside a tile, so a pair is 16 lanes apart), a gate per head, and the
+// What follows a matmul in its model runs on the accumulators (fb_dense_epilogue): SiLU on the first columns, a squared
+// ReLU, a clamped or a GELU-gated unit (gate and up rows alternate in runs of 16 inside a tile, so a pair is 16 lanes apart), a gate per head, and the
 // Dynamic Tanh - residual add - Dynamic Tanh between two branches, which needs no sum over the row and therefore no
 // kernel of its own.  Every wait is bounded (sm100.cuh).
 //
@@ -102,6 +102,13 @@ __device__ __forceinline__ void emit(const DenseParams& p, const Column& c, int 
   if constexpr (EPI == FB_DENSE_SILU) {
     if (n < p.e.act_cols) v = __fdividef(v, 1.f + __expf(-v));
   }
+  if constexpr (EPI == FB_DENSE_GLU || EPI == FB_DENSE_RELU2) {
+    if (p.e.row_scale) {
+      const float s = p.e.row_scale[t];
+      v *= s, up *= s;
+    }
+  }
+  if constexpr (EPI == FB_DENSE_RELU2) v = fmaxf(v, 0.f), v *= v;
   if constexpr (EPI == FB_DENSE_GLU) {
     const float g = fminf(v, p.e.limit), u = fminf(fmaxf(up, -p.e.limit), p.e.limit);
     v = g / (1.f + __expf(-p.e.slope * g)) * (u + p.shift);
@@ -375,6 +382,7 @@ static int run_dense(fb::DenseParams& p, const void* x, int64_t x_rows, int64_t 
     case FB_DENSE_SILU: return launch_dense<FB_DENSE_SILU>(tw, tx, p, grid, smem, s);
     case FB_DENSE_GLU: return launch_dense<FB_DENSE_GLU>(tw, tx, p, grid, smem, s);
     case FB_DENSE_GEGLU: return launch_dense<FB_DENSE_GEGLU>(tw, tx, p, grid, smem, s);
+    case FB_DENSE_RELU2: return launch_dense<FB_DENSE_RELU2>(tw, tx, p, grid, smem, s);
     case FB_DENSE_GATE: return launch_dense<FB_DENSE_GATE>(tw, tx, p, grid, smem, s);
     case FB_DENSE_DYT_ADD: return launch_dense<FB_DENSE_DYT_ADD>(tw, tx, p, grid, smem, s);
     default: return launch_dense<FB_DENSE_NONE>(tw, tx, p, grid, smem, s);
@@ -393,7 +401,7 @@ extern "C" int fb_dense(const void* x, int64_t M, int64_t K, int64_t ldx, int64_
   using namespace fb;
   FB_REQUIRE(x && W && out && M >= 1 && batch >= 1 && M < (1 << 30) && N < (1 << 30), "fb_dense: null pointer or empty");
   fb_dense_epilogue e = epilogue_host ? *epilogue_host : fb_dense_epilogue{};
-  FB_REQUIRE(e.kind >= FB_DENSE_NONE && e.kind <= FB_DENSE_GEGLU, "fb_dense: unknown epilogue %d", e.kind);
+  FB_REQUIRE(e.kind >= FB_DENSE_NONE && e.kind <= FB_DENSE_RELU2, "fb_dense: unknown epilogue %d", e.kind);
   const float shift = settle_unit(e);
   FB_REQUIRE(K >= 8 && K % 8 == 0 && ldx % 8 == 0 && ldw % 8 == 0 && x_batch % 8 == 0 && w_batch % 8 == 0 && ldx >= K && ldw >= K && (uintptr_t)x % 16 == 0 &&
                  (uintptr_t)W % 16 == 0 && N >= 1,
@@ -425,7 +433,8 @@ extern "C" int fb_dense_grouped(const void* x, int64_t x_rows, int64_t K, int64_
   using namespace fb;
   FB_REQUIRE(x && W && out && tile_expert && live && tiles >= 1 && n >= 1 && x_rows >= 1 && tiles * tile < (1 << 30) && N < (1 << 30), "fb_dense_grouped: null pointer or empty");
   fb_dense_epilogue e = epilogue_host ? *epilogue_host : fb_dense_epilogue{};
-  FB_REQUIRE(e.kind == FB_DENSE_NONE || e.kind == FB_DENSE_GLU || e.kind == FB_DENSE_SWIGLU, "fb_dense_grouped: plain, or a gated unit");
+  FB_REQUIRE(e.kind == FB_DENSE_NONE || e.kind == FB_DENSE_GLU || e.kind == FB_DENSE_SWIGLU || e.kind == FB_DENSE_RELU2, "fb_dense_grouped: plain, a gated unit or a squared ReLU");
+  FB_REQUIRE(!e.row_scale || e.kind != FB_DENSE_NONE, "fb_dense_grouped: weights on the input of a unit take one");
   FB_REQUIRE(tile >= 16 && tile <= 256 && tile % 16 == 0 && (shared_rows ? x_rows <= tile : x_rows >= tiles * tile), "fb_dense_grouped: tiles of 16 to 256 rows, all of them there");
   FB_REQUIRE(fb_dense_supports(x, ldx, 0, W, ldw, n > 1 ? w_batch : 0, K, N, e.kind), "fb_dense_grouped: rows of x and W 16-byte aligned, K a multiple of 8, a gated unit's halves whole runs of 16");
   FB_REQUIRE(out_dtype == FB_BF16 || out_dtype == FB_FP32, "fb_dense_grouped: out is bf16 or fp32");

@@ -1,5 +1,5 @@
 // A mixture of experts around its matmuls, for weights kept as bf16 or fp32:
-//   fb_route            router logits -> each token's k largest (by logit, or by corrected score), their weights, and where each
+//   fb_route            router logits -> each token's k largest (by logit, or by softmax or sigmoid score), their weights, and where each
 //                       choice's row goes (an identity expert's: nowhere): the touched experts' rows in whole tiles, a list of the tiles' experts, how many there are
 //   fb_spread_rows      the tokens' rows to their choices' places
 //   fb_grouped_matmul   rows of tiles by each tile's own matrix, any sizes, bf16 or fp32 (the tensor cores' form: fb_dense_grouped)
@@ -16,14 +16,16 @@ struct RouteArgs {
   int64_t T, ld;
   const float* bias;  // [n] or null
   int n, k, tile, shared;
-  int real, scored;  // outputs 0 .. real - 1 are experts with rows
+  int real, scored;  // outputs 0 .. real - 1 are experts with rows; scored: 1 softmax, 2 sigmoid
   float scale;
+  int as_scored;     // the weights are the scores, not over their sum
   int tiles;  // entries of tile_expert
   float* weights;       // [T, k]
   int32_t* ids;         // [T, k]
   int32_t* slots;       // [T, k]: the row of each choice
   int32_t* tile_expert; // [tiles, 3]: a tile's expert (n past those used), its expert's first tile and how many it has
   int32_t* live;        // [1] tiles used
+  float* row_weights;   // each choice's weight at its row, or null
 };
 
 // a float as a number that orders like it (-0 as 0), above 0 for all of them
@@ -39,8 +41,8 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
   const float* z = a.logits + t * a.ld;
   float mine[2] = {-INFINITY, -INFINITY};  // lane j keeps the picks j and 32 + j
   int my_id[2] = {0, 0};
-  float most = 0.f, norm = 1.f;  // scored: a score is exp(z - most) * norm
-  if (a.scored) {
+  float most = 0.f, norm = 1.f;  // scored by softmax: a score is exp(z - most) * norm
+  if (a.scored == 1) {
     most = -INFINITY;
     for (int c = lane; c < a.n; c += 32) most = fmaxf(most, z[c]);
     most = warp_max(most);
@@ -48,7 +50,9 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
     for (int c = lane; c < a.n; c += 32) sum += expf(z[c] - most);
     norm = 1.f / warp_sum(sum);
   }
-  auto chosen_by = [&](int c) { return (a.scored ? expf(z[c] - most) * norm : z[c]) + (a.bias ? a.bias[c] : 0.f); };
+  auto score = [&](int c) { return a.scored == 1 ? expf(z[c] - most) * norm : sigmoid_f(z[c]); };
+  // (sigmoids without a correction order as their logits do, which are never equal where those are not)
+  auto chosen_by = [&](int c) { return (a.scored == 1 || (a.scored == 2 && a.bias) ? score(c) : z[c]) + (a.bias ? a.bias[c] : 0.f); };
   auto keep = [&](int j, float v, int at) {
     if (j < 32 && lane == j) mine[0] = v, my_id[0] = at;
     if (j >= 32 && lane == j - 32) mine[1] = v, my_id[1] = at;
@@ -95,8 +99,8 @@ __device__ __forceinline__ void route_token(const RouteArgs& a, int64_t t, int l
     }
   }
   const float top = __shfl_sync(0xffffffffu, mine[0], 0);
-  auto weight = [&](int i) { return lane + 32 * i >= a.k ? 0.f : a.scored ? expf(z[min(my_id[i], a.n - 1)] - most) * norm : expf(mine[i] - top); };
-  const float e0 = weight(0), e1 = weight(1), sum = warp_sum(e0 + e1) + (a.scored ? 1e-20f : 0.f);
+  auto weight = [&](int i) { return lane + 32 * i >= a.k ? 0.f : a.scored ? score(min(my_id[i], a.n - 1)) : expf(mine[i] - top); };
+  const float e0 = weight(0), e1 = weight(1), sum = a.as_scored ? 1.f : warp_sum(e0 + e1) + (a.scored ? 1e-20f : 0.f);
   if (lane < a.k) a.weights[t * a.k + lane] = e0 / sum * a.scale, a.ids[t * a.k + lane] = my_id[0];
   if (lane + 32 < a.k) a.weights[t * a.k + lane + 32] = e1 / sum * a.scale, a.ids[t * a.k + lane + 32] = my_id[1];
 }
@@ -170,7 +174,12 @@ __global__ void __launch_bounds__(1024) route_places_kernel(const RouteArgs a, c
     for (int b = 0; b < BATCH; ++b) e[b] = i0 + b * 1024 < choices ? a.ids[i0 + b * 1024] : -1;
 #pragma unroll
     for (int b = 0; b < BATCH; ++b)
-      if (e[b] >= 0) a.slots[i0 + b * 1024] = e[b] >= a.real ? -1 : a.shared ? count[e[b]] + (int)((i0 + b * 1024) / a.k) : atomicAdd(count + e[b], 1);
+      if (e[b] >= 0) {
+        const int64_t i = i0 + b * 1024;
+        const int slot = e[b] >= a.real ? -1 : a.shared ? count[e[b]] + (int)(i / a.k) : atomicAdd(count + e[b], 1);
+        a.slots[i] = slot;
+        if (a.row_weights && slot >= 0) a.row_weights[slot] = a.weights[i];
+      }
   }
 }
 
@@ -202,6 +211,7 @@ struct GroupedArgs {
   int64_t ldo, N, K;
   int tile, n;
   const int32_t *tile_expert, *live;
+  const float* row_scale;
 };
 
 __device__ __forceinline__ float typed(const void* p, int dtype, int64_t at) {
@@ -229,6 +239,7 @@ __global__ void __launch_bounds__(256) grouped_matmul_kernel(const GroupedArgs g
     __syncthreads();
   }
   if (col >= g.N) return;
+  if (g.row_scale) acc *= g.row_scale[(int64_t)i * g.tile + r0 + ty];
   const int64_t at = ((int64_t)i * g.tile + r0 + ty) * g.ldo + col;
   if (g.out_dtype == FB_FP32) static_cast<float*>(g.out)[at] = acc;
   else static_cast<uint16_t*>(g.out)[at] = (uint16_t)float_to_bf16_bits(acc);
@@ -244,15 +255,16 @@ extern "C" int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_
 }
 
 extern "C" int fb_route(const fb_router* router_host, const float* logits, int64_t T, int64_t ld, int tile, int shared_rows, float* weights, int32_t* ids, int32_t* slots,
-                        int32_t* tile_expert, int32_t* live, void* stream) {
+                        int32_t* tile_expert, int32_t* live, float* row_weights, void* stream) {
   FB_REQUIRE(router_host && logits && weights && ids && slots && tile_expert && live && T >= 1 && T <= (1 << 24), "fb_route: null pointer or no tokens");
   const int n = router_host->n, k = router_host->k, real = n - router_host->identity;
   FB_REQUIRE(router_host->identity >= 0 && real >= 1, "fb_route: at least one expert with rows");
+  FB_REQUIRE(router_host->scored >= 0 && router_host->scored <= 2 && (router_host->scored || !router_host->as_scored), "fb_route: choices by logit, or scores by softmax or sigmoid, which may be the weights");
   FB_REQUIRE(n >= 1 && n <= 8192 && k >= 1 && k <= 64 && k <= n && ld >= n, "fb_route: up to 64 choices among up to 8192 experts (got %d of %d)", k, n);
   FB_REQUIRE(tile >= 16 && tile % 16 == 0 && (!shared_rows || T <= tile), "fb_route: tiles of whole runs of 16 rows; shared rows: all the tokens in one");
   const int64_t tiles = fb_route_tiles(T, real, k, tile, shared_rows);
   FB_REQUIRE(tiles * tile < (1ll << 31), "fb_route: too many rows");
-  const fb::RouteArgs a{logits, T, ld, router_host->bias, n, k, tile, shared_rows, real, router_host->scored, router_host->scale, (int)tiles, weights, ids, slots, tile_expert, live};
+  const fb::RouteArgs a{logits, T, ld, router_host->bias, n, k, tile, shared_rows, real, router_host->scored, router_host->scale, router_host->as_scored, (int)tiles, weights, ids, slots, tile_expert, live, row_weights};
   const auto s = (cudaStream_t)stream;
   const int pick = T <= 32;
   if (!pick)
@@ -271,11 +283,11 @@ extern "C" int fb_spread_rows(const void* x, int64_t T, int64_t row_bytes, int64
 }
 
 extern "C" int fb_grouped_matmul(int x_dtype, const void* x, int64_t x_rows, int64_t ldx, int shared_rows, int w_dtype, const void* W, const int64_t* w_strides_host, int n, int64_t K, int64_t N,
-                                 const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, int out_dtype, void* out, int64_t ldo, void* stream) {
+                                 const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, const float* row_scale, int out_dtype, void* out, int64_t ldo, void* stream) {
   FB_REQUIRE(x && W && w_strides_host && tile_expert && live && out && tiles >= 1 && K >= 1 && N >= 1 && n >= 1, "fb_grouped_matmul: null pointer or empty");
   FB_REQUIRE(tile >= 16 && tile % 16 == 0 && ldx >= K && ldo >= N && tiles * (tile / 16) <= 65535, "fb_grouped_matmul: tiles of whole runs of 16 rows, at most 65535 such runs");
   FB_REQUIRE(shared_rows ? x_rows >= 1 && x_rows <= tile : x_rows >= tiles * tile, "fb_grouped_matmul: all the tiles' rows there");
   for (int d : {x_dtype, w_dtype, out_dtype}) FB_REQUIRE(d == FB_BF16 || d == FB_FP32, "fb_grouped_matmul: bf16 or fp32");
-  const fb::GroupedArgs g{x, x_dtype, ldx, x_rows, shared_rows, W, w_dtype, {w_strides_host[0], w_strides_host[1], w_strides_host[2]}, out, out_dtype, ldo, N, K, tile, n, tile_expert, live};
+  const fb::GroupedArgs g{x, x_dtype, ldx, x_rows, shared_rows, W, w_dtype, {w_strides_host[0], w_strides_host[1], w_strides_host[2]}, out, out_dtype, ldo, N, K, tile, n, tile_expert, live, row_scale};
   return fb::launch_after(fb::grouped_matmul_kernel, dim3((unsigned)fb::ceil_div(N, 16), (unsigned)(tiles * (tile / 16))), dim3(256), 0, (cudaStream_t)stream, "fb_grouped_matmul", g);
 }

@@ -17,6 +17,8 @@ struct HeadsArgs {
   int window; // 0: none; else a token sees the last `window` places only
   float scale, softcap;  // softcap > 0: a scaled score s becomes softcap tanh(s / softcap)
   const float* sink;  // [heads] or null
+  const float* key_bias;  // [heads] or null; given: no softmax, a key's weight is sigmoid(score + key_bias[h])
+  float out_scale;    // of the result
   int gate_dtype;
   const void* gate;  // [T, ld_g]: head h at h * vdim; the output times its sigmoid
   int64_t ld_g;
@@ -33,13 +35,6 @@ __device__ __forceinline__ int first_seen(const HeadsArgs& a, int place) {
   return a.window > 0 ? max(lo, place - a.window + 1) : lo;
 }
 
-// 2^x, the hardware's (x far below: 0)
-__device__ __forceinline__ float exp2_of(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
 // an unscaled score s as the unscaled score that the cap leaves: (softcap / scale) tanh(s scale / softcap), tanh by one exponential
 // (to about 2e-7 of 1)
 struct SoftCap {
@@ -47,6 +42,12 @@ struct SoftCap {
 };
 __device__ __forceinline__ SoftCap soft_cap(const HeadsArgs& a) { return {a.softcap > 0.f ? 2.8853900817779268f * a.scale / a.softcap : 0.f, a.softcap > 0.f ? a.softcap / a.scale : 0.f}; }
 __device__ __forceinline__ float capped(const SoftCap& c, float s) { return fmaf(-2.f * c.out, __fdividef(1.f, 1.f + exp2_of(fminf(s * c.in, 80.f))), c.out); }
+
+// sigmoids of two numbers given times log2(e), by two exponentials and one reciprocal
+__device__ __forceinline__ void sigmoid_pair(float x, float y, float& a, float& b) {
+  const float u = 1.f + exp2_of(fminf(-x, 60.f)), v = 1.f + exp2_of(fminf(-y, 60.f)), r = __fdividef(1.f, u * v);
+  a = r * v, b = r * u;
+}
 
 __device__ __forceinline__ float gate_value(const HeadsArgs& a, int64_t at) {
   return a.gate_dtype == FB_FP32 ? static_cast<const float*>(a.gate)[at] : bf16_bits_to_float(static_cast<const uint16_t*>(a.gate)[at]);

@@ -1,7 +1,7 @@
 // Attention with grouped key heads over a cache whose rows are a key and then its value: the two may differ in width, the
 // keys a token sees may be confined to its own span of the sequence (spans of `span` places, counted from its start) or to the
 // last `window` places, scores may be capped, a number per head may join the softmax's denominator, and the output may be gated
-// column by column.
+// column by column.  Or there is no softmax: a key's weight is a sigmoid of its own score and a number of the head.
 //
 // A CTA has one key head, a tile of (token, query head) pairs that share it - the pairs of one token in a decode step, those
 // of consecutive tokens in a prompt's chunk - and a run of the keys that they see; tiles of 64 keys and their values come in by
@@ -57,8 +57,16 @@ __global__ void __launch_bounds__(32 * PLAIN_HEADS) heads_attention_plain_kernel
       s *= a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
     }
-    const float m_new = fmaxf(m, warp_max(s)), corr = expf(m - m_new), p = lane < n ? expf(s - m_new) : 0.f;
-    m = m_new, l = l * corr + warp_sum(p);
+    if (a.key_bias) {
+      m = 0.f, l = 1.f;
+      s = lane < n ? sigmoid_f(s + a.key_bias[h]) : 0.f;
+    }
+    float corr = 1.f, p = s;
+    if (!a.key_bias) {
+      const float m_new = fmaxf(m, warp_max(s));
+      corr = expf(m - m_new), p = lane < n ? expf(s - m_new) : 0.f;
+      m = m_new, l = l * corr + warp_sum(p);
+    }
 #pragma unroll
     for (int i = 0; i < COLS; ++i) acc[i] *= corr;
     for (int j = 0; j < n; ++j) {
@@ -69,7 +77,7 @@ __global__ void __launch_bounds__(32 * PLAIN_HEADS) heads_attention_plain_kernel
         if (i * 32 + lane < a.vdim) acc[i] = fmaf(pj, value_of(v[i * 32 + lane]), acc[i]);
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = l > 0.f ? a.out_scale / l : 0.f;
 #pragma unroll
   for (int i = 0; i < COLS; ++i) {
     const int64_t col = (int64_t)h * a.vdim + i * 32 + lane;
@@ -87,7 +95,7 @@ static int launch_plain(const HeadsArgs& a, cudaStream_t s) {
 
 extern "C" int fb_heads_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int kv_heads, int dim, int vdim, const void* cache, int64_t cache_rows,
                                   int64_t head_stride, const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk, int span, int window, float scale,
-                                  float softcap, const float* sink, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o, void* stream) {
+                                  float softcap, const float* sink, const float* key_bias, float out_scale, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o, void* stream) {
   using namespace fb;
   FB_REQUIRE(q && cache && last && out && T >= 1 && max_keys >= 1 && cache_rows >= 1, "fb_heads_attention: null pointer or empty");
   FB_REQUIRE(heads >= 1 && kv_heads >= 1 && heads % kv_heads == 0 && dim >= 1 && vdim >= 1 && kv_heads <= 65535, "fb_heads_attention: whole groups of query heads per key head (got %d / %d)", heads, kv_heads);
@@ -97,7 +105,8 @@ extern "C" int fb_heads_attention(int dtype, const void* q, int64_t T, int64_t l
   FB_REQUIRE(!gate || ((gate_dtype == FB_BF16 || gate_dtype == FB_FP32) && ld_g >= (int64_t)heads * vdim), "fb_heads_attention: gates, bf16 or fp32, one a column of the result");
   FB_REQUIRE(!chunk || !base, "fb_heads_attention: a chunk is one sequence's (no base)");
   FB_REQUIRE(softcap >= 0.f, "fb_heads_attention: a cap of scores is positive (0: none)");
-  HeadsArgs a{q, T, ld_q, heads, kv_heads, dim, vdim, heads / kv_heads, cache, cache_rows, head_stride, base, last, row0, chunk, span, window, scale, softcap, sink, gate_dtype, gate, ld_g, out, ld_o, max_keys, 0, 0, 0, 0};
+  FB_REQUIRE(!key_bias || !sink, "fb_heads_attention: a sink joins a softmax's denominator");
+  HeadsArgs a{q, T, ld_q, heads, kv_heads, dim, vdim, heads / kv_heads, cache, cache_rows, head_stride, base, last, row0, chunk, span, window, scale, softcap, sink, key_bias, out_scale, gate_dtype, gate, ld_g, out, ld_o, max_keys, 0, 0, 0, 0};
   if (span > 0 && span < a.seen) a.seen = span;
   if (window > 0 && window + (chunk ? ceil_div(128, a.rep) : 0) < a.seen) a.seen = window + (chunk ? ceil_div(128, a.rep) : 0);  // (a tile's tokens' windows together)
   const auto s = (cudaStream_t)stream;

@@ -133,6 +133,16 @@ __global__ void __launch_bounds__(32 * WR * WK + 32) heads_attention_kernel(cons
   for (int mt = 0; mt < MT; ++mt) m_run[mt][0] = m_run[mt][1] = -INFINITY, l_run[mt][0] = l_run[mt][1] = 0.f;
   const float scale_log2 = a.scale * LOG2E;
   const SoftCap cap = soft_cap(a);
+  float bias_r[MT][2];  // weights by sigmoid: the rows' numbers; such parts have the maximum 0 and are added up as they are
+  if (a.key_bias) {
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int r = 16 * (WR * mt + wr) + (lane >> 2) + 8 * h;
+        bias_r[mt][h] = r < rows ? a.key_bias[g * a.rep + (pair0 + r) % a.rep] * LOG2E : 0.f, m_run[mt][h] = 0.f;
+      }
+  }
 
   // where a lane's 16 bytes stand within a swizzled row, for the four steps of 16 columns that a row has
   uint32_t k_off[4], v_off[4];
@@ -187,6 +197,17 @@ __global__ void __launch_bounds__(32 * WR * WK + 32) heads_attention_kernel(cons
             const int key = key_first + n * 8 + (e & 1);
             if (key >= k1 || key > place_r[mt][e >> 1] || key < lo_r[mt][e >> 1]) s[mt][n][e] = -INFINITY;
           }
+      }
+      if (a.key_bias) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            float x, y;
+            sigmoid_pair(fmaf(s[mt][n][2 * h], scale_log2, bias_r[mt][h]), fmaf(s[mt][n][2 * h + 1], scale_log2, bias_r[mt][h]), x, y);
+            pf[mt][n / 2][2 * (n & 1) + h] = pack_bf16x2(s[mt][n][2 * h] == -INFINITY ? 0.f : x, s[mt][n][2 * h + 1] == -INFINITY ? 0.f : y);
+          }
+        continue;
       }
       float mx[2] = {m_run[mt][0], m_run[mt][1]}, corr[2];
 #pragma unroll
@@ -247,7 +268,7 @@ __global__ void __launch_bounds__(32 * WR * WK + 32) heads_attention_kernel(cons
           const float sink = a.sink[head] * LOG2E;
           m = fmaxf(m, sink), f = exp2_of(m_run[mt][h] - m), l = l * f + exp2_of(sink - m);
         }
-        f = l > 0.f ? f / l : 0.f;
+        f = a.key_bias ? a.out_scale : l > 0.f ? f * a.out_scale / l : 0.f;
         uint16_t* out = static_cast<uint16_t*>(a.out) + t * a.ld_o;
 #pragma unroll
         for (int d = 0; d < DV / 8; ++d)
@@ -327,7 +348,7 @@ __global__ void __launch_bounds__(32 * WR * WK + 32) heads_attention_kernel(cons
       const float f = exp2_of(pm[p] - m);
       l = fmaf(pl[p], f, l), acc = fmaf(po[p], f, acc);
     }
-    static_cast<uint16_t*>(a.out)[t * a.ld_o + col] = (uint16_t)float_to_bf16_bits(l > 0.f ? acc / l * gate : 0.f);
+    static_cast<uint16_t*>(a.out)[t * a.ld_o + col] = (uint16_t)float_to_bf16_bits(a.key_bias ? acc * a.out_scale * gate : l > 0.f ? acc / l * a.out_scale * gate : 0.f);
   }
   if (splits > 1) cluster_barrier();  // the others have read this CTA's part
 }

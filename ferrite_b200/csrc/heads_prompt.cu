@@ -9,6 +9,7 @@
 //
 // A softmax thread owns a pair: its scores, its probabilities (written over the scores, as bf16) and its sums are one lane of
 // tensor memory.  The sums stand under a reference maximum that moves only when the scores outgrow it by a factor of 256.
+// Where weights are sigmoids (SIGMOID) there is neither a maximum nor a denominator.
 //
 //   warps 0-3, 4-7   softmax of the two groups       warp 8   TMA        warp 9   MMAs (the whole warp issues them, written out)
 //
@@ -25,7 +26,7 @@ namespace {
 constexpr int HP_KEYS = 64, HP_MAX_STAGES = 6, HP_ROWS = 128;
 constexpr size_t HP_SMEM = 224 * 1024, HP_SMEM_HALF = 112 * 1024;  // a CTA's alone on its SM, one of two
 constexpr int HP_Q_CHUNK = HP_ROWS * 128, HP_K_CHUNK = HP_KEYS * 128;  // 64 columns of a group's queries, of a tile's keys or values
-constexpr int HP_COLS = 2 * HP_KEYS + 128;                             // tensor memory of a group: two tiles of scores, the sums
+constexpr int HP_COLS = 2 * HP_KEYS + 128;                             // tensor memory of a group (of two): two tiles of scores, the sums
 constexpr float HP_SLACK = 8.f;                                        // log2 of how far scores may outgrow the reference maximum
 constexpr float HP_LOG2E = 1.4426950408889634f;
 
@@ -41,7 +42,7 @@ struct PromptParams {
 // v times the sigmoid of g
 __device__ __forceinline__ float gated(float v, float g) { return __fdividef(v, 1.f + __expf(-g)); }
 
-template <int GROUPS>
+template <int GROUPS, bool SIGMOID>
 __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) heads_prompt_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tkv, const PromptParams p) {
   constexpr int HP_WARP_LOAD = 4 * GROUPS, HP_WARP_MMA = HP_WARP_LOAD + 1;
   extern __shared__ uint8_t prompt_smem[];
@@ -165,6 +166,7 @@ __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) he
     const uint32_t lanes = (uint32_t)(32 * (warp & 3)) << 16, tS = tmem + lanes + gr * HP_COLS, tO = tS + 2 * HP_KEYS;
     const float scale_log2 = a.scale * HP_LOG2E;
     const SoftCap cap = soft_cap(a);
+    const float bias = SIGMOID && live ? a.key_bias[head] * HP_LOG2E : 0.f;
     float m = -INFINITY, l = 0.f;  // the reference maximum of the unscaled scores, and the sum under it
     for (int t = 0; t < n_tiles; ++t) {
       mbar_wait(smem_u32(s_full + 2 * gr + (t & 1)), (t >> 1) & 1, abort_flag, PW_S);
@@ -183,24 +185,34 @@ __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) he
         for (int j = 0; j < HP_KEYS; ++j)
           if (j >= seen || j < hidden) s[j] = -INFINITY;
       }
-      float tops[4] = {s[0], s[1], s[2], s[3]};
-#pragma unroll
-      for (int j = 4; j < HP_KEYS; ++j) tops[j & 3] = fmaxf(tops[j & 3], s[j]);
-      const float top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
       float corr = 1.f;
-      const bool grown = (top - m) * scale_log2 > HP_SLACK || (m == -INFINITY && top > m);
-      if (grown) corr = exp2_of((m - top) * scale_log2), m = top;
-      const bool any = __any_sync(0xffffffffu, grown);
-      const float at = m == -INFINITY ? 0.f : -m * scale_log2;
-      float sums[4] = {0.f, 0.f, 0.f, 0.f};
+      bool any = false;
       uint32_t pair[HP_KEYS / 2];
+      if constexpr (SIGMOID) {
 #pragma unroll
-      for (int j = 0; j < HP_KEYS; j += 2) {
-        const float x = exp2_of(fmaf(s[j], scale_log2, at)), y = exp2_of(fmaf(s[j + 1], scale_log2, at));
-        sums[j & 2] += x, sums[(j & 2) + 1] += y;
-        pair[j / 2] = pack_bf16x2(x, y);
+        for (int j = 0; j < HP_KEYS; j += 2) {
+          float x, y;
+          sigmoid_pair(fmaf(s[j], scale_log2, bias), fmaf(s[j + 1], scale_log2, bias), x, y);
+          pair[j / 2] = pack_bf16x2(s[j] == -INFINITY ? 0.f : x, s[j + 1] == -INFINITY ? 0.f : y);
+        }
+      } else {
+        float tops[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+        for (int j = 4; j < HP_KEYS; ++j) tops[j & 3] = fmaxf(tops[j & 3], s[j]);
+        const float top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
+        const bool grown = (top - m) * scale_log2 > HP_SLACK || (m == -INFINITY && top > m);
+        if (grown) corr = exp2_of((m - top) * scale_log2), m = top;
+        any = __any_sync(0xffffffffu, grown);
+        const float at = m == -INFINITY ? 0.f : -m * scale_log2;
+        float sums[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int j = 0; j < HP_KEYS; j += 2) {
+          const float x = exp2_of(fmaf(s[j], scale_log2, at)), y = exp2_of(fmaf(s[j + 1], scale_log2, at));
+          sums[j & 2] += x, sums[(j & 2) + 1] += y;
+          pair[j / 2] = pack_bf16x2(x, y);
+        }
+        l = l * corr + ((sums[0] + sums[1]) + (sums[2] + sums[3]));
       }
-      l = l * corr + ((sums[0] + sums[1]) + (sums[2] + sums[3]));
       if (t > 0) {  // the sums stand still once the last tile's MMAs are done
         mbar_wait(smem_u32(pv_done + gr), (t - 1) & 1, abort_flag, PW_PV);
         tc_fence_after();
@@ -232,7 +244,7 @@ __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) he
         const float sink = a.sink[head] * HP_LOG2E, top = fmaxf(mine, sink);
         f = exp2_of(mine - top), total = l * f + exp2_of(sink - top);
       }
-      f = total > 0.f ? f / total : 0.f;
+      f = SIGMOID ? a.out_scale : total > 0.f ? f * a.out_scale / total : 0.f;
     }
     if (n_tiles) {
       mbar_wait(smem_u32(pv_done + gr), (n_tiles - 1) & 1, abort_flag, PW_PV);
@@ -317,18 +329,19 @@ bool prompt_sizes(PromptParams& p, int groups) {
   const HeadsArgs& a = p.a;
   p.groups = groups, p.tokens = HP_ROWS / a.rep, p.ck = (a.dim + 63) / 64, p.cv = (a.vdim + 63) / 64, p.nv = (a.vdim + 15) / 16 * 16;
   p.q_bytes = p.ck * HP_Q_CHUNK > 17 * 1024 ? p.ck * HP_Q_CHUNK : 17 * 1024;  // (17 KB: what the result takes on its way out)
-  p.tmem_cols = groups * HP_COLS;
+  p.tmem_cols = p.nv > 128 ? 512 : groups * HP_COLS;  // (sums of more than 128 columns: one group, all of tensor memory)
+  if (p.nv > 128 && groups > 1) return false;
   const int64_t stage = (p.ck + p.cv) * HP_K_CHUNK, rest = 1024 + groups * p.q_bytes;
-  p.smem = groups == 1 && rest + 2 * stage <= (int64_t)HP_SMEM_HALF ? HP_SMEM_HALF : HP_SMEM;
+  p.smem = groups == 1 && p.nv <= 128 && rest + 2 * stage <= (int64_t)HP_SMEM_HALF ? HP_SMEM_HALF : HP_SMEM;
   const int64_t room = ((int64_t)p.smem - rest) / stage;
   p.stages = (int)(room < HP_MAX_STAGES ? room : HP_MAX_STAGES);
   return p.stages >= 2;
 }
 
-template <int GROUPS>
+template <int GROUPS, bool SIGMOID>
 int launch_prompt(const PromptParams& p, const CUtensorMap& tq, const CUtensorMap& tkv, cudaStream_t s) {
   static std::atomic<uint64_t> opted{0};
-  if (first_on_device(opted)) cudaFuncSetAttribute(heads_prompt_kernel<GROUPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)HP_SMEM);
+  if (first_on_device(opted)) cudaFuncSetAttribute(heads_prompt_kernel<GROUPS, SIGMOID>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)HP_SMEM);
   cudaLaunchConfig_t cfg{};
   cfg.gridDim = dim3((unsigned)p.a.kv_heads, (unsigned)ceil_div(p.a.T, GROUPS * p.tokens)), cfg.blockDim = dim3((4 * GROUPS + 2) * 32);
   cfg.dynamicSmemBytes = p.smem, cfg.stream = s;
@@ -336,7 +349,7 @@ int launch_prompt(const PromptParams& p, const CUtensorMap& tq, const CUtensorMa
   attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   attr[0].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr, cfg.numAttrs = 1;
-  cudaLaunchKernelEx(&cfg, heads_prompt_kernel<GROUPS>, tq, tkv, p);
+  cudaLaunchKernelEx(&cfg, heads_prompt_kernel<GROUPS, SIGMOID>, tq, tkv, p);
   return launch_status("fb_heads_attention");
 }
 
@@ -347,7 +360,7 @@ static const StatusWord g_status_reader(read_and_clear_status_word);
 // a chunk of one sequence with tiles enough for half the SMs (fewer: heads_attention.cu splits the keys), heads that tensor
 // memory takes, rows that TMA takes (the caller has checked that q and the cache are whole 16-byte pieces)
 bool heads_prompt_supports(const HeadsArgs& a) {
-  if (!a.chunk || a.rep > HP_ROWS || a.dim > 256 || a.vdim > 128 || a.ld_o % 2 || ceil_div(a.T, HP_ROWS / a.rep) > 65535 || a.cache_rows >= (1ll << 31)) return false;
+  if (!a.chunk || a.rep > HP_ROWS || a.dim > 256 || a.vdim > 256 || a.ld_o % 2 || ceil_div(a.T, HP_ROWS / a.rep) > 65535 || a.cache_rows >= (1ll << 31)) return false;
   PromptParams p{};
   p.a = a;
   return ceil_div(a.T, HP_ROWS / a.rep) * a.kv_heads >= 74 && prompt_sizes(p, 1) && tma_encoder() != nullptr;
@@ -367,7 +380,8 @@ int heads_prompt(const HeadsArgs& a, cudaStream_t s) {
   const int64_t kd[3] = {a.dim + a.vdim, a.cache_rows, a.kv_heads}, ks[2] = {a.dim + a.vdim, a.head_stride};
   const int kb[3] = {64, HP_KEYS, 1};
   if (int rc = tma_map_bf16(&tkv, a.cache, 3, kd, ks, kb, "fb_heads_attention (cache)")) return rc;
-  return two ? launch_prompt<2>(p, tq, tkv, s) : launch_prompt<1>(p, tq, tkv, s);
+  if (a.key_bias) return two ? launch_prompt<2, true>(p, tq, tkv, s) : launch_prompt<1, true>(p, tq, tkv, s);
+  return two ? launch_prompt<2, false>(p, tq, tkv, s) : launch_prompt<1, false>(p, tq, tkv, s);
 }
 
 }  // namespace fb

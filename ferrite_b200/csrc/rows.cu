@@ -3,8 +3,8 @@
 //   fb_heads_put   after a joint q | k | v projection: biases, a short convolution over time, RMSNorm of each query and key head or
 //                  of all of them together, the turn by the token's place, values mixed with another layer's or the keys
 //                  themselves, the new cache row
-//   fb_add_norm    a layer's end: the branches' results scaled by column, a mixture's chosen rows weighted and summed, all
-//                  added to the stream, and the next layer's RMSNorm of it
+//   fb_add_norm    a layer's end: the branches' results scaled by column, a mixture's chosen rows weighted and summed, all of that
+//                  gated and normed where the design says so and added to the stream, and the next layer's RMSNorm of it
 #include "launch.cuh"
 #include "values.cuh"
 
@@ -40,6 +40,11 @@ struct HeadsPutArgs {
   void* cache;  // [kv_heads, cache_rows, dim + vdim]: a key, then its value
   int64_t cache_rows, head_stride;
 };
+
+// what a token's queries are multiplied by after their norm
+__device__ __forceinline__ float temperature_of(const fb_heads& s, int64_t t) {
+  return s.temp_coef != 0.f ? fmaf(s.temp_coef, logf(floorf((float)(s.places[t] + 1) / s.temp_every) + 1.f), 1.f) : 1.f;
+}
 
 constexpr int HEADS_WARPS = 8, HEADS_REGS = 8;  // a lane keeps up to 8 columns (heads of up to 256) between the two passes
 
@@ -84,7 +89,7 @@ __global__ void __launch_bounds__(32 * HEADS_WARPS) heads_put_kernel(const Heads
     const float v = value_of(x[c]) + (bias ? bias[c] : 0.f);
     ss = fmaf(v, v, ss);
   }
-  const float r = w ? 1.f / sqrtf(warp_sum(ss) / (float)n + s.eps) : 1.f;
+  const float r = (w ? 1.f / sqrtf(warp_sum(ss) / (float)n + s.eps) : 1.f) * (is_q ? temperature_of(s, t) : 1.f);
 #pragma unroll
   for (int i = 0; i < HEADS_REGS; ++i) {
     const int c = 32 * i + lane;
@@ -118,7 +123,7 @@ __global__ void __launch_bounds__(128) heads_put4_kernel(const HeadsPutArgs a) {
       v[i][j] = four(x + at + c);
       if (u >= keys && s.first) f[i][j] = four(static_cast<const In*>(s.first) + t * s.ld_first + (int64_t)(u - keys) * s.vdim + c);
     }
-  const float share = s.first ? *s.share : 0.f;
+  const float share = s.first ? *s.share : 0.f, temp = temperature_of(s, t);
 #pragma unroll
   for (int i = 0; i < UNITS; ++i) {
     const int u = u0 + i, n = u < keys ? s.dim : s.vdim;
@@ -141,7 +146,7 @@ __global__ void __launch_bounds__(128) heads_put4_kernel(const HeadsPutArgs a) {
       ss = fmaf(v[i][j].x, v[i][j].x, fmaf(v[i][j].y, v[i][j].y, fmaf(v[i][j].z, v[i][j].z, fmaf(v[i][j].w, v[i][j].w, ss))));
     }
     const float* w = u < s.heads ? s.q_norm : u < keys ? s.k_norm : nullptr;
-    const float r = w ? 1.f / sqrtf(warp_sum(ss) / (float)n + s.eps) : 1.f;
+    const float r = (w ? 1.f / sqrtf(warp_sum(ss) / (float)n + s.eps) : 1.f) * (u < s.heads ? temp : 1.f);
     if (u >= s.heads && !inside) continue;
     Act* out = u < s.heads ? static_cast<Act*>(a.q_out) + t * a.ld_q + (int64_t)u * s.dim
                            : static_cast<Act*>(a.cache) + (u < keys ? u - s.heads : u - keys) * a.head_stride + row * (s.dim + s.vdim) + (u < keys ? 0 : s.dim);
@@ -248,6 +253,7 @@ __global__ void __launch_bounds__(512) heads_turn_kernel(const HeadsTurnArgs arg
     const float joint = s.norm_all ? 1.f / sqrtf(block_sum(ss, red) / (float)((blockIdx.y ? s.kv_heads : s.heads) * s.dim) + s.eps) : 1.f;
     __syncthreads();
     const bool inside = row >= 0 && row < a.cache_rows;  // nothing is written outside the cache
+    const float temp = temperature_of(s, t);
     for (int u = u0 + warp; u < u1; u += blockDim.x / 32) {
       const bool is_q = u < s.heads, is_v = u >= keys;
       const int n = is_v ? s.vdim : s.dim, g = is_q ? u : is_v ? u - keys : u - s.heads;
@@ -273,6 +279,10 @@ __global__ void __launch_bounds__(512) heads_turn_kernel(const HeadsTurnArgs arg
 #pragma unroll
           for (int e = 0; e < N; ++e) v[e] *= r * g4[e];
         }
+        if (is_q) {
+#pragma unroll
+          for (int e = 0; e < N; ++e) v[e] *= temp;
+        }
         if (!is_v && c < s.turned) {
           if constexpr (N == 4) {
 #pragma unroll
@@ -282,7 +292,7 @@ __global__ void __launch_bounds__(512) heads_turn_kernel(const HeadsTurnArgs arg
                 v[e] = x0 * cs - x1 * sn, v[e + 1] = x1 * cs + x0 * sn;
               }
           } else {
-            const float other = mine[c ^ 1] * (w ? r * w[c ^ 1] : 1.f), cs = turns[c >> 1], sn = turns[half + (c >> 1)];
+            const float other = mine[c ^ 1] * (w ? r * w[c ^ 1] : 1.f) * (is_q ? temp : 1.f), cs = turns[c >> 1], sn = turns[half + (c >> 1)];
             v[0] = c & 1 ? v[0] * cs + other * sn : v[0] * cs - other * sn;
           }
         }
@@ -355,7 +365,7 @@ __device__ __forceinline__ void chosen_rows(const fb_branches& a, int64_t t, con
     const int64_t slot = a.slots[t * a.k + j];
     const bool own = slot < 0 && a.own;
     from[j] = own ? static_cast<const Act*>(a.own) + t * a.ld_own : static_cast<const Act*>(a.chosen) + (slot < 0 ? 0 : slot) * a.ld_chosen;
-    weight[j] = slot < 0 && !own ? 0.f : a.weights[t * a.k + j];
+    weight[j] = slot < 0 && !own ? 0.f : a.weights ? a.weights[t * a.k + j] : 1.f;
   }
 }
 
@@ -374,9 +384,10 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, cons
   const float* x = a.x + t * a.ld_x;
   const In* y1 = a.mixer ? static_cast<const In*>(a.mixer) + t * a.ld_mixer : nullptr;
   const In* y2 = a.other ? static_cast<const In*>(a.other) + t * a.ld_other : nullptr;
+  const bool apart = a.gate || a.post;  // the branches' sum is finished before the stream joins
   float ss = 0.f;
   for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) {
-    float v = x[c];
+    float v = apart ? 0.f : x[c];
     if (y1 || a.mixer_bias) v = fmaf((y1 ? value_of(y1[c]) : 0.f) + (a.mixer_bias ? a.mixer_bias[c] : 0.f), a.mixer_scale ? a.mixer_scale[c] : 1.f, v);
     if (a.chosen || y2) {
       float f = y2 ? value_of(y2[c]) : 0.f;
@@ -384,9 +395,20 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, cons
         for (int j = 0; j < a.k; ++j) f = fmaf(weight[j], value_of(from[j][c]), f);
       v = fmaf(f, a.other_scale ? a.other_scale[c] : 1.f, v);
     }
+    if (a.gate) v *= sigmoid_f(a.gate[t * a.ld_gate + c] + (a.gate_bias ? a.gate_bias[c] : 0.f));
     row[c] = v;
-    if (a.x_out) a.x_out[t * a.ld_x_out + c] = v;
+    if (a.x_out && !apart) a.x_out[t * a.ld_x_out + c] = v;
     ss = fmaf(v, v, ss);
+  }
+  if (apart) {
+    const float r = a.post ? 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps) : 1.f;
+    ss = 0.f;
+    for (int64_t c = threadIdx.x; c < cols; c += blockDim.x) {
+      const float v = fmaf(row[c] * r, a.post ? a.post[c] : 1.f, x[c]);
+      row[c] = v;
+      if (a.x_out) a.x_out[t * a.ld_x_out + c] = v;
+      ss = fmaf(v, v, ss);
+    }
   }
   if (!a.h) return;
   const float r = a.w ? 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps) : 1.f;
@@ -396,7 +418,7 @@ __global__ void __launch_bounds__(512) add_norm_kernel(const fb_branches a, cons
 
 // the same for rows of whole groups of four columns, 16-byte aligned: a thread keeps its groups in registers, everything it
 // reads on its way at once
-template <typename In, typename Act, int GROUPS>
+template <typename In, typename Act, int GROUPS, bool APART>
 __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, const int64_t cols) {
   griddep_launch_dependents();
   griddep_wait();
@@ -409,14 +431,19 @@ __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, con
     __syncthreads();
   }
   const float4 one = make_float4(1.f, 1.f, 1.f, 1.f), none = make_float4(0.f, 0.f, 0.f, 0.f);
-  float4 v[GROUPS], f[GROUPS];
+  float4 v[GROUPS], f[GROUPS], x[APART ? GROUPS : 1], gate[APART ? GROUPS : 1];  // APART: the branches' sum is finished before the stream joins
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < GROUPS; ++i) {
     const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
     v[i] = f[i] = none;
     if (c >= cols) continue;
-    v[i] = four(a.x + t * a.ld_x + c);
+    if constexpr (APART) {
+      x[i] = four(a.x + t * a.ld_x + c), gate[i] = none;
+      if (a.gate) gate[i] = four(a.gate + t * a.ld_gate + c);
+    } else {
+      v[i] = four(a.x + t * a.ld_x + c);
+    }
     if (a.mixer) v[i] = fma4(four(static_cast<const In*>(a.mixer) + t * a.ld_mixer + c), a.mixer_scale ? four(a.mixer_scale + c) : one, v[i]);
     if (a.mixer_bias) v[i] = fma4(four(a.mixer_bias + c), a.mixer_scale ? four(a.mixer_scale + c) : one, v[i]);
     if (a.other) f[i] = four(static_cast<const In*>(a.other) + t * a.ld_other + c);
@@ -444,8 +471,28 @@ __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, con
     const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
     if (c >= cols) continue;
     if (a.chosen || a.other) v[i] = fma4(f[i], a.other_scale ? four(a.other_scale + c) : one, v[i]);
+    if constexpr (APART) {
+      if (a.gate) {
+        const float4 b = a.gate_bias ? four(a.gate_bias + c) : none;
+        v[i].x *= sigmoid_f(gate[i].x + b.x), v[i].y *= sigmoid_f(gate[i].y + b.y), v[i].z *= sigmoid_f(gate[i].z + b.z), v[i].w *= sigmoid_f(gate[i].w + b.w);
+      }
+      ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
+      continue;
+    }
     if (a.x_out) put_four(a.x_out + t * a.ld_x_out + c, v[i]);
     ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
+  }
+  if constexpr (APART) {
+    const float r = a.post ? 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps) : 1.f;
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < GROUPS; ++i) {
+      const int64_t c = 4 * (threadIdx.x + (int64_t)i * blockDim.x);
+      if (c >= cols) continue;
+      v[i] = fma4(make_float4(v[i].x * r, v[i].y * r, v[i].z * r, v[i].w * r), a.post ? four(a.post + c) : one, x[i]);
+      if (a.x_out) put_four(a.x_out + t * a.ld_x_out + c, v[i]);
+      ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
+    }
   }
   if (!a.h) return;
   const float r = a.w ? 1.f / sqrtf(block_sum(ss, red) / (float)cols + a.eps) : 1.f;
@@ -463,13 +510,20 @@ __global__ void __launch_bounds__(512) add_norm4_kernel(const fb_branches a, con
   }
 }
 
+template <typename In, typename Act, int GROUPS>
+static int launch_add_norm4(const fb_branches& a, int64_t T, dim3 block, int64_t cols, cudaStream_t s) {
+  if (a.gate || a.post) return launch_after(add_norm4_kernel<In, Act, GROUPS, true>, dim3((unsigned)T), block, 0, s, "fb_add_norm", a, cols);
+  return launch_after(add_norm4_kernel<In, Act, GROUPS, false>, dim3((unsigned)T), block, 0, s, "fb_add_norm", a, cols);
+}
+
 template <typename In, typename Act>
 static int launch_add_norm(const fb_branches& a, int64_t T, int64_t cols, cudaStream_t s) {
   static std::atomic<uint64_t> opted{0};
   if (first_on_device(opted)) cudaFuncSetAttribute(add_norm_kernel<In, Act>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
   const bool fours = cols % 4 == 0 && cols <= 4 * 4 * 512 && whole(a.x, a.ld_x, 4) && whole(a.mixer, a.ld_mixer, sizeof(In)) && whole(a.mixer_scale, 0, 4) &&
-                     whole(a.other, a.ld_other, sizeof(In)) && whole(a.other_scale, 0, 4) && whole(a.chosen, a.ld_chosen, sizeof(Act)) && whole(a.x_out, a.ld_x_out, 4) && whole(a.w, 0, 4) && whole(a.mixer_bias, 0, 4) && whole(a.own, a.ld_own, sizeof(Act)) &&
+                     whole(a.other, a.ld_other, sizeof(In)) && whole(a.other_scale, 0, 4) && whole(a.chosen, a.ld_chosen, sizeof(Act)) && whole(a.x_out, a.ld_x_out, 4) && whole(a.w, 0, 4) && whole(a.mixer_bias, 0, 4) && whole(a.own, a.ld_own, sizeof(Act)) && whole(a.gate, a.ld_gate, 4) &&
+                     whole(a.gate_bias, 0, 4) && whole(a.post, 0, 4) &&
                      whole(a.h, a.ld_h, sizeof(Act));
   const dim3 grid((unsigned)T);
   auto warps = [](int64_t work) { return dim3((unsigned)(work >= 512 ? 512 : ceil_div(work, 32) * 32)); };
@@ -477,9 +531,9 @@ static int launch_add_norm(const fb_branches& a, int64_t T, int64_t cols, cudaSt
   // few rows: a thread a group of four columns; many: fewer threads with more on their way each
   const int groups = cols > 4 * 1024 ? 4 : cols > 4 * 512 || T >= 512 ? 2 : 1;
   const dim3 block = warps(ceil_div(cols / 4, groups));
-  if (groups == 4) return launch_after(add_norm4_kernel<In, Act, 4>, grid, block, 0, s, "fb_add_norm", a, cols);
-  if (groups == 2) return launch_after(add_norm4_kernel<In, Act, 2>, grid, block, 0, s, "fb_add_norm", a, cols);
-  return launch_after(add_norm4_kernel<In, Act, 1>, grid, block, 0, s, "fb_add_norm", a, cols);
+  if (groups == 4) return launch_add_norm4<In, Act, 4>(a, T, block, cols, s);
+  if (groups == 2) return launch_add_norm4<In, Act, 2>(a, T, block, cols, s);
+  return launch_add_norm4<In, Act, 1>(a, T, block, cols, s);
 }
 
 }  // namespace fb
@@ -506,6 +560,7 @@ extern "C" int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void
   FB_REQUIRE(h.turned >= 0 && h.turned % 2 == 0 && h.turned <= h.dim && (!h.turned || (h.freq && h.places)), "fb_heads_put: an even number of a head's columns turn, by frequencies and places");
   FB_REQUIRE(!h.conv || (h.taps >= 1 && h.state && h.places && h.sequences >= 1 && T % h.sequences == 0 && (h.sequences == 1 || h.state_stride >= (h.taps - 1) * cols)),
              "fb_heads_put: a convolution takes its state, the places, and as many rows of each sequence");
+  FB_REQUIRE(h.temp_coef == 0.f || (h.places && h.temp_every > 0.f), "fb_heads_put: a temperature by place takes the places and a positive step");
   FB_REQUIRE(!h.norm_all || (h.q_norm && h.k_norm), "fb_heads_put: a norm over all heads takes its weights");
   FB_REQUIRE(!h.first || !(h.turned || h.conv || h.norm_all || h.keys_are_values), "fb_heads_put: mixed values go with plain heads");
   FB_REQUIRE(ld >= cols && ld_q >= (int64_t)h.heads * h.dim && cache_rows >= 1 && head_stride >= cache_rows * (h.dim + h.vdim), "fb_heads_put: row strides too small");
@@ -523,7 +578,8 @@ extern "C" int fb_add_norm(const fb_branches* branches_host, int64_t T, int64_t 
   FB_REQUIRE(branches_host && branches_host->x && T >= 1 && cols >= 1 && cols * 4 <= 200 * 1024, "fb_add_norm: null pointer, empty or rows past 51200 columns");
   const fb_branches& a = *branches_host;
   FB_REQUIRE(a.x_out || a.h, "fb_add_norm: no result");
-  FB_REQUIRE(!a.chosen || (a.slots && a.weights && a.k >= 1 && a.k <= 64), "fb_add_norm: chosen rows take their places and weights, up to 64 a token");
+  FB_REQUIRE(!a.gate || a.ld_gate >= cols, "fb_add_norm: a gate a column");
+  FB_REQUIRE(!a.chosen || (a.slots && a.k >= 1 && a.k <= 64), "fb_add_norm: chosen rows take their places, up to 64 a token");
   FB_REQUIRE((in_dtype == FB_BF16 || in_dtype == FB_FP32) && (dtype == FB_BF16 || dtype == FB_FP32) && (in_dtype == FB_FP32 || dtype == FB_BF16),
              "fb_add_norm: bf16 or fp32; fp32 results come from fp32");
   const auto s = (cudaStream_t)stream;

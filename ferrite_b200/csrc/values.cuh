@@ -22,6 +22,13 @@ __device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) { return ma
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
+// 2^x, the hardware's (x far below: 0)
+__device__ __forceinline__ float exp2_of(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // tanh by one exponential, and by its power series where that would cancel: about 2e-7 of the result either way
 __device__ __forceinline__ float tanh_of(float x) {
   const float y = x * x;

@@ -180,8 +180,7 @@ def kv_cache(c, size, zeros, slots=1):
 
 def slot(c, caches, u, slots):
     """Sequence u's part of caches made for several, in place."""
-    part = caches.size // slots
-    return mixers.Caches(part, [x[:, u * part:(u + 1) * part, :] for x in caches])
+    return mixers.slot(caches, u, slots)
 
 
 def random_weights(rt, c, prec=None, seed=0, scale=0.02):

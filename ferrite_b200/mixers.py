@@ -1,10 +1,10 @@
 """Layer parts beside the Llama block's (llama.attention, llama.mlp, llama.rms): token mixers that keep something per
-sequence, feed-forwards, a norm.  Every constant is a parameter; a design's module (binutar.py, labepel.py, vunadra.py) says which parts
-it is made of.
+sequence, feed-forwards, a norm.  Every constant is a parameter; a design's module (binutar.py, labepel.py, vunadra.py, ronavik.py) says
+which parts it is made of.
 
 They are: attention over cached latents, grouped-query attention within spans or windows of the sequence, with or without a
-rotation and a short convolution, linear attention with a decaying state; a clamped, a SiLU- and a GELU-gated unit, a mixture of
-experts; Dynamic Tanh.
+rotation and a short convolution, or weighted by sigmoids, linear attention with a decaying state, a state space whose decay is a token's
+own, a gated linear recurrence, and that beside attention; a clamped, a SiLU- and a GELU-gated unit, a mixture of experts; Dynamic Tanh.
 
 A mixer is a pair of functions: `*_cache(m, size, zeros, slots)` makes what it keeps for `slots` sequences of size / slots
 places each, and the mixer itself maps normed rows to rows, given its weights, its sizes m and where the tokens stand
@@ -23,6 +23,20 @@ class Caches(list):
     def __init__(self, size, caches):
         super().__init__(caches)
         self.size = size
+
+
+def slot(caches, u, slots):
+    """Sequence u's part of caches made for several, in place: of cached rows its run, of states (what follows the rows in a tuple; None stands
+    for no rows) its own."""
+    part = caches.size // slots
+    rows = lambda x: None if x is None else x[:, u * part:(u + 1) * part, :]
+    return Caches(part, [(rows(x[0]), *(s[u:u + 1, :, :] for s in x[1:])) if isinstance(x, tuple) else rows(x) for x in caches])
+
+
+def project(h, w):
+    """h @ w in fp32, its rows whole 16-byte pieces apart whatever w's width: parts of them are read four columns at a time."""
+    out = Tensor(h.rt, h.rows, -(-w.cols // 8) * 8, dtype="fp32")[:, :, :w.cols]
+    return h.matmul(w, dtype="fp32").realize(into=out)
 
 
 def dyt(x, p, name):
@@ -51,19 +65,21 @@ def gelu_mlp(h, p, pre):
     return unit.matmul(p[pre + "down"], dtype=h.dtype)
 
 
-def mixture(h, logits, p, pre, k, scored=False, identity=0, scale=1.0, clamp=None):
+def mixture(h, logits, p, pre, k, scored=False, identity=0, scale=1.0, clamp=None, as_scored=False, on_input=False):
     """A mixture of experts for rows h with their router logits (fp32): the k largest of each row's, weighted by their softmax.
     p: gate_up and down as batches of experts, the router's bias if it has one (router.b), a shared expert's own pair
-    (shared.gate_up, shared.down) if there is one.  scored: the softmax of all logits, with the bias, chooses, and without it
-    weighs; identity: the router's last so many outputs stand for experts that give back their input; scale: of the weights; clamp:
+    (shared.gate_up, shared.down) if there is one.  scored: the softmax of all logits ("sigmoid": each one's own sigmoid), with the bias,
+    chooses, and without it weighs, over the chosen ones' sum unless as_scored; on_input: a weight is on its expert's input; experts with an `up` instead of gate_up have
+    the unit max(up, 0)^2; identity: the router's last so many outputs stand for experts that give back their input; scale: of the weights; clamp:
     the experts' units are clamped ones (limit, slope).  Returns (the shared expert's result or None, (the chosen experts' rows,
     their routes)) as Tensor.add_norm adds them up."""
-    gate_up, down = p[pre + "gate_up"], p[pre + "down"]
-    routes = logits.route(gate_up.batch + identity, k, p.get(pre + "router.b"), scored, identity, scale)
+    relu2 = pre + "up" in p
+    gate_up, down = p[pre + ("up" if relu2 else "gate_up")], p[pre + "down"]
+    routes = logits.route(gate_up.batch + identity, k, p.get(pre + "router.b"), scored, identity, scale, as_scored, on_input)
     shared = gated_mlp(h, p, pre + "shared.") if pre + "shared.gate_up" in p else None
     if gate_up.dtype not in BFP:
-        return shared, (h.experts(routes, gate_up, down, clamp), routes)
-    assert not (identity or clamp), "block-float experts are plain ones"
+        return shared, (h.experts(routes, gate_up, down, clamp, relu2), routes)
+    assert not (identity or clamp or relu2 or on_input), "block-float experts are plain ones"
     of = lambda buf, dtype: Tensor(h.rt, routes.T, routes.k, dtype=dtype, buf=buf.view(1, routes.T, routes.k))
     y = llama.experts(h, {"experts.gate_up": gate_up, "experts.down": down}, of(routes.ids, "int32"), of(routes.weights, "fp32"))
     return (y if shared is None else shared + y), None
@@ -193,6 +209,19 @@ def turned_attention(h, p, m, eps, at, cache):
     return o.matmul(p["mix.o"], dtype=o.dtype)
 
 
+def sigmoid_width(m):
+    """Columns of the joint projection: queries, keys, values."""
+    return (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim
+
+
+def sigmoid_attention(joint, p, m, eps, at, cache, scale=1.0, into=None):
+    """Attention without a softmax: a key's weight is the sigmoid of its score and a number of the head (mix.pb).  joint: q | k | v, fp32; p: the heads'
+    norms (mix.q.norm, mix.k.norm); queries by the temperature of their place (m.q_temp).  The heads side by side times scale (into: there)."""
+    base, last, length, _ = at.seen
+    q = joint.heads_put(m.heads, m.dim, m.vdim, at.rows, cache, None, p["mix.q.norm"], p["mix.k.norm"], eps, places=at.places, temperature=m.q_temp and (m.q_temp.coef, m.q_temp.every))
+    return q.attend_heads(cache, base, last, m.vdim, m.scale, length, chunk=at.chunk, key_bias=p["mix.pb"], out_scale=scale, into=into)
+
+
 # -------------------------------------------------------------------- linear attention with a decaying state
 
 def decay_cache(m, size, zeros, slots):
@@ -210,3 +239,65 @@ def decay_attention(h, p, m, eps, at, state):
     qkvg = h.matmul(p["mix.qkvg"], dtype=h.dtype).silu_columns(n).realize()
     o = qkvg.decay_scan(H, m.dim, m.vdim, h.rt.numbers[key], at.places, state, at.dead)
     return o.gated_rms(qkvg[:, :, n:], p["mix.norm"], eps).matmul(p["mix.o"], dtype="fp32")
+
+
+# -------------------------------------------------------------------- a state space whose decay is a token's own
+
+def state_space_width(m):
+    """Columns of the joint projection: a gate and values (heads x vdim each), keys and queries (groups x state each), step sizes (heads)."""
+    return 2 * m.heads * m.vdim + 2 * m.groups * m.state + m.heads
+
+
+def state_space_cache(m, size, zeros, slots):
+    """No rows; what the convolution needs of earlier tokens, and a [state, vdim] matrix a head, fp32."""
+    return None, zeros((slots, max(m.conv - 1, 1), m.heads * m.vdim + 2 * m.groups * m.state), "fp32"), zeros((slots, m.heads * m.state, m.vdim), "fp32")
+
+
+def state_space(joint, p, m, eps, at, cache):
+    """joint: z | x | B | C | dt, fp32.  x, B and C through a short convolution and SiLU, the recurrence, the values beside it (mix.D), SiLU of z, RMSNorm in
+    m.norm_groups parts.  p: mix.conv, mix.conv.b, mix.dt_bias, mix.A_log, mix.D, mix.norm, mix.o."""
+    _, conv, state = cache
+    inner = m.heads * m.vdim
+    n = 2 * inner + 2 * m.groups * m.state
+    dtype = at.dtype
+    xbc = joint[:, :, inner:n].short_conv(p["mix.conv"], at.places, conv, at.dead, bias=p["mix.conv.b"], silu=True, dtype=dtype)
+    y = xbc.selective_scan(m.heads, m.groups, m.state, m.vdim, joint[:, :, n:n + m.heads], p["mix.dt_bias"], p["mix.A_log"], p["mix.D"], at.places, state, at.dead)
+    return y.gated_rms(joint[:, :, :inner], p["mix.norm"], eps, before=True, parts=m.norm_groups, dtype=dtype).matmul(p["mix.o"], dtype=dtype)
+
+
+# -------------------------------------------------------------------- a gated linear recurrence, and that beside attention
+
+LRU_RATE = -8.0  # log of the decay: this times a gate times the softplus of a number a column
+
+
+def recurrent_cache(m, size, zeros, slots):
+    """No rows; what the convolution needs of earlier tokens, and a number a column, fp32."""
+    return None, zeros((slots, max(m.conv - 1, 1), m.width), "fp32"), zeros((slots, 1, m.width), "fp32")
+
+
+def recurrent_block(joint, p, m, at, cache, scale=1.0, into=None):
+    """joint: y | x, fp32.  x through a short convolution, a gated linear recurrence whose gates are m.blocks matrices of their own (mix.gates: each block's
+    r | i), times the GELU of y.  p: mix.y.b, mix.x.b, mix.conv, mix.conv.b, mix.gates, mix.gates.b, mix.lam.  The result times scale (into: there)."""
+    _, conv, state = cache
+    u = joint[:, :, m.width:2 * m.width].short_conv(p["mix.conv"], at.places, conv, at.dead, bias=p["mix.conv.b"], in_bias=p["mix.x.b"], dtype=at.dtype)
+    gates = Tensor(joint.rt, joint.rows, 2 * m.width, dtype="fp32")
+    u.split(m.blocks).matmul(p["mix.gates"], dtype="fp32").realize(into=gates.split(m.blocks))
+    return u.lru_scan(gates, joint[:, :, :m.width], p["mix.lam"], LRU_RATE, m.blocks, at.places, state, at.dead, p["mix.gates.b"], p["mix.y.b"], scale, into)
+
+
+def parallel_width(m):
+    return sigmoid_width(m.left) + 2 * m.right.width
+
+
+def parallel_cache(m, size, zeros, slots):
+    return (heads_cache(m.left, size, zeros, slots), *recurrent_cache(m.right, size, zeros, slots)[1:])
+
+
+def parallel(joint, p, m, eps, at, cache):
+    """Attention and a recurrent block that read the same rows, each by a scale of its own.  joint: q | k | v | y | x, fp32; their output matrices are one
+    (mix.o), the attention's rows above the block's."""
+    n, wide = sigmoid_width(m.left), m.left.heads * m.left.vdim
+    both = Tensor(joint.rt, joint.rows, wide + m.right.width, dtype=at.dtype)
+    sigmoid_attention(joint[:, :, :n], p, m.left, eps, at, cache[0], m.left_scale, both[:, :, :wide])
+    recurrent_block(joint[:, :, n:], p, m.right, at, cache, m.right_scale, both[:, :, wide:])
+    return both.matmul(p["mix.o"], dtype=at.dtype)

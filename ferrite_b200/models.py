@@ -4,8 +4,8 @@ line) finds it here: by a config's `family`, or, when a checkpoint is opened, by
 import importlib
 from types import SimpleNamespace
 
-FAMILIES = {"llama": "llama", "binutar": "binutar", "labepel": "labepel", "vunadra": "vunadra"}  # a config's family -> its module of this package
-ARCHITECTURES = {"Binutar": "binutar", "Labepel": "labepel", "Vunadra": "vunadra"}  # config.json's "architecture" -> family (Hugging Face configs, which have none, are Llama-like)
+FAMILIES = {"llama": "llama", "binutar": "binutar", "labepel": "labepel", "vunadra": "vunadra", "ronavik": "ronavik"}  # a config's family -> its module of this package
+ARCHITECTURES = {"Binutar": "binutar", "Labepel": "labepel", "Vunadra": "vunadra", "Ronavik": "ronavik"}  # config.json's "architecture" -> family (Hugging Face configs, which have none, are Llama-like)
 
 
 def module(family):

@@ -312,9 +312,42 @@ def decay_scan(qkv, heads, dim, vdim, decay, places, dead, state, out):
     return out
 
 
-def gated_rmsnorm(x, gate, w, eps, out):
-    check(lib().fb_gated_rmsnorm(x.data_ptr(), x.shape[0], x.shape[1], x.stride(0), _CODES[gate.dtype], gate.data_ptr(), gate.stride(0), w.data_ptr(), eps,
-                                 out.data_ptr(), out.stride(0), _stream()))
+def selective_scan(xbc, heads, groups, dim, vdim, step, step_bias, a_log, skip, places, dead, state, out):
+    """A state space whose decay and step size are a token's own, over state [sequences, heads * dim, vdim] (fb_selective_scan)."""
+    sequences = state.shape[0]
+    assert state.stride(2) == 1 and state.stride(1) == vdim and places.dtype == torch.int32 and places.numel() == xbc.shape[0] and step.dtype == torch.float32 and step.stride(1) == 1
+    check(lib().fb_selective_scan(_CODES[xbc.dtype], xbc.data_ptr(), xbc.stride(0), heads, groups, dim, vdim, step.data_ptr(), step.stride(0), step_bias.data_ptr(), a_log.data_ptr(), skip.data_ptr(),
+                                  places.data_ptr(), dead, sequences, xbc.shape[0] // sequences, state.data_ptr(), state.stride(0), out.data_ptr(), out.stride(0), _stream()))
+    count()
+    return out
+
+
+def short_conv(x, w, out, places, dead, state=None, bias=None, in_bias=None, silu=False):
+    """A causal convolution over time of each column (fb_short_conv): w [taps, columns], state [sequences, >= taps - 1, columns]."""
+    taps, cols = w.shape
+    sequences = 1 if state is None else state.shape[0]
+    assert x.shape[1] == out.shape[1] == cols and w.is_contiguous() and (state is None or (state.dtype == torch.float32 and state.shape[1] >= taps - 1 and state.shape[2] == state.stride(1) == cols and state.stride(2) == 1))
+    c = _lib.Conv(cols, taps, w.data_ptr(), _ptr(bias), _ptr(in_bias), int(silu), places.data_ptr(), dead, sequences, x.shape[0] // sequences, _ptr(state), state.stride(0) if state is not None else 0)
+    check(lib().fb_short_conv(ctypes.byref(c), _CODES[x.dtype], x.data_ptr(), x.stride(0), _CODES[out.dtype], out.data_ptr(), out.stride(0), _stream()))
+    count()
+    return out
+
+
+def lru_scan(u, gates, y, out, lam, rate, blocks, places, dead, state, gate_bias=None, y_bias=None, scale=1.0):
+    """A gated linear recurrence per column times the GELU of y (fb_lru_scan): state [sequences, 1, width]."""
+    sequences, width = state.shape[0], u.shape[1]
+    assert state.shape[2] == width and state.stride(2) == 1 and state.dtype == gates.dtype == torch.float32 and u.dtype == out.dtype and gates.shape[1] == 2 * width and lam.numel() == width
+    l = _lib.Lru(width, blocks, lam.data_ptr(), rate, _ptr(gate_bias), _ptr(y_bias), scale, places.data_ptr(), dead, sequences, u.shape[0] // sequences, state.data_ptr(), state.stride(0))
+    check(lib().fb_lru_scan(ctypes.byref(l), _CODES[u.dtype], u.data_ptr(), u.stride(0), gates.data_ptr(), gates.stride(0), _CODES[y.dtype], y.data_ptr(), y.stride(0), out.data_ptr(), out.stride(0),
+                            _stream()))
+    count()
+    return out
+
+
+def gated_rmsnorm(x, gate, w, eps, out, before=False, parts=1):
+    """RMSNorm of x's rows in equal parts by w, times the sigmoid of gate (before: of x times its SiLU) (fb_gated_rmsnorm)."""
+    check(lib().fb_gated_rmsnorm(x.data_ptr(), x.shape[0], x.shape[1], x.stride(0), _CODES[gate.dtype], gate.data_ptr(), gate.stride(0), int(before), w.data_ptr(), eps, parts,
+                                 _CODES[out.dtype], out.data_ptr(), out.stride(0), _stream()))
     count()
     return out
 
@@ -346,13 +379,14 @@ def embed(table, ids, places_table, places, out, scale=1.0):
 
 
 def heads_put(qkv, heads, kv_heads, dim, vdim, rows, cache, q_out, bias=None, q_norm=None, k_norm=None, eps=0.0, first=None, first_bias=None, share=None,
-              norm_all=False, keys_are_values=False, rotation=None, places=None, conv=None, state=None, dead=-1):
+              norm_all=False, keys_are_values=False, rotation=None, places=None, conv=None, state=None, dead=-1, temperature=(0.0, 1.0)):
     """Biases, convolution, norms, turn, values and the cache write after a joint projection of heads (fb_heads_put); cache [kv_heads,
-    rows, dim + vdim]; rotation: (frequencies, columns that turn, factor); conv [taps, columns] and state [sequences, taps - 1, columns]."""
+    rows, dim + vdim]; rotation: (frequencies, columns that turn, factor); conv [taps, columns] and state [sequences, taps - 1, columns];
+    temperature: (coefficient, places a step)."""
     freq, dims, mag = rotation or (None, 0, 1.0)
     h = _lib.Heads(heads, kv_heads, dim, vdim, _ptr(bias), _ptr(q_norm), _ptr(k_norm), eps, _ptr(first), first.stride(0) if first is not None else 0, _ptr(first_bias), _ptr(share),
                    int(norm_all), int(keys_are_values), dims, _ptr(freq) if dims else None, mag, _ptr(places), conv.shape[0] if conv is not None else 0, _ptr(conv), _ptr(state),
-                   state.stride(0) if state is not None else 0, state.shape[0] if state is not None else 1, dead)
+                   state.stride(0) if state is not None else 0, state.shape[0] if state is not None else 1, dead, *temperature)
     assert conv is None or (conv.is_contiguous() and state.dtype == conv.dtype == torch.float32 and state.shape[2] == state.stride(1) == conv.shape[1] and state.stride(2) == 1 and state.shape[1] >= conv.shape[0] - 1)
     assert cache.shape[0] == kv_heads and cache.shape[2] == dim + vdim and cache.stride(2) == 1 and cache.stride(1) == dim + vdim and q_out.dtype == cache.dtype
     check(lib().fb_heads_put(ctypes.byref(h), _CODES[qkv.dtype], qkv.data_ptr(), qkv.shape[0], qkv.stride(0), rows.data_ptr(), _CODES[cache.dtype], q_out.data_ptr(), q_out.stride(0),
@@ -361,7 +395,8 @@ def heads_put(qkv, heads, kv_heads, dim, vdim, rows, cache, q_out, bias=None, q_
     return q_out
 
 
-def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, span=0, sink=None, gate=None, row0=0, out=None, window=0, softcap=0.0):
+def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, span=0, sink=None, gate=None, row0=0, out=None, window=0, softcap=0.0, key_bias=None,
+                    out_scale=1.0):
     """q [T, heads * dim] over cache [kv_heads, rows, dim + vdim] (fb_heads_attention)."""
     T, dim = q.shape[0], cache.shape[2] - vdim
     assert q.shape[1] == heads * dim and q.dtype == cache.dtype and cache.stride(2) == 1 and cache.stride(1) == cache.shape[2]
@@ -369,7 +404,7 @@ def heads_attention(q, cache, base, last, heads, vdim, scale, max_keys, chunk, s
     if out is None:
         out = torch.empty(T, heads * vdim, dtype=q.dtype, device=q.device)
     check(lib().fb_heads_attention(_CODES[q.dtype], q.data_ptr(), T, q.stride(0), heads, cache.shape[0], dim, vdim, cache.data_ptr(), cache.shape[1], cache.stride(0), _ptr(base), row0,
-                                   last.data_ptr(), max_keys, int(chunk), span, window, scale, softcap, _ptr(sink), _CODES[gate.dtype] if gate is not None else 0, _ptr(gate),
+                                   last.data_ptr(), max_keys, int(chunk), span, window, scale, softcap, _ptr(sink), _ptr(key_bias), out_scale, _CODES[gate.dtype] if gate is not None else 0, _ptr(gate),
                                    gate.stride(0) if gate is not None else 0, out.data_ptr(), out.stride(0), _stream()))
     count()
     return out
@@ -385,6 +420,7 @@ class Routes:
         i32 = lambda *shape: torch.empty(*shape, dtype=torch.int32, device=device)
         self.weights, self.ids, self.slots = torch.empty(T, k, dtype=torch.float32, device=device), i32(T, k), i32(T, k)
         self.tile_expert, self.live = i32(self.tiles, 3), i32(1)
+        self.row_weights = None  # where weights go on the experts' inputs: each row's
 
 
 @functools.lru_cache
@@ -401,14 +437,20 @@ def route_tile(T, n, k):
     return min(range(32, 257, 16), key=work), False
 
 
-def route(logits, n, k, bias=None, scored=False, identity=0, scale=1.0):
-    """Router logits (fp32 [T, >= n]) to Routes; scored, identity, scale: fb_router's."""
+SCORES = {False: 0, None: 0, True: 1, "softmax": 1, "sigmoid": 2}  # fb_router's scored
+
+
+def route(logits, n, k, bias=None, scored=False, identity=0, scale=1.0, as_scored=False, on_input=False):
+    """Router logits (fp32 [T, >= n]) to Routes; scored, identity, scale, as_scored: fb_router's; on_input: the weights by row, too."""
     T = logits.shape[0]
     tile, shared = route_tile(T, n, k)
     r = Routes(logits.device, T, n - identity, k, tile, shared)
-    router = _lib.Router(n, k, identity, _ptr(bias), int(scored), scale)
+    router = _lib.Router(n, k, identity, _ptr(bias), SCORES[scored], scale, int(as_scored))
+    if on_input:
+        assert not identity, "weights on the inputs go with experts that have rows"
+        r.row_weights = torch.empty(r.tiles * tile, dtype=torch.float32, device=logits.device)
     check(lib().fb_route(ctypes.byref(router), logits.data_ptr(), T, logits.stride(0), tile, int(shared), r.weights.data_ptr(), r.ids.data_ptr(), r.slots.data_ptr(),
-                         r.tile_expert.data_ptr(), r.live.data_ptr(), _stream()))
+                         r.tile_expert.data_ptr(), r.live.data_ptr(), _ptr(r.row_weights), _stream()))
     count(1 if T <= 32 else 2)
     return r
 
@@ -436,26 +478,27 @@ def grouped(x, w, routes, out, kind=_lib.DENSE_NONE, shared=False, **extra):
     return True
 
 
-def grouped_matmul(x, w, routes, out, shared=False):
-    """The same without a unit for any sizes, bf16 or fp32 (fb_grouped_matmul)."""
+def grouped_matmul(x, w, routes, out, shared=False, row_scale=None):
+    """The same without a unit for any sizes, bf16 or fp32 (fb_grouped_matmul); row_scale: a number a row of the result."""
     n, K, N = w.shape
     assert x.stride(1) == 1 and out.stride(1) == 1
     check(lib().fb_grouped_matmul(_CODES[x.dtype], x.data_ptr(), x.shape[0], x.stride(0), int(shared), _CODES[w.dtype], w.data_ptr(), (ctypes.c_int64 * 3)(*w.stride()), n, K, N,
-                                  routes.tile_expert.data_ptr(), routes.live.data_ptr(), routes.tiles, routes.tile, _CODES[out.dtype], out.data_ptr(), out.stride(0), _stream()))
+                                  routes.tile_expert.data_ptr(), routes.live.data_ptr(), routes.tiles, routes.tile, _ptr(row_scale), _CODES[out.dtype], out.data_ptr(), out.stride(0), _stream()))
     count()
     return out
 
 
 def add_norm(x, x_out, mixer=None, mixer_scale=None, other=None, other_scale=None, chosen=None, routes=None, w=None, plus=0.0, eps=0.0, h=None,
-             mixer_bias=None, own=None):
-    """A layer's end (fb_add_norm): x [T, cols] fp32 plus its branches into x_out, and that normed by w + plus (w None: as it is) into h."""
+             mixer_bias=None, own=None, gate=None, gate_bias=None, post=None):
+    """A layer's end (fb_add_norm): x [T, cols] fp32 plus its branches (their sum gated and normed, where given) into x_out, and that normed by
+    w + plus (w None: as it is) into h."""
     ld = lambda t: t.stride(0) if t is not None else 0
     of = lambda *ts: next((t.dtype for t in ts if t is not None), None)
     dtype = of(h, chosen) or torch.float32
     kind = of(mixer, other) or dtype if dtype == torch.bfloat16 else torch.float32
     assert all(t is None or t.dtype == kind for t in (mixer, other)) and all(t is None or t.dtype == dtype for t in (h, chosen, own))
     b = _lib.Branches(x.data_ptr(), ld(x), _ptr(mixer), ld(mixer), _ptr(mixer_scale), _ptr(other), ld(other), _ptr(other_scale), _ptr(chosen), ld(chosen),
-                      _ptr(routes.slots) if routes else None, _ptr(routes.weights) if routes else None, routes.k if routes else 0, _ptr(x_out), ld(x_out), _ptr(w), plus, eps, _ptr(h), ld(h),
-                      _ptr(mixer_bias), _ptr(own), ld(own))
+                      _ptr(routes.slots) if routes else None, _ptr(routes.weights) if routes and routes.row_weights is None else None, routes.k if routes else 0, _ptr(x_out), ld(x_out), _ptr(w), plus, eps, _ptr(h), ld(h),
+                      _ptr(mixer_bias), _ptr(own), ld(own), _ptr(gate), ld(gate), _ptr(gate_bias), _ptr(post))
     check(lib().fb_add_norm(ctypes.byref(b), x.shape[0], x.shape[1], _CODES[kind], _CODES[dtype], _stream()))
     count()

@@ -619,11 +619,47 @@ class Tensor:
         self.rt.launched("decay scan")
         return out
 
-    def gated_rms(self, gate, w, eps):
-        """RMSNorm of self (fp32 rows) by w, times the sigmoid of gate, as gate is stored."""
+    def selective_scan(self, heads, groups, dim, vdim, step, step_bias, a_log, skip, places, state, dead=-1):
+        """self: rows of values (heads x vdim) | keys (groups x dim) | queries (groups x dim), as decay_scan's sequences; step: fp32, a number a row and
+        head.  With d = softplus(step + step_bias): S = exp(-exp(a_log) d) S + d k v^T, o = S^T q + skip v per head.  Returns fp32 [1, tokens, heads vdim]."""
+        x, step, places = self.realize(), step.realize(), places.realize()
+        assert x.batch == 1 and x.buf.stride(2) == 1 and state.dtype == "fp32" and state.shape[1:] == (heads * dim, vdim) and x.rows % state.batch == 0
+        assert step.dtype == "fp32" and step.shape == (1, x.rows, heads) and all(t.dtype == "fp32" and t.cols == heads for t in (step_bias, a_log, skip))
+        out = Tensor(self.rt, x.rows, heads * vdim, dtype="fp32")
+        ops.selective_scan(x.buf[0], heads, groups, dim, vdim, step.buf[0], step_bias.buf, a_log.buf, skip.buf, places.buf.reshape(-1), dead, state.buf, out.buf[0])
+        self.rt.launched("selective scan")
+        return out
+
+    def short_conv(self, w, places, state, dead=-1, bias=None, in_bias=None, silu=False, dtype="bf16"):
+        """self: rows of one sequence, or one row of each of state.batch sequences.  A causal convolution over time of every column by w ([taps,
+        columns], fp32; in_bias joins before it, bias after), then SiLU; state ([sequences, >= taps - 1, columns], fp32, read and written): the inputs
+        of earlier tokens - zeros at place 0; a sequence at place `dead` leaves it alone."""
+        x, places = self.realize(), places.realize()
+        assert x.batch == 1 and x.buf.stride(2) == 1 and all(t is None or (t.dtype == "fp32" and t.cols == x.cols) for t in (w, bias, in_bias, state)) and x.rows % state.batch == 0
+        out = Tensor(self.rt, x.rows, x.cols, dtype=dtype)
+        buf = lambda t: None if t is None else t.buf
+        ops.short_conv(x.buf[0], w.buf[0], out.buf[0], places.buf.reshape(-1), dead, state.buf, buf(bias), buf(in_bias), silu)
+        self.rt.launched("short conv")
+        return out
+
+    def lru_scan(self, gates, y, lam, rate, blocks, places, state, dead=-1, gate_bias=None, y_bias=None, scale=1.0, into=None):
+        """self: rows as short_conv's; gates: fp32, a block's r columns and then its i columns, block after block.  With r and i their sigmoids and
+        log a = rate r softplus(lam): S = a S + sqrt(1 - a^2) i self per column, and the result is scale S gelu(y); state: fp32 [sequences, 1, columns]."""
+        x, gates, y, places = self.realize(), gates.realize(), y.realize(), places.realize()
+        out = into if into is not None else Tensor(self.rt, x.rows, x.cols, dtype=x.dtype)
+        assert x.batch == 1 and x.buf.stride(2) == gates.buf.stride(2) == y.buf.stride(2) == out.buf.stride(2) == 1 and y.shape == x.shape == out.shape and gates.shape == (1, x.rows, 2 * x.cols)
+        assert all(t is None or t.dtype == "fp32" for t in (lam, gate_bias, y_bias, state)) and (gate_bias is None or gate_bias.buf.is_contiguous()) and x.rows % state.batch == 0
+        buf = lambda t: None if t is None else t.buf
+        ops.lru_scan(x.buf[0], gates.buf[0], y.buf[0], out.buf[0], lam.buf, rate, blocks, places.buf.reshape(-1), dead, state.buf, buf(gate_bias), buf(y_bias), scale)
+        self.rt.launched("lru scan")
+        return out
+
+    def gated_rms(self, gate, w, eps, before=False, parts=1, dtype=None):
+        """RMSNorm of self (fp32 rows), each of its equal parts by its own root mean square, by w, times the sigmoid of gate; before: self times the
+        SiLU of gate is what is normed.  As gate is stored, or as dtype."""
         x, gate = self.realize(), gate.realize()
-        out = Tensor(self.rt, x.rows, x.cols, dtype=gate.dtype)
-        ops.gated_rmsnorm(x.buf[0], gate.buf[0], w.buf, eps, out.buf[0])
+        out = Tensor(self.rt, x.rows, x.cols, dtype=dtype or gate.dtype)
+        ops.gated_rmsnorm(x.buf[0], gate.buf[0], w.buf, eps, out.buf[0], before, parts)
         self.rt.launched("gated rmsnorm")
         return out
 
@@ -639,14 +675,14 @@ class Tensor:
         return out
 
     def heads_put(self, heads, dim, vdim, rows, cache, bias=None, q_norm=None, k_norm=None, eps=0.0, mix=None, norm_all=False,
-                  keys_are_values=False, rotation=None, places=None, conv=None, state=None, dead=-1):
+                  keys_are_values=False, rotation=None, places=None, conv=None, state=None, dead=-1, temperature=None):
         """self: a joint projection [1, tokens, q (heads x dim) | k | v (| more)]; its keys and values go into `cache` ([key
         heads, size, dim + vdim]) at `rows`, its queries come back, as the cache is stored.  bias: a number a column of q | k | v;
         q_norm, k_norm: RMSNorm of each head (norm_all: of all of them together); mix: (other values of the tokens, their bias or
         None, share): the values become (1 - share) own + share other; keys_are_values: there is no v, the keys as projected are the
         values; rotation: mixers.rotation's, by `places`; conv ([taps, columns]): a short convolution over time of every column, state
         ([sequences, taps - 1, columns], fp32, read and written) what it needs of earlier tokens - nothing at place 0, and a sequence
-        at place `dead` leaves it alone."""
+        at place `dead` leaves it alone; temperature: (coef, every): queries, after their norm, times 1 + coef ln(floor((place + 1) / every) + 1)."""
         x, rows = self.realize(), rows.realize()
         wide = (heads + cache.batch) * dim + (0 if keys_are_values else cache.batch * vdim)
         assert x.batch == 1 and x.buf.stride(2) == 1 and rows.cols == x.rows and x.cols >= wide, f"{self.shape} into a cache {cache.shape}"
@@ -658,41 +694,44 @@ class Tensor:
         out = Tensor(self.rt, x.rows, heads * dim, dtype=cache.dtype)
         ops.heads_put(x.buf[0], heads, cache.batch, dim, vdim, rows.buf.reshape(-1), cache.buf, out.buf[0], buf(bias), buf(q_norm), buf(k_norm), eps,
                       None if first is None else first.buf[0], buf(first_bias), buf(share), norm_all, keys_are_values, rotation, None if places is None else places.realize().buf.reshape(-1),
-                      None if conv is None else conv.realize().buf[0], buf(state), dead)
+                      None if conv is None else conv.realize().buf[0], buf(state), dead, temperature or (0.0, 1.0))
         self.rt.launched("heads put")
         return out
 
-    def attend_heads(self, cache, base, last, vdim, scale, length=None, span=0, sink=None, gate=None, chunk=False, window=0, softcap=0.0):
+    def attend_heads(self, cache, base, last, vdim, scale, length=None, span=0, sink=None, gate=None, chunk=False, window=0, softcap=0.0, key_bias=None,
+                     out_scale=1.0, into=None):
         """self: [1, tokens, heads x dim] over such a cache.  Token t, which stands at place last[t], attends the rows from base[t]
         on up to its own; with span, only those of its own span of that many places, with window, only the last so many.  softcap: c
         > 0 makes a scaled score s c tanh(s / c).  sink: a number per head that joins the
-        softmax's denominator; gate: the result is multiplied by its sigmoid, column by column; chunk: one sequence's tokens,
-        its first cache row 0.  Returns [1, tokens, heads x vdim]."""
+        softmax's denominator; key_bias: a number per head, no softmax: a key's weight is the sigmoid of its score and that; gate: the result is multiplied by
+        its sigmoid, column by column; chunk: one sequence's tokens, its first cache row 0.  Returns [1, tokens, heads x vdim] times out_scale (into: there)."""
         q, last = self.realize(), last.realize()
         dim = cache.cols - vdim
         assert q.batch == 1 and q.cols % dim == 0 and q.dtype == cache.dtype and (q.cols // dim) % cache.batch == 0, f"{q.shape} over a cache {cache.shape}"
         heads = q.cols // dim
-        out = Tensor(self.rt, q.rows, heads * vdim, dtype=q.dtype)
-        assert gate is None or gate.shape == out.shape
+        out = into if into is not None else Tensor(self.rt, q.rows, heads * vdim, dtype=q.dtype)
+        assert (gate is None or gate.shape == out.shape) and out.shape == (1, q.rows, heads * vdim) and out.dtype == q.dtype and out.buf.stride(2) == 1
         ops.heads_attention(q.buf[0], cache.buf, None if chunk else base.realize().buf.reshape(-1), last.buf.reshape(-1), heads, vdim, scale, min(length or cache.rows, cache.rows), chunk, span,
-                            None if sink is None else sink.realize().buf, None if gate is None else gate.realize().buf[0], out=out.buf[0], window=window, softcap=softcap)
+                            None if sink is None else sink.realize().buf, None if gate is None else gate.realize().buf[0], out=out.buf[0], window=window, softcap=softcap,
+                            key_bias=None if key_bias is None else key_bias.realize().buf, out_scale=out_scale)
         self.rt.launched("attention")
         return out
 
-    def route(self, n, k, bias=None, scored=False, identity=0, scale=1.0):
-        """self: fp32 router logits, n a token: each token's k experts, their weights and where their rows go (ops.Routes).  scored: chosen
-        by softmax + bias, weighted by the softmax; identity: the last so many give back their input; scale: of the weights."""
+    def route(self, n, k, bias=None, scored=False, identity=0, scale=1.0, as_scored=False, on_input=False):
+        """self: fp32 router logits, n a token: each token's k experts, their weights and where their rows go (ops.Routes).  scored ("softmax",
+        "sigmoid"): chosen by score + bias, weighted by the scores, over their sum unless as_scored; identity: the last so many give back their input; scale: of
+        the weights; on_input: they go on the experts' inputs."""
         x = self.realize()
         assert x.dtype == "fp32" and x.batch == 1 and x.cols == n and x.buf.stride(2) == 1 and (bias is None or (bias.dtype == "fp32" and bias.cols == n))
         self.rt.launched("route")
-        return ops.route(x.buf[0], n, k, None if bias is None else bias.realize().buf, scored, identity, scale)
+        return ops.route(x.buf[0], n, k, None if bias is None else bias.realize().buf, scored, identity, scale, as_scored, on_input)
 
-    def experts(self, routes, gate_up, down, clamp=None):
+    def experts(self, routes, gate_up, down, clamp=None, relu2=False):
         """self: rows of tokens.  Every chosen expert's down(silu(gate) * up) of its tokens' rows, a row a choice where `routes`
         puts it; gate and up side by side in gate_up [n, K, 2 m], down [n, m, N].  clamp: (limit, slope) of clamped_glu in the
-        unit's place."""
+        unit's place; relu2: max(up, 0)^2, and gate_up [n, K, m] is up alone.  A weight on an input scales the products of its row before the unit."""
         rt, h, m = self.rt, self.realize(), down.rows
-        assert h.batch == 1 and gate_up.cols == 2 * m and gate_up.batch == down.batch == routes.n and h.rows == routes.T
+        assert h.batch == 1 and gate_up.cols == (m if relu2 else 2 * m) and gate_up.batch == down.batch == routes.n and h.rows == routes.T
         if not routes.shared:
             x = Tensor(rt, routes.tiles * routes.tile, h.cols, dtype=h.dtype)
             ops.spread_rows(h.buf[0], routes, x.buf[0])
@@ -700,15 +739,20 @@ class Tensor:
             h = x
         act = Tensor(rt, routes.tiles * routes.tile, m, dtype=h.dtype)
         out = Tensor(rt, routes.tiles * routes.tile, down.cols, dtype=h.dtype)
-        unit = dict(kind=_lib.DENSE_GLU, limit=clamp[0], slope=clamp[1]) if clamp else dict(kind=_lib.DENSE_SWIGLU)
-        if ops.grouped(h.buf[0], gate_up.buf, routes, act.buf[0], shared=routes.shared, **unit):
-            rt.launched("experts glu" if clamp else "experts swiglu")
+        weights = routes.row_weights
+        unit = dict(kind=_lib.DENSE_RELU2) if relu2 else dict(kind=_lib.DENSE_GLU, limit=clamp[0], slope=clamp[1]) if clamp else dict(kind=_lib.DENSE_SWIGLU)
+        if ops.grouped(h.buf[0], gate_up.buf, routes, act.buf[0], shared=routes.shared, row_scale=None if weights is None else weights.data_ptr(), **unit):
+            rt.launched("experts relu2" if relu2 else "experts glu" if clamp else "experts swiglu")
         else:
-            both = Tensor(rt, act.rows, 2 * m, dtype="fp32")
-            ops.grouped_matmul(h.buf[0], gate_up.buf, routes, both.buf[0], routes.shared)
+            both = Tensor(rt, act.rows, gate_up.cols, dtype="fp32")
+            ops.grouped_matmul(h.buf[0], gate_up.buf, routes, both.buf[0], routes.shared, weights)
             rt.launched("experts matmul")
-            gate, up = both[:, :m], both[:, m:]
-            (clamped_glu(gate, up, *clamp) if clamp else gate.silu() * up).cast(h.dtype).realize(into=act)
+            if relu2:
+                up = both.relu()
+                (up * up).cast(h.dtype).realize(into=act)
+            else:
+                gate, up = both[:, :m], both[:, m:]
+                (clamped_glu(gate, up, *clamp) if clamp else gate.silu() * up).cast(h.dtype).realize(into=act)
         if ops.grouped(act.buf[0], down.buf, routes, out.buf[0]):
             rt.launched("experts")
         else:
@@ -717,19 +761,22 @@ class Tensor:
         return out
 
     def add_norm(self, w, eps, plus=0.0, dtype="bf16", mixer=None, mixer_scale=None, other=None, other_scale=None, experts=None,
-                 mixer_bias=None, own=None, into=None):
+                 mixer_bias=None, own=None, into=None, gate=None, gate_bias=None, post=None):
         """self: an fp32 residual stream.  (self + (mixer + mixer_bias) * mixer_scale + (other + the experts' rows by their weights) *
         other_scale, and that as RMSNorm by w + plus leaves it, or, w None, as it is); experts: (rows, routes), own: the row that an
-        identity expert gives back.  Without branches: (self, its norm).  into: where the second goes."""
+        identity expert gives back.  gate (fp32, with gate_bias): the branches' sum is multiplied by its sigmoid, and post: goes through RMSNorm by it, before it joins
+        the stream.  Without branches: (self, its norm).  into: where the second goes."""
         x = self.realize()
         get = lambda t: None if t is None else t.realize().buf[0]
-        assert x.dtype == "fp32" and x.batch == 1 and all(t is None or (t.shape == x.shape and t.buf.stride(2) == 1) for t in (mixer and mixer.realize(), other and other.realize()))
+        assert x.dtype == "fp32" and x.batch == 1 and all(t is None or (t.shape == x.shape and t.buf.stride(2) == 1) for t in (mixer and mixer.realize(), other and other.realize(), gate and gate.realize()))
+        assert gate is None or gate.dtype == "fp32"
         bare = mixer is other is experts is mixer_bias is None
         out, h = x if bare else Tensor(self.rt, x.rows, x.cols, dtype="fp32"), into if into is not None else Tensor(self.rt, x.rows, x.cols, dtype=dtype)
         assert h.shape == x.shape and h.dtype == dtype and h.buf.stride(2) == 1
         scale = lambda t: None if t is None else t.realize().buf
         rows, routes = experts or (None, None)
-        ops.add_norm(x.buf[0], None if bare else out.buf[0], get(mixer), scale(mixer_scale), get(other), scale(other_scale), get(rows), routes, scale(w), plus, eps, h.buf[0], scale(mixer_bias), get(own))
+        ops.add_norm(x.buf[0], None if bare else out.buf[0], get(mixer), scale(mixer_scale), get(other), scale(other_scale), get(rows), routes, scale(w), plus, eps, h.buf[0], scale(mixer_bias), get(own),
+                     get(gate), scale(gate_bias), scale(post))
         self.rt.launched("norm" if bare else "add norm")
         return out, h
 

@@ -173,7 +173,7 @@ def layer(x, h, p, b, c, at, cache, norm, into=None):
         return x.add_norm(norm, mixer=mixers.gelu_mlp(h, p, "mlp."), mixer_bias=p["mlp.down.b"], into=into, **ends)
     r = b.mlp.router
     logits = h.matmul(p["mlp.router"], dtype="fp32")
-    _, experts = mixers.mixture(h, logits, p, "mlp.", r.top, scored=True, identity=r.identity, scale=r.scale, clamp=(b.mlp.expert.limit, GLU_SLOPE))
+    _, experts = mixers.mixture(h, logits, p, "mlp.", r.top, scored="softmax", identity=r.identity, scale=r.scale, clamp=(b.mlp.expert.limit, GLU_SLOPE))
     return x.add_norm(norm, experts=experts, own=h, into=into, **ends)
 
 
@@ -219,9 +219,7 @@ def kv_cache(c, size, zeros, slots=1):
 
 def slot(c, caches, u, slots):
     """Sequence u's part of caches made for several, in place."""
-    part = caches.size // slots
-    rows = lambda x: x[:, u * part:(u + 1) * part, :]
-    return mixers.Caches(part, [(rows(x[0]), x[1][u:u + 1, :, :]) if isinstance(x, tuple) else rows(x) for x in caches])
+    return mixers.slot(caches, u, slots)
 
 
 def random_weights(rt, c, prec=None, seed=0, scale=0.02):

@@ -152,7 +152,8 @@ enum fb_dense_epilogue_kind {
   FB_DENSE_DYT_ADD = 4, /* out (fp32) = residual + tanh(alpha acc) w + b, and, with h_out given, h_out (bf16) = tanh(alpha2 out) w2 + b2: a Dynamic
                            Tanh on a branch, the residual add, and the Dynamic Tanh that the next branch starts with */
   FB_DENSE_SWIGLU = 5,  /* as FB_DENSE_GLU, the plain unit: out = g sigmoid(g) u */
-  FB_DENSE_GEGLU = 6    /* as FB_DENSE_GLU: out = gelu(gate + gate_bias) (up + up_bias), GELU's tanh form */
+  FB_DENSE_GEGLU = 6,   /* as FB_DENSE_GLU: out = gelu(gate + gate_bias) (up + up_bias), GELU's tanh form */
+  FB_DENSE_RELU2 = 7    /* out = max(v, 0)^2 */
 };
 typedef struct {
   int kind;
@@ -167,6 +168,7 @@ typedef struct {
   int64_t ld_h;
   const float *alpha2, *w2, *b2;
   const float *gate_bias, *up_bias; /* GEGLU: [N / 2] each, or null */
+  const float* row_scale;           /* GLU, SWIGLU, RELU2: row t's sums times row_scale[t] before the unit (a weight on its input), or null */
 } fb_dense_epilogue;
 /* batch independent matmuls: x, W and out move on by x_batch, w_batch and out_batch elements an entry (x_batch 0: all take the
  * same rows).  ldx, ldw, x_batch, w_batch multiples of 8 elements, x and W 16-byte aligned, K a multiple of 8 (GLU: N / 2 a
@@ -183,18 +185,20 @@ typedef struct {
   int identity;      /* the last so many outputs stand for experts that give back their input: they have no rows */
   const float* bias; /* [n] or null: joins what the choice goes by and, unless scored, the weights */
   int scored;        /* 0: choices by logit + bias, weights the softmax of the chosen; 1: scores = softmax of all logits, choices by
-                        score + bias, weights the chosen scores over their sum (+ 1e-20) */
+                        score + bias, weights the chosen scores over their sum (+ 1e-20); 2: likewise, scores = sigmoid of each logit */
   float scale;       /* the weights times this */
+  int as_scored;     /* the weights are the chosen scores themselves, not over their sum */
 } fb_router;
 /* Each token's k largest of its router's n outputs (fp32 logits; the lower column first among equals), their weights, and
  * where each choice's row goes (slots, both [T, k]; -1: an identity expert's) in rows of whole tiles of `tile` (a multiple of 16):
  *   shared_rows   a tile a touched expert, holding all the tokens (T <= tile): the choice's row is the token's in its expert's tile
  *   otherwise     each expert's choices in tiles of their own
  * tile_expert[tiles, 3]: each tile's expert, ascending (past those used: the number of experts with rows), that expert's first tile and its number
- * of tiles; live[0]: how many are used; tiles = fb_route_tiles(...) of the experts with rows, the most there can be.  ids [T, k]: the choices. */
+ * of tiles; live[0]: how many are used; tiles = fb_route_tiles(...) of the experts with rows, the most there can be.  ids [T, k]: the choices.
+ * row_weights (or null): each choice's weight once more, at its row (rows that are no choice's are left alone). */
 int64_t fb_route_tiles(int64_t T, int n, int k, int tile, int shared_rows);
 int fb_route(const fb_router* router_host, const float* logits, int64_t T, int64_t ld, int tile, int shared_rows, float* weights, int32_t* ids,
-             int32_t* slots, int32_t* tile_expert, int32_t* live, void* stream);
+             int32_t* slots, int32_t* tile_expert, int32_t* live, float* row_weights, void* stream);
 
 /* Row t of x (row_bytes bytes, rows ldx_bytes apart) into the rows slots[t, 0 .. k) of out (rows one after another): the
  * tokens' rows to their choices' places. */
@@ -204,12 +208,13 @@ int fb_spread_rows(const void* x, int64_t T, int64_t row_bytes, int64_t ldx_byte
 /* Rows of tiles by each tile's own matrix: rows i * tile .. of out = rows i * tile .. of x (shared_rows: x's `x_rows` rows, the
  * same for every tile) @ W[tile_expert[i, 0]]^T for the tiles i < live[0]; the other rows of out are left alone.
  * fb_dense_grouped: on the tensor cores, operands as fb_dense takes them (W [n, N, K], w_batch elements apart), epilogues
- * FB_DENSE_NONE, FB_DENSE_GLU and FB_DENSE_SWIGLU.  fb_grouped_matmul: any sizes, bf16 or fp32, W by strides (matrix, row of K, column). */
+ * FB_DENSE_NONE, FB_DENSE_GLU, FB_DENSE_SWIGLU and FB_DENSE_RELU2 (row_scale: one a row of out).  fb_grouped_matmul: any sizes, bf16 or
+ * fp32, W by strides (matrix, row of K, column); row_scale (or null): each row of the result times its own. */
 int fb_dense_grouped(const void* x, int64_t x_rows, int64_t K, int64_t ldx, int shared_rows, const void* W, int64_t N, int64_t ldw, int64_t w_batch,
                      int n, const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, void* out, int out_dtype, int64_t ldo,
                      const fb_dense_epilogue* epilogue_host, void* stream);
 int fb_grouped_matmul(int x_dtype, const void* x, int64_t x_rows, int64_t ldx, int shared_rows, int w_dtype, const void* W, const int64_t* w_strides_host, int n,
-                      int64_t K, int64_t N, const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, int out_dtype, void* out,
+                      int64_t K, int64_t N, const int32_t* tile_expert, const int32_t* live, int64_t tiles, int tile, const float* row_scale, int out_dtype, void* out,
                       int64_t ldo, void* stream);
 
 /* Tensor.matmul(index=) (ferrite/tensor.py:450-460; ferrite/compiler.py:704-706): a mixture of experts' matmul.  W is
@@ -406,9 +411,55 @@ int fb_latent_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int h
 int fb_decay_scan(int dtype, const void* qkv, int64_t ld, int heads, int dim, int vdim, const float* decay, const int32_t* places, int dead,
                   int64_t sequences, int64_t tokens, float* state, int64_t state_stride, float* out, int64_t ld_o, void* stream);
 
-/* out = RMSNorm(x) * w * sigmoid(gate), row by row; x, w fp32, gate and out of `dtype` */
-int fb_gated_rmsnorm(const float* x, int64_t rows, int64_t cols, int64_t ldx, int dtype, const void* gate, int64_t ld_g, const float* w, float eps,
-                     void* out, int64_t ldo, void* stream);
+/* The same with a decay and a step size per head and token (a state space): with d = softplus(step[t * ld_step + h] + step_bias[h]),
+ * S = exp(-exp(a_log[h]) d) S + d k v^T, out = S^T q + skip[h] v.  A row of xbc is v (heads x vdim) | k (groups x dim) | q (groups x
+ * dim); head h reads group h / (heads / groups).  The state, places and `dead` as above. */
+int fb_selective_scan(int dtype, const void* xbc, int64_t ld, int heads, int groups, int dim, int vdim, const float* step, int64_t ld_step, const float* step_bias,
+                      const float* a_log, const float* skip, const int32_t* places, int dead, int64_t sequences, int64_t tokens, float* state,
+                      int64_t state_stride, float* out, int64_t ld_o, void* stream);
+
+/* out = RMSNorm(x) * w * sigmoid(gate), or, before, RMSNorm(x silu(gate)) * w, row by row, each of a row's `parts` equal parts by its
+ * own root mean square; x, w fp32, gate of gate_dtype, out of `dtype` */
+int fb_gated_rmsnorm(const float* x, int64_t rows, int64_t cols, int64_t ldx, int gate_dtype, const void* gate, int64_t ld_g, int before, const float* w, float eps, int parts,
+                     int dtype, void* out, int64_t ldo, void* stream);
+
+/* ---- short convolutions over time and a gated linear recurrence ------------------------------------------- */
+
+typedef struct {
+  int64_t cols;
+  int taps;
+  const float* w;       /* [taps, cols]; the last row is the current token's */
+  const float* bias;    /* [cols] or null: added to the sum */
+  const float* in_bias; /* [cols] or null: added to what goes in */
+  int silu;             /* the result goes through SiLU */
+  const int32_t* places;
+  int dead;             /* as fb_decay_scan's */
+  int64_t sequences, tokens; /* `sequences` sequences of `tokens` rows each, in turn */
+  float* state;         /* a sequence's last taps - 1 inputs (with in_bias), [taps - 1, cols], state_stride elements apart, read and left for */
+  int64_t state_stride; /* the next call; taps 1: none */
+} fb_conv;
+/* out[t, c] = bias[c] + sum over j of w[j, c] in[t - taps + 1 + j, c], a causal convolution per column, zeros before a sequence's first
+ * token; x of in_dtype, out of dtype */
+int fb_short_conv(const fb_conv* conv_host, int in_dtype, const void* x, int64_t ld, int dtype, void* out, int64_t ld_o, void* stream);
+
+typedef struct {
+  int64_t width;
+  int blocks;                  /* gate columns come in so many equal blocks of (r | i) */
+  const float* lam;            /* [width] */
+  float rate;                  /* the decay: log a = rate r softplus(lam) */
+  const float* gate_bias;      /* [2 width], laid out as the gates, or null */
+  const float* y_bias;         /* [width] or null */
+  float scale;                 /* of the output */
+  const int32_t* places;
+  int dead;
+  int64_t sequences, tokens;
+  float* state;                /* [width] a sequence, state_stride elements apart */
+  int64_t state_stride;
+} fb_lru;
+/* A gated linear recurrence per column: r and i sigmoids of the gates, a = exp(log a), S = a S + sqrt(1 - a^2) i u, out = scale S
+ * gelu(y + y_bias), GELU's tanh form.  u and out of dtype, gates fp32 [rows, 2 width], y of y_dtype. */
+int fb_lru_scan(const fb_lru* lru_host, int dtype, const void* u, int64_t ld_u, const float* gates, int64_t ld_gates, int y_dtype, const void* y, int64_t ld_y,
+                void* out, int64_t ld_o, void* stream);
 
 /* ---- grouped-query attention over rows of a key and its value, and what stands around it ------------------- */
 
@@ -437,6 +488,7 @@ typedef struct {
   int64_t state_stride;            /* each sequence, read and left for the next call, state_stride elements a sequence.  The T rows are */
   int sequences, dead;             /* `sequences` sequences' in turn; one whose first token stands at place 0 starts from zeros, one whose
                                       first token stands at place `dead` (-1: none) leaves its state alone */
+  float temp_coef, temp_every;     /* queries, after their norm, times 1 + temp_coef ln(floor((places[t] + 1) / temp_every) + 1); 0: no such factor */
 } fb_heads;
 /* After a joint projection q (heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim) (| more): biases and norms in fp32, queries
  * to q_out, and (key | value) into row rows[t] of each key head of cache [kv_heads, cache_rows, dim + vdim] (heads head_stride
@@ -446,11 +498,13 @@ int fb_heads_put(const fb_heads* heads_host, int in_dtype, const void* qkv, int6
 
 /* Attention over such a cache: query head h reads key head h / (heads / kv_heads); token t, whose place is last[t], sees the cache
  * rows base[t] + row0 + lo .. + last[t] (base null: row0 alone), lo = 0, or, with span, the first place of its span of `span`
- * places; with window, only the last `window` of them.  softcap c > 0: a scaled score s becomes c tanh(s / c).  sink (fp32 [heads], or null): exp(sink[h]) joins head h's denominator.  gate (or null): the result times its sigmoid,
+ * places; with window, only the last `window` of them.  softcap c > 0: a scaled score s becomes c tanh(s / c).  sink (fp32 [heads], or null): exp(sink[h]) joins head h's denominator.  key_bias (fp32 [heads], or null): no softmax,
+ * a key's weight is sigmoid(score + key_bias[h]), and the result is the weighted sum as it is (then no sink).  The result times
+ * out_scale.  gate (or null): the result times its sigmoid,
  * column by column.  chunk: the tokens are consecutive ones of one sequence.  max_keys: an upper bound of last[t] + 1. */
 int fb_heads_attention(int dtype, const void* q, int64_t T, int64_t ld_q, int heads, int kv_heads, int dim, int vdim, const void* cache,
                        int64_t cache_rows, int64_t head_stride, const int32_t* base, int64_t row0, const int32_t* last, int64_t max_keys, int chunk,
-                       int span, int window, float scale, float softcap, const float* sink, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o,
+                       int span, int window, float scale, float softcap, const float* sink, const float* key_bias, float out_scale, int gate_dtype, const void* gate, int64_t ld_g, void* out, int64_t ld_o,
                        void* stream);
 
 typedef struct {
@@ -465,7 +519,7 @@ typedef struct {
   const void* chosen;
   int64_t ld_chosen;
   const int32_t* slots;
-  const float* weights;
+  const float* weights; /* null: each 1 */
   int k;
   float* x_out; /* x + mixer * mixer_scale + (other + chosen) * other_scale, or null */
   int64_t ld_x_out;
@@ -476,6 +530,10 @@ typedef struct {
   const float* mixer_bias; /* added to the mixer's result (where there is none, in its place), one a column */
   const void* own;         /* the row of a choice with slot -1: token t's is row t */
   int64_t ld_own;
+  const float* gate;       /* the branches' sum times sigmoid(gate[t * ld_gate + c] + gate_bias[c]), or null */
+  int64_t ld_gate;
+  const float* gate_bias;
+  const float* post;       /* and then as RMSNorm by it leaves it (one a column, the same eps), or null: before it joins the stream */
 } fb_branches;
 /* A layer's end and the next one's start.  Branches null: not there; h without w: the sum itself.  in_dtype: mixer and other; dtype:
  * chosen, own and h. */
