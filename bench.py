@@ -3,7 +3,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--workload llama8b|smollm] [--layers L] [--impl reference]
     python bench.py --matmul 32,4096,14336,bfp8,6      (one isolated matmul, a few calls: what the ncu captures run)
     python bench.py --attend 32,32,8,128,2048,6        (the decode attention alone, likewise)
-    python bench.py --design binutar|labepel|vunadra   (prefill, decode and kernels of that design beside the Llama decoder)
+    python bench.py --design binutar|labepel|vunadra|ronavik   (prefill, decode and kernels of that design beside the Llama decoder)
 
 The default workload is the Llama-3.1-8B-shape batched decode (32 sequences, 2048 tokens of context each, bfp8 weights,
 bf16 KV cache), tensor-parallel over N GPUs with an NCCL all-reduce after o_proj and down_proj.  A step is one decode
@@ -64,7 +64,7 @@ def parse():
     ap.add_argument("--sweep", type=int, default=1, help="0: leave the isolated matmul sweep out of the line (a profiling run)")
     ap.add_argument("--attend", default="", help="T,H,KV,hd,context[,calls]: only the decode attention, e.g. 32,32,8,128,2048,6")
     ap.add_argument("--matmul", default="", help="M,K,N,fmt[,calls]: only that isolated matmul (RMSNorm + SwiGLU fused), e.g. 32,4096,14336,bfp8,6")
-    ap.add_argument("--design", default="", help="binutar[:SIZE], labepel[:SIZE] or vunadra[:SIZE]: instead of the workload, prefill and decode of that design at sizes like a real model's layers, "
+    ap.add_argument("--design", default="", help="binutar[:SIZE], labepel[:SIZE], vunadra[:SIZE] or ronavik[:SIZE]: instead of the workload, prefill and decode of that design at sizes like a real model's layers, "
                                                  "and each of its kernels, beside the Llama decoder at equal size (one GPU)")
     return ap.parse_args()
 
@@ -434,6 +434,26 @@ VUNADRA_SIZES = {
 }
 
 
+# state spaces of Mamba-2's usual shape and attention beside a gated recurrence in turn, each before a mixture; a Llama-like mixture of the
+# same heads, experts and depth beside it
+RONAVIK_SIZES = {
+    "4096": dict(width=4096, layers=6, vocab=32000, heads=32, kv=8, dim=128, vdim=128, lru=4096, blocks=32, conv=4, ssm_heads=128, ssm_vdim=64, state=128, groups=8, experts=8, top=2, ff=14336),
+    "2048": dict(width=2048, layers=8, vocab=32000, heads=32, kv=4, dim=128, vdim=128, lru=2048, blocks=16, conv=4, ssm_heads=64, ssm_vdim=64, state=128, groups=8, experts=128, top=8, ff=768),
+}
+
+
+def ronavik_models(s, places):
+    """(Ronavik config, Llama config of a mixture) of one size."""
+    from ferrite_b200 import llama, ronavik
+    mlp = dict(kind="moe", router=dict(experts=s["experts"], top=s["top"]), expert=dict(ff=s["ff"]))
+    space = dict(type="mamba2", mixer=dict(heads=s["ssm_heads"], vdim=s["ssm_vdim"], state=s["state"], groups=s["groups"], conv=s["conv"], norm_groups=s["groups"]), mlp=mlp)
+    left = dict(heads=s["heads"], kv_heads=s["kv"], dim=s["dim"], vdim=s["vdim"], scale=s["dim"] ** -0.5, q_temp=dict(coef=0.1, every=8192))
+    side = dict(type="parallel", mixer=dict(left=left, right=dict(width=s["lru"], blocks=s["blocks"], conv=s["conv"]), left_scale=1.0, right_scale=1.0), mlp=mlp)
+    return (ronavik.model(vocab=s["vocab"], dim=s["width"], eps=1e-5, blocks=[space, side] * (s["layers"] // 2), positions=places, places=places),
+            llama.model(dim=s["width"], heads=s["heads"], kv=s["kv"], head_dim=s["dim"], layers=s["layers"], vocab=s["vocab"], ffn=0, experts=s["experts"], k=s["top"], moe=s["ff"], theta=10000.0,
+                        eps=1e-5, places=places))
+
+
 def vunadra_models(s, places):
     """(Vunadra config, Llama config of a mixture) of one size."""
     from ferrite_b200 import llama, vunadra
@@ -504,7 +524,7 @@ def design_steps(rt, c, prec, S, ctx, prompt, steps):
     part += -part % 64
     kv = family.kv_cache(c, S * part, llama.zeros(rt), S)
     gen = torch.Generator(device=rt.device).manual_seed(1)
-    for t in [t for x in kv for t in (x if isinstance(x, tuple) else (x,))]:  # (what the prompts would have left)
+    for t in [t for x in kv for t in (x if isinstance(x, tuple) else (x,)) if t is not None]:  # (what the prompts would have left)
         t.buf.normal_(0, 1, generator=gen)
     on = lambda row: Tensor.of(rt, [row], "int32")
     step = jit(lambda ids, at: llama.next_tokens(family.forward(ids, at, w, c, kv, S), c))
@@ -835,6 +855,98 @@ def vunadra_kernels(rt, s, T, ctx, peaks):
     return rows
 
 
+def ronavik_kernels(rt, s, T, ctx, peaks):
+    """Each kernel of the Ronavik layers, as design_kernels does it; beside the state space's scan the fixed decay's over as many heads of that size."""
+    import torch
+    from ferrite_b200 import _lib, ops
+    dev, gen = rt.device, torch.Generator(device=rt.device).manual_seed(0)
+    f32 = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.float32).normal_(0, 1, generator=gen)
+    bf = lambda *shape: torch.empty(*shape, device=dev, dtype=torch.bfloat16).normal_(0, 1, generator=gen)
+    rows, prompt = [], ctx == 0
+    d, H, G, dim, vd, W, blocks, taps = (s[n] for n in ("width", "heads", "kv", "dim", "vdim", "lru", "blocks", "conv"))
+    SH, P, N, SG, E, k, ff = (s[n] for n in ("ssm_heads", "ssm_vdim", "state", "groups", "experts", "top", "ff"))
+    inner, n = SH * P, (H + G) * dim + G * vd
+    wide = inner + 2 * SG * N
+
+    def row(name, us, nbytes, flops=0.0, like=None):
+        floor = max(nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6)
+        rows.append({"kernel": name, "us": round(us, 2), "roofline_us": round(floor, 2), "frac": round(floor / us, 3)} | ({"like": like} if like else {}))
+
+    def dense(name, K, N, out_dtype=torch.bfloat16, batch=1):
+        copies = max(1, min(16, int(3e8 // (2 * batch * K * N))))
+        ws, x = [bf(batch, N, K) for _ in range(copies)], bf(T, batch, K).permute(1, 0, 2)
+        out = torch.empty(T, batch, N + -N % 8, device=dev, dtype=out_dtype).permute(1, 0, 2)[:, :, :N]
+        us = timed(40, copies, lambda i: ops.dense(x, ws[i].transpose(1, 2), out, True))
+        row(f"fb_dense {name} " + (f"{batch}x" if batch > 1 else "") + f"[{K}, {N}]", us, batch * (2 * K * N + 2 * T * K + out.element_size() * T * N), 2.0 * T * batch * K * N, "fb_linear")
+
+    dense("parallel: gate, q, k, v, y, x", d, d + n + 2 * W, torch.float32)
+    dense("mamba2: gate, z, x, B, C, dt", d, d + inner + wide + SH, torch.float32)
+    dense("gates by block", W // blocks, 2 * W // blocks, torch.float32, blocks)
+    dense("parallel o", H * vd + W, d)
+    dense("mamba2 o", inner, d)
+    dense("gate, router", d, d + E, torch.float32)
+    dense("head", d, s["vocab"], torch.float32)
+
+    places = torch.arange(T, device=dev, dtype=torch.int32) if prompt else torch.full((T,), ctx - 1, device=dev, dtype=torch.int32)
+    slots, keys, dead = 1 if prompt else T, T if prompt else ctx, -1
+    part = keys + -keys % 64
+    base = torch.arange(T, device=dev, dtype=torch.int32) * part
+    pairs = T * (T + 1) / 2 if prompt else T * ctx
+    for v in (vd, 2 * vd):
+        caches, m = [bf(G, slots * part, dim + v) for _ in range(4)], (H + G) * dim + G * v
+        joint, q, both = f32(T, d + m + 2 * W), bf(T, H * dim), bf(T, H * v + W)
+        us = timed(40, 1, lambda i: ops.heads_put(joint[:, d:d + m], H, G, dim, v, places if prompt else base + places, caches[0], q, q_norm=f32_ones(dev, dim), k_norm=f32_ones(dev, dim), eps=1e-5, places=places,
+                                                  temperature=(0.1, 8192.0)))
+        if v == vd:
+            row("fb_heads_put, temperature", us, T * 6 * m, like="fb_rope_kv_write")
+        us = timed(20, 4, lambda i: ops.heads_attention(q, caches[i], None if prompt else base, places, H, v, 0.1, keys, prompt, key_bias=f32_ones(dev, H), out=both[:, :H * v]))
+        row("fb_heads_attention by sigmoids" + ("" if v == vd else f", values of {v} columns"), us, 2 * (slots * keys * G * (dim + v) + T * H * (dim + v)), 2.0 * pairs * H * (dim + v), "attention")
+
+    joint, u, gates = f32(T, d + n + 2 * W), bf(T, W), f32(T, 2 * W)
+    x, y = joint[:, d + n + W:d + n + 2 * W], joint[:, d + n:d + n + W]
+    conv, w = f32(slots, taps - 1, max(W, wide)), f32(taps, max(W, wide))
+    us = timed(40, 1, lambda i: ops.short_conv(x, w.view(-1)[:taps * W].view(taps, W), u, places, dead, conv.view(-1)[:slots * (taps - 1) * W].view(slots, taps - 1, W), f32_ones(dev, W), f32_ones(dev, W)))
+    row("fb_short_conv, recurrence", us, T * W * 6 + slots * (taps - 1) * W * 8, like="fb_rope_kv_write")
+    state = f32(slots, 1, W)
+    us = timed(40, 1, lambda i: ops.lru_scan(u, gates, y, both[:, -W:], f32_ones(dev, W), -8.0, blocks, places, dead, state, f32_ones(dev, 2 * W), f32_ones(dev, W)))
+    row("fb_lru_scan", us, T * W * 16 + slots * W * 8, like="fb_decay_scan")
+
+    joint, xbc, out = f32(T, d + inner + wide + SH + -SH % 8), bf(T, wide), f32(T, inner)
+    us = timed(40, 1, lambda i: ops.short_conv(joint[:, d + inner:d + inner + wide], w.view(-1)[:taps * wide].view(taps, wide), xbc, places, dead, conv.view(-1)[:slots * (taps - 1) * wide].view(slots, taps - 1, wide),
+                                               f32_ones(dev, wide), None, True))
+    row("fb_short_conv, state space", us, T * wide * 6 + slots * (taps - 1) * wide * 8, like="fb_rope_kv_write")
+    step, states, low = joint[:, d + inner + wide:d + inner + wide + SH], [f32(slots, SH * N, P) for _ in range(1 if prompt else 4)], f32_ones(dev, SH) * -2
+    us = timed(20, len(states), lambda i: ops.selective_scan(xbc, SH, SG, N, P, step, low, low, low, places, dead, states[i], out))
+    row("fb_selective_scan", us, T * (2 * wide + 4 * SH + 4 * inner) + slots * SH * N * P * 8, 2.0 * T * SH * 2 * N * P, "fb_decay_scan")
+    qkv, decay = bf(T, SH * (2 * N + P)), torch.full((SH,), 0.95, device=dev)
+    us = timed(20, len(states), lambda i: ops.decay_scan(qkv, SH, N, P, decay, places, dead, states[i], out))
+    row("fb_decay_scan, the fixed decay's", us, T * (2 * SH * (2 * N + P) + 4 * inner) + slots * SH * N * P * 8, 2.0 * T * SH * 2 * N * P)
+    h = bf(T, inner)
+    us = timed(40, 1, lambda i: ops.gated_rmsnorm(out, joint[:, d:d + inner], f32_ones(dev, inner), 1e-5, h, True, SG))
+    row("fb_gated_rmsnorm, gate before, in parts", us, T * inner * 10, like="fb_rmsnorm")
+
+    logits = f32(T, E)
+    us = timed(40, 1, lambda i: ops.route(logits, E, k, None, "sigmoid", as_scored=True, on_input=True))
+    row("fb_route, sigmoids", us, T * (4 * E + 12 * k), like="fb_topk and fb_touched (fb_group)")
+    r = ops.route(logits, E, k, None, "sigmoid", as_scored=True, on_input=True)
+    touched, live = len(set(r.ids.cpu().reshape(-1).tolist())), int(r.live)
+    copies = max(1, min(4, int(3e8 // (4 * touched * d * ff)) + 1))
+    up, down, h = [bf(E, ff, d).transpose(1, 2) for _ in range(copies)], [bf(E, d, ff).transpose(1, 2) for _ in range(copies)], bf(T, d)
+    x, act, y = bf(r.tiles * r.tile, d), bf(r.tiles * r.tile, ff), bf(r.tiles * r.tile, d)
+    if not r.shared:
+        us = timed(20, 1, lambda i: ops.spread_rows(h, r, x))
+        row("fb_spread_rows", us, 2 * T * (k + 1) * d, like="fb_gather_rows")
+    us = timed(20, copies, lambda i: ops.grouped(h if r.shared else x, up[i], r, act, _lib.DENSE_RELU2, r.shared, row_scale=r.row_weights.data_ptr()))
+    row(f"fb_dense_grouped up, squared ReLU ({touched} experts, {live} tiles of {r.tile})", us, 2 * touched * d * ff + T * k * 2 * (d + ff), 2.0 * T * k * d * ff, "fb_linear_indexed")
+    us = timed(20, copies, lambda i: ops.grouped(act, down[i], r, y))
+    row("fb_dense_grouped down", us, 2 * touched * d * ff + T * k * 2 * (d + ff), 2.0 * T * k * d * ff, "fb_linear_indexed")
+    res, sums, one, gate = f32(T, d), f32(T, d), f32_ones(dev, d), f32(T, d + E + -E % 8)
+    for what, more in (("mixer", dict(mixer=h)), ("chosen rows", dict(chosen=y, routes=r))):
+        us = timed(40, 1, lambda i: ops.add_norm(res, sums, w=one, eps=1e-5, h=x[:T], gate=gate[:, :d], gate_bias=one, post=one, **more))
+        row(f"fb_add_norm, {what}, gated and normed", us, T * d * (8 + 4 + 2 + 2 * (1 if what == "mixer" else k)), like="fb_rmsnorm")
+    return rows
+
+
 def llama_expert_kernels(rt, s, T, peaks):
     """The Llama mixture's own kernels at the same size (bfp8 experts): its router's and its experts', decode or prompt."""
     import torch
@@ -890,7 +1002,8 @@ def run_design(args):
     from ferrite_b200 import llama, models
     from ferrite_b200.tensor import Runtime
     name, _, size = args.design.partition(":")
-    designs = {"binutar": (DESIGN_SIZES, design_models, design_kernels), "labepel": (LABEPEL_SIZES, labepel_models, labepel_kernels), "vunadra": (VUNADRA_SIZES, vunadra_models, vunadra_kernels)}
+    designs = {"binutar": (DESIGN_SIZES, design_models, design_kernels), "labepel": (LABEPEL_SIZES, labepel_models, labepel_kernels), "vunadra": (VUNADRA_SIZES, vunadra_models, vunadra_kernels),
+               "ronavik": (RONAVIK_SIZES, ronavik_models, ronavik_kernels)}
     assert name in designs and args.gpus == 1, "--design " + " or ".join(f"{n}[:SIZE]" for n in designs) + ", one GPU"
     sizes, make, kernels = designs[name]
     rt, (peaks, kind), family = Runtime(0), measured_peaks(), models.module(name)

@@ -5,7 +5,9 @@ import math
 
 import numpy as np
 
-f64 = np.float64
+
+def f64(x):
+    return np.asarray(x, np.float64)
 
 
 def sigmoid(x):

@@ -63,3 +63,11 @@ def test_vunadra_models_are_of_equal_size():
         e = b.blocks[1]
         assert (e.mixer.heads, e.mixer.kv_heads, e.mixer.dim, e.mlp.router.experts, e.mlp.router.top, e.mlp.expert.ff) == (l.heads, l.kv, l.head_dim, l.experts, l.k, l.moe)
         assert [e.type for e in b.blocks] == ["attention", "attention_2", "latent_attention"]
+
+
+def test_ronavik_models_are_of_equal_size():
+    for s in bench.RONAVIK_SIZES.values():
+        b, l = bench.ronavik_models(s, 512)
+        assert (b.dim, b.vocab, b.layers, b.positions) == (l.dim, l.vocab, l.layers, 512) and [e.type for e in b.blocks[:2]] == ["mamba2", "parallel"]
+        m, f = b.blocks[1].mixer.left, b.blocks[0].mlp
+        assert (m.heads, m.kv_heads, m.dim, f.router.experts, f.router.top, f.expert.ff) == (l.heads, l.kv, l.head_dim, l.experts, l.k, l.moe)
