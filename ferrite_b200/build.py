@@ -21,10 +21,10 @@ FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std
 
 
 # what a family runs on where that is a part of the whole: its kernels, the sampling head, the general operators
-FAMILY_SOURCES = {"binutar": ["api.cu", "decode_misc.cu", "dense.cu", "generic.cu", "latent.cu", "latent_tcgen05.cu", "recurrent.cu", "router.cu"],
+FAMILY_SOURCES = {"binutar": ["api.cu", "decode_misc.cu", "dense.cu", "generic.cu", "latent.cu", "latent_tcgen05.cu", "recurrent.cu", "router.cu", "selective_prompt.cu"],
                   "labepel": ["api.cu", "decode_misc.cu", "dense.cu", "experts.cu", "generic.cu", "heads_attention.cu", *(f"heads_attention_{n}.cu" for n in (64, 128, 192, 256)), "heads_prompt.cu", "router.cu", "rows.cu"]}
 FAMILY_SOURCES["vunadra"] = sorted({*FAMILY_SOURCES["labepel"], "latent.cu", "latent_tcgen05.cu"})
-FAMILY_SOURCES["ronavik"] = sorted({*FAMILY_SOURCES["labepel"], "recurrent.cu", "short_conv.cu"})
+FAMILY_SOURCES["ronavik"] = sorted({*FAMILY_SOURCES["labepel"], "recurrent.cu", "selective_prompt.cu", "short_conv.cu"})
 LINKED = os.path.join(HERE, "lib", "sources.txt")  # the sources a part of a library holds (no such file: all of them)
 
 

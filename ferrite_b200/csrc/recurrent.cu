@@ -7,31 +7,12 @@
 //   fb_gated_rmsnorm    RMSNorm over the heads' outputs, together or in equal parts, with a gate after or before it
 //
 // Both scans go token after token - a decode step's one token a sequence, and prompts in fp32 or of odd sizes - or, for bf16
-// prompts, in chunks of 64 tokens on tensor-core MMAs (decay_chunk_kernel).
+// prompts, in chunks of 64 tokens on tensor-core MMAs (decay_chunk_kernel); longer selective ones in selective_prompt.cu.
 #include "launch.cuh"
 #include "mma_sync.cuh"
-#include "values.cuh"
+#include "scan.cuh"
 
 namespace fb {
-
-struct ScanArgs {
-  const void* x;  // [tokens, ld]: of head h the query at q0 + h / rep * dim, the key at k0 + h / rep * dim, the value at v0 + h * vdim
-  int64_t ld, q0, k0, v0;
-  int rep, heads, dim, vdim;
-  const float* decay;     // [heads] (a selective scan: none)
-  const int32_t* places;  // a sequence whose first token is at place 0 starts from a zero state
-  int dead;               // a sequence whose first token is at this place has no token (its state stays, its output is 0); -1: none
-  int64_t tokens;         // per sequence, one sequence's after the other's
-  float* state;           // [sequences, heads, dim, vdim], sequences state_stride apart
-  int64_t state_stride;
-  float* out;  // [tokens, ld_o]
-  int64_t ld_o;
-  const float* step;  // selective: [tokens, ld_step], head h's step size before its bias and softplus
-  int64_t ld_step;
-  const float *step_bias, *a_log, *skip;  // [heads]
-};
-
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // A CTA keeps 32 columns of one head's state of one sequence in registers: thread (group g, lane) the rows
 // 16 g .. 16 g + 15 of column `lane`.  The groups' parts of an output meet in shared memory.
@@ -356,6 +337,9 @@ static int run_scan(int dtype, const ScanArgs& a, int64_t sequences, cudaStream_
   FB_REQUIRE(dtype == FB_BF16 || dtype == FB_FP32, "%s: bf16 or fp32", what);
   FB_REQUIRE(a.dim <= 512, "%s: heads of up to 512 query columns (got %d)", what, a.dim);
   FB_REQUIRE(a.ld_o >= (int64_t)a.heads * a.vdim && a.state_stride >= (int64_t)a.heads * a.dim * a.vdim && sequences <= 65535 && a.heads <= 65535, "%s: row strides too small", what);
+  if constexpr (SELECTIVE) {
+    if (dtype == FB_BF16 && selective_prompt_supports(a, sequences)) return selective_prompt(a, sequences, s);
+  }
   // (a few tokens are done sooner one by one)
   if (dtype == FB_BF16 && a.tokens >= 16 && a.dead < 0 && a.dim % 16 == 0 && a.dim <= 256 && a.vdim % 8 == 0 && a.ld % 8 == 0 && a.q0 % 8 == 0 && a.k0 % 8 == 0 && a.v0 % 8 == 0 && a.ld_o % 2 == 0 &&
       a.state_stride % 2 == 0 && (uintptr_t)a.x % 16 == 0 && (uintptr_t)a.state % 8 == 0 && (uintptr_t)a.out % 8 == 0)

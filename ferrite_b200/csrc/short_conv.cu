@@ -33,7 +33,7 @@ __device__ __forceinline__ void set_some(T* p, const float v[N]) {
   else store_value(p, v[0]);
 }
 
-constexpr int CONV_THREADS = 128, CONV_KEPT = 4;  // up to so many taps the inputs go through registers, each read once a block
+constexpr int CONV_THREADS = 128, CONV_KEPT = 4, CONV_AHEAD = 2;  // up to CONV_KEPT taps the inputs go through registers, each read once a block
 
 // A block has N columns a thread and a run of one sequence's tokens.  The first run's block alone reads and leaves the state.
 template <typename In, typename Act, int N, int TAPS>  // TAPS 0: any number, inputs read anew for every token
@@ -71,20 +71,20 @@ __global__ void __launch_bounds__(CONV_THREADS) short_conv_kernel(const ConvArgs
   auto finish = [&](int64_t i, float y[N]) {
 #pragma unroll
     for (int e = 0; e < N; ++e)
-      if (a.silu) y[e] *= sigmoid_f(y[e]);
+      if (a.silu) y[e] *= sizeof(Act) == 4 ? sigmoid_f(y[e]) : sigmoid_near(y[e]);
     set_some<N>(static_cast<Act*>(args.out) + (row0 + i) * args.ld_o + col, y);
   };
   if constexpr (TAPS > 0) {
     float past[TAPS][N];  // the inputs of the last TAPS tokens, the current one's last
 #pragma unroll
     for (int j = 1; j < TAPS; ++j) input(begin - TAPS + j, past[j]);
-    for (int64_t i0 = begin; i0 < end; i0 += 4) {  // (four tokens' inputs on their way at once)
-      float next[4][N];
+    for (int64_t i0 = begin; i0 < end; i0 += CONV_AHEAD) {  // (so many tokens' inputs on their way at once; more, and the loop outgrows the instruction cache)
+      float next[CONV_AHEAD][N];
 #pragma unroll
-      for (int k = 0; k < 4; ++k)
+      for (int k = 0; k < CONV_AHEAD; ++k)
         if (i0 + k < end) input(i0 + k, next[k]);
 #pragma unroll
-      for (int k = 0; k < 4; ++k) {
+      for (int k = 0; k < CONV_AHEAD; ++k) {
         if (i0 + k >= end) break;
         float y[N];
 #pragma unroll
@@ -135,8 +135,8 @@ static int launch_conv(const ConvArgs& a, cudaStream_t s) {
 template <typename In, typename Act>
 static int run_conv(ConvArgs a, cudaStream_t s) {
   const fb_conv& c = a.c;
-  a.first = (int)(c.taps - 1 < 1 ? 1 : c.taps - 1 < c.tokens ? c.taps - 1 : c.tokens), a.group = 4;
-  while (a.group < 32 && ceil_div(c.sequences * c.tokens, 2 * a.group) * ceil_div(c.cols, CONV_THREADS * 4) >= 8 * 148) a.group *= 2;  // (a run's first token reads the taps - 1 before it)
+  a.first = (int)(c.taps - 1 < 1 ? 1 : c.taps - 1 < c.tokens ? c.taps - 1 : c.tokens), a.group = CONV_AHEAD;
+  while (a.group < 32 && ceil_div(c.sequences * c.tokens, 2 * a.group) * ceil_div(c.cols, CONV_THREADS * 4) >= 32 * 148) a.group *= 2;  // (a run's first token reads the taps - 1 before it)
   auto whole = [](const void* p, int64_t ld, int bytes) { return (uintptr_t)p % (4 * bytes) == 0 && ld % 4 == 0; };
   const bool fours = c.cols % 4 == 0 && whole(a.x, a.ld, sizeof(In)) && whole(a.out, a.ld_o, sizeof(Act)) && whole(c.w, 0, 4) && whole(c.state, c.state_stride, 4);
   return fours ? launch_conv<In, Act, 4>(a, s) : launch_conv<In, Act, 1>(a, s);
@@ -171,11 +171,26 @@ __device__ __forceinline__ LruColumn lru_column(const LruArgs& a, int64_t col) {
   return c;
 }
 
-// a token's step: the state becomes a S + b
+__device__ __forceinline__ float sqrt_near(float x) {
+  float y;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// a token's step: the state becomes a S + b.  1 - a^2 is formed from log a, so that it holds where a is all but 1; NEAR: by the
+// hardware's exponential, and there by its power series
+template <bool NEAR>
 __device__ __forceinline__ void lru_step(const LruColumn& c, float r, float i, float u, float& a, float& b) {
-  const float log_a = c.slope * sigmoid_f(r + c.r_bias);
-  a = expf(log_a);
-  b = sqrtf(-expm1f(2.f * log_a)) * sigmoid_f(i + c.i_bias) * u;  // (1 - a^2, also where a is all but 1)
+  if constexpr (NEAR) {
+    const float log_a = c.slope * sigmoid_near(r + c.r_bias), z = 2.f * log_a;
+    a = __expf(log_a);
+    const float series = -z * fmaf(z, fmaf(z, fmaf(z, fmaf(z, fmaf(z, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
+    b = sqrt_near(z > -0.3f ? series : fmaf(-a, a, 1.f)) * sigmoid_near(i + c.i_bias) * u;
+  } else {
+    const float log_a = c.slope * sigmoid_f(r + c.r_bias);
+    a = expf(log_a);
+    b = sqrtf(-expm1f(2.f * log_a)) * sigmoid_f(i + c.i_bias) * u;
+  }
 }
 
 __device__ __forceinline__ float gelu_of(float z) { return 0.5f * z * (1.f + tanh_of(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
@@ -194,7 +209,7 @@ __global__ void __launch_bounds__(128) lru_token_kernel(const LruArgs a) {
   const float before = *state, r = a.gates[seq * a.ld_gates + c.r_at], i = a.gates[seq * a.ld_gates + c.r_at + a.part];
   const float u = value_of(static_cast<const Act*>(a.u)[seq * a.ld_u + col]), y = value_of(static_cast<const Y*>(a.y)[seq * a.ld_y + col]);
   float decay, in;
-  lru_step(c, r, i, u, decay, in);
+  lru_step<sizeof(Act) == 2>(c, r, i, u, decay, in);
   const float s = place ? fmaf(decay, before, in) : in;
   *state = s;
   store_value(out, a.l.scale * s * gelu_of(y + c.y_bias));
@@ -202,8 +217,8 @@ __global__ void __launch_bounds__(128) lru_token_kernel(const LruArgs a) {
 
 constexpr int LRU_COLS = 16, LRU_RUNS = 32, LRU_TOKENS = 8;
 
-template <typename Act, typename Y>
-__global__ void __launch_bounds__(LRU_COLS* LRU_RUNS) lru_scan_kernel(const LruArgs a) {
+template <typename Act, typename Y, int BLOCKS>  // BLOCKS: of them an SM (one alone has registers enough to have more on its way)
+__global__ void __launch_bounds__(LRU_COLS* LRU_RUNS, BLOCKS) lru_scan_kernel(const LruArgs a) {
   griddep_launch_dependents();
   griddep_wait();
   __shared__ float2 parts[2][LRU_RUNS][LRU_COLS];  // of each run: the product of its a, the state it ends in from zero
@@ -218,26 +233,26 @@ __global__ void __launch_bounds__(LRU_COLS* LRU_RUNS) lru_scan_kernel(const LruA
   const LruColumn c = lru_column(a, mine ? col : 0);
   float* state = a.l.state + seq * a.l.state_stride + col;
   float carry = mine && place ? *state : 0.f;
+  const int64_t first = row0 + run * LRU_TOKENS, stride = LRU_RUNS * LRU_TOKENS;
+  const Act* u = static_cast<const Act*>(a.u) + first * a.ld_u + col;
+  const Y* y = static_cast<const Y*>(a.y) + first * a.ld_y + col;
+  const float* gates = a.gates + first * a.ld_gates + c.r_at;
+  Act* out = static_cast<Act*>(a.out) + first * a.ld_o + col;
   int buf = 0;
-  for (int64_t s0 = 0; s0 < a.l.tokens; s0 += LRU_RUNS * LRU_TOKENS, buf ^= 1) {
-    float decay[LRU_TOKENS], in[LRU_TOKENS], u[LRU_TOKENS], y[LRU_TOKENS];
-    const int64_t t0 = s0 + run * LRU_TOKENS;
-    const int n = mine ? (int)min((int64_t)LRU_TOKENS, max((int64_t)0, a.l.tokens - t0)) : 0;
+  for (int64_t s0 = 0; s0 < a.l.tokens; s0 += stride, buf ^= 1) {
+    float decay[LRU_TOKENS], in[LRU_TOKENS], v[LRU_TOKENS], z[LRU_TOKENS];
+    const int n = mine ? (int)min((int64_t)LRU_TOKENS, max((int64_t)0, a.l.tokens - s0 - run * LRU_TOKENS)) : 0;
 #pragma unroll
     for (int k = 0; k < LRU_TOKENS; ++k) {  // (all on their way before the first is needed)
-      decay[k] = in[k] = u[k] = y[k] = 0.f;
-      if (k < n) {
-        const int64_t t = row0 + t0 + k;
-        decay[k] = a.gates[t * a.ld_gates + c.r_at], in[k] = a.gates[t * a.ld_gates + c.r_at + a.part];
-        u[k] = value_of(static_cast<const Act*>(a.u)[t * a.ld_u + col]), y[k] = value_of(static_cast<const Y*>(a.y)[t * a.ld_y + col]);
-      }
+      decay[k] = in[k] = v[k] = z[k] = 0.f;
+      if (k < n) decay[k] = gates[k * a.ld_gates], in[k] = gates[k * a.ld_gates + a.part], v[k] = value_of(u[k * a.ld_u]), z[k] = value_of(y[k * a.ld_y]);
     }
     float whole = 1.f, end = 0.f;
 #pragma unroll
     for (int k = 0; k < LRU_TOKENS; ++k) {
       if (k >= n) break;
       float d, b;
-      lru_step(c, decay[k], in[k], u[k], d, b);
+      lru_step<sizeof(Act) == 2>(c, decay[k], in[k], v[k], d, b);
       decay[k] = d, in[k] = b, whole *= d, end = fmaf(d, end, b);
     }
     parts[buf][run][lane] = make_float2(whole, end);
@@ -253,8 +268,9 @@ __global__ void __launch_bounds__(LRU_COLS* LRU_RUNS) lru_scan_kernel(const LruA
     for (int k = 0; k < LRU_TOKENS; ++k) {
       if (k >= n) break;
       s = fmaf(decay[k], s, in[k]);
-      store_value(static_cast<Act*>(a.out) + (row0 + t0 + k) * a.ld_o + col, a.l.scale * s * gelu_of(y[k] + c.y_bias));
+      store_value(out + k * a.ld_o, a.l.scale * s * gelu_of(z[k] + c.y_bias));
     }
+    u += stride * a.ld_u, y += stride * a.ld_y, gates += stride * a.ld_gates, out += stride * a.ld_o;
   }
   if (run == 0 && mine) *state = carry;
 }
@@ -262,7 +278,9 @@ __global__ void __launch_bounds__(LRU_COLS* LRU_RUNS) lru_scan_kernel(const LruA
 template <typename Act, typename Y>
 static int launch_lru(const LruArgs& a, cudaStream_t s) {
   if (a.l.tokens == 1) return launch_after(lru_token_kernel<Act, Y>, dim3((unsigned)ceil_div(a.l.width, 128), (unsigned)a.l.sequences), dim3(128), 0, s, "fb_lru_scan", a);
-  return launch_after(lru_scan_kernel<Act, Y>, dim3((unsigned)ceil_div(a.l.width, LRU_COLS), (unsigned)a.l.sequences), dim3(LRU_COLS * LRU_RUNS), 0, s, "fb_lru_scan", a);
+  const dim3 grid((unsigned)ceil_div(a.l.width, LRU_COLS), (unsigned)a.l.sequences), block(LRU_COLS * LRU_RUNS);
+  if ((int64_t)grid.x * grid.y <= 148) return launch_after(lru_scan_kernel<Act, Y, 1>, grid, block, 0, s, "fb_lru_scan", a);
+  return launch_after(lru_scan_kernel<Act, Y, 2>, grid, block, 0, s, "fb_lru_scan", a);
 }
 
 }  // namespace fb

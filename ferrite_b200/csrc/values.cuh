@@ -22,6 +22,9 @@ __device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) { return ma
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 
+// the same by the hardware's exponential and reciprocal (about 1e-6 of the result): beside bf16 values
+__device__ __forceinline__ float sigmoid_near(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+
 // 2^x, the hardware's (x far below: 0)
 __device__ __forceinline__ float exp2_of(float x) {
   float y;

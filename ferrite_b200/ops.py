@@ -498,7 +498,7 @@ def add_norm(x, x_out, mixer=None, mixer_scale=None, other=None, other_scale=Non
     kind = of(mixer, other) or dtype if dtype == torch.bfloat16 else torch.float32
     assert all(t is None or t.dtype == kind for t in (mixer, other)) and all(t is None or t.dtype == dtype for t in (h, chosen, own))
     b = _lib.Branches(x.data_ptr(), ld(x), _ptr(mixer), ld(mixer), _ptr(mixer_scale), _ptr(other), ld(other), _ptr(other_scale), _ptr(chosen), ld(chosen),
-                      _ptr(routes.slots) if routes else None, _ptr(routes.weights) if routes and routes.row_weights is None else None, routes.k if routes else 0, _ptr(x_out), ld(x_out), _ptr(w), plus, eps, _ptr(h), ld(h),
+                      _ptr(routes.slots) if routes else None, _ptr(routes.weights) if routes and getattr(routes, "row_weights", None) is None else None, routes.k if routes else 0, _ptr(x_out), ld(x_out), _ptr(w), plus, eps, _ptr(h), ld(h),
                       _ptr(mixer_bias), _ptr(own), ld(own), _ptr(gate), ld(gate), _ptr(gate_bias), _ptr(post))
     check(lib().fb_add_norm(ctypes.byref(b), x.shape[0], x.shape[1], _CODES[kind], _CODES[dtype], _stream()))
     count()

@@ -42,7 +42,7 @@ def in_portions(torch, on, T, run, state, mine=1):
 
 # ---- the state space
 
-@pytest.mark.parametrize("H,G,dim,vdim", [(5, 5, 32, 96), (6, 2, 16, 48), (4, 1, 128, 64), (3, 3, 64, 32), (4, 2, 20, 33), (2, 1, 96, 256), (8, 4, 1, 1), (3, 1, 240, 40), (2, 2, 300, 24)])
+@pytest.mark.parametrize("H,G,dim,vdim", [(5, 5, 32, 96), (6, 2, 16, 48), (4, 1, 128, 64), (3, 3, 64, 32), (4, 2, 20, 33), (2, 1, 96, 256), (8, 4, 1, 1), (3, 1, 240, 40), (2, 2, 300, 24), (6, 3, 48, 72), (2, 1, 128, 136), (9, 3, 112, 8), (2, 2, 96, 64)])
 @pytest.mark.parametrize("bf16", [True, False])
 def test_selective_scan(torch, H, G, dim, vdim, bf16):
     from ferrite_b200 import ops
@@ -70,6 +70,29 @@ def test_selective_scan(torch, H, G, dim, vdim, bf16):
         assert np.abs(to_numpy(state)[1].reshape(H, dim, vdim)[h] - last[h]).max() < 5e-5 * np.abs(last[h]).max(), h
     np.testing.assert_allclose(to_numpy(three)[0].reshape(H, vdim), want[0], rtol=1e-4, atol=1e-4 * np.abs(want[0]).max())
     assert torch.equal(state[2], left) and not three[2].any(), "a slot without a token keeps its state"
+
+
+def test_selective_scan_of_a_long_prompt_and_of_several(torch):
+    # chunk after chunk, a state that lasts, and rows of another sequence right after a sequence's last
+    from ferrite_b200 import ops
+    rng, on, (H, G, dim, vdim) = np.random.default_rng(15), Device(torch, True), (4, 2, 64, 48)
+    for sequences, T in ((1, 1500), (3, 200), (2, 129), (5, 65)):
+        n = H * vdim + 2 * G * dim
+        x, dt = rounded(rng.normal(0, 0.6, (sequences * T, n)), True), f32(rng.normal(-1, 1.5, (sequences * T, H)))
+        bias, a_log, skip = f32(rng.normal(-3, 1, H)), f32([-7.0, -4, -1, 1]), f32(rng.normal(1, 1, H))
+        state, out = torch.randn(sequences, H * dim, vdim, device="cuda"), torch.empty(sequences * T, H * vdim, device="cuda")
+        before = to_numpy(state).reshape(sequences, H, dim, vdim)
+        places = np.concatenate([np.arange(T) + 10 * (s == 1) for s in range(sequences)])  # (the second goes on, the others begin)
+        ops.selective_scan(on(x), H, G, dim, vdim, on.f32(dt), on.f32(bias), on.f32(a_log), on.f32(skip), on.i32(places), -1, state, out)
+        for s in range(sequences):
+            v = x[s * T:(s + 1) * T]
+            parts = v[:, :H * vdim].reshape(-1, H, vdim), v[:, H * vdim:H * vdim + G * dim].reshape(-1, G, dim), v[:, H * vdim + G * dim:].reshape(-1, G, dim)
+            want, last = oracle.state_space(*parts, oracle.softplus(dt[s * T:(s + 1) * T] + bias), a_log, before[s] if s == 1 else np.zeros((H, dim, vdim)))
+            want += skip[:, None] * parts[0]
+            got = to_numpy(out)[s * T:(s + 1) * T].reshape(T, H, vdim)
+            for h in range(H):
+                assert np.abs(got[:, h] - want[:, h]).max() < 5e-5 * np.abs(want[:, h]).max(), (sequences, T, s, h)
+                assert np.abs(to_numpy(state)[s].reshape(H, dim, vdim)[h] - last[h]).max() < 5e-5 * np.abs(last[h]).max(), (sequences, T, s, h)
 
 
 @pytest.mark.parametrize("cols,parts,skip", [(333, 3, 7), (96, 8, 8), (2048, 1, 0), (6000, 1, 4), (6000, 4, 4), (5001, 1, 3), (64, 64, 4)])
