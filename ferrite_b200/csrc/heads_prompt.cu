@@ -171,6 +171,38 @@ __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) he
     for (int t = 0; t < n_tiles; ++t) {
       mbar_wait(smem_u32(s_full + 2 * gr + (t & 1)), (t >> 1) & 1, abort_flag, PW_S);
       tc_fence_after();
+      if constexpr (SIGMOID) {  // 32 keys at a time over the columns read before, in a loop that stays in the instruction cache
+        const int seen = place + 1 - (k0 + t * HP_KEYS), hidden = first - (k0 + t * HP_KEYS);
+        const bool whole = __all_sync(0xffffffffu, seen >= HP_KEYS && hidden <= 0);
+#pragma unroll 1
+        for (int b = 0; b < HP_KEYS; b += 32) {
+          float s[32], p[16];
+          tmem_ld32_nowait(tS + (t & 1) * HP_KEYS + b, s);
+          tmem_ld_wait();
+          if (cap.in > 0.f) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) s[j] = capped(cap, s[j]);
+          }
+          if (!whole) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              if (b + j >= seen || b + j < hidden) s[j] = -INFINITY;
+          }
+#pragma unroll
+          for (int j = 0; j < 32; j += 2) {
+            float x, y;
+            sigmoid_pair(fmaf(s[j], scale_log2, bias), fmaf(s[j + 1], scale_log2, bias), x, y);
+            p[j / 2] = __uint_as_float(pack_bf16x2(s[j] == -INFINITY ? 0.f : x, s[j + 1] == -INFINITY ? 0.f : y));
+          }
+          tmem_st16(tS + (t & 1) * HP_KEYS + b / 2, p);
+        }
+        tmem_st_wait();
+        if (t > 0) mbar_wait(smem_u32(pv_done + gr), (t - 1) & 1, abort_flag, PW_PV);  // (each tile's in turn: a phase two on looks like this one)
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(p_full + gr));
+        continue;
+      }
       float s[HP_KEYS];
       tmem_ld32_nowait(tS + (t & 1) * HP_KEYS, s);
       tmem_ld32_nowait(tS + (t & 1) * HP_KEYS + 32, s + 32);
@@ -185,34 +217,24 @@ __global__ void __launch_bounds__((4 * GROUPS + 2) * 32, GROUPS == 1 ? 2 : 1) he
         for (int j = 0; j < HP_KEYS; ++j)
           if (j >= seen || j < hidden) s[j] = -INFINITY;
       }
+      float tops[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+      for (int j = 4; j < HP_KEYS; ++j) tops[j & 3] = fmaxf(tops[j & 3], s[j]);
+      const float top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
       float corr = 1.f;
-      bool any = false;
+      const bool grown = (top - m) * scale_log2 > HP_SLACK || (m == -INFINITY && top > m);
+      if (grown) corr = exp2_of((m - top) * scale_log2), m = top;
+      const bool any = __any_sync(0xffffffffu, grown);
+      const float at = m == -INFINITY ? 0.f : -m * scale_log2;
+      float sums[4] = {0.f, 0.f, 0.f, 0.f};
       uint32_t pair[HP_KEYS / 2];
-      if constexpr (SIGMOID) {
 #pragma unroll
-        for (int j = 0; j < HP_KEYS; j += 2) {
-          float x, y;
-          sigmoid_pair(fmaf(s[j], scale_log2, bias), fmaf(s[j + 1], scale_log2, bias), x, y);
-          pair[j / 2] = pack_bf16x2(s[j] == -INFINITY ? 0.f : x, s[j + 1] == -INFINITY ? 0.f : y);
-        }
-      } else {
-        float tops[4] = {s[0], s[1], s[2], s[3]};
-#pragma unroll
-        for (int j = 4; j < HP_KEYS; ++j) tops[j & 3] = fmaxf(tops[j & 3], s[j]);
-        const float top = fmaxf(fmaxf(tops[0], tops[1]), fmaxf(tops[2], tops[3]));
-        const bool grown = (top - m) * scale_log2 > HP_SLACK || (m == -INFINITY && top > m);
-        if (grown) corr = exp2_of((m - top) * scale_log2), m = top;
-        any = __any_sync(0xffffffffu, grown);
-        const float at = m == -INFINITY ? 0.f : -m * scale_log2;
-        float sums[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-        for (int j = 0; j < HP_KEYS; j += 2) {
-          const float x = exp2_of(fmaf(s[j], scale_log2, at)), y = exp2_of(fmaf(s[j + 1], scale_log2, at));
-          sums[j & 2] += x, sums[(j & 2) + 1] += y;
-          pair[j / 2] = pack_bf16x2(x, y);
-        }
-        l = l * corr + ((sums[0] + sums[1]) + (sums[2] + sums[3]));
+      for (int j = 0; j < HP_KEYS; j += 2) {
+        const float x = exp2_of(fmaf(s[j], scale_log2, at)), y = exp2_of(fmaf(s[j + 1], scale_log2, at));
+        sums[j & 2] += x, sums[(j & 2) + 1] += y;
+        pair[j / 2] = pack_bf16x2(x, y);
       }
+      l = l * corr + ((sums[0] + sums[1]) + (sums[2] + sums[3]));
       if (t > 0) {  // the sums stand still once the last tile's MMAs are done
         mbar_wait(smem_u32(pv_done + gr), (t - 1) & 1, abort_flag, PW_PV);
         tc_fence_after();
