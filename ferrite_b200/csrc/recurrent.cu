@@ -84,10 +84,10 @@ __global__ void decay_scan_kernel(const ScanArgs a) {
 // ---- a prompt in chunks of 64 tokens.  Within a chunk that starts from the state S,
 //     o_i = decay^(i+1) S^T q_i + sum over j <= i of decay^(i-j) (q_i . k_j) v_j,    S' = decay^n S + sum decay^(n-1-j) k_j v_j^T,
 // all of it matrix products; where the decay is a token's own, decay^(i-j) is the product of those after token j up to token i,
-// exp2 of a difference of running sums of their logarithms, and v_j comes times its step.  A CTA walks one sequence's chunks for one head and 32 of its value columns, with its part of the
-// state in registers as the accumulators of the last product.  q, k and v are bf16 as they come; what is not - the state, the
-// decayed scores, the decayed values - enters a product as two bf16 parts, so the recurrence keeps fp32's range and 16 bits
-// of mantissa in every factor, with sums in fp32.
+// exp2 of a difference of running sums of their logarithms, and v_j comes times its step.  A CTA walks one sequence's chunks for
+// one head and 32 of its value columns, with its part of the state in registers as the accumulators of the last product.  q, k and
+// v are bf16 as they come; what is not - the state, the decayed scores, the decayed values - enters a product as two bf16 parts, so
+// the recurrence keeps fp32's range and 16 bits of mantissa in every factor, with sums in fp32.
 constexpr int CH_TOKENS = 64, CH_COLS = 32, CH_PITCH = CH_COLS * 2 + 16;  // (rows an odd number of 16-byte pieces apart: no bank conflicts)
 
 template <int TILES, bool SELECTIVE>  // TILES: 16-row tiles of the state a warp owns
@@ -95,8 +95,8 @@ __global__ void __launch_bounds__(128) decay_chunk_kernel(const ScanArgs a) {
   griddep_launch_dependents();
   griddep_wait();
   extern __shared__ __align__(128) uint8_t chunk_smem[];
-  __shared__ float power[CH_TOKENS + 1];                      // a fixed decay's powers
-  __shared__ float2 logs[2][CH_TOKENS];                       // selective: log2 of the decays up to and with each token, and its step
+  __shared__ float power[CH_TOKENS + 1];  // a fixed decay's powers
+  __shared__ float2 logs[2][CH_TOKENS];   // selective: log2 of the decays up to and with each token, and its step
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, v0 = blockIdx.x * CH_COLS;
   const int dim = a.dim, pitch = dim * 2 + 16, pieces = dim / 8;
   const int64_t seq = blockIdx.z, t0 = seq * a.tokens;
@@ -327,8 +327,9 @@ template <int TILES, bool SELECTIVE>
 static int launch_chunks(const ScanArgs& a, int64_t sequences, cudaStream_t s) {
   static std::atomic<uint64_t> opted{0};
   if (first_on_device(opted)) cudaFuncSetAttribute(decay_chunk_kernel<TILES, SELECTIVE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-  return launch_after(decay_chunk_kernel<TILES, SELECTIVE>, dim3((unsigned)ceil_div(a.vdim, CH_COLS), (unsigned)a.heads, (unsigned)sequences), dim3(128), chunk_smem_bytes(a.dim), s,
-                      SELECTIVE ? "fb_selective_scan (chunks)" : "fb_decay_scan (chunks)", a);
+  // (not ahead of the kernel before: long CTAs that find the GPU half full stand two on one SM and none on another)
+  decay_chunk_kernel<TILES, SELECTIVE><<<dim3((unsigned)ceil_div(a.vdim, CH_COLS), (unsigned)a.heads, (unsigned)sequences), 128, chunk_smem_bytes(a.dim), s>>>(a);
+  return launch_status(SELECTIVE ? "fb_selective_scan (chunks)" : "fb_decay_scan (chunks)");
 }
 
 template <bool SELECTIVE>
